@@ -36,7 +36,7 @@ NVCC_FLAGS = [
     "-I", str(CSRC / "kernels"), "-I", str(CSRC / "include"),
 ]
 # bandwidth-bound generic kernels keep IEEE-accurate transcendentals (they are compared against f32 / f64 references at tight tolerances)
-PRECISE_MATH = {"elementwise.cu", "reduce_index.cu", "nn_ops.cu"}
+PRECISE_MATH = {"elementwise.cu", "reduce_index.cu", "nn_ops.cu", "stream_ops.cu", "moe.cu", "latent_attn.cu"}
 # no errno / trap bookkeeping for the math builtins (lets the Box-Muller and Philox loops vectorise); no FMA contraction, so the random streams are
 # the same on every x86-64 machine whatever instruction set the vector path picks
 CXX_FLAGS = ["-O3", "-fno-math-errno", "-fno-trapping-math", "-ffp-contract=off", "-std=c++20", "-fPIC", "-fvisibility=hidden", "-pthread", "-I", str(CSRC / "include"), "-I", str(CSRC / "runtime")]
@@ -110,6 +110,12 @@ def build_runtime(verbose=False):
     link = [CXX, "-shared", "-pthread"]
     lib = _build_lib("libft_runtime.so", srcs, CXX, CXX_FLAGS, link, [CSRC / "runtime", CSRC / "include"], verbose)
     return lib
+
+
+def build_one(name: str):
+    """Builds the one library a process asks for (the loader's way in a fresh checkout)."""
+    OUT.mkdir(parents=True, exist_ok=True)
+    return build_kernels() if name == "libft_kernels.so" else build_runtime()
 
 
 SANITIZERS = {"thread": "thread", "address": "address,undefined"}

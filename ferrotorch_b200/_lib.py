@@ -36,7 +36,7 @@ def _load(name: str):
     if not path.exists():
         if os.environ.get("FT_NO_AUTOBUILD") != "1":
             from . import _build
-            _build.build_all()
+            _build.build_one(name)
     if not path.exists():
         raise NativeLibraryMissing(f"{path} is missing; run `python -m ferrotorch_b200._build`")
     # local binding: the kernels library carries its own static CUDA runtime, whose symbols must not interpose on the ones other

@@ -16,13 +16,18 @@ constexpr int TM = 64, TN = 64, TK = 16;
 // op(A)[m][k]: ta == 0 -> A[m * lda + k], ta == 1 -> A[k * lda + m]; same for B with (k, n).
 template <typename T>
 __global__ void __launch_bounds__(256) gemm_simt_kernel(const T* __restrict__ A, const T* __restrict__ B, T* __restrict__ C, int M, int N, int K, int64_t lda, int64_t ldb,
-                                                        int64_t ldc, int64_t sA, int64_t sB, int64_t sC, int ta, int tb, T alpha, T beta) {
+                                                        int64_t ldc, int64_t sA, int64_t sB, int64_t sC, int ta, int tb, T alpha, T beta, const int* __restrict__ group) {
   __shared__ T As[TK][TM + 1], Bs[TK][TN + 1];
   const int bz = blockIdx.z;
   A += (size_t)bz * sA;
   B += (size_t)bz * sB;
   C += (size_t)bz * sC;
   const int m0 = blockIdx.y * TM, n0 = blockIdx.x * TN;
+  if (group != nullptr) {                                       // rows in 128-row tiles of one group each: the group's B matrix, -1 = unused rows
+    const int g = group[m0 / 128];
+    if (g < 0) return;
+    B += (size_t)g * sB;
+  }
   const int tx = threadIdx.x % 16, ty = threadIdx.x / 16;       // each thread owns a 4 x 4 patch
   T acc[4][4] = {};
   for (int k0 = 0; k0 < K; k0 += TK) {
@@ -95,9 +100,19 @@ FT_EXPORT int ft_gemm_simt(int dtype, const void* A, const void* B, void* C, int
   if (batch < 1 || M < 1 || N < 1 || K < 1 || batch > 65535) return FT_ERR_ARG;
   const dim3 grid((N + TN - 1) / TN, (M + TM - 1) / TM, batch);
   if (grid.y > 65535) return FT_ERR_ARG;
-  if (dtype == 0) gemm_simt_kernel<float><<<grid, 256, 0, st>>>((const float*)A, (const float*)B, (float*)C, M, N, K, lda, ldb, ldc, sA, sB, sC, ta, tb, (float)alpha, (float)beta);
-  else if (dtype == 3) gemm_simt_kernel<double><<<grid, 256, 0, st>>>((const double*)A, (const double*)B, (double*)C, M, N, K, lda, ldb, ldc, sA, sB, sC, ta, tb, alpha, beta);
+  if (dtype == 0) gemm_simt_kernel<float><<<grid, 256, 0, st>>>((const float*)A, (const float*)B, (float*)C, M, N, K, lda, ldb, ldc, sA, sB, sC, ta, tb, (float)alpha, (float)beta, nullptr);
+  else if (dtype == 3) gemm_simt_kernel<double><<<grid, 256, 0, st>>>((const double*)A, (const double*)B, (double*)C, M, N, K, lda, ldb, ldc, sA, sB, sC, ta, tb, alpha, beta, nullptr);
   else return FT_ERR_ARG;
+  return (int)cudaGetLastError();
+}
+
+// f32 form of ft_gemm_grouped: C[m][n] = sum_k A[m][k] B[g][n][k], g = tile_group[m / 128] (-1: rows unused); group_stride elements between groups.
+FT_EXPORT int ft_gemm_simt_grouped(const float* A, const float* B, float* C, int M, int N, int K, int64_t lda, int64_t ldb, int64_t ldc, const int* tile_group,
+                                   int64_t group_stride, cudaStream_t st) {
+  if (M < 1 || N < 1 || K < 1 || tile_group == nullptr) return FT_ERR_ARG;
+  const dim3 grid((N + TN - 1) / TN, (M + TM - 1) / TM, 1);
+  if (grid.y > 65535) return FT_ERR_ARG;
+  gemm_simt_kernel<float><<<grid, 256, 0, st>>>(A, B, C, M, N, K, lda, ldb, ldc, 0, group_stride, 0, 0, 1, 1.f, 0.f, tile_group);
   return (int)cudaGetLastError();
 }
 

@@ -99,7 +99,18 @@ struct TailArgs {
   // A's columns (kb % a_atoms_per_tap) * 64 at rows m + a_shift[t] (zeros outside A).
   int a_atoms_per_tap;
   int a_shift[9];
+  // Grouped product (group null: off): the rows of A come in 128-row tiles that belong to one group each, B stacks the groups' [group_rows, K]
+  // matrices, and tile row i multiplies with group[i]'s (-1: the tile is unused and skipped by every role).
+  const int* group;
+  int group_rows;
 };
+
+// B row offset of a work item's group, -1 when the tile is unused
+FT_DEVICE int group_offset(const TailArgs& t, int m0) {
+  if (t.group == nullptr) return 0;
+  const int g = __ldg(t.group + m0 / BM);
+  return g < 0 ? -1 : g * t.group_rows;
+}
 
 struct WorkItem {
   int tile, split, kb0, kb1;
@@ -189,6 +200,8 @@ ft_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
         int m0, n0;
         const WorkItem wi = decode_item(tile, k_splits, kb_per, num_kb_total, full_items, tail);
         tile_coords(wi.tile, tiles_m, tiles_n, m0, n0);
+        const int b_row0 = group_offset(tail, m0);
+        if (b_row0 < 0) continue;
         const int kb0 = wi.kb0, kb1 = wi.kb1;
         for (int kb = kb0; kb < kb1; kb++) {
           if (!mbar_wait_deadline(&empty_bar[s], phase ^ 1)) { ft_set_status(status, FT_K_GEMM, 1, s); ok = false; break; }
@@ -203,7 +216,7 @@ ft_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
             for (int j = 0; j < BM / 64; j++) tma_load_2d(a_dst + j * (BK * 128), &tmA, &full_bar[s], m0 + j * 64, kb * BK);
           }
           if constexpr (!B_MN) {
-            tma_load_2d(b_dst, &tmB, &full_bar[s], kb * BK, n0);
+            tma_load_2d(b_dst, &tmB, &full_bar[s], kb * BK, n0 + b_row0);
           } else if (tail.b_atoms_per_tap == 0) {
 #pragma unroll
             for (int j = 0; j < BN / 64; j++) tma_load_2d(b_dst + j * (BK * 128), &tmB, &full_bar[s], n0 + j * 64, kb * BK);
@@ -233,6 +246,11 @@ ft_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       uint32_t s = 0, phase = 0, acc = 0, acc_phase = 0;
       bool ok = true;
       for (int tile = blockIdx.x; tile < num_tiles && ok; tile += gridDim.x) {
+        if (tail.group != nullptr) {
+          int gm0, gn0;
+          tile_coords(decode_item(tile, k_splits, kb_per, num_kb_total, full_items, tail).tile, tiles_m, tiles_n, gm0, gn0);
+          if (group_offset(tail, gm0) < 0) continue;
+        }
         if (!mbar_wait_deadline(&tempty_bar[acc], acc_phase ^ 1)) { ft_set_status(status, FT_K_GEMM, 2, acc); ok = false; break; }
         tc_fence_after();
         const uint32_t d_tmem = tmem_base + acc * BN;
@@ -283,6 +301,7 @@ ft_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ 
       int m0, n0;
       const WorkItem wi = decode_item(tile, k_splits, kb_per, num_kb_total, full_items, tail);
       tile_coords(wi.tile, tiles_m, tiles_n, m0, n0);
+      if (group_offset(tail, m0) < 0) continue;
       const int split = wi.split;
       const bool empty_split = wi.kb0 >= wi.kb1;
       if (!mbar_wait_deadline(&tfull_bar[acc], acc_phase)) { if (lane == 0) ft_set_status(status, FT_K_GEMM, 4, acc); ok = false; break; }
@@ -436,7 +455,7 @@ TailWs g_tail_ws[64][TAIL_SLOTS] = {};
 int g_tail_enabled = -1;
 
 TailArgs plan_tail(int dev, int tiles, int num_kb, int k_splits, int sms, cudaStream_t stream) {
-  TailArgs t{0, 1, nullptr, nullptr, 0, {0, 0, 0, 0, 0, 0, 0, 0, 0}, 0, {0, 0, 0, 0, 0, 0, 0, 0, 0}};
+  TailArgs t{0, 1, nullptr, nullptr, 0, {0, 0, 0, 0, 0, 0, 0, 0, 0}, 0, {0, 0, 0, 0, 0, 0, 0, 0, 0}, nullptr, 0};
   if (g_tail_enabled < 0) {
     const char* e = getenv("FT_GEMM_TAIL");
     g_tail_enabled = (e && e[0] == '1') ? 1 : 0;
@@ -498,14 +517,14 @@ int g_num_sms[64] = {0};
 static int gemm_impl(const void* A, const void* B, void* D, const void* bias, int M, int N, int K, int64_t lda, int64_t ldb,
                      int64_t ldd, int a_mn, int b_mn, int out_f32, int k_splits, cudaStream_t stream, EpiArgs epi = EpiArgs{0, nullptr, 0, 0},
                      int b_cols = 0, int b_atoms_per_tap = 0, const int* b_shift = nullptr, int a_cols = 0, int64_t a_rows = 0, int a_taps = 0,
-                     const int* a_shift = nullptr, int64_t b_rows = 0) {
+                     const int* a_shift = nullptr, int64_t b_rows = 0, const int* group = nullptr, int groups = 0, int group_rows = 0) {
   if (epi.act < 0 || epi.act > 4) return FT_ERR_ARG;
   const bool in_bf16 = !epi.in_f16;
   if (M <= 0 || N <= 0 || K <= 0 || k_splits < 1 || k_splits > 256) return FT_ERR_ARG;
   if ((lda & 7) || (ldb & 7) || ((ldd * (out_f32 ? 4 : 2)) & 15)) return FT_ERR_ARG;
   // Large-M problems without a row-shift table go to the CTA-pair kernel (256 x 256 tiles, tcgen05 cta_group::2); FT_ERR_DRIVER from it means
   // that this device cannot co-schedule pairs, and the one-SM kernel below takes over.
-  if (a_cols == 0 && b_atoms_per_tap == 0 && ft_gemm2_wanted(M, N, K, k_splits)) {
+  if (a_cols == 0 && b_atoms_per_tap == 0 && group == nullptr && ft_gemm2_wanted(M, N, K, k_splits)) {
     const int r2 = ft_gemm2_launch(A, B, D, bias, M, N, K, lda, ldb, ldd, a_mn, b_mn, out_f32, k_splits, stream, Gemm2Epi{epi.act, epi.residual, epi.ldr, epi.in_f16});
     if (r2 != FT_ERR_DRIVER) return r2;
   }
@@ -523,7 +542,7 @@ static int gemm_impl(const void* A, const void* B, void* D, const void* bias, in
                                  CU_TENSOR_MAP_SWIZZLE_128B);
   else       r = ft_make_tmap_2d(&tA, A, 2, in_bf16, (uint64_t)M, (uint64_t)K, (uint64_t)lda * 2, 64, BK, CU_TENSOR_MAP_SWIZZLE_128B);
   if (r) return r;
-  if (!b_mn) r = ft_make_tmap_2d(&tB, B, 2, in_bf16, (uint64_t)K, (uint64_t)N, (uint64_t)ldb * 2, BK, BN, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!b_mn) r = ft_make_tmap_2d(&tB, B, 2, in_bf16, (uint64_t)K, group ? (uint64_t)groups * group_rows : (uint64_t)N, (uint64_t)ldb * 2, BK, BN, CU_TENSOR_MAP_SWIZZLE_128B);
   else       r = ft_make_tmap_2d(&tB, B, 2, in_bf16, (uint64_t)(b_cols > 0 ? b_cols : N), (uint64_t)(b_rows > 0 ? b_rows : K), (uint64_t)ldb * 2, 64, BK,
                                  CU_TENSOR_MAP_SWIZZLE_128B);
   if (r) return r;
@@ -533,7 +552,9 @@ static int gemm_impl(const void* A, const void* B, void* D, const void* bias, in
   if (r) return r;
 
   const int sms = g_num_sms[dev];
-  TailArgs tail = plan_tail(dev, ((M + BM - 1) / BM) * ((N + BN - 1) / BN), (K + BK - 1) / BK, k_splits, sms, stream);
+  TailArgs tail = plan_tail(dev, group ? 1 : ((M + BM - 1) / BM) * ((N + BN - 1) / BN), (K + BK - 1) / BK, k_splits, sms, stream);
+  tail.group = group;
+  tail.group_rows = group_rows;
   if (a_cols > 0) {
     tail.a_atoms_per_tap = a_cols / 64;
     for (int t = 0; t < 9; t++) tail.a_shift[t] = t < a_taps ? a_shift[t] : 0;
@@ -608,6 +629,16 @@ FT_EXPORT int ft_gemm_gated_a(const void* A, const void* B, void* D, int M, int 
   if (!ft_gemm2_wanted(M, N, K, 1)) return FT_ERR_ARG;
   const Gemm2Gate gate{(const uint32_t*)counters, expected, 1, 0, (long long)M, (long long)rows_per_piece, 1, m_rot % ((M + 255) / 256)};
   return ft_gemm2_launch(A, B, D, nullptr, M, N, K, lda, ldb, ldd, 0, 0, out_f32, 1, stream, Gemm2Epi{0, nullptr, 0, 0}, gate);
+}
+
+// Grouped product over ragged groups of rows: D[m][n] = sum_k A[m][k] B[g][n][k] with g = tile_group[m / 128] (device array, one entry per 128 rows of
+// A; -1: rows unused, D keeps its contents there). B: [groups][group_rows][ldb] bf16, group_rows >= N. Used by the experts of a mixture, whose token
+// segments start at multiples of 128 rows.
+FT_EXPORT int ft_gemm_grouped(const void* A, const void* B, void* D, int M, int N, int K, int64_t lda, int64_t ldb, int64_t ldd, int out_f32, const int* tile_group,
+                              int groups, int group_rows, cudaStream_t stream) {
+  if (tile_group == nullptr || groups < 1 || group_rows < N || (int64_t)groups * group_rows > 0x7fffffffll) return FT_ERR_ARG;
+  return gemm_impl(A, B, D, nullptr, M, N, K, lda, ldb, ldd, 0, 0, out_f32, 1, stream, EpiArgs{0, nullptr, 0, 0}, 0, 0, nullptr, 0, 0, 0, nullptr, 0, tile_group, groups,
+                   group_rows);
 }
 
 // Split-K form: partial[s][M][N] (f32, contiguous planes of M*ldd elements) = A (x) B restricted to the s-th slice of K.

@@ -52,6 +52,16 @@ class KvCache:
         for l in self.layers:
             l.truncate(n)
 
+    def expand(self, n: int) -> None:
+        """One cached sequence becomes ``n`` equal ones (the start of a beam search)."""
+        for l in self.layers:
+            l.k, l.v = l.k.repeat(n, 1, 1, 1), l.v.repeat(n, 1, 1, 1)
+
+    def reorder(self, index: torch.Tensor) -> None:
+        """Sequence ``i`` becomes a copy of sequence ``index[i]``."""
+        for l in self.layers:
+            l.k, l.v = l.k[index], l.v[index]
+
     def clone(self) -> "KvCache":
         c = KvCache(len(self.layers))
         for a, b in zip(c.layers, self.layers):
@@ -281,8 +291,7 @@ def beam_search(model, new_cache, ids: torch.Tensor, cfg: GenerationConfig) -> t
     top = logp.topk(nb, -1)
     seqs = torch.cat([ids.repeat(nb, 1), top.indices.view(nb, 1)], 1)
     scores = top.values.view(nb)
-    for l in cache.layers:
-        l.k, l.v = l.k.repeat(nb, 1, 1, 1), l.v.repeat(nb, 1, 1, 1)
+    cache.expand(nb)
     finished: List[Tuple[float, torch.Tensor]] = []
     for step in range(1, cfg.max_new_tokens):
         logp = model(seqs[:, -1:], cache)[:, -1].log_softmax(-1)
@@ -291,8 +300,7 @@ def beam_search(model, new_cache, ids: torch.Tensor, cfg: GenerationConfig) -> t
         beam, tok = top.indices // logp.shape[-1], top.indices % logp.shape[-1]
         seqs = torch.cat([seqs[beam], tok[:, None]], 1)
         scores = top.values
-        for l in cache.layers:
-            l.k, l.v = l.k[beam], l.v[beam]
+        cache.reorder(beam)
         if cfg.eos_token_id is not None:
             ended = tok == cfg.eos_token_id
             for b in torch.where(ended)[0].tolist():
@@ -304,6 +312,13 @@ def beam_search(model, new_cache, ids: torch.Tensor, cfg: GenerationConfig) -> t
         if scores[b] > float("-inf"):
             finished.append((float(scores[b]) / (seqs.shape[1] - ids.shape[1]) ** cfg.length_penalty, seqs[b]))
     return max(finished, key=lambda t: t[0])[1][None]
+
+
+def _device_of(model):
+    """Device a cached model takes its token ids on."""
+    if hasattr(model, "W"):
+        return model.W["model.embed_tokens.weight"].device
+    return getattr(model, "device", "cpu")
 
 
 @torch.no_grad()
@@ -323,7 +338,7 @@ def generate_with_streamer(model, prompt_ids: Sequence[int], config: GenerationC
     if config.repetition_penalty <= 0.0:
         raise InvalidArgument(f"generate: repetition_penalty must be > 0, got {config.repetition_penalty}")
     cache = (new_cache or model.new_cache)()
-    dev = getattr(model, "W", {}).get("model.embed_tokens.weight").device if hasattr(model, "W") else "cpu"
+    dev = _device_of(model)
     rng = XorShift64(config.seed)
     ids, produced, stops = list(int(t) for t in prompt_ids), [], set(config.stop_ids())
     feed = ids
@@ -411,7 +426,7 @@ class LlamaHandle(ModelHandle):
     def __init__(self, model, new_cache: Optional[Callable[[], "KvCache"]] = None, vocab_size: Optional[int] = None):
         self.model, self._new_cache = model, new_cache or model.new_cache
         self._vocab = vocab_size if vocab_size is not None else model.cfg.vocab_size
-        self._dev = model.W["model.embed_tokens.weight"].device if hasattr(model, "W") else "cpu"
+        self._dev = _device_of(model)
         self._seen: List[int] = []
         self._cache = None
 

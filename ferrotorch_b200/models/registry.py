@@ -1,0 +1,92 @@
+"""Architectures by name: which configuration and engine a checkpoint directory (``config.json`` + safetensors) takes.
+
+``load_engine(directory)`` reads ``config.json``, finds the architecture (its ``architecture``, ``architectures`` or ``model_type`` entry), loads the weights and
+returns an engine with ``step`` / ``generate`` / ``release``; ``register_architecture`` adds another one.
+"""
+from __future__ import annotations
+
+import json
+from dataclasses import dataclass
+from pathlib import Path
+from typing import Callable, Dict, List
+
+import torch
+
+from ..errors import InvalidArgument
+
+
+@dataclass
+class Architecture:
+    """``config(dict)`` parses ``config.json``; ``engine(config, weights, device, dtype, max_tokens)`` builds the engine."""
+    name: str
+    config: Callable[[dict], object]
+    engine: Callable[..., object]
+    aliases: tuple = ()
+
+
+_ARCHITECTURES: Dict[str, Architecture] = {}
+
+
+def register_architecture(arch: Architecture) -> None:
+    for n in (arch.name, *arch.aliases):
+        _ARCHITECTURES[n.lower()] = arch
+
+
+def architectures() -> List[str]:
+    return sorted({a.name for a in _ARCHITECTURES.values()})
+
+
+def architecture_of(config: dict) -> Architecture:
+    names = [config.get("architecture"), *(config.get("architectures") or []), config.get("model_type")]
+    for n in names:
+        if n and str(n).lower() in _ARCHITECTURES:
+            return _ARCHITECTURES[str(n).lower()]
+    raise InvalidArgument(f"no registered architecture for {[n for n in names if n]}; known: {', '.join(architectures())}")
+
+
+def load_model_config(directory):
+    """``(architecture, parsed configuration)`` of a checkpoint directory."""
+    d = json.loads((Path(directory) / "config.json").read_text())
+    arch = architecture_of(d)
+    return arch, arch.config(d)
+
+
+def load_checkpoint_weights(directory) -> Dict[str, torch.Tensor]:
+    """All tensors of ``model.safetensors`` or of the shards that ``model.safetensors.index.json`` lists (host memory)."""
+    from ..serialize import load_safetensors, load_safetensors_sharded
+    d = Path(directory)
+    idx = d / "model.safetensors.index.json"
+    return load_safetensors_sharded(idx) if idx.exists() else load_safetensors(d / "model.safetensors")
+
+
+def load_engine(directory, device="cuda", dtype: torch.dtype = torch.bfloat16, max_tokens: int = 4096):
+    arch, cfg = load_model_config(directory)
+    return arch.engine(cfg, load_checkpoint_weights(directory), device, dtype, max_tokens)
+
+
+def _ginisun_config(d: dict):
+    from .ginisun import GinisunConfig
+    return GinisunConfig.from_dict(d)
+
+
+def _ginisun_engine(cfg, weights, device, dtype, max_tokens):
+    from .ginisun import GinisunModel
+    from .serving import ServingEngine
+    return ServingEngine(GinisunModel(cfg, weights, device, dtype), max_tokens=max_tokens)
+
+
+def _llama_config(d: dict):
+    from .llama import LlamaConfig
+    return LlamaConfig.from_hf(d)
+
+
+def _llama_engine(cfg, weights, device, dtype, max_tokens):
+    from .llama_gen import CachedLlama
+    from .serving import CachedModelEngine
+    if max_tokens > cfg.max_position_embeddings:
+        cfg.max_position_embeddings = max_tokens
+    return CachedModelEngine(CachedLlama(cfg, {k: v.to(device, dtype) for k, v in weights.items()}), cfg.vocab_size, device)
+
+
+register_architecture(Architecture("Ginisun", _ginisun_config, _ginisun_engine))
+register_architecture(Architecture("LlamaForCausalLM", _llama_config, _llama_engine, ("llama",)))

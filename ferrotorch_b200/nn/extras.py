@@ -115,6 +115,76 @@ class PagedKVCache:
         return t.to(self.k.device)
 
 
+class PagedRowCache:
+    """Paged storage of one row per token and layer, ``[num_pages, page_size, row]`` per layer with its own row length, behind one page table per
+    sequence that all layers share: for mixers that cache a single vector per token (latent attention). Pages come from a :class:`PagePool`; a
+    shared page is copied before it is written (:meth:`fork`)."""
+
+    def __init__(self, pool: PagePool, row_sizes: Sequence[int], device="cpu", dtype=torch.float32):
+        self.pool = pool
+        n, ps = len(pool.pages), pool.page_size
+        self.rows = [torch.zeros(n, ps, r, device=device, dtype=dtype) for r in row_sizes]
+        self.tables: Dict[object, List[int]] = {}
+        self.lengths: Dict[object, int] = {}
+
+    def add_sequence(self, seq_id) -> None:
+        if seq_id in self.tables:
+            raise InvalidArgument(f"sequence {seq_id!r} is already in the cache")
+        self.tables[seq_id], self.lengths[seq_id] = [], 0
+
+    def free_sequence(self, seq_id) -> None:
+        for p in self.tables.pop(seq_id, []):
+            self.pool.release(p)
+        self.lengths.pop(seq_id, None)
+
+    def pages_for(self, seq_id, tokens: int) -> int:
+        """Pages that :meth:`reserve` would take from the pool."""
+        return max(0, -(-tokens // self.pool.page_size) - len(self.tables.get(seq_id, ())))
+
+    def reserve(self, seq_id, tokens: int) -> None:
+        """Makes room for ``tokens`` tokens in all, with every page from the current length on owned by this sequence alone."""
+        table, ps = self.tables[seq_id], self.pool.page_size
+        for i in range(self.lengths[seq_id] // ps, min(len(table), -(-tokens // ps))):
+            if self.pool.pages[table[i]].ref_count > 1:
+                fresh = self.pool.allocate()
+                for r in self.rows:
+                    r[fresh].copy_(r[table[i]])
+                self.pool.release(table[i])
+                table[i] = fresh
+        while len(table) * ps < tokens:
+            table.append(self.pool.allocate())
+
+    def slots(self, seq_id, start: int, count: int) -> List[int]:
+        """Row indices (page * page_size + offset) of positions ``start .. start + count - 1``."""
+        t, ps = self.tables[seq_id], self.pool.page_size
+        return [t[p // ps] * ps + p % ps for p in range(start, start + count)]
+
+    def truncate(self, seq_id, n: int) -> None:
+        """Forgets every token from position ``n`` on; pages that hold none of the rest go back to the pool."""
+        table, ps = self.tables[seq_id], self.pool.page_size
+        while len(table) > -(-n // ps):
+            self.pool.release(table.pop())
+        self.lengths[seq_id] = min(self.lengths[seq_id], n)
+
+    def fork(self, src, dst) -> None:
+        self.add_sequence(dst)
+        self.tables[dst], self.lengths[dst] = list(self.tables[src]), self.lengths[src]
+        for p in self.tables[dst]:
+            self.pool.retain(p)
+
+    def gather(self, layer: int, seq_id) -> torch.Tensor:
+        n = self.lengths[seq_id]
+        idx = torch.tensor(self.slots(seq_id, 0, n), device=self.rows[layer].device, dtype=torch.long)
+        return self.rows[layer].flatten(0, 1)[idx]
+
+    def block_table(self, seq_ids: Sequence, max_blocks: int) -> torch.Tensor:
+        """Host table ``[sequences, max_blocks]`` (int32, -1 past a sequence's pages)."""
+        t = torch.full((len(seq_ids), max_blocks), -1, dtype=torch.int32)
+        for i, s in enumerate(seq_ids):
+            t[i, : len(self.tables[s])] = torch.tensor(self.tables[s], dtype=torch.int32)
+        return t
+
+
 class PagedAttentionManager:
     """One :class:`PagedKVCache` per layer sharing a page pool; tracks live sequences."""
 
