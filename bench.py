@@ -43,6 +43,9 @@ def _parse():
     ap.add_argument("--breakdown", action="store_true",
                     help="after the timed runs, time every kernel class of one step with CUDA events (optimizer serialised on the compute "
                          "stream so that the classes add up to the step) and add the table to the JSON line")
+    ap.add_argument("--serving", nargs="?", const="1k,2k,4k", default=None, metavar="SIZES",
+                    help="instead of the headline: prefill and decode throughput of the serving models (Ginisun beside Llama) on a few layers of "
+                         "the named sizes with random weights, and every kernel class against its roofline")
     return ap.parse_args()
 
 
@@ -160,6 +163,13 @@ def main():
     args = _parse()
     if args.impl == "reference":
         return reference_arm(args)
+    if args.serving:
+        sampler = ClockSampler(0)
+        sampler.start()
+        from benchmarks.serving_bench import main as serving
+        rc = serving(args.serving)
+        print(json.dumps({"clocks": sampler.stop()}))
+        return rc
     import torch
     import torch.distributed as dist
     world = int(os.environ.get("WORLD_SIZE", "1"))

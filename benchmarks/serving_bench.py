@@ -1,0 +1,224 @@
+"""Prefill and decode throughput of the serving models on layers of realistic size with random weights: the Ginisun decoder beside a Llama decoder of the
+same width and the same number of feed-forward neurons per token. Run through ``bench.py --serving``.
+
+Every kernel class is also timed (CUDA events around its launches, L2 flushed by the step's own traffic) against its roofline, the slower of algorithmic
+bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate. Times of single launches below ~5 us are dominated by launch overhead.
+"""
+from __future__ import annotations
+
+import json
+import statistics
+from pathlib import Path
+
+import torch
+
+from ferrotorch_b200 import _lib
+from ferrotorch_b200.models import GenerationConfig, LlamaConfig
+from ferrotorch_b200.models.ginisun import GinisunConfig, GinisunModel, RandomGinisunWeights
+from ferrotorch_b200.models.llama_infer import LlamaTPEngine, TPContext
+from ferrotorch_b200.models.serving import ServingEngine, StepEntry
+
+SIZES = {
+    "1k": dict(width=1024, heads=8, dim=64, rot_dim=32, vdim=64, kv_rank=256, experts=16, top=2, ff=1024, shared_ff=1024),
+    "2k": dict(width=2048, heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, experts=64, top=6, ff=1408, shared_ff=2816),
+    "4k": dict(width=4096, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, experts=32, top=4, ff=2048, shared_ff=4096),
+}
+VOCAB = 32768
+
+
+def peaks():
+    p = Path(__file__).resolve().parents[1] / "MEASURED_PEAKS.json"
+    if p.exists():
+        d = json.loads(p.read_text())
+        return d["hbm_gbs"] * 1e9, d["bf16_tflops"] * 1e12, "measured"
+    return 6.65e12, 1.59e15, "fallback"
+
+
+def timed(fn, reps=7, warm=3):
+    for _ in range(warm):
+        fn()
+    out = []
+    for _ in range(reps):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        fn()
+        e1.record()
+        torch.cuda.synchronize()
+        out.append(e0.elapsed_time(e1))
+    return statistics.median(out)
+
+
+def kernel_table(fn, classify, roofs, bw, fl, reps=5):
+    """us per call and roofline fraction by kernel class; ``roofs[label] = (bytes, flops)`` per call."""
+    rows = {}
+    for i in range(reps):
+        _lib.trace_begin(classify)
+        fn()
+        for k, v in _lib.trace_end().items():
+            rows.setdefault(k, []).append((v["ms"] * 1e3 / v["calls"], v["calls"]))
+    out = {}
+    for k, v in rows.items():
+        us = statistics.median(x[0] for x in v)
+        out[k] = {"us": round(us, 1), "calls": v[0][1]}
+        if k in roofs:
+            b, f = roofs[k]
+            out[k]["roofline"] = round(max(b / bw, f / fl) * 1e6 / us, 3)
+    return out
+
+
+def _by_shape(names):
+    """GEMM launches by (N, K) -> label, everything else by launcher name."""
+    def c(fn, raw):
+        if fn in ("ft_gemm_bf16", "ft_gemm_bf16_splitk"):
+            o = 4 if fn == "ft_gemm_bf16" else 3
+            return names.get((raw[o + 1], raw[o + 2]), f"gemm n={raw[o + 1]} k={raw[o + 2]}")
+        if fn == "ft_gemm_grouped":
+            return names.get((raw[4], raw[5]), "grouped gemm")
+        return names.get(fn, fn)
+    return c
+
+
+def run_ginisun(size, layers, batch, prompt, ctx, steps, kernels=True):
+    bw, fl, _ = peaks()
+    s = SIZES[size]
+    cfg = GinisunConfig.uniform(layers, VOCAB, streams=4, **s)
+    eng = ServingEngine(GinisunModel(cfg, RandomGinisunWeights(cfg)), max_tokens=max(batch * (ctx + steps * 4 + 64), prompt + 64), max_sequences=batch + 1)
+    g = torch.Generator().manual_seed(1)
+    ids = torch.randint(0, VOCAB, (prompt,), generator=g).tolist()
+    def prefill():
+        eng.step([StepEntry("p", ids, [prompt - 1])], ["p"])
+    from ferrotorch_b200.models.serving import RowBatch
+    eng._admit([StepEntry("p", ids, [prompt - 1])])
+    rb = RowBatch([StepEntry("p", ids, [prompt - 1])], eng.cache, eng.device, eng.max_blocks)
+    rb.tiles_for(eng.model.subs[0].attn.dims)
+    device_prefill = lambda: eng.model.forward_rows(rb, eng.cache)          # the device part: tables of the batch are built once
+    pre_ms, pre_e2e = timed(device_prefill), timed(lambda: (eng.release("p"), prefill()))
+    W, H, T = s["width"], s["heads"], prompt
+    D = eng.model.subs[0].attn.dims
+    F, SF, E, top = s["ff"], s["shared_ff"], s["experts"], s["top"]
+    nkv = H * (D.dim8 + D.v8)
+    table = None
+    if kernels:
+        eng._admit([StepEntry("p", ids, [])])
+        names = {(D.proj_cols, W): "projection gemm", (nkv, D.rank): "key/value expansion gemm", (W, H * D.v8): "output gemm", (E, W): "router gemm",
+                 (2 * F, W): "experts gate/up gemm", (W, F): "experts down gemm", (2 * SF, W): "shared gate/up gemm", (W, SF): "shared down gemm"}
+        pairs = T * top
+        def g_(n, k, out=2, m=T): return (2 * (m * k + n * k) + out * m * n, 2 * m * n * k)
+        roofs = {"projection gemm": g_(D.proj_cols, W), "key/value expansion gemm": g_(nkv, D.rank), "output gemm": g_(W, H * D.v8, 4),
+                 "experts gate/up gemm": (2 * (pairs * W + E * 2 * F * W + pairs * 2 * F), 4 * pairs * F * W), "experts down gemm": (2 * (pairs * W + E * F * W + pairs * F), 2 * pairs * F * W),
+                 "shared gate/up gemm": g_(2 * SF, W), "shared down gemm": g_(W, SF, 4),
+                 "ft_latent_flash": (2 * T * (H * (D.dim8 + D.rot8) + nkv + H * D.v8), H * T * T * (D.dim + D.rot_dim + D.vdim)),
+                 "ft_latent_prep": (2 * T * (2 * H * D.rot8 + D.rank + D.rot8 + 2 * D.row), 0),
+                 "ft_hyper_update": (T * W * (32 + 2 + 4 + top) if SF else T * W * (34 + 2 * top), 0),   # average of the two sublayers, see below
+                 "ft_moe_gather": (4 * pairs * W, 0), "ft_moe_act": ((pairs * F * 6 + T * SF * 6) / 2, 0)}
+        # streams read and written in f32 (8 bytes each), bf16 operand out; attention adds one f32 plane, the mixture its bf16 rows (+ one f32 plane)
+        roofs["ft_hyper_update"] = (T * W * (4 * 8 + 2 + (4 + (2 * top + (4 if SF else 0))) / 2), 0)
+        table = kernel_table(device_prefill, _by_shape(names), roofs, bw, fl)
+    eng.release("p")
+    # decode
+    seqs = [f"s{i}" for i in range(batch)]
+    for q in seqs:
+        eng.step([StepEntry(q, torch.randint(0, VOCAB, (ctx,), generator=g).tolist(), [])])
+    eng.decode_greedy(seqs, [1] * batch, 4)
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    best = []
+    for _ in range(3):
+        torch.cuda.synchronize()
+        e0.record()
+        eng.decode_greedy(seqs, [1] * batch, steps)
+        e1.record()
+        torch.cuda.synchronize()
+        best.append(e0.elapsed_time(e1) / steps)
+    dec_ms = statistics.median(best)
+    dtable = None
+    if kernels:
+        eng.use_graph = False
+        for q in seqs:
+            eng.cache.reserve(q, eng.cache.lengths[q] + 1)
+        eng.state.load([1 + i for i in range(batch)], [eng.cache.lengths[q] for q in seqs], eng.cache.block_table(seqs, eng.max_blocks))
+        positions, lens = eng.state.positions.clone(), eng.state.seq_lens.clone()
+        tokens = eng.state.tokens.clone()
+        def one():
+            eng.state.positions.copy_(positions); eng.state.seq_lens.copy_(lens); eng.state.tokens.copy_(tokens)
+            eng.model.decode(eng.state, batch, eng.cache)
+        one()
+        active = int(eng.model._moe_buffers.n_active)               # experts in use (of the last layer; the layers are alike)
+        L = eng.cache.lengths[seqs[0]] + 1
+        names = {(D.proj_cols, W): "projection gemm", (W, H * D.v8): "output gemm", (VOCAB, W): "head gemm"}
+        roofs = {"projection gemm": (2 * D.proj_cols * W, 0), "output gemm": (2 * H * D.v8 * W, 0), "head gemm": (2 * VOCAB * W, 0),
+                 "ft_latent_decode": (2 * batch * L * D.row, 2 * batch * H * L * (D.row + D.r16)), "ft_latent_decode_prep": (2 * H * D.dim8 * D.rank, 0),
+                 "ft_skinny_heads": (2 * H * D.v8 * D.rank, 0), "ft_moe_gate_up_small": (4 * W * (active * F + SF), 0), "ft_moe_down_small": (2 * W * (active * F + SF), 0),
+                 "ft_hyper_update": (batch * W * 40, 0)}
+        dtable = kernel_table(one, _by_shape(names), roofs, bw, fl)
+        eng.use_graph = True
+    eng.check()
+    return {"prefill_ms": round(pre_ms, 3), "prefill_tokens_per_s": round(prompt / pre_ms * 1e3), "prefill_e2e_ms": round(pre_e2e, 3), "decode_ms_per_step": round(dec_ms, 4),
+            "decode_tokens_per_s": round(batch / dec_ms * 1e3), "active_experts": active if kernels else None, "prefill_kernels": table,
+            "decode_kernels": dtable}
+
+
+def run_llama(size, layers, batch, prompt, ctx, steps, kernels=True):
+    bw, fl, _ = peaks()
+    s = SIZES[size]
+    W, H = s["width"], s["width"] // 128
+    kvh = max(1, H // 4)
+    F = s["top"] * s["ff"] + s["shared_ff"]
+    cfg = LlamaConfig(vocab_size=VOCAB, hidden_size=W, intermediate_size=F, num_hidden_layers=layers, num_attention_heads=H, num_key_value_heads=kvh)
+    g = torch.Generator().manual_seed(1)
+    eng = LlamaTPEngine(cfg, TPContext("cuda"), max_batch=1, max_seq=prompt + 16)
+    ids = torch.randint(0, VOCAB, (1, prompt), generator=g).cuda()
+    pre_ms = timed(lambda: eng.prefill(ids))
+    T, nq = prompt, (H + 2 * kvh) * 128
+    table = dtable = None
+    def g_(n, k, m=T): return (2 * (m * k + n * k + m * n), 2 * m * n * k)
+    if kernels:
+        names = {(nq, W): "qkv gemm", (W, H * 128): "output gemm", (2 * F, W): "gate/up gemm", (W, F): "down gemm"}
+        roofs = {"qkv gemm": g_(nq, W), "output gemm": g_(W, H * 128), "gate/up gemm": g_(2 * F, W), "down gemm": g_(W, F),
+                 "ft_flash_fwd": (2 * T * (nq + H * 128), H * T * T * 256), "ft_rmsnorm_fwd": (6 * T * W, 0), "ft_swiglu_fwd": (6 * T * F, 0), "ft_add_bf16": (6 * T * W, 0),
+                 "ft_rope_inplace": (4 * T * (H + kvh) * 128, 0)}
+        table = kernel_table(lambda: eng.prefill(ids), _by_shape(names), roofs, bw, fl)
+    del eng
+    torch.cuda.empty_cache()
+    eng = LlamaTPEngine(cfg, TPContext("cuda"), max_batch=batch, max_seq=ctx + 4 * steps + 64)
+    eng.prefill(torch.randint(0, VOCAB, (batch, ctx), generator=g).cuda())
+    for _ in range(4):
+        eng.decode_step()
+    best = []
+    for _ in range(3):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        for _ in range(steps):
+            eng.decode_step()
+        e1.record()
+        torch.cuda.synchronize()
+        best.append(e0.elapsed_time(e1) / steps)
+    dec_ms = statistics.median(best)
+    if kernels:
+        L = ctx + 4
+        names = {(nq, W): "qkv gemm", (W, H * 128): "output gemm", (2 * F, W): "gate/up gemm", (W, F): "down gemm", (VOCAB, W): "head gemm"}
+        roofs = {"qkv gemm": (2 * nq * W, 0), "output gemm": (2 * W * H * 128, 0), "gate/up gemm": (4 * F * W, 0), "down gemm": (2 * F * W, 0), "head gemm": (2 * VOCAB * W, 0),
+                 "ft_paged_attn_decode": (4 * batch * L * kvh * 128, 0)}
+        eng.use_graph = False
+        import os
+        os.environ["FT_DECODE_PDL"] = "0"
+        dtable = kernel_table(lambda: eng.decode_step(), _by_shape(names), roofs, bw, fl)
+        os.environ.pop("FT_DECODE_PDL")
+    eng.check()
+    return {"prefill_ms": round(pre_ms, 3), "prefill_tokens_per_s": round(prompt / pre_ms * 1e3), "decode_ms_per_step": round(dec_ms, 4),
+            "decode_tokens_per_s": round(batch / dec_ms * 1e3), "prefill_kernels": table, "decode_kernels": dtable}
+
+
+def main(sizes="1k,2k,4k", layers=4, batch=8, prompt=4096, ctx=2048, steps=64, kernels=True) -> int:
+    torch.cuda.set_device(0)
+    _, _, of = peaks()
+    res = {}
+    for size in sizes.split(","):
+        res[size] = {}
+        for name, run in (("ginisun", run_ginisun), ("llama", run_llama)):
+            res[size][name] = run(size, layers, batch, prompt, ctx, steps, kernels)
+            torch.cuda.empty_cache()
+    print(json.dumps({"bench": "serving", "layers": layers, "decode_batch": batch, "prompt": prompt, "context": ctx, "dtype": "bf16", "peaks": of,
+                      "data": "synthetic (uniform random token ids, random weights)", "sizes": res, "kernel_status": _lib.read_status()}))
+    return 0

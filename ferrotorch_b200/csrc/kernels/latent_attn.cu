@@ -39,49 +39,65 @@ struct LatentDims {
 };
 
 // ------------------------------------------------------------------------------------------------------------
-// prompt rows: grid rows, 256 threads
+// prompt rows: grid rows, 128 threads; a warp takes whole heads, a lane neighbouring pairs (two elements at a time everywhere: all offsets are even)
 // ------------------------------------------------------------------------------------------------------------
+template <typename T> FT_DEVICE float2 load2(const T* p);
+template <> FT_DEVICE float2 load2<float>(const float* p) { return *reinterpret_cast<const float2*>(p); }
+template <> FT_DEVICE float2 load2<__nv_bfloat16>(const __nv_bfloat16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+template <typename T> FT_DEVICE void store2(T* p, float a, float b);
+template <> FT_DEVICE void store2<float>(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+template <> FT_DEVICE void store2<__nv_bfloat16>(__nv_bfloat16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+
 template <typename T>
-__global__ void __launch_bounds__(256) latent_prep_kernel(T* __restrict__ qkv, int64_t ld, LatentDims D, const float* __restrict__ w, float eps,
+__global__ void __launch_bounds__(128) latent_prep_kernel(T* __restrict__ qkv, int64_t ld, LatentDims D, const float* __restrict__ w, float eps,
                                                           const int* __restrict__ positions, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
                                                           const int* __restrict__ slots, const int* __restrict__ ctx_rows, T* __restrict__ cache, T* __restrict__ ctx) {
   __shared__ float red[32];
-  const int r = blockIdx.x, half = D.dr / 2;
+  const int r = blockIdx.x, half = D.dr / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pos = positions[r];
   T* row = qkv + (size_t)r * ld;
-  const float* c = cos_t + (size_t)pos * half;
-  const float* s = sin_t + (size_t)pos * half;
-  for (int i = threadIdx.x; i < D.H * half; i += 256) {
-    const int hd = i / half, p = i % half;
-    T* q = row + hd * (D.d8 + D.dr8) + D.d8 + 2 * p;
-    const float u = to_f(q[0]), v = to_f(q[1]);
-    q[0] = from_f<T>(u * c[p] - v * s[p]);
-    q[1] = from_f<T>(v * c[p] + u * s[p]);
-  }
+  const float* ct = cos_t + (size_t)pos * half;
+  const float* st = sin_t + (size_t)pos * half;
   const T* lat = row + D.H * (D.d8 + D.dr8);
   float ss = 0.f;
-  for (int i = threadIdx.x; i < D.rank; i += 256) { const float v = to_f(lat[i]); ss += v * v; }
+  for (int i = threadIdx.x * 2; i < D.rank; i += 256) {
+    const float2 v = load2(lat + i);
+    ss += v.x * v.x + (i + 1 < D.rank ? v.y * v.y : 0.f);
+  }
+  for (int p = lane; p < half; p += 32) {
+    const float c = ct[p], s = st[p];
+#pragma unroll 4
+    for (int hd = warp; hd < D.H; hd += 4) {
+      T* q = row + hd * (D.d8 + D.dr8) + D.d8 + 2 * p;
+      const float2 v = load2(q);
+      store2(q, v.x * c - v.y * s, v.y * c + v.x * s);
+    }
+  }
   ss = block_sum(ss, red);
   const float rstd = 1.f / sqrtf(ss / (float)D.rank + eps);
   T* dst = cache + (size_t)slots[r] * D.row;
   T* dense = ctx ? ctx + (size_t)ctx_rows[r] * D.row : nullptr;
-  for (int i = threadIdx.x; i < D.r16; i += 256) {
-    const T v = from_f<T>(i < D.rank ? to_f(lat[i]) * rstd * w[i] : 0.f);
-    dst[i] = v;
-    if (dense) dense[i] = v;
+  for (int i = threadIdx.x * 2; i < D.r16; i += 256) {
+    float a = 0.f, b = 0.f;
+    if (i < D.rank) {
+      const float2 v = load2(lat + i);
+      a = v.x * rstd * w[i];
+      if (i + 1 < D.rank) b = v.y * rstd * w[i + 1];
+    }
+    store2(dst + i, a, b);
+    if (dense) store2(dense + i, a, b);
   }
   const T* kr = lat + D.rank8;
-  for (int i = threadIdx.x; i < (D.row - D.r16) / 2; i += 256) {
+  for (int i = threadIdx.x; i < (D.row - D.r16) / 2; i += 128) {
     float a = 0.f, b = 0.f;
     if (i < half) {
-      const float u = to_f(kr[2 * i]), v = to_f(kr[2 * i + 1]);
-      a = u * c[i] - v * s[i];
-      b = v * c[i] + u * s[i];
+      const float2 v = load2(kr + 2 * i);
+      const float c = ct[i], s = st[i];
+      a = v.x * c - v.y * s;
+      b = v.y * c + v.x * s;
     }
-    const T ta = from_f<T>(a), tb = from_f<T>(b);
-    dst[D.r16 + 2 * i] = ta;
-    dst[D.r16 + 2 * i + 1] = tb;
-    if (dense) { dense[D.r16 + 2 * i] = ta; dense[D.r16 + 2 * i + 1] = tb; }
+    store2(dst + D.r16 + 2 * i, a, b);
+    if (dense) store2(dense + D.r16 + 2 * i, a, b);
   }
 }
 
@@ -151,56 +167,68 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const T* __restrict__ 
 // ------------------------------------------------------------------------------------------------------------
 // decode preparation on split-K planes: CTAs [0, H * slices) absorb 64 latent columns of one head for every token, the rest handle one token's cache row
 // ------------------------------------------------------------------------------------------------------------
-constexpr int DEC_TOK = 16, ABS_COLS = 64;
+constexpr int DEC_TOK = 16, ABS_COLS = 64, PREP_THREADS = 256;
 FT_DEVICE float plane_sum(const float* __restrict__ p, int splits, size_t stride, size_t idx) {
   float a = 0.f;
-  for (int s = 0; s < splits; s++) a += p[s * stride + idx];
+  int s = 0;
+  for (; s + 4 <= splits; s += 4) {
+    float v[4];
+#pragma unroll
+    for (int j = 0; j < 4; j++) v[j] = __ldcg(p + (s + j) * stride + idx);
+    a += (v[0] + v[1]) + (v[2] + v[3]);
+  }
+  for (; s < splits; s++) a += __ldcg(p + s * stride + idx);
   return a;
 }
-__global__ void __launch_bounds__(128) latent_decode_prep_kernel(const float* __restrict__ planes, int splits, int64_t ldp, size_t pstride, LatentDims D, int B,
-                                                                 const __nv_bfloat16* __restrict__ wuk, int64_t ldw, const float* __restrict__ w, float eps,
-                                                                 const int* __restrict__ positions, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
-                                                                 const int* __restrict__ block_table, int max_blocks, __nv_bfloat16* __restrict__ q,
-                                                                 __nv_bfloat16* __restrict__ cache) {
-  pdl_wait();
-  pdl_launch_dependents();
-  extern __shared__ float sq[];     // [DEC_TOK][d]
+__global__ void __launch_bounds__(PREP_THREADS) latent_decode_prep_kernel(const float* __restrict__ planes, int splits, int64_t ldp, size_t pstride, LatentDims D, int B,
+                                                                          const __nv_bfloat16* __restrict__ wuk, int64_t ldw, const float* __restrict__ w, float eps,
+                                                                          const int* __restrict__ positions, const float* __restrict__ cos_t,
+                                                                          const float* __restrict__ sin_t, const int* __restrict__ block_table, int max_blocks,
+                                                                          __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache) {
+  extern __shared__ __align__(16) uint8_t prep_smem[];
   __shared__ float red[32];
   const int slices = (D.r16 + ABS_COLS - 1) / ABS_COLS, half = D.dr / 2;
-  if ((int)blockIdx.x < D.H * slices) {
-    const int hd = blockIdx.x / slices, sl = blockIdx.x % slices;
+  const bool absorb = (int)blockIdx.x < D.H * slices;
+  const int hd = blockIdx.x / slices, sl = blockIdx.x % slices;
+  __nv_bfloat16* sw = reinterpret_cast<__nv_bfloat16*>(prep_smem);             // [d][ABS_COLS]
+  float* sq = reinterpret_cast<float*>(prep_smem + (size_t)D.d * ABS_COLS * 2);   // [d][DEC_TOK]
+  if (absorb) {
+    // the weight slice does not depend on the predecessor: it is on its way before the wait
+    const __nv_bfloat16* wp = wuk + (size_t)hd * D.d8 * ldw + sl * ABS_COLS;
+    const int vecs = min(ABS_COLS, (int)(ldw - sl * ABS_COLS)) / 8;
+    for (int i = threadIdx.x; i < D.d * vecs; i += PREP_THREADS) {
+      const int k = i / vecs, v = i % vecs;
+      asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_u32(sw + k * ABS_COLS + v * 8)), "l"(wp + (size_t)k * ldw + v * 8) : "memory");
+    }
+    asm volatile("cp.async.commit_group;" ::: "memory");
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  if (absorb) {
     const size_t qcol = (size_t)hd * (D.d8 + D.dr8);
-    for (int i = threadIdx.x; i < B * D.d; i += 128) {
+    for (int i = threadIdx.x; i < B * D.d; i += PREP_THREADS) {
       const int b = i / D.d, k = i % D.d;
       // the query as the bf16 operand that the prompt kernels see
-      sq[b * D.d + k] = __bfloat162float(__float2bfloat16(plane_sum(planes, splits, pstride, (size_t)b * ldp + qcol + k)));
+      sq[k * DEC_TOK + b] = __bfloat162float(__float2bfloat16(plane_sum(planes, splits, pstride, (size_t)b * ldp + qcol + k)));
     }
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
     __syncthreads();
-    const int cp = threadIdx.x & 31, tg = threadIdx.x >> 5, c0 = sl * ABS_COLS + cp * 2;
-    if (c0 < D.r16) {
-      float acc[DEC_TOK / 4][2];
-#pragma unroll
-      for (int i = 0; i < DEC_TOK / 4; i++) acc[i][0] = acc[i][1] = 0.f;
-      const __nv_bfloat16* wp = wuk + (size_t)hd * D.d8 * ldw + c0;
+    const int cp = threadIdx.x & 31, tg = (threadIdx.x >> 5) * 2, c0 = sl * ABS_COLS + cp * 2;   // two columns of two tokens
+    if (c0 < D.r16 && tg < B) {
+      float a00 = 0.f, a01 = 0.f, a10 = 0.f, a11 = 0.f;
 #pragma unroll 8
       for (int k = 0; k < D.d; k++) {
-        const float2 wv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(wp + (size_t)k * ldw));
-#pragma unroll
-        for (int i = 0; i < DEC_TOK / 4; i++)
-          if (tg + 4 * i < B) {
-            const float x = sq[(tg + 4 * i) * D.d + k];
-            acc[i][0] += x * wv.x;
-            acc[i][1] += x * wv.y;
-          }
+        const float2 wv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sw + k * ABS_COLS + cp * 2));
+        const float2 x = *reinterpret_cast<const float2*>(sq + k * DEC_TOK + tg);
+        a00 += x.x * wv.x; a01 += x.x * wv.y;
+        a10 += x.y * wv.x; a11 += x.y * wv.y;
       }
-#pragma unroll
-      for (int i = 0; i < DEC_TOK / 4; i++)
-        if (tg + 4 * i < B)
-          *reinterpret_cast<__nv_bfloat162*>(q + ((size_t)(tg + 4 * i) * D.H + hd) * D.row + c0) = __floats2bfloat162_rn(acc[i][0], acc[i][1]);
+      *reinterpret_cast<__nv_bfloat162*>(q + ((size_t)tg * D.H + hd) * D.row + c0) = __floats2bfloat162_rn(a00, a01);
+      if (tg + 1 < B) *reinterpret_cast<__nv_bfloat162*>(q + ((size_t)(tg + 1) * D.H + hd) * D.row + c0) = __floats2bfloat162_rn(a10, a11);
     }
     if (sl == 0) {
       const int pairs = (D.row - D.r16) / 2;
-      for (int i = threadIdx.x; i < B * pairs; i += 128) {
+      for (int i = threadIdx.x; i < B * pairs; i += PREP_THREADS) {
         const int b = i / pairs, p = i % pairs;
         float a = 0.f, bb = 0.f;
         if (p < half) {
@@ -217,9 +245,9 @@ __global__ void __launch_bounds__(128) latent_decode_prep_kernel(const float* __
   }
   const int b = blockIdx.x - D.H * slices, pos = positions[b];
   const size_t base = (size_t)b * ldp + (size_t)D.H * (D.d8 + D.dr8);
-  float* lat = sq;                  // rank floats (the launcher sizes the buffer for both uses)
+  float* lat = reinterpret_cast<float*>(prep_smem);     // rank floats (the launcher sizes the buffer for both uses)
   float ss = 0.f;
-  for (int i = threadIdx.x; i < D.rank; i += 128) {
+  for (int i = threadIdx.x; i < D.rank; i += PREP_THREADS) {
     const float v = plane_sum(planes, splits, pstride, base + i);
     lat[i] = v;
     ss += v * v;
@@ -229,8 +257,8 @@ __global__ void __launch_bounds__(128) latent_decode_prep_kernel(const float* __
   const int blk = block_table[(size_t)b * max_blocks + pos / KV_BLOCK];
   if (blk < 0) return;
   __nv_bfloat16* dst = cache + ((size_t)blk * KV_BLOCK + pos % KV_BLOCK) * D.row;
-  for (int i = threadIdx.x; i < D.r16; i += 128) dst[i] = __float2bfloat16(i < D.rank ? lat[i] * rstd * w[i] : 0.f);
-  for (int p = threadIdx.x; p < (D.row - D.r16) / 2; p += 128) {
+  for (int i = threadIdx.x; i < D.r16; i += PREP_THREADS) dst[i] = __float2bfloat16(i < D.rank ? lat[i] * rstd * w[i] : 0.f);
+  for (int p = threadIdx.x; p < (D.row - D.r16) / 2; p += PREP_THREADS) {
     float a = 0.f, bb = 0.f;
     if (p < half) {
       const float u = plane_sum(planes, splits, pstride, base + D.rank8 + 2 * p), v = plane_sum(planes, splits, pstride, base + D.rank8 + 2 * p + 1);
@@ -537,15 +565,17 @@ struct FlashDims {
   int dv8;
 };
 
-template <int NT>
-__global__ void __launch_bounds__(64 + 128 * NT, 1)
+// NQ, NV: 64-column blocks of the query / key and value dimensions at compile time (the issuing thread's descriptors then are constants added to a base;
+// built at run time they cost more than the MMAs themselves), or 0 to read them from F.
+template <int NT, int NQ, int NV>
+__global__ void __launch_bounds__(64 + 128 * NT, (NT == 1 && NV == 1) ? 2 : 1)
 latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmQr, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmKr, const __grid_constant__ CUtensorMap tmV, const int4* __restrict__ tiles, FlashDims F, float scale_log2,
                     __nv_bfloat16* __restrict__ out, int64_t ldo, uint32_t* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  const int nq = F.nn + F.nr;
-  const int k_bytes = nq * LF_KB, v_bytes = F.nv * LF_KB;
+  const int nq = NQ > 0 ? NQ : F.nn + F.nr, nv = NV > 0 ? NV : F.nv;
+  const int k_bytes = nq * LF_KB, v_bytes = nv * LF_KB;
   uint8_t* sQ = smem;                               // [NT][nq]
   uint8_t* sK = sQ + NT * nq * LF_QB;               // [2][nq]
   uint8_t* sV = sK + 2 * k_bytes;                   // [2][nv]
@@ -578,7 +608,8 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     mbar_fence_init();
   }
   if (warp == 0 && lane == 0) { tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmQr); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmKr); tma_prefetch_desc(&tmV); }
-  if (warp == 1) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
+  constexpr uint32_t TMEM = (NT == 1 && NV == 1) ? 256 : 512;       // small heads leave room for a second CTA
+  if (warp == 1) { tmem_alloc(tmem_slot, TMEM); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
@@ -609,7 +640,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         const int s = j & 1;
         if (!lf_wait(&v_empty[s], ((j >> 1) & 1) ^ 1)) { ft_set_status(status, FT_K_LATENT, 2, j); ok = false; break; }
         mbar_expect_tx(&v_full[s], v_bytes);
-        for (int c = 0; c < F.nv; c++) tma_load_3d(sV + s * v_bytes + c * LF_KB, &tmV, &v_full[s], c * 64, hd, tl.w + j * LF_BN);
+        for (int c = 0; c < nv; c++) tma_load_3d(sV + s * v_bytes + c * LF_KB, &tmV, &v_full[s], c * 64, hd, tl.w + j * LF_BN);
       }
       if (!ok)
         for (int i = 0; i < 64; i++) __nanosleep(1000);      // copies in flight land before the shared memory goes away
@@ -617,18 +648,17 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   } else if (warp == 1) {
     if (lane == 0) {
       const uint32_t idesc_s = make_idesc_f16(LF_BM, LF_BN, 1, 0, 0);
-      const uint32_t idesc_o = make_idesc_f16(LF_BM, F.nv * 64, 1, 0, 1);
+      const uint32_t idesc_o = make_idesc_f16(LF_BM, nv * 64, 1, 0, 1);
+      // a descriptor's start address counts 16-byte units in its low bits: moving inside the operand is an addition
+      const uint64_t q_desc = make_smem_desc(smem_u32(sQ), 16, 1024, FT_SWZ_128B), k_desc = make_smem_desc(smem_u32(sK), 16, 1024, FT_SWZ_128B);
+      const uint64_t p_desc = make_smem_desc(smem_u32(sP), 16, 1024, FT_SWZ_128B), v_desc = make_smem_desc(smem_u32(sV), LF_KB, 1024, FT_SWZ_128B);
       auto issue_s = [&](int t, int j) {
-        const uint32_t qb = smem_u32(sQ) + t * nq * LF_QB, kb = smem_u32(sK) + (j & 1) * k_bytes;
+        const uint64_t qd = q_desc + (uint32_t)(t * nq) * (LF_QB / 16), kd = k_desc + (uint32_t)(j & 1) * (k_bytes / 16);
         const uint32_t d = tS + t * 2 * LF_BN + (j & 1) * LF_BN;
-        uint32_t acc = 0;
+#pragma unroll
         for (int c = 0; c < nq; c++) {
-          const int left = c < F.nn ? F.d - c * 64 : F.dr - (c - F.nn) * 64;
-          const int steps = left >= 64 ? 4 : (left + 15) / 16;
-          for (int k = 0; k < steps; k++) {
-            umma_f16_ss(d, make_smem_desc(qb + c * LF_QB + k * 32, 16, 1024, FT_SWZ_128B), make_smem_desc(kb + c * LF_KB + k * 32, 16, 1024, FT_SWZ_128B), idesc_s, acc);
-            acc = 1;
-          }
+#pragma unroll
+          for (int k = 0; k < 4; k++) umma_f16_ss(d, qd + c * (LF_QB / 16) + k * 2, kd + c * (LF_KB / 16) + k * 2, idesc_s, (c | k) != 0);
         }
         umma_commit(&s_full[2 * t + (j & 1)]);
       };
@@ -650,7 +680,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             umma_commit(&k_empty[(j + 1) & 1]);
           }
           if (!lf_wait(&v_full[j & 1], (j >> 1) & 1)) { ft_set_status(status, FT_K_LATENT, 5, j); break; }
-          const uint32_t vb = smem_u32(sV) + (j & 1) * v_bytes;
+          const uint64_t vd = v_desc + (uint32_t)(j & 1) * (v_bytes / 16);
 #pragma unroll
           for (int t = 0; t < NT; t++) {
             if (j >= nblk[t] || !ok) continue;
@@ -658,8 +688,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
             tc_fence_after();
 #pragma unroll
             for (int k = 0; k < LF_BN / 16; k++)
-              umma_f16_ss(tO + t * F.nv * 64, make_smem_desc(smem_u32(sP) + t * LF_PB + k * 32, 16, 1024, FT_SWZ_128B),
-                          make_smem_desc(vb + k * 2048, LF_KB, 1024, FT_SWZ_128B), idesc_o, (j | k) != 0);
+              umma_f16_ss(tO + t * nv * 64, p_desc + t * (LF_PB / 16) + k * 2, vd + k * 128, idesc_o, (j | k) != 0);
             umma_commit(&pv_done[t]);
           }
           umma_commit(&v_empty[j & 1]);
@@ -677,6 +706,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     for (int j = 0; j < nb && ok; j++) {
       if (!lf_wait(&s_full[2 * t + (j & 1)], (j >> 1) & 1)) { if (lane == 0) ft_set_status(status, FT_K_LATENT, 7, j); ok = false; break; }
       tc_fence_after();
+      __syncwarp();                                            // the TMEM loads are warp-wide: every lane is here
       uint32_t sv[64];
       tmem_ld_32x32b_x32(tS + lane_off + t * 2 * LF_BN + (j & 1) * LF_BN, sv);
       tmem_ld_32x32b_x32(tS + lane_off + t * 2 * LF_BN + (j & 1) * LF_BN + 32, sv + 32);
@@ -715,11 +745,12 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       if (j > 0) {
         if (!lf_wait(&pv_done[t], (j - 1) & 1)) { if (lane == 0) ft_set_status(status, FT_K_LATENT, 8, j); ok = false; break; }
         tc_fence_after();
+        __syncwarp();
         if (rescale) {
 #pragma unroll 1
-          for (int c = 0; c < F.nv * 2; c++) {
+          for (int c = 0; c < nv * 2; c++) {
             uint32_t ov[32];
-            const uint32_t addr = tO + lane_off + t * F.nv * 64 + c * 32;
+            const uint32_t addr = tO + lane_off + t * nv * 64 + c * 32;
             tmem_ld_32x32b_x32(addr, ov);
             tmem_ld_wait();
 #pragma unroll
@@ -744,24 +775,28 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
       const float inv_l = 1.f / l;
       const bool live = t * LF_BM + r < tl.y;
       __nv_bfloat16* dst = out + (size_t)(tl.x + t * LF_BM + r) * ldo + (size_t)hd * F.dv8;
+      // rows past the end of the sequence only skip the stores: the warp-wide TMEM loads stay in code that all lanes run together
 #pragma unroll 1
-      for (int c = 0; c < F.nv * 2; c++) {
+      for (int c = 0; c < nv * 2; c++) {
         uint32_t ov[32];
-        tmem_ld_32x32b_x32(tO + lane_off + t * F.nv * 64 + c * 32, ov);
+        __syncwarp();
+        tmem_ld_32x32b_x32(tO + lane_off + t * nv * 64 + c * 32, ov);
         tmem_ld_wait();
-        if (live) {
+        uint4 w[4];
 #pragma unroll
-          for (int c8 = 0; c8 < 4; c8++) {
-            if (c * 32 + c8 * 8 + 8 > F.dv8) continue;
-            uint32_t w[4];
+        for (int c8 = 0; c8 < 4; c8++) {
+          uint32_t e[4];
 #pragma unroll
-            for (int e = 0; e < 4; e++) {
-              __nv_bfloat162 hh = __floats2bfloat162_rn(__uint_as_float(ov[8 * c8 + 2 * e]) * inv_l, __uint_as_float(ov[8 * c8 + 2 * e + 1]) * inv_l);
-              w[e] = *reinterpret_cast<uint32_t*>(&hh);
-            }
-            *reinterpret_cast<uint4*>(dst + c * 32 + c8 * 8) = make_uint4(w[0], w[1], w[2], w[3]);
+          for (int i = 0; i < 4; i++) {
+            __nv_bfloat162 hh = __floats2bfloat162_rn(__uint_as_float(ov[8 * c8 + 2 * i]) * inv_l, __uint_as_float(ov[8 * c8 + 2 * i + 1]) * inv_l);
+            e[i] = *reinterpret_cast<uint32_t*>(&hh);
           }
+          w[c8] = make_uint4(e[0], e[1], e[2], e[3]);
         }
+#pragma unroll
+        for (int c8 = 0; c8 < 4; c8++)
+          if (live && c * 32 + c8 * 8 + 8 <= F.dv8) *reinterpret_cast<uint4*>(dst + c * 32 + c8 * 8) = w[c8];
+        __syncwarp();
       }
     }
   }
@@ -769,7 +804,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   __syncthreads();
   if (warp == 1) {
     tc_fence_after();
-    tmem_dealloc(tS, 512);
+    tmem_dealloc(tS, TMEM);
   }
 }
 
@@ -787,14 +822,14 @@ bool dims_ok(int H, int d, int dr, int rank) { return H >= 1 && d >= 1 && dr >= 
 int flash_smem(int NT, int nq, int nv) { return NT * nq * LF_QB + 2 * (nq + nv) * LF_KB + NT * LF_PB + 256 + 1024; }
 constexpr int SMEM_MAX = 232448;
 
-template <int NT>
+template <int NT, int NQ, int NV>
 int launch_flash(const CUtensorMap (&m)[5], const int* tiles, int ntiles, int H, const FlashDims& F, float scale, void* out, int64_t ldo, int smem, cudaStream_t st) {
   static bool configured = false;
   if (!configured) {
-    FT_CUDA_TRY(cudaFuncSetAttribute(latent_flash_kernel<NT>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX));
+    FT_CUDA_TRY(cudaFuncSetAttribute(latent_flash_kernel<NT, NQ, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX));
     configured = true;
   }
-  latent_flash_kernel<NT><<<dim3(ntiles, H), 64 + 128 * NT, smem, st>>>(m[0], m[1], m[2], m[3], m[4], reinterpret_cast<const int4*>(tiles), F,
+  latent_flash_kernel<NT, NQ, NV><<<dim3(ntiles, H), 64 + 128 * NT, smem, st>>>(m[0], m[1], m[2], m[3], m[4], reinterpret_cast<const int4*>(tiles), F,
                                                                        scale * 1.4426950408889634f, (__nv_bfloat16*)out, ldo, ft_status_ptr());
   return (int)cudaGetLastError();
 }
@@ -821,9 +856,9 @@ FT_EXPORT int ft_latent_prep(void* qkv, int64_t ld, int rows, int H, int d, int 
                              const float* sin_t, const int* slots, const int* ctx_rows, void* cache, void* ctx, int is_f32, cudaStream_t st) {
   if (rows < 1 || !dims_ok(H, d, dr, rank) || (ctx && !ctx_rows)) return FT_ERR_ARG;
   const LatentDims D = make_dims(H, d, dr, rank);
-  if (ld < (int64_t)H * (D.d8 + D.dr8) + D.rank8 + dr) return FT_ERR_ARG;
-  if (is_f32) latent_prep_kernel<float><<<rows, 256, 0, st>>>((float*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (float*)cache, (float*)ctx);
-  else latent_prep_kernel<__nv_bfloat16><<<rows, 256, 0, st>>>((__nv_bfloat16*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (__nv_bfloat16*)cache,
+  if (ld < (int64_t)H * (D.d8 + D.dr8) + D.rank8 + dr || (ld & 7)) return FT_ERR_ARG;
+  if (is_f32) latent_prep_kernel<float><<<rows, 128, 0, st>>>((float*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (float*)cache, (float*)ctx);
+  else latent_prep_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>((__nv_bfloat16*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (__nv_bfloat16*)cache,
                                                                (__nv_bfloat16*)ctx);
   return (int)cudaGetLastError();
 }
@@ -856,11 +891,12 @@ FT_EXPORT int ft_latent_decode_prep(const float* planes, int splits, int64_t ldp
                                     int max_blocks, void* q, void* cache, cudaStream_t st) {
   if (B < 1 || B > DEC_TOK || splits < 1 || !dims_ok(H, d, dr, rank)) return FT_ERR_ARG;
   const LatentDims D = make_dims(H, d, dr, rank);
-  if ((ldw & 1) || ldw < D.r16) return FT_ERR_ARG;
+  if ((ldw & 7) || ldw < D.r16) return FT_ERR_ARG;
   const int slices = (D.r16 + ABS_COLS - 1) / ABS_COLS;
-  const size_t smem = sizeof(float) * (size_t)(B * d > rank ? B * d : rank);
+  const size_t absorb = (size_t)d * (ABS_COLS * 2 + DEC_TOK * 4), norm = sizeof(float) * (size_t)rank;
+  const size_t smem = absorb > norm ? absorb : norm;
   if (smem > 48 * 1024) return FT_ERR_TOO_LARGE;
-  return (int)ft_launch_pdl(latent_decode_prep_kernel, dim3(H * slices + B), dim3(128), smem, st, planes, splits, ldp, (size_t)plane_stride, D, B,
+  return (int)ft_launch_pdl(latent_decode_prep_kernel, dim3(H * slices + B), dim3(PREP_THREADS), smem, st, planes, splits, ldp, (size_t)plane_stride, D, B,
                             (const __nv_bfloat16*)wuk, ldw, w, eps, positions, cos_t, sin_t, block_table, max_blocks, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
 }
 
@@ -898,6 +934,7 @@ FT_EXPORT int ft_latent_combine(const float* ws, int B, int H, int rank, int nsp
 // Query rows of one tile of ft_latent_flash for these head sizes: 256 or 128; 0 when the sizes do not fit the kernel (use ft_latent_rows).
 FT_EXPORT int ft_latent_flash_tile(int d, int dr, int dv) {
   const int nq = (d + 63) / 64 + (dr + 63) / 64, nv = (dv + 63) / 64;
+  if (nq == 2 && nv == 1) return 128;                  // two CTAs of one tile per SM
   if (nv <= 2 && flash_smem(2, nq, nv) <= SMEM_MAX) return 256;
   if (nv <= 4 && flash_smem(1, nq, nv) <= SMEM_MAX) return 128;
   return 0;
@@ -927,6 +964,15 @@ FT_EXPORT int ft_latent_flash(const void* q, int64_t ldq, int q_rows, const void
   if (r) return r;
   const FlashDims F{d, dr, dv, (d + 63) / 64, (dr + 63) / 64, (dv + 63) / 64, dv8};
   const int nq = F.nn + F.nr;
-  if (tile == 256) return launch_flash<2>(m, tiles, ntiles, H, F, scale, out, ldo, flash_smem(2, nq, F.nv), st);
-  return launch_flash<1>(m, tiles, ntiles, H, F, scale, out, ldo, flash_smem(1, nq, F.nv), st);
+  const int smem = flash_smem(tile / 128, nq, F.nv);
+#define FT_LF(T, Q, V) return launch_flash<T, Q, V>(m, tiles, ntiles, H, F, scale, out, ldo, smem, st)
+  if (tile == 256) {
+    if (nq == 2 && F.nv == 2) FT_LF(2, 2, 2);
+    if (nq == 3 && F.nv == 1) FT_LF(2, 3, 1);
+    if (nq == 3 && F.nv == 2) FT_LF(2, 3, 2);
+    FT_LF(2, 0, 0);
+  }
+  if (nq == 2 && F.nv == 1) FT_LF(1, 2, 1);
+  FT_LF(1, 0, 0);
+#undef FT_LF
 }

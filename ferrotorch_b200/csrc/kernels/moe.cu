@@ -28,6 +28,13 @@ FT_DEVICE float gated_clamped(float g, float u, float limit, float slope) {
   return g * sigmoid_f(slope * g) * (u + 1.f);
 }
 
+// the same on the fast exponential and division, for results that are rounded to bf16
+FT_DEVICE float gated_clamped_fast(float g, float u, float limit, float slope) {
+  g = fminf(g, limit);
+  u = fminf(fmaxf(u, -limit), limit);
+  return __fdividef(g * (u + 1.f), 1.f + __expf(-slope * g));
+}
+
 // whole warp: (value, index) of the largest logit that comes after (pv, pi) in the order "value descending, index ascending"
 FT_DEVICE void next_best(const float* z, int E, float pv, int pi, float& bv, int& bi) {
   bv = -INFINITY;
@@ -114,29 +121,44 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict
   for (int i = threadIdx.x; i < vecs; i += 128) dst[i] = src[i];
 }
 
-// gu: [rows][2 * fp] in blocks of eight gate | eight up columns -> act [rows][ld_act]
+// gu: [rows][2 * fp] in blocks of eight gate | eight up columns -> act [rows][ld_act]. grid (column blocks, row groups): a thread keeps its eight neurons.
 template <typename T>
-__global__ void __launch_bounds__(256) moe_act_kernel(const T* __restrict__ gu, int64_t ld_gu, const float* __restrict__ row_score, const int* __restrict__ rows_used,
+__global__ void __launch_bounds__(128) moe_act_kernel(const T* __restrict__ gu, int64_t ld_gu, const float* __restrict__ row_score, const int* __restrict__ rows_used,
                                                       int rows, int fp, float limit, float slope, T* __restrict__ act, int64_t ld_act) {
   const int n = rows_used ? min(rows, *rows_used) : rows;
-  const int per_row = fp / 8;
-  const size_t total = (size_t)n * per_row;
-  for (size_t i = blockIdx.x * (size_t)256 + threadIdx.x; i < total; i += (size_t)gridDim.x * 256) {
-    const int r = (int)(i / per_row), blk = (int)(i % per_row);
-    const float s = row_score ? row_score[r] : 1.f;
-    const T* src = gu + (size_t)r * ld_gu + blk * 16;
-    T* dst = act + (size_t)r * ld_act + blk * 8;
-    float o[8];
-    if constexpr (sizeof(T) == 2) {
-      float g[8], u[8];
-      bf16x8_to_float(*reinterpret_cast<const bf16x8*>(src), g);
-      bf16x8_to_float(*reinterpret_cast<const bf16x8*>(src + 8), u);
+  const int blk = blockIdx.x * 128 + threadIdx.x;
+  if (blk * 8 >= fp) return;
+  if constexpr (sizeof(T) == 2) {
+    constexpr int RU = 4;                              // rows in flight
+    for (int r0 = blockIdx.y; r0 < n; r0 += gridDim.y * RU) {
+      bf16x8 gr[RU], ur[RU];
+      float sc[RU];
 #pragma unroll
-      for (int e = 0; e < 8; e++) o[e] = gated_clamped(s * g[e], s * u[e], limit, slope);
-      *reinterpret_cast<bf16x8*>(dst) = float_to_bf16x8(o);
-    } else {
+      for (int i = 0; i < RU; i++) {
+        const int r = min(r0 + i * (int)gridDim.y, n - 1);
+        const T* src = gu + (size_t)r * ld_gu + blk * 16;
+        gr[i] = *reinterpret_cast<const bf16x8*>(src);
+        ur[i] = *reinterpret_cast<const bf16x8*>(src + 8);
+        sc[i] = row_score ? row_score[r] : 1.f;
+      }
 #pragma unroll
-      for (int e = 0; e < 8; e++) dst[e] = gated_clamped(s * src[e], s * src[8 + e], limit, slope);
+      for (int i = 0; i < RU; i++) {
+        const int r = r0 + i * (int)gridDim.y;
+        if (r >= n) break;
+        float g[8], u[8], o[8];
+        bf16x8_to_float(gr[i], g);
+        bf16x8_to_float(ur[i], u);
+#pragma unroll
+        for (int e = 0; e < 8; e++) o[e] = gated_clamped_fast(sc[i] * g[e], sc[i] * u[e], limit, slope);
+        *reinterpret_cast<bf16x8*>(act + (size_t)r * ld_act + blk * 8) = float_to_bf16x8(o);
+      }
+    }
+  } else {
+    for (int r = blockIdx.y; r < n; r += gridDim.y) {
+      const float s = row_score ? row_score[r] : 1.f;
+      const T* src = gu + (size_t)r * ld_gu + blk * 16;
+#pragma unroll
+      for (int e = 0; e < 8; e++) act[(size_t)r * ld_act + blk * 8 + e] = gated_clamped(s * src[e], s * src[8 + e], limit, slope);
     }
   }
 }
@@ -144,48 +166,56 @@ __global__ void __launch_bounds__(256) moe_act_kernel(const T* __restrict__ gu, 
 // ------------------------------------------------------------------------------------------------------------
 // decode
 // ------------------------------------------------------------------------------------------------------------
-// Routing of a decode step in device memory: n[0] active experts; id[a], cnt[a] and pair[a][i] = token * top + slot of active expert a;
-// score[token * top + slot].
+// Routing of a decode step in device memory: n[0] active experts; id[a], cnt[a], pair[a][i] = token * top + slot of active expert a in token order, and
+// pair_of[a][token] (-1: the token did not choose it); score[token * top + slot].
 struct SmallRoute {
   int* n;
   int* id;
   int* cnt;
   int* pair;                       // [experts][SMALL_TOK]
+  int* pair_of;                    // [experts][SMALL_TOK]
   float* score;
 };
 
-// grid ceil(E / 8): one warp per expert computes its logit for every token; the last CTA chooses and builds the lists
-__global__ void __launch_bounds__(256) moe_route_small_kernel(const __nv_bfloat16* __restrict__ h, int64_t ldh, const __nv_bfloat16* __restrict__ router, int64_t ldr,
+constexpr int ROUTE_LOGITS = 8192;   // logits of the choosing CTA that fit its shared memory
+
+// grid E: one CTA per expert computes its logit for every token; the last CTA chooses and builds the lists
+__global__ void __launch_bounds__(128) moe_route_small_kernel(const __nv_bfloat16* __restrict__ h, int64_t ldh, const __nv_bfloat16* __restrict__ router, int64_t ldr,
                                                               int B, int W, int E, int top, float* __restrict__ logits, int* __restrict__ counter, SmallRoute R) {
   pdl_wait();
   pdl_launch_dependents();
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, e = blockIdx.x * 8 + warp;
-  if (e < E) {
-    const __nv_bfloat16* w = router + (size_t)e * ldr;
-    for (int b0 = 0; b0 < B; b0 += 8) {
-      float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-      for (int k = lane * 8; k < W; k += 256) {
-        float wv[8];
-        bf16x8_to_float(*reinterpret_cast<const bf16x8*>(w + k), wv);
-        const int lim = W - k;
+  __shared__ float part[4][SMALL_TOK];
+  __shared__ float zs[ROUTE_LOGITS];
+  __shared__ int chosen[SMALL_TOK * MAX_TOP];
+  __shared__ int is_last;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, e = blockIdx.x;
+  const __nv_bfloat16* w = router + (size_t)e * ldr;
+  for (int b0 = 0; b0 < B; b0 += 8) {
+    float acc[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+    for (int k = threadIdx.x * 8; k < W; k += 1024) {
+      float wv[8];
+      const bf16x8 wr = *reinterpret_cast<const bf16x8*>(w + k);
+      bf16x8 hr[8];
 #pragma unroll
-        for (int b = 0; b < 8; b++) {
-          if (b0 + b < B) {
-            float hv[8];
-            bf16x8_to_float(*reinterpret_cast<const bf16x8*>(h + (size_t)(b0 + b) * ldh + k), hv);
-#pragma unroll
-            for (int j = 0; j < 8; j++) acc[b] += j < lim ? wv[j] * hv[j] : 0.f;
-          }
-        }
-      }
+      for (int b = 0; b < 8; b++) hr[b] = *reinterpret_cast<const bf16x8*>(h + (size_t)min(b0 + b, B - 1) * ldh + k);
+      bf16x8_to_float(wr, wv);
+      const int lim = W - k;
 #pragma unroll
       for (int b = 0; b < 8; b++) {
-        acc[b] = warp_sum(acc[b]);
-        if (lane == 0 && b0 + b < B) logits[(size_t)(b0 + b) * E + e] = acc[b];
+        float hv[8];
+        bf16x8_to_float(hr[b], hv);
+#pragma unroll
+        for (int j = 0; j < 8; j++) acc[b] += j < lim ? wv[j] * hv[j] : 0.f;
       }
     }
+#pragma unroll
+    for (int b = 0; b < 8; b++) {
+      acc[b] = warp_sum(acc[b]);
+      if (lane == 0) part[warp][b0 + b] = acc[b];
+    }
   }
-  __shared__ int is_last;
+  __syncthreads();
+  if (threadIdx.x < B) logits[(size_t)threadIdx.x * E + e] = (part[0][threadIdx.x] + part[1][threadIdx.x]) + (part[2][threadIdx.x] + part[3][threadIdx.x]);
   __threadfence();
   __syncthreads();
   if (threadIdx.x == 0) {
@@ -195,14 +225,19 @@ __global__ void __launch_bounds__(256) moe_route_small_kernel(const __nv_bfloat1
   __syncthreads();
   if (!is_last) return;
   __threadfence();
-  __shared__ int chosen[SMALL_TOK * MAX_TOP];
-  for (int b = warp; b < B; b += 8) {
+  const bool staged = B * E <= ROUTE_LOGITS;
+  if (staged) {
+    for (int i = threadIdx.x; i < B * E; i += 128) zs[i] = __ldcg(logits + i);
+    __syncthreads();
+  }
+  for (int b = warp; b < B; b += 4) {
+    const float* z = staged ? zs + (size_t)b * E : logits + (size_t)b * E;
     float pv = INFINITY;
     int pi = -1;
     for (int j = 0; j < top; j++) {
       float v;
       int c;
-      next_best(logits + (size_t)b * E, E, pv, pi, v, c);
+      next_best(z, E, pv, pi, v, c);
       if (c >= E) c = j;
       if (lane == 0) { chosen[b * top + j] = c; R.score[b * top + j] = sigmoid_f(v); }
       pv = v;
@@ -210,175 +245,152 @@ __global__ void __launch_bounds__(256) moe_route_small_kernel(const __nv_bfloat1
     }
   }
   __syncthreads();
-  if (warp == 0) {                                   // active experts in ascending order
-    int n = 0;
-    for (int e0 = 0; e0 < E; e0 += 32) {
-      const int x = e0 + lane;
-      int cnt = 0;
-      if (x < E)
-        for (int p = 0; p < B * top; p++) cnt += chosen[p] == x;
-      const unsigned m = __ballot_sync(0xffffffffu, cnt > 0);
-      if (cnt > 0) {
-        const int a = n + __popc(m & ((1u << lane) - 1));
-        R.id[a] = x;
-        R.cnt[a] = cnt;
-        int i = 0;
-        for (int p = 0; p < B * top; p++)
-          if (chosen[p] == x && i < SMALL_TOK) R.pair[a * SMALL_TOK + i++] = p;
+  // active experts in ascending order; thread t of a round looks at expert e0 + t
+  __shared__ int warp_n[4];
+  int base = 0;
+  for (int e0 = 0; e0 < E; e0 += 128) {
+    const int x = e0 + threadIdx.x;
+    int cnt = 0;
+    if (x < E)
+      for (int q = 0; q < B * top; q++) cnt += chosen[q] == x;
+    const unsigned m = __ballot_sync(0xffffffffu, cnt > 0);
+    if (lane == 0) warp_n[warp] = __popc(m);
+    __syncthreads();
+    int a = base + __popc(m & ((1u << lane) - 1u));
+    for (int i = 0; i < warp; i++) a += warp_n[i];
+    if (cnt > 0) {
+      R.id[a] = x;
+      R.cnt[a] = min(cnt, SMALL_TOK);
+      int i = 0;
+      for (int b = 0; b < B; b++) {
+        int mine = -1;
+        for (int j = 0; j < top; j++)
+          if (chosen[b * top + j] == x) mine = b * top + j;
+        R.pair_of[a * SMALL_TOK + b] = mine;
+        if (mine >= 0) R.pair[a * SMALL_TOK + i++] = mine;
       }
-      n += __popc(m);
     }
-    if (lane == 0) *R.n = n;
+    base += (warp_n[0] + warp_n[1]) + (warp_n[2] + warp_n[3]);
+    __syncthreads();
   }
+  if (threadIdx.x == 0) *R.n = base;
 }
 
 // One side of a decode launch: a stack of experts (or the one shared expert) in the packed layout
 struct ExpertSet {
-  const __nv_bfloat16* gu;         // [experts][2 * fp][ld_in]
-  const __nv_bfloat16* down;       // [experts][rows_out][ld_mid]
+  const __nv_bfloat16* w;          // gate / up: [experts][2 * fp][ld] interleaved; down: [experts][rows][ld]
   int f, fp;                       // neurons, padded to a multiple of 8
-  int64_t ld_in, ld_mid;           // padded to multiples of 32
+  int64_t ld, stride;              // row pitch, elements between experts
   float limit;
 };
 
-// grid (blocks of 64 neurons, groups + shared), 256 threads: warp w computes 8 neurons (16 interleaved rows) for all tokens; tokens that did not
-// choose the expert are computed along (the tensor tile has room for eight) and dropped.
-template <int NT>
-__global__ void __launch_bounds__(256) moe_gate_up_small_kernel(const __nv_bfloat16* __restrict__ h, int64_t ldh, int B, int W, int top, SmallRoute R, int groups,
-                                                                ExpertSet ex, ExpertSet sh, float slope, __nv_bfloat16* __restrict__ act, int64_t ld_act,
-                                                                __nv_bfloat16* __restrict__ act_sh, int64_t ld_act_sh, int tok0) {
-  pdl_wait();
-  pdl_launch_dependents();
-  extern __shared__ __align__(128) uint8_t xs[];
-  __shared__ int pair_of[8 * NT];
-  __shared__ float sc[8 * NT];
-  const int a = blockIdx.y;
-  const bool shared_ex = a == groups;
-  if (!shared_ex && a >= *R.n) return;
-  const ExpertSet& S = shared_ex ? sh : ex;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  if ((int)blockIdx.x * 64 >= S.fp) return;
-  const int nb = min(8 * NT, B - tok0), kp = (W + 31) & ~31, pitch = skinny_pitch(kp);
-  if (threadIdx.x < 8 * NT) {
-    pair_of[threadIdx.x] = shared_ex && (int)threadIdx.x < nb ? tok0 + threadIdx.x : -1;
-    sc[threadIdx.x] = 1.f;
+// Gate and up rows of eight neurons per item; all tokens are multiplied (the tensor tile has room for eight), those that chose the expert kept. Groups:
+// the active experts, then the shared one.
+struct GateUpWork {
+  const __nv_bfloat16* h;
+  int64_t ldh;
+  int B, W, tok0;
+  SmallRoute R;
+  ExpertSet ex, sh;
+  int has_shared;
+  float slope;
+  __nv_bfloat16 *act, *act_sh;
+  int64_t ld_act, ld_act_sh;
+
+  FT_DEVICE SkinnyShape shape() const { return SkinnyShape{{*R.n, has_shared}, {ex.fp / 8, has_shared ? sh.fp / 8 : 1}, {1, 1}}; }
+  FT_DEVICE bool shared(int g) const { return has_shared && g == *R.n; }
+  FT_DEVICE int K(int) const { return W; }
+  FT_DEVICE int64_t ldw(int g) const { return shared(g) ? sh.ld : ex.ld; }
+  FT_DEVICE const __nv_bfloat16* w(int g, int blk) const {
+    return shared(g) ? sh.w + (size_t)blk * 16 * sh.ld : ex.w + (size_t)R.id[g] * ex.stride + (size_t)blk * 16 * ex.ld;
   }
-  __syncthreads();
-  if (!shared_ex && threadIdx.x < R.cnt[a]) {
-    const int p = R.pair[a * SMALL_TOK + threadIdx.x], tk = p / top - tok0;
-    if (tk >= 0 && tk < 8 * NT) { pair_of[tk] = p; sc[tk] = R.score[p]; }
-  }
-  for (int n = 0; n < 8 * NT; n++) skinny_fill_row(xs, pitch, n, n < nb ? h + (size_t)(tok0 + n) * ldh : nullptr, W, kp, threadIdx.x, 256);
-  __syncthreads();
-  const int blk = blockIdx.x * 8 + warp;
-  if (blk * 8 >= S.fp) return;
-  float acc[NT][4];
-#pragma unroll
-  for (int n = 0; n < NT; n++) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-  const __nv_bfloat16* w = S.gu + ((size_t)(shared_ex ? 0 : R.id[a]) * 2 * S.fp + (size_t)blk * 16) * S.ld_in;
-  skinny_rows16<NT>(w, S.ld_in, kp, xs, pitch, acc);
-  const int f = blk * 8 + (lane >> 2);
-  if (f >= S.f) return;
-  __nv_bfloat16* dst = shared_ex ? act_sh : act;
-  const int64_t ld = shared_ex ? ld_act_sh : ld_act;
-#pragma unroll
-  for (int n = 0; n < NT; n++)
+  FT_DEVICE int x_id(int) const { return 0; }
+  FT_DEVICE const __nv_bfloat16* x_row(int, int n) const { return tok0 + n < B ? h + (size_t)(tok0 + n) * ldh : nullptr; }
+  FT_DEVICE void finish(int g, int blk, int nt, float4 c, int lane) const {
+    const bool s = shared(g);
+    const ExpertSet& S = s ? sh : ex;
+    const int f = blk * 8 + (lane >> 2), tk = tok0 + nt * 8 + (lane & 3) * 2;
+    if (f >= S.f) return;
 #pragma unroll
     for (int j = 0; j < 2; j++) {
-      const int tk = n * 8 + (lane & 3) * 2 + j, p = pair_of[tk];
-      if (p >= 0) dst[(size_t)p * ld + f] = __float2bfloat16(gated_clamped(sc[tk] * acc[n][j], sc[tk] * acc[n][2 + j], S.limit, slope));
+      if (tk + j >= B) break;
+      const int pr = s ? tk + j : R.pair_of[g * SMALL_TOK + tk + j];
+      if (pr < 0) continue;
+      const float k = s ? 1.f : R.score[pr];
+      (s ? act_sh + (size_t)pr * ld_act_sh : act + (size_t)pr * ld_act)[f] =
+          __float2bfloat16(gated_clamped_fast(k * (j ? c.y : c.x), k * (j ? c.w : c.z), S.limit, slope));
     }
-}
-
-// grid (blocks of 128 output columns, groups + shared), 256 threads: plane `slot` of out gets the expert's contribution to its tokens, plane `top`
-// the shared expert's. out: [top + 1][tok_stride][ldo] f32.
-template <int NT>
-__global__ void __launch_bounds__(256) moe_down_small_kernel(const __nv_bfloat16* __restrict__ act, int64_t ld_act, const __nv_bfloat16* __restrict__ act_sh,
-                                                             int64_t ld_act_sh, int B, int W, int top, SmallRoute R, int groups, ExpertSet ex, ExpertSet sh,
-                                                             int rows_out, float* __restrict__ out, int64_t plane_stride, int64_t ldo) {
-  pdl_wait();
-  pdl_launch_dependents();
-  extern __shared__ __align__(128) uint8_t xs[];
-  __shared__ int pair_sh[SMALL_TOK];
-  const int a = blockIdx.y;
-  const bool shared_ex = a == groups;
-  if (!shared_ex && a >= *R.n) return;
-  const ExpertSet& S = shared_ex ? sh : ex;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int cnt = shared_ex ? B : min(R.cnt[a], SMALL_TOK), kp = (S.f + 31) & ~31, pitch = skinny_pitch(kp);
-  if (threadIdx.x < SMALL_TOK) pair_sh[threadIdx.x] = (int)threadIdx.x < cnt ? (shared_ex ? (int)threadIdx.x : R.pair[a * SMALL_TOK + threadIdx.x]) : -1;
-  __syncthreads();
-  const int row0 = blockIdx.x * 128 + warp * 16;
-  const __nv_bfloat16* w = S.down + ((size_t)(shared_ex ? 0 : R.id[a]) * rows_out + row0) * S.ld_mid;
-  for (int i0 = 0; i0 < cnt; i0 += 8 * NT) {
-    if (i0) __syncthreads();
-    for (int n = 0; n < 8 * NT; n++) {
-      const int p = i0 + n < SMALL_TOK ? pair_sh[i0 + n] : -1;
-      const __nv_bfloat16* src = p < 0 ? nullptr : (shared_ex ? act_sh + (size_t)p * ld_act_sh : act + (size_t)p * ld_act);
-      skinny_fill_row(xs, pitch, n, src, S.f, kp, threadIdx.x, 256);
-    }
-    __syncthreads();
-    if (row0 >= rows_out) continue;
-    float acc[NT][4];
-#pragma unroll
-    for (int n = 0; n < NT; n++) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-    skinny_rows16<NT>(w, S.ld_mid, kp, xs, pitch, acc);
-#pragma unroll
-    for (int n = 0; n < NT; n++)
-#pragma unroll
-      for (int j = 0; j < 2; j++) {
-        const int i = i0 + n * 8 + (lane & 3) * 2 + j;
-        const int p = i < SMALL_TOK ? pair_sh[i] : -1;
-        if (p < 0) continue;
-        float* o = out + (shared_ex ? (size_t)top * plane_stride + (size_t)p * ldo : (size_t)(p % top) * plane_stride + (size_t)(p / top) * ldo);
-        const int r = row0 + (lane >> 2);
-        if (r < W) o[r] = acc[n][j];
-        if (r + 8 < W) o[r + 8] = acc[n][2 + j];
-      }
   }
-}
+};
 
-// one product of a few tokens per group (group = attention head: latent output -> value): grid (rows / 128, groups)
-template <int NT>
-__global__ void __launch_bounds__(256) skinny_heads_kernel(const __nv_bfloat16* __restrict__ x, int64_t ldx, int64_t head_x, const __nv_bfloat16* __restrict__ w,
-                                                           int64_t ldw, int64_t head_w, int B, int N, int K, __nv_bfloat16* __restrict__ out, int64_t ldo,
-                                                           int64_t head_o) {
-  pdl_wait();
-  pdl_launch_dependents();
-  extern __shared__ __align__(128) uint8_t xs[];
-  const int hd = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int kp = (K + 31) & ~31, pitch = skinny_pitch(kp);
-  for (int n = 0; n < 8 * NT; n++) skinny_fill_row(xs, pitch, n, n < B ? x + (size_t)n * ldx + hd * head_x : nullptr, K, kp, threadIdx.x, 256);
-  __syncthreads();
-  const int row0 = blockIdx.x * 128 + warp * 16;
-  if (row0 >= N) return;
-  float acc[NT][4];
-#pragma unroll
-  for (int n = 0; n < NT; n++) acc[n][0] = acc[n][1] = acc[n][2] = acc[n][3] = 0.f;
-  skinny_rows16<NT>(w + (size_t)hd * head_w + (size_t)row0 * ldw, ldw, kp, xs, pitch, acc);
-#pragma unroll
-  for (int n = 0; n < NT; n++)
+// Sixteen output columns per item, the expert's own tokens as columns: plane `slot` of out gets its contribution, plane `top` the shared expert's.
+struct DownWork {
+  const __nv_bfloat16 *act, *act_sh;
+  int64_t ld_act, ld_act_sh;
+  int B, W, top, col0;
+  SmallRoute R;
+  ExpertSet ex, sh;
+  int has_shared, blocks;
+  float* out;
+  int64_t plane_stride, ldo;
+
+  FT_DEVICE SkinnyShape shape() const { return SkinnyShape{{*R.n, has_shared}, {blocks, blocks}, {(ex.f + 31) >> 5, has_shared ? (sh.f + 31) >> 5 : 1}}; }
+  FT_DEVICE bool shared(int g) const { return has_shared && g == *R.n; }
+  FT_DEVICE int K(int g) const { return shared(g) ? sh.f : ex.f; }
+  FT_DEVICE int64_t ldw(int g) const { return shared(g) ? sh.ld : ex.ld; }
+  FT_DEVICE const __nv_bfloat16* w(int g, int blk) const {
+    return shared(g) ? sh.w + (size_t)blk * 16 * sh.ld : ex.w + (size_t)R.id[g] * ex.stride + (size_t)blk * 16 * ex.ld;
+  }
+  FT_DEVICE int x_id(int g) const { return g; }
+  FT_DEVICE int pair(int g, int n) const {
+    if (shared(g)) return n < B ? n : -1;
+    return n < SMALL_TOK && n < R.cnt[g] ? R.pair[g * SMALL_TOK + n] : -1;
+  }
+  FT_DEVICE const __nv_bfloat16* x_row(int g, int n) const {
+    const int pr = pair(g, col0 + n);
+    return pr < 0 ? nullptr : (shared(g) ? act_sh + (size_t)pr * ld_act_sh : act + (size_t)pr * ld_act);
+  }
+  FT_DEVICE void finish(int g, int blk, int nt, float4 c, int lane) const {
+    const bool s = shared(g);
+    const int r = blk * 16 + (lane >> 2), i = col0 + nt * 8 + (lane & 3) * 2;
 #pragma unroll
     for (int j = 0; j < 2; j++) {
-      const int tk = n * 8 + (lane & 3) * 2 + j;
-      if (tk >= B) continue;
-      __nv_bfloat16* o = out + (size_t)tk * ldo + hd * head_o;
-      const int r = row0 + (lane >> 2);
-      if (r < N) o[r] = __float2bfloat16(acc[n][j]);
-      if (r + 8 < N) o[r + 8] = __float2bfloat16(acc[n][2 + j]);
+      const int pr = pair(g, i + j);
+      if (pr < 0) continue;
+      float* o = out + (s ? (size_t)top * plane_stride + (size_t)pr * ldo : (size_t)(pr % top) * plane_stride + (size_t)(pr / top) * ldo);
+      if (r < W) o[r] = j ? c.y : c.x;
+      if (r + 8 < W) o[r + 8] = j ? c.w : c.z;
     }
-}
+  }
+};
 
-constexpr int SMALL_SMEM_MAX = 220 * 1024;
-template <typename K>
-cudaError_t allow_smem(K kernel, bool (&done)[64]) {
-  int dev = 0;
-  cudaGetDevice(&dev);
-  if (dev < 64 && done[dev]) return cudaSuccess;
-  const cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, SMALL_SMEM_MAX);
-  if (e == cudaSuccess && dev < 64) done[dev] = true;
-  return e;
-}
+// One matrix per group with the same tokens in every group (attention heads: latent output -> value)
+struct HeadsWork {
+  const __nv_bfloat16 *x, *weights;
+  int64_t ldx, head_x, ld, head_w;
+  int B, heads, N, Kin;
+  __nv_bfloat16* out;
+  int64_t ldo, head_o;
+
+  FT_DEVICE SkinnyShape shape() const { return SkinnyShape{{heads, 0}, {(N + 15) / 16, 1}, {1, 1}}; }
+  FT_DEVICE int K(int) const { return Kin; }
+  FT_DEVICE int64_t ldw(int) const { return ld; }
+  FT_DEVICE const __nv_bfloat16* w(int g, int blk) const { return weights + (size_t)g * head_w + (size_t)blk * 16 * ld; }
+  FT_DEVICE int x_id(int g) const { return g; }
+  FT_DEVICE const __nv_bfloat16* x_row(int g, int n) const { return n < B ? x + (size_t)n * ldx + (size_t)g * head_x : nullptr; }
+  FT_DEVICE void finish(int g, int blk, int nt, float4 c, int lane) const {
+    const int r = blk * 16 + (lane >> 2), tk = nt * 8 + (lane & 3) * 2;
+#pragma unroll
+    for (int j = 0; j < 2; j++) {
+      if (tk + j >= B) break;
+      __nv_bfloat16* o = out + (size_t)(tk + j) * ldo + (size_t)g * head_o;
+      if (r < N) o[r] = __float2bfloat16(j ? c.y : c.x);
+      if (r + 8 < N) o[r + 8] = __float2bfloat16(j ? c.w : c.z);
+    }
+  }
+};
+
+bool skinny_fits(int nt, int kmax) { return 8 * nt * skinny_pitch((kmax + 31) & ~31) + 64 <= SKINNY_SMEM_MAX; }
 
 }  // namespace
 
@@ -413,48 +425,40 @@ FT_EXPORT int ft_moe_gather(const void* h, int64_t ldh_bytes, const int* expert,
 FT_EXPORT int ft_moe_act(const void* gu, int64_t ld_gu, const float* row_score, const int* rows_used, int rows, int fp, float limit, float slope, void* act,
                          int64_t ld_act, int is_f32, cudaStream_t st) {
   if (rows < 1 || fp < 8 || (fp & 7) || (ld_gu & 7) || (ld_act & 7) || ld_gu < 2 * fp || ld_act < fp) return FT_ERR_ARG;
-  const size_t work = ((size_t)rows * (fp / 8) + 255) / 256;
-  const int grid = (int)(work > 148 * 16 ? 148 * 16 : work);
-  if (is_f32) moe_act_kernel<float><<<grid, 256, 0, st>>>((const float*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (float*)act, ld_act);
-  else moe_act_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((const __nv_bfloat16*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (__nv_bfloat16*)act, ld_act);
+  const int gx = (fp / 8 + 127) / 128;
+  int gy = (148 * 16 + gx - 1) / gx;
+  const dim3 grid(gx, gy < rows ? gy : rows);
+  if (is_f32) moe_act_kernel<float><<<grid, 128, 0, st>>>((const float*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (float*)act, ld_act);
+  else moe_act_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>((const __nv_bfloat16*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (__nv_bfloat16*)act, ld_act);
   return (int)cudaGetLastError();
 }
 
 // Decode routing (B <= 16 tokens, bf16 operands, f32 accumulation): logits [B][E] f32 scratch, counter int zero before the first launch. Outputs:
-// n_active int[1], id int[E], cnt int[E], pair int[E][16], score f32 [B * top].
+// n_active int[1], id int[E], cnt int[E], pair int[E][16], pair_of int[E][16], score f32 [B * top].
 FT_EXPORT int ft_moe_route_small(const void* h, int64_t ldh, const void* router, int64_t ldr, int B, int W, int E, int top, float* logits, int* counter, int* n_active,
-                                 int* id, int* cnt, int* pair, float* score, cudaStream_t st) {
+                                 int* id, int* cnt, int* pair, int* pair_of, float* score, cudaStream_t st) {
   if (B < 1 || B > SMALL_TOK || E < 1 || top < 1 || top > E || top > MAX_TOP || (ldh & 7) || (ldr & 7)) return FT_ERR_ARG;
-  return (int)ft_launch_pdl(moe_route_small_kernel, dim3((E + 7) / 8), dim3(256), 0, st, (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)router, ldr, B, W, E, top,
-                            logits, counter, SmallRoute{n_active, id, cnt, pair, score});
+  return (int)ft_launch_pdl(moe_route_small_kernel, dim3(E), dim3(128), 0, st, (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)router, ldr, B, W, E, top, logits,
+                            counter, SmallRoute{n_active, id, cnt, pair, pair_of, score});
 }
 
 // Gate / up projections and activation of a decode step. gu: [E][2 * fp][ld_in] interleaved rows, ld_in >= W rounded up to 32; act: bf16 [B * top][ld_act],
-// row = token * top + slot. Shared expert (shared_gu null: none): act_sh bf16 [B][ld_act_sh]. fp and fp_sh are the neuron counts rounded up to 8.
-FT_EXPORT int ft_moe_gate_up_small(const void* h, int64_t ldh, int B, int W, int E, int top, int* n_active, int* id, int* cnt, int* pair, float* score, const void* gu,
-                                   int f, int64_t ld_in, float limit, const void* shared_gu, int f_sh, int64_t ld_in_sh, float limit_sh, float slope, void* act,
-                                   int64_t ld_act, void* act_sh, int64_t ld_act_sh, cudaStream_t st) {
-  const int kp = (W + 31) & ~31;
-  if (B < 1 || B > SMALL_TOK || f < 1 || (ldh & 7) || (ld_in & 7) || ld_in < kp || ld_act < f || (shared_gu && ((ld_in_sh & 7) || ld_in_sh < kp || ld_act_sh < f_sh)))
+// row = token * top + slot. Shared expert (shared_gu null: none): act_sh bf16 [B][ld_act_sh]. fp is the neuron count rounded up to 8.
+FT_EXPORT int ft_moe_gate_up_small(const void* h, int64_t ldh, int B, int W, int E, int top, int* n_active, int* id, int* cnt, int* pair, int* pair_of, float* score,
+                                   const void* gu, int f, int64_t ld_in, float limit, const void* shared_gu, int f_sh, int64_t ld_in_sh, float limit_sh, float slope,
+                                   void* act, int64_t ld_act, void* act_sh, int64_t ld_act_sh, cudaStream_t st) {
+  const int kp = (W + 31) & ~31, fp = (f + 7) & ~7, fps = (f_sh + 7) & ~7;
+  if (B < 1 || B > SMALL_TOK || f < 1 || (ldh & 7) || (ld_in & 7) || ld_in < kp || ld_act < f || (shared_gu && (f_sh < 1 || (ld_in_sh & 7) || ld_in_sh < kp || ld_act_sh < f_sh)))
     return FT_ERR_ARG;
-  const SmallRoute R{n_active, id, cnt, pair, score};
-  const ExpertSet ex{(const __nv_bfloat16*)gu, nullptr, f, (f + 7) & ~7, ld_in, 0, limit};
-  const ExpertSet sh{(const __nv_bfloat16*)shared_gu, nullptr, f_sh, (f_sh + 7) & ~7, ld_in_sh, 0, limit_sh};
-  const int groups = E < B * top ? E : B * top, fmax = shared_gu && sh.fp > ex.fp ? sh.fp : ex.fp;
-  const dim3 grid((fmax + 63) / 64, groups + (shared_gu ? 1 : 0));
-  const int pitch = skinny_pitch(kp);
-  static bool done1[64] = {}, done2[64] = {};
-  if (B > 8 && 16 * pitch <= SMALL_SMEM_MAX) {
-    FT_CUDA_TRY(allow_smem(moe_gate_up_small_kernel<2>, done2));
-    return (int)ft_launch_pdl(moe_gate_up_small_kernel<2>, grid, dim3(256), (size_t)16 * pitch, st, (const __nv_bfloat16*)h, ldh, B, W, top, R, groups, ex, sh, slope,
-                              (__nv_bfloat16*)act, ld_act, (__nv_bfloat16*)act_sh, ld_act_sh, 0);
-  }
-  if (8 * pitch > SMALL_SMEM_MAX) return FT_ERR_TOO_LARGE;
-  FT_CUDA_TRY(allow_smem(moe_gate_up_small_kernel<1>, done1));
-  for (int t0 = 0; t0 < B; t0 += 8) {
-    const cudaError_t e = ft_launch_pdl(moe_gate_up_small_kernel<1>, grid, dim3(256), (size_t)8 * pitch, st, (const __nv_bfloat16*)h, ldh, B, W, top, R, groups, ex, sh,
-                                        slope, (__nv_bfloat16*)act, ld_act, (__nv_bfloat16*)act_sh, ld_act_sh, t0);
-    if (e != cudaSuccess) return (int)e;
+  if (!skinny_fits(1, W)) return FT_ERR_TOO_LARGE;
+  GateUpWork p{(const __nv_bfloat16*)h, ldh, B, W, 0, SmallRoute{n_active, id, cnt, pair, pair_of, score},
+               ExpertSet{(const __nv_bfloat16*)gu, f, fp, ld_in, 2 * fp * ld_in, limit}, ExpertSet{(const __nv_bfloat16*)shared_gu, f_sh, fps, ld_in_sh, 0, limit_sh},
+               shared_gu ? 1 : 0, slope, (__nv_bfloat16*)act, (__nv_bfloat16*)act_sh, ld_act, ld_act_sh};
+  const int items = (E < B * top ? E : B * top) * (fp / 8) + (shared_gu ? fps / 8 : 0);
+  if (B > 8 && skinny_fits(2, W)) return skinny_launch<GateUpWork, 2>(p, W, items, st);
+  for (p.tok0 = 0; p.tok0 < B; p.tok0 += 8) {
+    const int r = skinny_launch<GateUpWork, 1>(p, W, items, st);
+    if (r) return r;
   }
   return FT_OK;
 }
@@ -462,28 +466,23 @@ FT_EXPORT int ft_moe_gate_up_small(const void* h, int64_t ldh, int B, int W, int
 // Down projections of a decode step: out[slot][token][W] f32 (plane_stride, ldo in elements), the shared expert in plane `top`. down: [E][rows_out][ld_mid]
 // with rows_out >= W a multiple of 16 and ld_mid >= f rounded up to 32 (zeros past f).
 FT_EXPORT int ft_moe_down_small(const void* act, int64_t ld_act, const void* act_sh, int64_t ld_act_sh, int B, int W, int E, int top, int* n_active, int* id, int* cnt,
-                                int* pair, float* score, const void* down, int f, int64_t ld_mid, const void* shared_down, int f_sh, int64_t ld_mid_sh, int rows_out,
-                                float* out, int64_t plane_stride, int64_t ldo, cudaStream_t st) {
+                                int* pair, int* pair_of, float* score, const void* down, int f, int64_t ld_mid, const void* shared_down, int f_sh, int64_t ld_mid_sh,
+                                int rows_out, float* out, int64_t plane_stride, int64_t ldo, cudaStream_t st) {
   if (B < 1 || B > SMALL_TOK || f < 1 || (rows_out & 15) || rows_out < W || (ld_act & 7) || ld_mid < ((f + 31) & ~31) || (ld_mid & 7) ||
-      (shared_down && ((ld_act_sh & 7) || (ld_mid_sh & 7) || ld_mid_sh < ((f_sh + 31) & ~31))))
+      (shared_down && (f_sh < 1 || (ld_act_sh & 7) || (ld_mid_sh & 7) || ld_mid_sh < ((f_sh + 31) & ~31))))
     return FT_ERR_ARG;
-  const SmallRoute R{n_active, id, cnt, pair, score};
-  const ExpertSet ex{nullptr, (const __nv_bfloat16*)down, f, (f + 7) & ~7, 0, ld_mid, 0.f};
-  const ExpertSet sh{nullptr, (const __nv_bfloat16*)shared_down, f_sh, (f_sh + 7) & ~7, 0, ld_mid_sh, 0.f};
-  const int groups = E < B * top ? E : B * top;
-  const int kmax = ((shared_down && f_sh > f ? f_sh : f) + 31) & ~31;
-  int smem = 8 * skinny_pitch(kmax);
-  if (smem > SMALL_SMEM_MAX) return FT_ERR_TOO_LARGE;
-  const dim3 grid((W + 127) / 128, groups + (shared_down ? 1 : 0));
-  static bool done1[64] = {}, done2[64] = {};
-  if (B > 8 && 2 * smem + 128 <= SMALL_SMEM_MAX) {
-    FT_CUDA_TRY(allow_smem(moe_down_small_kernel<2>, done2));
-    return (int)ft_launch_pdl(moe_down_small_kernel<2>, grid, dim3(256), (size_t)2 * smem + 128, st, (const __nv_bfloat16*)act, ld_act, (const __nv_bfloat16*)act_sh,
-                              ld_act_sh, B, W, top, R, groups, ex, sh, rows_out, out, plane_stride, ldo);
+  const int kmax = shared_down && f_sh > f ? f_sh : f, blocks = (W + 15) / 16;
+  if (!skinny_fits(1, kmax)) return FT_ERR_TOO_LARGE;
+  DownWork p{(const __nv_bfloat16*)act, (const __nv_bfloat16*)act_sh, ld_act, ld_act_sh, B, W, top, 0, SmallRoute{n_active, id, cnt, pair, pair_of, score},
+             ExpertSet{(const __nv_bfloat16*)down, f, 0, ld_mid, rows_out * ld_mid, 0.f}, ExpertSet{(const __nv_bfloat16*)shared_down, f_sh, 0, ld_mid_sh, 0, 0.f},
+             shared_down ? 1 : 0, blocks, out, plane_stride, ldo};
+  const int items = ((E < B * top ? E : B * top) + (shared_down ? 1 : 0)) * blocks;
+  if (B > 8 && skinny_fits(2, kmax)) return skinny_launch<DownWork, 2>(p, kmax, items, st);
+  for (p.col0 = 0; p.col0 < B; p.col0 += 8) {
+    const int r = skinny_launch<DownWork, 1>(p, kmax, items, st);
+    if (r) return r;
   }
-  FT_CUDA_TRY(allow_smem(moe_down_small_kernel<1>, done1));
-  return (int)ft_launch_pdl(moe_down_small_kernel<1>, grid, dim3(256), (size_t)smem + 64, st, (const __nv_bfloat16*)act, ld_act, (const __nv_bfloat16*)act_sh, ld_act_sh,
-                            B, W, top, R, groups, ex, sh, rows_out, out, plane_stride, ldo);
+  return FT_OK;
 }
 
 // out[b][head][n] = sum_k w[head][n][k] x[b][head][k] for B <= 16 tokens: x bf16 (ldx between tokens, head_x between heads, 16-byte aligned), w bf16 rows of
@@ -491,18 +490,9 @@ FT_EXPORT int ft_moe_down_small(const void* act, int64_t ld_act, const void* act
 // to the next multiple of 16), out bf16.
 FT_EXPORT int ft_skinny_heads(const void* x, int64_t ldx, int64_t head_x, const void* w, int64_t ldw, int64_t head_w, int B, int heads, int N, int K, void* out,
                               int64_t ldo, int64_t head_o, cudaStream_t st) {
-  const int kp = (K + 31) & ~31, pitch = skinny_pitch(kp);
-  if (B < 1 || B > SMALL_TOK || heads < 1 || N < 1 || K < 1 || (ldx & 7) || (head_x & 7) || (ldw & 7) || ldw < kp || (head_w & 7)) return FT_ERR_ARG;
-  static bool done1[64] = {}, done2[64] = {};
-  const dim3 grid((N + 127) / 128, heads);
-  if (B > 8) {
-    if (16 * pitch > SMALL_SMEM_MAX) return FT_ERR_TOO_LARGE;
-    FT_CUDA_TRY(allow_smem(skinny_heads_kernel<2>, done2));
-    return (int)ft_launch_pdl(skinny_heads_kernel<2>, grid, dim3(256), (size_t)16 * pitch, st, (const __nv_bfloat16*)x, ldx, head_x, (const __nv_bfloat16*)w, ldw, head_w,
-                              B, N, K, (__nv_bfloat16*)out, ldo, head_o);
-  }
-  if (8 * pitch > SMALL_SMEM_MAX) return FT_ERR_TOO_LARGE;
-  FT_CUDA_TRY(allow_smem(skinny_heads_kernel<1>, done1));
-  return (int)ft_launch_pdl(skinny_heads_kernel<1>, grid, dim3(256), (size_t)8 * pitch, st, (const __nv_bfloat16*)x, ldx, head_x, (const __nv_bfloat16*)w, ldw, head_w, B,
-                            N, K, (__nv_bfloat16*)out, ldo, head_o);
+  if (B < 1 || B > SMALL_TOK || heads < 1 || N < 1 || K < 1 || (ldx & 7) || (head_x & 7) || (ldw & 7) || ldw < ((K + 31) & ~31) || (head_w & 7)) return FT_ERR_ARG;
+  const HeadsWork p{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, ldx, head_x, ldw, head_w, B, heads, N, K, (__nv_bfloat16*)out, ldo, head_o};
+  const int items = heads * ((N + 15) / 16);
+  if (!skinny_fits(B > 8 ? 2 : 1, K)) return FT_ERR_TOO_LARGE;
+  return B > 8 ? skinny_launch<HeadsWork, 2>(p, K, items, st) : skinny_launch<HeadsWork, 1>(p, K, items, st);
 }

@@ -7,6 +7,10 @@ from .llama import (rope_tables, rope_inplace, apply_rope, swiglu, swiglu_fwd, s
 from .loss import cross_entropy, cross_entropy_fwd_bwd
 from .optim import adamw_flat_, sgd_flat_, grad_norm_, scale_
 from .attention import attention_packed, flash_fwd, flash_bwd
+from .streams import DynamicTanhWeights, HyperWeights, SublayerOutput, dynamic_tanh, hyper_embed, hyper_update
+from .moe import ExpertStack, MoeWeights, MoeSmallBuffers, MoeRouting, moe_rows, moe_small, gated_act, grouped_linear, interleave_gate_up
+from .latent_attention import (LatentDims, LatentWeights, LatentDecodeBuffers, latent_attention_rows, latent_attention_decode, absorb_queries, expand_values,
+                               rotary_pair_tables)
 from . import attention
 
 __all__ = [n for n in dir() if not n.startswith("_")]

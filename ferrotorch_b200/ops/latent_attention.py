@@ -52,6 +52,8 @@ class LatentDims:
     def flash_tile(self) -> int:
         """Query rows per tile of the flash kernel, 0 when these sizes do not fit it."""
         nq, nv = -(-self.dim // 64) + -(-self.rot_dim // 64), -(-self.vdim // 64)
+        if nq == 2 and nv == 1:
+            return 128
         for nt, limit in ((2, 2), (1, 4)):
             if nv <= limit and nt * nq * 16384 + 2 * (nq + nv) * 8192 + nt * 16384 + 1280 <= _SMEM_MAX:
                 return 128 * nt
@@ -67,8 +69,8 @@ class LatentDims:
         return 0
 
     def decode_supported(self) -> bool:
-        fits = max(SMALL_TOKENS * self.dim, self.rank) * 4 <= 48 * 1024
-        return self.head_tiles() > 0 and fits and SMALL_TOKENS * (2 * round_up(self.rank, 32) + 64) <= 220 * 1024
+        fits = max(self.dim * (128 + 4 * SMALL_TOKENS), self.rank * 4) <= 48 * 1024
+        return self.head_tiles() > 0 and fits and SMALL_TOKENS * (2 * round_up(self.rank, 32) + 64) + 64 <= 208 * 1024
 
 
 @dataclass
@@ -179,22 +181,22 @@ class LatentDecodeBuffers:
         D = dims
         self.mt = D.head_tiles()
         self.tiles = -(-D.heads // (16 * self.mt))
-        # one CTA per SM (the ring takes most of its shared memory), at least one 64-row chunk per split at the longest sequence
-        self.nsplit = splits or max(1, min(64, 148 // max(1, max_batch * self.tiles), -(-max_tokens // 64)))
+        # by batch size: one CTA per SM (the ring takes most of its shared memory), at least one 64-row chunk per split at the longest sequence
+        self.splits = [splits or max(1, min(64, 148 // (b * self.tiles), -(-max_tokens // 64))) for b in range(1, max_batch + 1)]
         self.q = torch.zeros(SMALL_TOKENS, D.heads, D.row, device=device, dtype=torch.bfloat16)
         self.lat = torch.zeros(SMALL_TOKENS, D.heads, D.r16, device=device, dtype=torch.bfloat16)
-        self.ws = torch.zeros(max_batch * self.tiles * self.nsplit * self.mt * 16 * (D.r16 + 4), device=device)
+        self.ws = torch.zeros(max(b * n for b, n in enumerate(self.splits, 1)) * self.tiles * self.mt * 16 * (D.r16 + 4), device=device)
         self.attn = torch.zeros(SMALL_TOKENS, D.heads * D.v8, device=device, dtype=torch.bfloat16)
 
 
 def latent_attention_decode(planes: torch.Tensor, splits: int, w: LatentWeights, b: LatentDecodeBuffers, state, cache: torch.Tensor, cos, sin, B: int) -> torch.Tensor:
     """One token per sequence from the split-K planes of the projection: returns the attention output rows ``[16, heads * v8]`` (bf16, in ``b``)."""
     D, S = w.dims, _lib.S()
-    bt, mb = state.block_table, state.block_table.shape[1]
+    bt, mb, nsplit = state.block_table, state.block_table.shape[1], b.splits[B - 1]
     _lib.call("ft_latent_decode_prep", planes, splits, planes.stride(1), planes.stride(0), B, D.heads, D.dim, D.rot_dim, D.rank, w.ukv, w.ukv.stride(0), w.norm, D.eps,
               state.positions, cos, sin, bt, mb, b.q, cache, S)
-    _lib.call("ft_latent_decode", b.q, cache, bt, mb, state.seq_lens, B, D.heads, D.rot_dim, D.rank, D.scale, b.nsplit, b.mt, b.ws, S)
-    _lib.call("ft_latent_combine", b.ws, B, D.heads, D.rank, b.nsplit, b.mt, b.lat, S)
+    _lib.call("ft_latent_decode", b.q, cache, bt, mb, state.seq_lens, B, D.heads, D.rot_dim, D.rank, D.scale, nsplit, b.mt, b.ws, S)
+    _lib.call("ft_latent_combine", b.ws, B, D.heads, D.rank, nsplit, b.mt, b.lat, S)
     _lib.call("ft_skinny_heads", b.lat, b.lat.stride(0), b.lat.stride(1), w.uv, w.uv.stride(0), D.v8 * w.uv.stride(0), B, D.heads, D.vdim, D.rank, b.attn,
               b.attn.stride(0), D.v8, S)
     return b.attn

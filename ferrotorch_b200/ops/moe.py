@@ -19,7 +19,7 @@ from .streams import SublayerOutput, round_up
 
 SMALL_TOKENS = 16
 MAX_TOP = 32
-_SMALL_SMEM = 220 * 1024
+_SMALL_SMEM = 208 * 1024
 SEGMENT = 128
 
 
@@ -111,6 +111,7 @@ class MoeSmallBuffers:
     ids: torch.Tensor
     cnt: torch.Tensor
     pair: torch.Tensor
+    pair_of: torch.Tensor
     score: torch.Tensor
     act: torch.Tensor
     act_sh: torch.Tensor
@@ -124,7 +125,7 @@ class MoeSmallBuffers:
 
         def ints(*s):
             return torch.zeros(*s, device=device, dtype=torch.int32)
-        return MoeSmallBuffers(torch.zeros(SMALL_TOKENS * E, device=device), ints(1), ints(1), ints(E), ints(E), ints(E * SMALL_TOKENS),
+        return MoeSmallBuffers(torch.zeros(SMALL_TOKENS * E, device=device), ints(1), ints(1), ints(E), ints(E), ints(E * SMALL_TOKENS), ints(E * SMALL_TOKENS),
                                torch.zeros(SMALL_TOKENS * top, device=device), torch.zeros(SMALL_TOKENS * top, round_up(f, 8), device=device, dtype=torch.bfloat16),
                                torch.zeros(SMALL_TOKENS, round_up(fs, 8), device=device, dtype=torch.bfloat16),
                                torch.zeros(top + 1, SMALL_TOKENS, round_up(width, 8), device=device))
@@ -133,7 +134,7 @@ class MoeSmallBuffers:
 def moe_small(h: torch.Tensor, w: MoeWeights, b: MoeSmallBuffers, tokens: int) -> SublayerOutput:
     """Decode step: ``tokens`` (<= 16) bf16 rows of ``h``. The result's planes live in ``b`` until the next call."""
     E, x, s, S = w.num_experts, w.experts, w.shared, _lib.S()
-    route = (b.n_active, b.ids, b.cnt, b.pair, b.score)
+    route = (b.n_active, b.ids, b.cnt, b.pair, b.pair_of, b.score)
     _lib.call("ft_moe_route_small", h, h.stride(0), w.router, w.router.stride(0), tokens, w.width, E, w.top, b.logits, b.counter, *route, S)
     _lib.call("ft_moe_gate_up_small", h, h.stride(0), tokens, w.width, E, w.top, *route, x.gu, x.ff, x.gu.stride(1), x.limit, s.gu if s else None, s.ff if s else 0,
               s.gu.stride(1) if s else 0, s.limit if s else 0.0, w.slope, b.act, b.act.stride(0), b.act_sh, b.act_sh.stride(0), S)
@@ -191,6 +192,6 @@ def moe_rows(h: torch.Tensor, w: MoeWeights) -> SublayerOutput:
     planes = None
     if s is not None:
         sgu = linear_rows(h, s.gu[0][:, : w.width])
-        planes = linear_rows(gated_act(sgu, s.fp, s.limit, w.slope), s.down[0][: w.width, : s.ff], out_f32=True)
+        planes = linear_rows(gated_act(sgu, s.fp, s.limit, w.slope)[:, : s.ff], s.down[0][: w.width, : s.ff], out_f32=True)
         planes = planes.as_strided((1, T, w.width), (0, planes.stride(0), 1))
     return SublayerOutput(planes=planes, rows=out, row_of=row_of, top=w.top)
