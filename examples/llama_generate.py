@@ -3,6 +3,9 @@
 
     python examples/llama_generate.py --prompt-len 16 --new 32 [--weights /path/to/model.safetensors --config /path/to/config.json]
 
+With `--model DIR` any registered architecture is loaded from its checkpoint directory (`config.json` + safetensors; Llama, Ginisun) and run by the
+serving engine: `python examples/llama_generate.py --model DIR --prompt 5,17,3 --prompt 8 --new 32 [--temperature 0.8 --top-k 50 --top-p 0.95]`.
+
 On a B200 the same model runs through the tensor-parallel engine (`LlamaTPEngine`: paged KV cache, CUDA-graph decode) with `--engine tp`
 (launch with torch.distributed.run for more than one GPU). Counterpart of ferrotorch-llama/examples/llama3_8b.rs and llama3_8b_gpu.rs.
 """
@@ -19,6 +22,16 @@ from ferrotorch_b200.models import CachedLlama, GenerationConfig, LlamaConfig, S
 from ferrotorch_b200.models.llama_infer import random_hf_weights
 
 
+def generate_from_directory(a):
+    from ferrotorch_b200.models import load_engine, load_model_config
+    _, cfg = load_model_config(a.model)
+    prompts = [[int(t) for t in p.split(",")] for p in a.prompt] if a.prompt else [torch.randint(0, cfg.vocab_size, (a.prompt_len,)).tolist()]
+    eng = load_engine(a.model, a.device, getattr(torch, a.dtype), max_tokens=sum(len(p) + a.new + 16 for p in prompts))
+    g = GenerationConfig(max_new_tokens=a.new, do_sample=a.temperature > 0, temperature=a.temperature, top_k=a.top_k, top_p=a.top_p, seed=a.seed)
+    for p, out in zip(prompts, eng.generate(prompts, g)):
+        print(",".join(map(str, p)), "->", ",".join(map(str, out)))
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--prompt-len", type=int, default=16)
@@ -27,7 +40,16 @@ def main():
     ap.add_argument("--config")
     ap.add_argument("--engine", choices=["cached", "tp"], default="cached")
     ap.add_argument("--device", default="cuda" if torch.cuda.is_available() else "cpu")
+    ap.add_argument("--model", help="checkpoint directory of a registered architecture")
+    ap.add_argument("--prompt", action="append", help="token ids with commas between them; several prompts form a batch (with --model)")
+    ap.add_argument("--dtype", choices=["bfloat16", "float32"], default="bfloat16")
+    ap.add_argument("--temperature", type=float, default=0.0)
+    ap.add_argument("--top-k", type=int, default=0)
+    ap.add_argument("--top-p", type=float, default=1.0)
+    ap.add_argument("--seed", type=int, default=0)
     a = ap.parse_args()
+    if a.model:
+        return generate_from_directory(a)
     if a.config:
         cfg = LlamaConfig.from_hf(json.load(open(a.config)))
     else:

@@ -121,44 +121,51 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict
   for (int i = threadIdx.x; i < vecs; i += 128) dst[i] = src[i];
 }
 
-// gu: [rows][2 * fp] in blocks of eight gate | eight up columns -> act [rows][ld_act]. grid (column blocks, row groups): a thread keeps its eight neurons.
+// gu: [rows][2 * fp] in blocks of eight gate | eight up columns -> act [rows][ld_act]. grid (column blocks, row groups). bf16: neighbouring lanes load the
+// gate and the up half of a block (16 bytes each, a warp reads 512 contiguous bytes) and swap halves, so each ends up with four neurons.
 template <typename T>
-__global__ void __launch_bounds__(128) moe_act_kernel(const T* __restrict__ gu, int64_t ld_gu, const float* __restrict__ row_score, const int* __restrict__ rows_used,
+__global__ void __launch_bounds__(256) moe_act_kernel(const T* __restrict__ gu, int64_t ld_gu, const float* __restrict__ row_score, const int* __restrict__ rows_used,
                                                       int rows, int fp, float limit, float slope, T* __restrict__ act, int64_t ld_act) {
   const int n = rows_used ? min(rows, *rows_used) : rows;
-  const int blk = blockIdx.x * 128 + threadIdx.x;
-  if (blk * 8 >= fp) return;
+  const int unit = blockIdx.x * blockDim.x + threadIdx.x, units = fp / 4;
   if constexpr (sizeof(T) == 2) {
     constexpr int RU = 4;                              // rows in flight
+    const bool live = unit < units;
+    const int u = live ? unit : units - 2 + (unit & 1);
+    const bool odd = unit & 1;
     for (int r0 = blockIdx.y; r0 < n; r0 += gridDim.y * RU) {
-      bf16x8 gr[RU], ur[RU];
+      uint4 v[RU];
       float sc[RU];
 #pragma unroll
       for (int i = 0; i < RU; i++) {
         const int r = min(r0 + i * (int)gridDim.y, n - 1);
-        const T* src = gu + (size_t)r * ld_gu + blk * 16;
-        gr[i] = *reinterpret_cast<const bf16x8*>(src);
-        ur[i] = *reinterpret_cast<const bf16x8*>(src + 8);
+        v[i] = *reinterpret_cast<const uint4*>(gu + (size_t)r * ld_gu + u * 8);
         sc[i] = row_score ? row_score[r] : 1.f;
       }
 #pragma unroll
       for (int i = 0; i < RU; i++) {
         const int r = r0 + i * (int)gridDim.y;
-        if (r >= n) break;
-        float g[8], u[8], o[8];
-        bf16x8_to_float(gr[i], g);
-        bf16x8_to_float(ur[i], u);
-#pragma unroll
-        for (int e = 0; e < 8; e++) o[e] = gated_clamped_fast(sc[i] * g[e], sc[i] * u[e], limit, slope);
-        *reinterpret_cast<bf16x8*>(act + (size_t)r * ld_act + blk * 8) = float_to_bf16x8(o);
+        // even lane: gate 0..3 kept, up 0..3 received; odd lane: gate 4..7 received, up 4..7 kept
+        const uint32_t m0 = __shfl_xor_sync(0xffffffffu, odd ? v[i].x : v[i].z, 1), m1 = __shfl_xor_sync(0xffffffffu, odd ? v[i].y : v[i].w, 1);
+        const uint32_t g0 = odd ? m0 : v[i].x, g1 = odd ? m1 : v[i].y, u0 = odd ? v[i].z : m0, u1 = odd ? v[i].w : m1;
+        const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g0)), gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g1));
+        const float2 ua = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u0)), ub = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u1));
+        const float k = sc[i];
+        __nv_bfloat162 o0 = __floats2bfloat162_rn(gated_clamped_fast(k * ga.x, k * ua.x, limit, slope), gated_clamped_fast(k * ga.y, k * ua.y, limit, slope));
+        __nv_bfloat162 o1 = __floats2bfloat162_rn(gated_clamped_fast(k * gb.x, k * ub.x, limit, slope), gated_clamped_fast(k * gb.y, k * ub.y, limit, slope));
+        uint2 pk;
+        pk.x = *reinterpret_cast<uint32_t*>(&o0);
+        pk.y = *reinterpret_cast<uint32_t*>(&o1);
+        if (live && r < n) *reinterpret_cast<uint2*>(act + (size_t)r * ld_act + unit * 4) = pk;
       }
     }
   } else {
+    if (unit >= units) return;
     for (int r = blockIdx.y; r < n; r += gridDim.y) {
       const float s = row_score ? row_score[r] : 1.f;
-      const T* src = gu + (size_t)r * ld_gu + blk * 16;
+      const T* src = gu + (size_t)r * ld_gu + (unit / 2) * 16 + (unit % 2) * 4;
 #pragma unroll
-      for (int e = 0; e < 8; e++) act[(size_t)r * ld_act + blk * 8 + e] = gated_clamped(s * src[e], s * src[8 + e], limit, slope);
+      for (int e = 0; e < 4; e++) act[(size_t)r * ld_act + unit * 4 + e] = gated_clamped(s * src[e], s * src[8 + e], limit, slope);
     }
   }
 }
@@ -425,11 +432,11 @@ FT_EXPORT int ft_moe_gather(const void* h, int64_t ldh_bytes, const int* expert,
 FT_EXPORT int ft_moe_act(const void* gu, int64_t ld_gu, const float* row_score, const int* rows_used, int rows, int fp, float limit, float slope, void* act,
                          int64_t ld_act, int is_f32, cudaStream_t st) {
   if (rows < 1 || fp < 8 || (fp & 7) || (ld_gu & 7) || (ld_act & 7) || ld_gu < 2 * fp || ld_act < fp) return FT_ERR_ARG;
-  const int gx = (fp / 8 + 127) / 128;
-  int gy = (148 * 16 + gx - 1) / gx;
+  const int units = fp / 4, gx = (units + 255) / 256, threads = ((units + gx - 1) / gx + 31) / 32 * 32;
+  const int gy = (148 * 8 * (256 / threads) + gx - 1) / gx;
   const dim3 grid(gx, gy < rows ? gy : rows);
-  if (is_f32) moe_act_kernel<float><<<grid, 128, 0, st>>>((const float*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (float*)act, ld_act);
-  else moe_act_kernel<__nv_bfloat16><<<grid, 128, 0, st>>>((const __nv_bfloat16*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (__nv_bfloat16*)act, ld_act);
+  if (is_f32) moe_act_kernel<float><<<grid, threads, 0, st>>>((const float*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (float*)act, ld_act);
+  else moe_act_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>((const __nv_bfloat16*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (__nv_bfloat16*)act, ld_act);
   return (int)cudaGetLastError();
 }
 

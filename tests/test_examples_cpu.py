@@ -94,3 +94,10 @@ def test_learner_example_trains_on_synthetic_digits(tmp_path):
     losses = [float(l.split("train_loss")[1].split()[0]) for l in out.splitlines() if l.startswith("epoch")]
     assert len(losses) == 3 and losses[-1] < losses[0]
     assert any((tmp_path / "run").rglob("*")), "checkpoints / event files were written"
+
+
+def test_generation_from_a_checkpoint_directory(tmp_path):
+    _run(ROOT / "examples/llm_inference_dump.py", "--write-random", tmp_path / "ckpt")
+    out = _run(ROOT / "examples/llama_generate.py", "--model", tmp_path / "ckpt", "--device", "cpu", "--dtype", "float32", "--prompt", "5,17,3", "--prompt", "8", "--new", "4")
+    lines = [l for l in out.splitlines() if "->" in l]
+    assert lines[0].startswith("5,17,3 -> ") and lines[1].startswith("8 -> ") and all(len(l.split("-> ")[1].split(",")) == 4 for l in lines)
