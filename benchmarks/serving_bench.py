@@ -74,7 +74,7 @@ def _by_shape(names):
             o = 4 if fn == "ft_gemm_bf16" else 3
             return names.get((raw[o + 1], raw[o + 2]), f"gemm n={raw[o + 1]} k={raw[o + 2]}")
         if fn == "ft_gemm_grouped":
-            return names.get((raw[4], raw[5]), "grouped gemm")
+            return names.get(("grouped", raw[4], raw[5]), "grouped gemm")
         return names.get(fn, fn)
     return c
 
@@ -102,15 +102,15 @@ def run_ginisun(size, layers, batch, prompt, ctx, steps, kernels=True):
     if kernels:
         eng._admit([StepEntry("p", ids, [])])
         names = {(D.proj_cols, W): "projection gemm", (nkv, D.rank): "key/value expansion gemm", (W, H * D.v8): "output gemm", (E, W): "router gemm",
-                 (2 * F, W): "experts gate/up gemm", (W, F): "experts down gemm", (2 * SF, W): "shared gate/up gemm", (W, SF): "shared down gemm"}
+                 ("grouped", 2 * F, W): "experts gate/up gemm", ("grouped", W, F): "experts down gemm", (2 * SF, W): "shared gate/up gemm"}
+        names[(W, SF)] = "output and shared down gemm" if SF == H * D.v8 else "shared down gemm"      # one shape: one label
         pairs = T * top
         def g_(n, k, out=2, m=T): return (2 * (m * k + n * k) + out * m * n, 2 * m * n * k)
         roofs = {"projection gemm": g_(D.proj_cols, W), "key/value expansion gemm": g_(nkv, D.rank), "output gemm": g_(W, H * D.v8, 4),
                  "experts gate/up gemm": (2 * (pairs * W + E * 2 * F * W + pairs * 2 * F), 4 * pairs * F * W), "experts down gemm": (2 * (pairs * W + E * F * W + pairs * F), 2 * pairs * F * W),
-                 "shared gate/up gemm": g_(2 * SF, W), "shared down gemm": g_(W, SF, 4),
+                 "shared gate/up gemm": g_(2 * SF, W), "shared down gemm": g_(W, SF, 4), "output and shared down gemm": g_(W, SF, 4),
                  "ft_latent_flash": (2 * T * (H * (D.dim8 + D.rot8) + nkv + H * D.v8), H * T * T * (D.dim + D.rot_dim + D.vdim)),
                  "ft_latent_prep": (2 * T * (2 * H * D.rot8 + D.rank + D.rot8 + 2 * D.row), 0),
-                 "ft_hyper_update": (T * W * (32 + 2 + 4 + top) if SF else T * W * (34 + 2 * top), 0),   # average of the two sublayers, see below
                  "ft_moe_gather": (4 * pairs * W, 0), "ft_moe_act": ((pairs * F * 6 + T * SF * 6) / 2, 0)}
         # streams read and written in f32 (8 bytes each), bf16 operand out; attention adds one f32 plane, the mixture its bf16 rows (+ one f32 plane)
         roofs["ft_hyper_update"] = (T * W * (4 * 8 + 2 + (4 + (2 * top + (4 if SF else 0))) / 2), 0)

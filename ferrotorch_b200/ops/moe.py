@@ -8,7 +8,7 @@ weights of the experts in use through ``mma.sync`` with all tokens in shared mem
 from __future__ import annotations
 
 from dataclasses import dataclass
-from typing import List, Optional, Sequence
+from typing import Optional, Sequence
 
 import torch
 

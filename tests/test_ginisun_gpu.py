@@ -97,7 +97,7 @@ def test_streams_start_update_and_end(dtype, n, rows, width):
 # -- latent attention ------------------------------------------------------------------------------------------------------------------
 DIMS = [dict(heads=3, dim=16, rot_dim=8, vdim=24, rank=40), dict(heads=5, dim=20, rot_dim=6, vdim=12, rank=33), dict(heads=2, dim=64, rot_dim=64, vdim=64, rank=128),
         dict(heads=4, dim=128, rot_dim=64, vdim=128, rank=512), dict(heads=2, dim=96, rot_dim=32, vdim=72, rank=64), dict(heads=1, dim=160, rot_dim=64, vdim=200, rank=96),
-        dict(heads=40, dim=24, rot_dim=16, vdim=16, rank=48), dict(heads=17, dim=8, rot_dim=2, vdim=8, rank=8)]
+        dict(heads=40, dim=24, rot_dim=16, vdim=16, rank=48), dict(heads=17, dim=8, rot_dim=2, vdim=8, rank=8), dict(heads=2, dim=320, rot_dim=64, vdim=128, rank=64)]
 
 
 def make_attention(D, width=48, seed=0, scale=None):
