@@ -1,0 +1,1106 @@
+// Grouped-query attention with per-head key and value sizes, over a paged row cache: rotary positions on the first dimensions of a head (neighbouring pairs),
+// RMS norms on queries and keys (per head, or over the whole projection), an optional sliding window, softmax with an optional sink per head, values
+// optionally mixed with those of an earlier layer, and an output gate (per element or per head) with a scale.
+//
+// Head sizes are padded to multiples of 16 (zeros): d16, v16. A token's cache row is [G keys of d16 | G values of v16]; pages hold 16 rows.
+//
+//   ft_gqa_prep          projection rows of a prompt -> normalised, rotated queries (in place), keys and values -> cache rows
+//   ft_gqa_flash         prompts (tcgen05): ragged sequences, keys and values straight from the pages; the heads of a group share a tile
+//   ft_gqa_decode_prep   the same as ft_gqa_prep for one token per sequence, from split-K planes
+//   ft_gqa_decode        one query token per sequence, the heads of a group share every loaded row (mma.sync), split over the visible range; the last CTA
+//                        of a group merges the splits, adds the sink and applies the gate
+//   ft_gqa_rows          plain f32-arithmetic kernel for f32 or bf16 data and any sizes (the 32-bit path)
+// Compiled without fast-math.
+#include <cooperative_groups.h>
+
+#include "common.cuh"
+#include "host_common.h"
+
+namespace {
+
+constexpr int KV_BLOCK = 16;
+constexpr float LOG2E = 1.4426950408889634f;
+
+FT_DEVICE float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+FT_DEVICE float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+FT_DEVICE float sigmoid_fast(float x) { return 1.f / (1.f + __expf(-x)); }
+
+struct GqaDims {
+  int H, G, d, dv, d16, v16, rot;    // query heads, key / value heads, sizes and padded sizes, rotated dimensions
+  int row;                           // cache row: G * (d16 + v16)
+};
+enum { GATE_NONE = 0, GATE_ELEMENT = 1, GATE_HEAD = 2 };
+
+// eight consecutive elements
+template <typename T> FT_DEVICE void load8(const T* p, float (&v)[8]);
+template <> FT_DEVICE void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> FT_DEVICE void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) { bf16x8_to_float(*reinterpret_cast<const bf16x8*>(p), v); }
+template <typename T> FT_DEVICE void store8(T* p, const float (&v)[8]);
+template <> FT_DEVICE void store8<float>(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <> FT_DEVICE void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) { *reinterpret_cast<bf16x8*>(p) = float_to_bf16x8(v); }
+template <typename T> FT_DEVICE float one(T v);
+template <> FT_DEVICE float one<float>(float v) { return v; }
+template <> FT_DEVICE float one<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+// ------------------------------------------------------------------------------------------------------------
+// prompt rows: one CTA per row; a thread holds eight neighbouring columns (four rotation pairs) of a head. WHOLE: one norm over all heads.
+// ------------------------------------------------------------------------------------------------------------
+struct PrepArgs {
+  GqaDims D;
+  const float *wq, *wk;              // per head: [d16]; whole: [heads * d16]
+  float eps;
+  const int* positions;
+  const float *cos_t, *sin_t;
+  const int* slots;
+};
+constexpr int PREP_T = 128;
+
+template <typename T, bool WHOLE>
+__global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, int64_t ld, PrepArgs A, T* __restrict__ cache, const T* __restrict__ vfirst, int64_t ldf,
+                                                          const float* __restrict__ lambda) {
+  __shared__ float red[32];
+  const GqaDims& D = A.D;
+  const int r = blockIdx.x, pos = A.positions[r], half = D.rot / 2, hv = D.d16 / 8, nq = D.H * hv, nk = D.G * hv;
+  T* row = qkv + (size_t)r * ld;
+  T* dst = cache + (size_t)A.slots[r] * D.row;
+  const float* ct = A.cos_t + (size_t)pos * half;
+  const float* st = A.sin_t + (size_t)pos * half;
+  auto finish = [&](int head, int vi, bool is_q, const float (&x)[8], float rstd) {       // norm weight, rotation, store
+    const float* w = (is_q ? A.wq : A.wk) + (WHOLE ? (is_q ? head : head - D.H) * D.d16 : 0) + vi * 8;
+    float v[8];
+#pragma unroll
+    for (int e = 0; e < 8; e++) v[e] = x[e] * rstd * w[e];
+#pragma unroll
+    for (int e = 0; e < 4; e++) {
+      const int p = vi * 4 + e;
+      if (p < half) {
+        const float c = ct[p], s = st[p], a = v[2 * e], b = v[2 * e + 1];
+        v[2 * e] = a * c - b * s;
+        v[2 * e + 1] = b * c + a * s;
+      }
+    }
+    store8(is_q ? row + head * D.d16 + vi * 8 : dst + (head - D.H) * D.d16 + vi * 8, v);
+  };
+  if constexpr (WHOLE) {
+    float sq = 0.f, sk = 0.f, x[8];
+    for (int i = threadIdx.x; i < nq + nk; i += PREP_T) {
+      load8(row + i * 8, x);
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < 8; e++) s += x[e] * x[e];
+      if (i < nq) sq += s; else sk += s;
+    }
+    sq = block_sum(sq, red);
+    sk = block_sum(sk, red);
+    const float rq = 1.f / sqrtf(sq / (float)(D.H * D.d) + A.eps), rk = 1.f / sqrtf(sk / (float)(D.G * D.d) + A.eps);
+    for (int i = threadIdx.x; i < nq + nk; i += PREP_T) {
+      load8(row + i * 8, x);
+      finish(i / hv, i % hv, i < nq, x, i < nq ? rq : rk);
+    }
+  } else {
+    int lanes = 1;                                   // lanes of a head: a power of two that covers its columns, at most a warp
+    while (lanes < hv && lanes < 32) lanes *= 2;
+    const int l = threadIdx.x % lanes, groups = PREP_T / lanes;
+    for (int h0 = 0; h0 < D.H + D.G; h0 += groups) {
+      const int head = h0 + threadIdx.x / lanes;
+      const bool live = head < D.H + D.G;
+      float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, s = 0.f;
+      if (live)
+        for (int vi = l; vi < hv; vi += lanes) {
+          load8(row + head * D.d16 + vi * 8, x);
+#pragma unroll
+          for (int e = 0; e < 8; e++) s += x[e] * x[e];
+        }
+      for (int o = lanes / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
+      const float rstd = 1.f / sqrtf(s / (float)D.d + A.eps);
+      if (live)
+        for (int vi = l; vi < hv; vi += lanes) {
+          if (hv > lanes) load8(row + head * D.d16 + vi * 8, x);       // a single vector per lane is still in registers
+          finish(head, vi, head < D.H, x, rstd);
+        }
+    }
+  }
+  const float lam = lambda ? *lambda : 0.f;
+  for (int i = threadIdx.x; i < D.G * D.v16 / 8; i += PREP_T) {
+    float v[8];
+    load8(row + (D.H + D.G) * D.d16 + i * 8, v);
+    if (lambda) {
+      float f[8];
+      load8(vfirst + (size_t)r * ldf + i * 8, f);
+#pragma unroll
+      for (int e = 0; e < 8; e++) v[e] = (1.f - lam) * v[e] + lam * f[e];
+    }
+    store8(dst + D.G * D.d16 + i * 8, v);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// plain kernel: grid (rows, H), 128 threads
+// ------------------------------------------------------------------------------------------------------------
+struct MaskGate {
+  float scale;
+  int window;                        // keys a position sees, itself included (INT_MAX: all)
+  const float* sink;                 // [H] or null
+  const void* gate;                  // per element: rows of H * v16 in the data type; per head: f32 rows of H (pre-activation)
+  int64_t ldg;
+  int gate_kind;
+  float out_scale;
+};
+constexpr int ROWS_CHUNK = 64, ROWS_MAX_COLS = 8;
+template <typename T>
+__global__ void __launch_bounds__(128) gqa_rows_kernel(const T* __restrict__ q, int64_t ldq, const T* __restrict__ cache, const int* __restrict__ block_table, int max_blocks,
+                                                       const int* __restrict__ seq_of, const int* __restrict__ positions, GqaDims D, MaskGate M, T* __restrict__ out,
+                                                       int64_t ldo) {
+  extern __shared__ float sq[];      // d16
+  __shared__ float sp[ROWS_CHUNK];
+  const int r = blockIdx.x, hd = blockIdx.y, g = hd / (D.H / D.G), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int len = positions[r] + 1, first = M.window < len ? len - M.window : 0;
+  const int* bt = block_table + (size_t)seq_of[r] * max_blocks;
+  for (int i = threadIdx.x; i < D.d16; i += 128) sq[i] = one(q[(size_t)r * ldq + hd * D.d16 + i]);
+  float o[ROWS_MAX_COLS];
+#pragma unroll
+  for (int i = 0; i < ROWS_MAX_COLS; i++) o[i] = 0.f;
+  float m = -INFINITY, l = 0.f;
+  if (M.sink) { m = M.sink[hd]; l = 1.f; }           // the sink is a score without a value
+  __syncthreads();
+  for (int t0 = first; t0 < len; t0 += ROWS_CHUNK) {
+    const int cnt = min(ROWS_CHUNK, len - t0);
+    for (int k = warp; k < cnt; k += 4) {
+      const int t = t0 + k;
+      const T* kr = cache + ((size_t)bt[t / KV_BLOCK] * KV_BLOCK + t % KV_BLOCK) * D.row + g * D.d16;
+      float a = 0.f;
+      for (int i = lane; i < D.d16; i += 32) a += sq[i] * one(kr[i]);
+      a = warp_sum(a);
+      if (lane == 0) sp[k] = a * M.scale;
+    }
+    __syncthreads();
+    float mx = m;
+    for (int k = 0; k < cnt; k++) mx = fmaxf(mx, sp[k]);
+    const float alpha = expf(m - mx);
+    l *= alpha;
+#pragma unroll
+    for (int i = 0; i < ROWS_MAX_COLS; i++) o[i] *= alpha;
+    for (int k = 0; k < cnt; k++) {
+      const int t = t0 + k;
+      const T* vr = cache + ((size_t)bt[t / KV_BLOCK] * KV_BLOCK + t % KV_BLOCK) * D.row + D.G * D.d16 + g * D.v16;
+      const float p = expf(sp[k] - mx);
+      l += p;
+#pragma unroll
+      for (int i = 0; i < ROWS_MAX_COLS; i++)
+        if (threadIdx.x + 128 * i < D.v16) o[i] += p * one(vr[threadIdx.x + 128 * i]);
+    }
+    m = mx;
+    __syncthreads();
+  }
+#pragma unroll
+  for (int i = 0; i < ROWS_MAX_COLS; i++) {
+    const int c = threadIdx.x + 128 * i;
+    if (c < D.v16) {
+      float v = o[i] / l * M.out_scale;
+      if (M.gate_kind == GATE_ELEMENT) v *= sigmoid_exact(one(reinterpret_cast<const T*>(M.gate)[(size_t)r * M.ldg + hd * D.v16 + c]));
+      if (M.gate_kind == GATE_HEAD) v *= sigmoid_exact(reinterpret_cast<const float*>(M.gate)[(size_t)r * M.ldg + hd]);
+      if constexpr (sizeof(T) == 4) out[(size_t)r * ldo + hd * D.v16 + c] = v;
+      else out[(size_t)r * ldo + hd * D.v16 + c] = __float2bfloat16(v);
+    }
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// decode preparation from split-K planes: a warp takes one head (or 128 gate columns) of one token, four columns a lane. WHOLE: the CTAs of a token form a
+// cluster, sums of squares meet in distributed shared memory, the plane sums wait in shared memory meanwhile.
+// ------------------------------------------------------------------------------------------------------------
+constexpr int DEC_TOK = 16, DP_WARPS = 8, DP_MAXC = 4;       // head sizes up to 128 * DP_MAXC
+FT_DEVICE float4 plane_sum4(const float* __restrict__ p, int splits, size_t stride) {
+  float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+  int s = 0;
+  for (; s + 4 <= splits; s += 4) {
+    float4 t[4];
+#pragma unroll
+    for (int j = 0; j < 4; j++) t[j] = __ldcg(reinterpret_cast<const float4*>(p + (s + j) * stride));
+    a.x += (t[0].x + t[1].x) + (t[2].x + t[3].x);
+    a.y += (t[0].y + t[1].y) + (t[2].y + t[3].y);
+    a.z += (t[0].z + t[1].z) + (t[2].z + t[3].z);
+    a.w += (t[0].w + t[1].w) + (t[2].w + t[3].w);
+  }
+  for (; s < splits; s++) {
+    const float4 t = __ldcg(reinterpret_cast<const float4*>(p + s * stride));
+    a.x += t.x; a.y += t.y; a.z += t.z; a.w += t.w;
+  }
+  return a;
+}
+struct DecPrepArgs {
+  PrepArgs P;
+  const float* planes;
+  int splits;
+  int64_t ldp;
+  size_t pstride;
+  const int* block_table;
+  int max_blocks;
+  int gate_col, gate_kind;           // column of the gate's pre-activation in the planes
+  float* gate;                       // [16][H * v16] or [16][H]: sigmoid of it
+  float* vf_out;                     // [16][G * v16]: values kept for later layers, or
+  const float* vf_in;                //   mixed in with weight *lambda
+  const float* lambda;
+};
+FT_DEVICE void put_bf16x4(__nv_bfloat16* p, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 pk;
+  pk.x = *reinterpret_cast<uint32_t*>(&a);
+  pk.y = *reinterpret_cast<uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(p) = pk;
+}
+
+template <bool WHOLE>
+__global__ void __launch_bounds__(DP_WARPS * 32) gqa_decode_prep_kernel(DecPrepArgs A, __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache) {
+  namespace cg = cooperative_groups;
+  extern __shared__ __align__(16) float held[];      // WHOLE: plane sums of this CTA's query and key heads, [local unit][d16]
+  __shared__ float red[32];
+  __shared__ float cta_ss[2];
+  pdl_wait();
+  pdl_launch_dependents();
+  const GqaDims& D = A.P.D;
+  const int b = blockIdx.y, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, pos = A.P.positions[b], half = D.rot / 2, stride = gridDim.x * DP_WARPS;
+  const int u0 = blockIdx.x * DP_WARPS + warp, heads = D.H + D.G;
+  const float* src = A.planes + (size_t)b * A.ldp;
+  const int blk = A.block_table[(size_t)b * A.max_blocks + pos / KV_BLOCK];
+  __nv_bfloat16* dst = blk < 0 ? nullptr : cache + ((size_t)blk * KV_BLOCK + pos % KV_BLOCK) * D.row;
+  const float* ct = A.P.cos_t + (size_t)pos * half;
+  const float* st = A.P.sin_t + (size_t)pos * half;
+  auto finish = [&](int u, int c, float4 v, float rstd) {
+    const bool is_q = u < D.H;
+    const float* wp = (is_q ? A.P.wq : A.P.wk) + (WHOLE ? (is_q ? u : u - D.H) * D.d16 : 0) + c;
+    const float4 w = *reinterpret_cast<const float4*>(wp);
+    v = make_float4(v.x * rstd * w.x, v.y * rstd * w.y, v.z * rstd * w.z, v.w * rstd * w.w);
+    const int p = c / 2;
+    if (p < half) {
+      const float cc = ct[p], ss = st[p], a = v.x;
+      v.x = a * cc - v.y * ss;
+      v.y = v.y * cc + a * ss;
+    }
+    if (p + 1 < half) {
+      const float cc = ct[p + 1], ss = st[p + 1], a = v.z;
+      v.z = a * cc - v.w * ss;
+      v.w = v.w * cc + a * ss;
+    }
+    if (is_q) put_bf16x4(q + ((size_t)b * D.H + u) * D.d16 + c, v);
+    else if (dst) put_bf16x4(dst + (u - D.H) * D.d16 + c, v);
+  };
+  float ssq = 0.f, ssk = 0.f;
+  int local = warp;
+  for (int u = u0; u < heads; u += stride, local += DP_WARPS) {
+    float4 v[DP_MAXC];
+    float ss = 0.f;
+#pragma unroll
+    for (int i = 0; i < DP_MAXC; i++) {
+      const int c = lane * 4 + i * 128;
+      if (c < D.d16) {
+        v[i] = plane_sum4(src + (size_t)u * D.d16 + c, A.splits, A.pstride);
+        ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
+        if constexpr (WHOLE) *reinterpret_cast<float4*>(held + local * D.d16 + c) = v[i];
+      }
+    }
+    if constexpr (WHOLE) {
+      if (u < D.H) ssq += ss; else ssk += ss;
+    } else {
+      const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)D.d + A.P.eps);
+#pragma unroll
+      for (int i = 0; i < DP_MAXC; i++)
+        if (lane * 4 + i * 128 < D.d16) finish(u, lane * 4 + i * 128, v[i], rstd);
+    }
+  }
+  if constexpr (WHOLE) {
+    ssq = block_sum(ssq, red);
+    ssk = block_sum(ssk, red);
+    if (threadIdx.x == 0) { cta_ss[0] = ssq; cta_ss[1] = ssk; }
+  }
+  // values and gates: the first unit of this warp past the heads
+  const int gate_cols = A.gate_kind == GATE_ELEMENT ? D.H * D.v16 : A.gate_kind == GATE_HEAD ? D.H : 0;
+  const int units = heads + D.G + (gate_cols + 127) / 128;
+  const float lam = A.lambda ? *A.lambda : 0.f;
+  int u = u0;
+  if (u < heads) u += (heads - u + stride - 1) / stride * stride;
+  for (; u < units; u += stride) {
+    if (u < heads + D.G) {
+      const int g = u - heads;
+      for (int c = lane * 4; c < D.v16; c += 128) {
+        float4 v = plane_sum4(src + (size_t)heads * D.d16 + g * D.v16 + c, A.splits, A.pstride);
+        const size_t at = (size_t)b * D.G * D.v16 + g * D.v16 + c;
+        if (A.lambda) {
+          const float4 f = *reinterpret_cast<const float4*>(A.vf_in + at);
+          v = make_float4((1.f - lam) * v.x + lam * f.x, (1.f - lam) * v.y + lam * f.y, (1.f - lam) * v.z + lam * f.z, (1.f - lam) * v.w + lam * f.w);
+        } else if (A.vf_out) {
+          *reinterpret_cast<float4*>(A.vf_out + at) = v;
+        }
+        if (dst) put_bf16x4(dst + D.G * D.d16 + g * D.v16 + c, v);
+      }
+    } else {
+      const int c = (u - heads - D.G) * 128 + lane * 4;
+      if (c < gate_cols) {
+        const float4 v = plane_sum4(src + A.gate_col + c, A.splits, A.pstride);      // columns past a head gate's end: readable, not stored
+        const float e[4] = {sigmoid_exact(v.x), sigmoid_exact(v.y), sigmoid_exact(v.z), sigmoid_exact(v.w)};
+        for (int j = 0; j < 4; j++)
+          if (c + j < gate_cols) A.gate[(size_t)b * gate_cols + c + j] = e[j];
+      }
+    }
+  }
+  if constexpr (WHOLE) {
+    cg::cluster_group cluster = cg::this_cluster();
+    cluster.sync();
+    float tq = 0.f, tk = 0.f;
+    for (unsigned r = 0; r < gridDim.x; r++) {
+      const float* p = cluster.map_shared_rank(cta_ss, r);
+      tq += p[0];
+      tk += p[1];
+    }
+    const float rq = 1.f / sqrtf(tq / (float)(D.H * D.d) + A.P.eps), rk = 1.f / sqrtf(tk / (float)(D.G * D.d) + A.P.eps);
+    local = warp;
+    for (int v = u0; v < heads; v += stride, local += DP_WARPS)
+      for (int c = lane * 4; c < D.d16; c += 128) finish(v, c, *reinterpret_cast<const float4*>(held + local * D.d16 + c), v < D.H ? rq : rk);
+    cluster.sync();                                  // nobody leaves while a partner may still read its shared memory
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// decode attention: grid (nsplit, G * head tiles, B), 256 threads. Chunks of 64 visible rows go through a two-stage shared-memory ring (16-byte cp.async; rows an
+// odd number of 16-byte units apart, so the ldmatrix reads are conflict free). Scores: warp w takes eight rows against the 16 heads of the tile; softmax
+// statistics meet in shared memory; output: warp w takes NP * 16 value columns over all 64 rows. ws: [B][G * tiles][split][16][v16 + 4] f32 (accumulators,
+// running maximum in the log2 domain, running sum); counters: [B][G * tiles], zero between launches.
+// ------------------------------------------------------------------------------------------------------------
+constexpr int GD_CHUNK = 64, GD_STAGES = 2, GD_P_PITCH = 144, GD_MAX_SPLIT = 64, GD_HT = 16;
+FT_DEVICE void cp_async16(uint32_t dst, const void* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); }
+FT_DEVICE void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+template <int N>
+FT_DEVICE void cp_async_wait() { asm volatile("cp.async.wait_group %0;" ::"n"(N) : "memory"); }
+FT_DEVICE void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+FT_DEVICE void ldmatrix_x2(uint32_t& r0, uint32_t& r1, uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(r0), "=r"(r1) : "r"(addr));
+}
+FT_DEVICE void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
+  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+FT_DEVICE void mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__host__ __device__ inline int gd_pitch(int d16, int v16) { return (d16 + v16) * 2 + 16; }
+inline int gd_smem(int d16, int v16) {
+  const int p = gd_pitch(d16, v16), ring = GD_HT * p + GD_STAGES * GD_CHUNK * p + GD_HT * GD_P_PITCH, merge = 2 * GD_MAX_SPLIT * GD_HT * 4 + GD_HT * 4;
+  return ring > merge ? ring : merge;
+}
+
+template <int NP>
+__global__ void __launch_bounds__(256) gqa_decode_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache, const int* __restrict__ block_table,
+                                                         int max_blocks, const int* __restrict__ seq_lens, GqaDims D, MaskGate M, int tiles, float* __restrict__ ws,
+                                                         int* __restrict__ counters, __nv_bfloat16* __restrict__ out, int64_t ldo) {
+  pdl_wait();
+  pdl_launch_dependents();
+  extern __shared__ __align__(128) uint8_t smem[];
+  __shared__ float sm_mx[8][GD_HT], sm_l[8][GD_HT];
+  __shared__ int is_last;
+  const int split = blockIdx.x, nsplit = gridDim.x, g = blockIdx.y / tiles, tile = blockIdx.y % tiles, b = blockIdx.z;
+  const int R = D.H / D.G, h0 = g * R + tile * GD_HT, nh = min(GD_HT, R - tile * GD_HT);
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, t2 = (lane & 3) * 2;
+  const int len = seq_lens[b], first = M.window < len ? len - M.window : 0;
+  const int per = ((len - first + nsplit - 1) / nsplit + 15) & ~15;
+  const int t0 = first + split * per, t1 = min(len, t0 + per);
+  const int nchunks = t1 > t0 ? (t1 - t0 + GD_CHUNK - 1) / GD_CHUNK : 0;
+  const int wrow = D.v16 + 4;
+  float* base = ws + ((size_t)b * gridDim.y + blockIdx.y) * nsplit * GD_HT * wrow;
+  float* my_ws = base + (size_t)split * GD_HT * wrow;
+  const int pitch = gd_pitch(D.d16, D.v16), kvecs = D.d16 / 8, vecs = kvecs + D.v16 / 8;
+  const uint32_t sQ = smem_u32(smem), sK = sQ + GD_HT * pitch, sP = sK + GD_STAGES * GD_CHUNK * pitch;
+  const int* bt = block_table + (size_t)b * max_blocks;
+  const float sl2 = M.scale * LOG2E;
+
+  auto load_chunk = [&](int c, int stage) {
+    const int c0 = t0 + c * GD_CHUNK, cnt = min(GD_CHUNK, t1 - c0);
+    const uint32_t dst = sK + stage * GD_CHUNK * pitch;
+    for (int r = warp; r < cnt; r += 8) {
+      const int t = c0 + r;
+      const __nv_bfloat16* src = cache + ((size_t)__ldg(bt + t / KV_BLOCK) * KV_BLOCK + t % KV_BLOCK) * D.row;
+      for (int i = lane; i < vecs; i += 32)
+        cp_async16(dst + r * pitch + i * 16, i < kvecs ? src + g * D.d16 + i * 8 : src + D.G * D.d16 + g * D.v16 + (i - kvecs) * 8);
+    }
+    // rows up to the next multiple of 16 meet weight zero: they must be finite
+    for (int r = cnt + warp; r < ((cnt + 15) & ~15); r += 8)
+      for (int i = lane; i < vecs; i += 32) *reinterpret_cast<uint4*>(smem + (dst - sQ) + r * pitch + i * 16) = make_uint4(0, 0, 0, 0);
+  };
+  if (nchunks > 0) {
+    for (int r = warp; r < GD_HT; r += 8)
+      for (int i = lane; i < kvecs; i += 32) {
+        if (r < nh) cp_async16(sQ + r * pitch + i * 16, q + ((size_t)b * D.H + h0 + r) * D.d16 + i * 8);
+        else *reinterpret_cast<uint4*>(smem + r * pitch + i * 16) = make_uint4(0, 0, 0, 0);
+      }
+#pragma unroll
+    for (int s = 0; s < GD_STAGES; s++) {
+      if (s < nchunks) load_chunk(s, s);
+      cp_async_commit();
+    }
+  }
+  float o[NP][2][4];
+#pragma unroll
+  for (int p = 0; p < NP; p++)
+#pragma unroll
+    for (int e = 0; e < 4; e++) o[p][0][e] = o[p][1][e] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  const int npairs = D.v16 / 16, ksteps = D.d16 / 16;
+  for (int c = 0; c < nchunks; c++) {
+    cp_async_wait<GD_STAGES - 1>();
+    __syncthreads();
+    const int stage = c % GD_STAGES, cnt = min(GD_CHUNK, t1 - (t0 + c * GD_CHUNK));
+    const uint32_t kb = sK + stage * GD_CHUNK * pitch;
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
+    if (warp * 8 < cnt) {
+      const uint32_t krow = kb + (warp * 8 + (lane & 7)) * pitch, qrow = sQ + (lane & 15) * pitch + (lane >> 4) * 16;
+      for (int ks = 0; ks < ksteps; ks++) {
+        uint32_t k0, k1, qa[4];
+        ldmatrix_x2(k0, k1, krow + ks * 32 + ((lane >> 3) & 1) * 16);
+        ldmatrix_x4(qa, qrow + ks * 32);
+        mma_16816(s, qa, k0, k1);
+      }
+    }
+    const bool v0 = warp * 8 + t2 < cnt, v1 = warp * 8 + t2 + 1 < cnt;
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      float a = fmaxf(v0 ? s[2 * e] : -INFINITY, v1 ? s[2 * e + 1] : -INFINITY);
+      a = fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 1));
+      a = fmaxf(a, __shfl_xor_sync(0xffffffffu, a, 2));
+      if ((lane & 3) == 0) sm_mx[warp][gr + 8 * e] = a;
+    }
+    __syncthreads();
+    float alpha[2];
+#pragma unroll
+    for (int e = 0; e < 2; e++) {
+      float mx = m_run[e];
+#pragma unroll
+      for (int w = 0; w < 8; w++) mx = fmaxf(mx, sm_mx[w][gr + 8 * e]);
+      alpha[e] = ex2((m_run[e] - mx) * sl2);                        // 0 on the first chunk
+      m_run[e] = mx;
+      const float p0 = v0 ? ex2((s[2 * e] - mx) * sl2) : 0.f, p1 = v1 ? ex2((s[2 * e + 1] - mx) * sl2) : 0.f;
+      l_run[e] = l_run[e] * alpha[e] + p0 + p1;
+      *reinterpret_cast<__nv_bfloat162*>(smem + (sP - sQ) + (gr + 8 * e) * GD_P_PITCH + (warp * 8 + t2) * 2) = __floats2bfloat162_rn(p0, p1);
+    }
+    __syncthreads();
+    const int psteps = (cnt + 15) / 16;
+#pragma unroll
+    for (int p = 0; p < NP; p++)
+#pragma unroll
+      for (int n = 0; n < 2; n++) {
+        o[p][n][0] *= alpha[0]; o[p][n][1] *= alpha[0];
+        o[p][n][2] *= alpha[1]; o[p][n][3] *= alpha[1];
+      }
+    for (int ps = 0; ps < psteps; ps++) {
+      uint32_t pf[4];
+      ldmatrix_x4(pf, sP + (lane & 15) * GD_P_PITCH + ps * 32 + (lane >> 4) * 16);
+      const uint32_t vrow = kb + (ps * 16 + (lane & 7) + (((lane >> 3) & 1) << 3)) * pitch + D.d16 * 2 + (lane >> 4) * 16;
+#pragma unroll
+      for (int p = 0; p < NP; p++) {
+        const int pr = warp * NP + p;
+        if (pr < npairs) {
+          uint32_t vb[4];
+          ldmatrix_x4_trans(vb, vrow + pr * 32);
+          mma_16816(o[p][0], pf, vb[0], vb[1]);
+          mma_16816(o[p][1], pf, vb[2], vb[3]);
+        }
+      }
+    }
+    __syncthreads();
+    if (c + GD_STAGES < nchunks) load_chunk(c + GD_STAGES, stage);
+    cp_async_commit();
+  }
+  cp_async_wait<0>();
+#pragma unroll
+  for (int e = 0; e < 2; e++) {
+    float l = l_run[e];
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
+    const int hrow = gr + 8 * e;
+    if ((lane & 3) == 0) sm_l[warp][hrow] = l;
+    float* dst = my_ws + (size_t)hrow * wrow;
+    if (nchunks > 0 && hrow < nh) {
+#pragma unroll
+      for (int p = 0; p < NP; p++) {
+        const int pr = warp * NP + p;
+        if (pr < npairs) {
+          *reinterpret_cast<float2*>(dst + pr * 16 + t2) = make_float2(o[p][0][2 * e], o[p][0][2 * e + 1]);
+          *reinterpret_cast<float2*>(dst + pr * 16 + 8 + t2) = make_float2(o[p][1][2 * e], o[p][1][2 * e + 1]);
+        }
+      }
+    }
+    if (warp == 0 && (lane & 3) == 0) dst[D.v16] = nchunks > 0 ? m_run[e] * sl2 : -INFINITY;
+  }
+  __syncthreads();
+  if (threadIdx.x < GD_HT) {
+    float l = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; w++) l += sm_l[w][threadIdx.x];
+    my_ws[(size_t)threadIdx.x * wrow + D.v16 + 1] = l;
+  }
+  __threadfence();
+  __syncthreads();
+  if (threadIdx.x == 0) {
+    int* ctr = counters + (size_t)b * gridDim.y + blockIdx.y;
+    is_last = atomicAdd(ctr, 1) == nsplit - 1;
+    if (is_last) *ctr = 0;
+  }
+  __syncthreads();
+  if (!is_last) return;
+  __threadfence();
+  // merge: weights of the splits and the row sums first, then one pass over the value columns
+  float* fw = reinterpret_cast<float*>(smem);                       // [nsplit][16]
+  float* fl = fw + GD_MAX_SPLIT * GD_HT;
+  float* inv = fl + GD_MAX_SPLIT * GD_HT;                           // [16]
+  for (int i = threadIdx.x; i < nsplit * nh; i += 256) {
+    const int s = i / nh, r = i % nh;
+    const float2 ml = __ldcg(reinterpret_cast<const float2*>(base + ((size_t)s * GD_HT + r) * wrow + D.v16));
+    fw[s * GD_HT + r] = ml.x;
+    fl[s * GD_HT + r] = ml.y;
+  }
+  __syncthreads();
+  if (threadIdx.x < nh) {
+    const int r = threadIdx.x;
+    const float sink = M.sink ? M.sink[h0 + r] * LOG2E : -INFINITY;
+    float mx = sink, l = 0.f;
+    for (int s = 0; s < nsplit; s++) mx = fmaxf(mx, fw[s * GD_HT + r]);
+    if (M.sink) l = ex2(sink - mx);
+    for (int s = 0; s < nsplit; s++) {
+      const float f = fw[s * GD_HT + r] == -INFINITY ? 0.f : ex2(fw[s * GD_HT + r] - mx);
+      l += f * fl[s * GD_HT + r];
+      fw[s * GD_HT + r] = f;
+    }
+    float k = M.out_scale / l;
+    if (M.gate_kind == GATE_HEAD) k *= reinterpret_cast<const float*>(M.gate)[(size_t)b * D.H + h0 + r];
+    inv[r] = k;
+  }
+  __syncthreads();
+  const int vq = D.v16 / 4;
+  for (int i = threadIdx.x; i < nh * vq; i += 256) {
+    const int r = i / vq, c = (i % vq) * 4;
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int s0 = 0; s0 < nsplit; s0 += 8) {
+      float4 v[8];
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+        const bool live = s0 + j < nsplit && fw[min(s0 + j, GD_MAX_SPLIT - 1) * GD_HT + r] > 0.f;    // a split without rows left its accumulators unwritten
+        v[j] = live ? __ldcg(reinterpret_cast<const float4*>(base + ((size_t)(s0 + j) * GD_HT + r) * wrow + c)) : make_float4(0.f, 0.f, 0.f, 0.f);
+      }
+#pragma unroll
+      for (int j = 0; j < 8; j++) {
+        const float w = s0 + j < nsplit ? fw[(s0 + j) * GD_HT + r] : 0.f;
+        a.x += w * v[j].x; a.y += w * v[j].y; a.z += w * v[j].z; a.w += w * v[j].w;
+      }
+    }
+    const float k = inv[r];
+    a = make_float4(a.x * k, a.y * k, a.z * k, a.w * k);
+    if (M.gate_kind == GATE_ELEMENT) {
+      const float4 gt = *reinterpret_cast<const float4*>(reinterpret_cast<const float*>(M.gate) + ((size_t)b * D.H + h0 + r) * D.v16 + c);
+      a = make_float4(a.x * gt.x, a.y * gt.y, a.z * gt.z, a.w * gt.w);
+    }
+    put_bf16x4(out + (size_t)b * ldo + (h0 + r) * D.v16 + c, a);
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// prompt attention (tcgen05): one CTA per (tile of NT sub-tiles of one sequence, key / value head). A sub-tile's 128 rows are `tok` tokens times the R query heads
+// of the group, so a window costs the keys of `tok` tokens more than its size, and a group's heads share every loaded key and value.
+//   warp 0       TMA: the queries' column blocks once, then keys and values, 64 rows at a time (four pages; a lane per page and column block), two-stage rings.
+//                Heads are a tensor-map dimension of their own, so columns past a head's size arrive as zeros; pages past the end are out of bounds: zeros
+//   warp 1       TMEM owner; one lane issues S_t = Q_t K^T for the NT sub-tiles (double buffered) and O_t += P_t V
+//   warps 2..    one thread per row: causal and window mask, online softmax in the log2 domain, P (bf16) through swizzled shared memory
+// ------------------------------------------------------------------------------------------------------------
+constexpr int GF_BM = 128, GF_BN = 64;
+constexpr int GF_QB = GF_BM * 128;         // one 64-column block of 128 query rows
+constexpr int GF_KB = GF_BN * 128;         // one 64-column block of 64 keys
+constexpr int GF_PB = GF_BM * 128;
+constexpr int GF_PAGE = KV_BLOCK * 128;    // one page's share of a key block
+constexpr uint32_t FT_K_GQA = 10;
+
+FT_DEVICE bool gf_wait(uint64_t* bar, uint32_t parity) {
+  if (mbar_try_wait(bar, parity)) return true;
+  const uint64_t t0 = globaltimer_ns();
+  for (uint32_t i = 1;; i++) {
+    if (mbar_try_wait(bar, parity)) return true;
+    if ((i & 0xff) == 0 && globaltimer_ns() - t0 > 2000000000ull) return false;
+  }
+}
+
+struct FlashArgs {
+  GqaDims D;
+  MaskGate M;
+  int R, tok;                      // query heads per key / value head, tokens per sub-tile
+  int nq, nv;                      // 64-column blocks of key and value sizes
+  int max_blocks;
+};
+
+// NQ, NV: column blocks at compile time (the issuing thread's descriptors then are constants added to a base), or 0 to read them from A.
+template <int NT, int NQ, int NV>
+__global__ void __launch_bounds__(64 + 128 * NT, (NT == 1 && NV == 1) ? 2 : 1)
+gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const int4* __restrict__ tiles,
+                 const int* __restrict__ block_table, FlashArgs A, __nv_bfloat16* __restrict__ out, int64_t ldo, uint32_t* status) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  const int nq = NQ > 0 ? NQ : A.nq, nv = NV > 0 ? NV : A.nv;
+  const int k_bytes = nq * GF_KB, v_bytes = nv * GF_KB;
+  uint8_t* sQ = smem;                               // [NT][nq]
+  uint8_t* sK = sQ + NT * nq * GF_QB;               // [2][nq]
+  uint8_t* sV = sK + 2 * k_bytes;                   // [2][nv]
+  uint8_t* sP = sV + 2 * v_bytes;                   // [NT]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(sP + NT * GF_PB);
+  uint64_t* q_full = bars;
+  uint64_t* k_full = bars + 1;                      // [2]
+  uint64_t* k_empty = bars + 3;
+  uint64_t* v_full = bars + 5;
+  uint64_t* v_empty = bars + 7;
+  uint64_t* s_full = bars + 9;                      // [NT][2]
+  uint64_t* p_ready = bars + 9 + 2 * NT;            // [NT]
+  uint64_t* pv_done = bars + 9 + 3 * NT;            // [NT]
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 9 + 4 * NT);
+
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int4 tl = tiles[blockIdx.x];                // first query row, tokens, position of the first token, sequence
+  const int g = blockIdx.y, tok = A.tok, window = A.M.window;
+  // key blocks [j0, j0 + nblk[t]) of every sub-tile; the start is the window of the tile's first token
+  const int j0 = (tl.z - window >= 0 ? tl.z - window + 1 : 0) / GF_BN;
+  int nblk[NT], nmax = 0;
+#pragma unroll
+  for (int t = 0; t < NT; t++) {
+    const int n = min(tok, tl.y - t * tok);
+    nblk[t] = n > 0 ? (tl.z + t * tok + n + GF_BN - 1) / GF_BN - j0 : 0;
+    nmax = max(nmax, nblk[t]);
+  }
+  if (threadIdx.x == 0) {
+    mbar_init(q_full, 1);
+    for (int i = 0; i < 2; i++) { mbar_init(&k_full[i], 1); mbar_init(&k_empty[i], 1); mbar_init(&v_full[i], 1); mbar_init(&v_empty[i], 1); }
+    for (int t = 0; t < NT; t++) { mbar_init(&s_full[2 * t], 1); mbar_init(&s_full[2 * t + 1], 1); mbar_init(&p_ready[t], 128); mbar_init(&pv_done[t], 1); }
+    mbar_fence_init();
+  }
+  if (warp == 0 && lane == 0) { tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV); }
+  constexpr uint32_t TMEM = (NT == 1 && NV == 1) ? 256 : 512;       // small heads leave room for a second CTA
+  if (warp == 1) { tmem_alloc(tmem_slot, TMEM); tmem_relinquish(); }
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tS = *tmem_slot, tO = tS + NT * 2 * GF_BN;
+
+  if (warp == 0) {
+    if (lane == 0) {
+      int live = 0;
+      for (int t = 0; t < NT; t++) live += nblk[t] > 0;
+      mbar_expect_tx(q_full, live * nq * A.R * tok * 128);
+      for (int t = 0; t < NT; t++)
+        if (nblk[t] > 0)
+          for (int c = 0; c < nq; c++) tma_load_3d(sQ + (t * nq + c) * GF_QB, &tmQ, q_full, c * 64, g * A.R, tl.x + t * tok);
+    }
+    __syncwarp();
+    const int* bt = block_table + (size_t)tl.w * A.max_blocks;
+    const int pg = lane & 3, cb = lane >> 2;        // this lane's page of a key block, and its first column block
+    auto page_row = [&](int j) -> int {             // first row of that page in the cache, out of bounds past the sequence's pages
+      const int p = (j0 + j) * 4 + pg;
+      const int blk = p < A.max_blocks ? __ldg(bt + p) : -1;
+      return blk * KV_BLOCK;                        // -1: a negative coordinate, read as zeros
+    };
+    auto load_k = [&](int j, int y) -> bool {
+      const int s = j & 1;
+      const bool free_k = gf_wait(&k_empty[s], ((j >> 1) & 1) ^ 1);
+      if (!__all_sync(0xffffffffu, free_k)) { if (lane == 0) ft_set_status(status, FT_K_GQA, 1, j); return false; }   // the whole warp at once
+      if (lane == 0) mbar_expect_tx(&k_full[s], k_bytes);
+      __syncwarp();
+      for (int c = cb; c < nq; c += 8) tma_load_3d(sK + s * k_bytes + c * GF_KB + pg * GF_PAGE, &tmK, &k_full[s], c * 64, g, y);
+      return true;
+    };
+    int y = nmax > 0 ? page_row(0) : 0;
+    bool ok = nmax > 0 && load_k(0, y);
+    for (int j = 0; j < nmax && ok; j++) {
+      const int y_next = j + 1 < nmax ? page_row(j + 1) : 0;
+      if (j + 1 < nmax) ok = load_k(j + 1, y_next);
+      if (!ok) break;
+      const int s = j & 1;
+      const bool free_v = gf_wait(&v_empty[s], ((j >> 1) & 1) ^ 1);
+      if (!__all_sync(0xffffffffu, free_v)) { if (lane == 0) ft_set_status(status, FT_K_GQA, 2, j); ok = false; break; }
+      if (lane == 0) mbar_expect_tx(&v_full[s], v_bytes);
+      __syncwarp();
+      for (int c = cb; c < nv; c += 8) tma_load_3d(sV + s * v_bytes + c * GF_KB + pg * GF_PAGE, &tmV, &v_full[s], c * 64, g, y);
+      y = y_next;
+    }
+    if (!ok)
+      for (int i = 0; i < 64; i++) __nanosleep(1000);      // copies in flight land before the shared memory goes away
+  } else if (warp == 1) {
+    if (lane == 0) {
+      const uint32_t idesc_s = make_idesc_f16(GF_BM, GF_BN, 1, 0, 0);
+      const uint32_t idesc_o = make_idesc_f16(GF_BM, nv * 64, 1, 0, 1);
+      // a descriptor's start address counts 16-byte units in its low bits: moving inside the operand is an addition
+      const uint64_t q_desc = make_smem_desc(smem_u32(sQ), 16, 1024, FT_SWZ_128B), k_desc = make_smem_desc(smem_u32(sK), 16, 1024, FT_SWZ_128B);
+      const uint64_t p_desc = make_smem_desc(smem_u32(sP), 16, 1024, FT_SWZ_128B), v_desc = make_smem_desc(smem_u32(sV), GF_KB, 1024, FT_SWZ_128B);
+      auto issue_s = [&](int t, int j) {
+        const uint64_t qd = q_desc + (uint32_t)(t * nq) * (GF_QB / 16), kd = k_desc + (uint32_t)(j & 1) * (k_bytes / 16);
+        const uint32_t d = tS + t * 2 * GF_BN + (j & 1) * GF_BN;
+#pragma unroll
+        for (int c = 0; c < nq; c++) {
+#pragma unroll
+          for (int k = 0; k < 4; k++) umma_f16_ss(d, qd + c * (GF_QB / 16) + k * 2, kd + c * (GF_KB / 16) + k * 2, idesc_s, (c | k) != 0);
+        }
+        umma_commit(&s_full[2 * t + (j & 1)]);
+      };
+      bool ok = gf_wait(q_full, 0) && gf_wait(&k_full[0], 0);
+      if (!ok) ft_set_status(status, FT_K_GQA, 3, 0);
+      if (ok) {
+        tc_fence_after();
+#pragma unroll
+        for (int t = 0; t < NT; t++)
+          if (nblk[t] > 0) issue_s(t, 0);
+        umma_commit(&k_empty[0]);
+        for (int j = 0; j < nmax && ok; j++) {
+          if (j + 1 < nmax) {
+            if (!gf_wait(&k_full[(j + 1) & 1], ((j + 1) >> 1) & 1)) { ft_set_status(status, FT_K_GQA, 4, j); break; }
+            tc_fence_after();
+#pragma unroll
+            for (int t = 0; t < NT; t++)
+              if (j + 1 < nblk[t]) issue_s(t, j + 1);
+            umma_commit(&k_empty[(j + 1) & 1]);
+          }
+          if (!gf_wait(&v_full[j & 1], (j >> 1) & 1)) { ft_set_status(status, FT_K_GQA, 5, j); break; }
+          const uint64_t vd = v_desc + (uint32_t)(j & 1) * (v_bytes / 16);
+#pragma unroll
+          for (int t = 0; t < NT; t++) {
+            if (j >= nblk[t] || !ok) continue;
+            if (!gf_wait(&p_ready[t], j & 1)) { ft_set_status(status, FT_K_GQA, 6, j); ok = false; continue; }
+            tc_fence_after();
+#pragma unroll
+            for (int k = 0; k < GF_BN / 16; k++)
+              umma_f16_ss(tO + t * nv * 64, p_desc + t * (GF_PB / 16) + k * 2, vd + k * 128, idesc_o, (j | k) != 0);
+            umma_commit(&pv_done[t]);
+          }
+          umma_commit(&v_empty[j & 1]);
+        }
+      }
+    }
+  } else {
+    const int t = (warp - 2) >> 2, q = warp & 3, r = q * 32 + lane;
+    const int nb = t == 0 ? nblk[0] : nblk[NT - 1];
+    const int tk = r / A.R, head = g * A.R + r % A.R;      // token inside the sub-tile, query head
+    const bool live = tk < tok && t * tok + tk < tl.y;
+    const int qpos = tl.z + t * tok + tk;
+    const int lo_pos = tl.z + t * tok, hi_pos = tl.z + min(tl.y, (t + 1) * tok) - 1;      // positions of the sub-tile
+    const int wlow = qpos - window;                        // the last position that has left this row's window (far below zero without one)
+    const float scale_log2 = A.M.scale * LOG2E;
+    const uint32_t lane_off = (uint32_t)(q * 32) << 16;
+    uint8_t* prow = sP + t * GF_PB + r * 128;
+    float m_used = -INFINITY, l = 0.f;
+    bool ok = true;
+    for (int j = 0; j < nb && ok; j++) {
+      if (!gf_wait(&s_full[2 * t + (j & 1)], (j >> 1) & 1)) { if (lane == 0) ft_set_status(status, FT_K_GQA, 7, j); ok = false; break; }
+      tc_fence_after();
+      __syncwarp();                                            // the TMEM loads are warp-wide: every lane is here
+      uint32_t sv[64];
+      tmem_ld_32x32b_x32(tS + lane_off + t * 2 * GF_BN + (j & 1) * GF_BN, sv);
+      tmem_ld_32x32b_x32(tS + lane_off + t * 2 * GF_BN + (j & 1) * GF_BN + 32, sv + 32);
+      tmem_ld_wait();
+      const int kv0 = (j0 + j) * GF_BN;
+      if (kv0 + GF_BN - 1 > lo_pos || kv0 <= hi_pos - window) {   // the diagonal or the window's edge can cross this block
+#pragma unroll
+        for (int c = 0; c < 64; c++)
+          if (kv0 + c > qpos || kv0 + c <= wlow) sv[c] = __float_as_uint(-INFINITY);
+      }
+      float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
+#pragma unroll
+      for (int c = 0; c < 64; c++) mx4[c & 3] = fmaxf(mx4[c & 3], __uint_as_float(sv[c]));
+      const float m_new = fmaxf(m_used, fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])));
+      // a row that has seen no key yet (all of them outside its window) stays at minus infinity with weights zero
+      const bool grow = m_new != -INFINITY && (m_new - m_used) * scale_log2 > 8.f;
+      const bool rescale = __any_sync(0xffffffffu, grow);
+      float alpha = 1.f;
+      if (rescale && m_new != -INFINITY) {
+        alpha = ex2((m_used - m_new) * scale_log2);
+        m_used = m_new;
+      }
+      const float moff = m_used == -INFINITY ? 0.f : m_used * scale_log2;
+      float rs4[4] = {0.f, 0.f, 0.f, 0.f};
+      uint32_t pk[32];
+#pragma unroll
+      for (int c = 0; c < 32; c++) {
+        const float p0 = ex2(fmaf(__uint_as_float(sv[2 * c]), scale_log2, -moff));
+        const float p1 = ex2(fmaf(__uint_as_float(sv[2 * c + 1]), scale_log2, -moff));
+        rs4[c & 3] += p0 + p1;
+        __nv_bfloat162 hh = __floats2bfloat162_rn(p0, p1);
+        pk[c] = *reinterpret_cast<uint32_t*>(&hh);
+      }
+      l = l * alpha + ((rs4[0] + rs4[1]) + (rs4[2] + rs4[3]));
+      if (j > 0) {
+        if (!gf_wait(&pv_done[t], (j - 1) & 1)) { if (lane == 0) ft_set_status(status, FT_K_GQA, 8, j); ok = false; break; }
+        tc_fence_after();
+        __syncwarp();
+        if (rescale) {
+#pragma unroll 1
+          for (int c = 0; c < nv * 2; c++) {
+            uint32_t ov[32];
+            const uint32_t addr = tO + lane_off + t * nv * 64 + c * 32;
+            tmem_ld_32x32b_x32(addr, ov);
+            tmem_ld_wait();
+#pragma unroll
+            for (int e = 0; e < 32; e++) ov[e] = __float_as_uint(__uint_as_float(ov[e]) * alpha);
+            tmem_st_32x32b_x32(addr, ov);
+          }
+          tmem_st_wait();
+        }
+      }
+#pragma unroll
+      for (int c8 = 0; c8 < 8; c8++)
+        *reinterpret_cast<uint4*>(prow + ((c8 ^ (r & 7)) << 4)) = make_uint4(pk[4 * c8], pk[4 * c8 + 1], pk[4 * c8 + 2], pk[4 * c8 + 3]);
+      fence_proxy_async_smem();
+      tc_fence_before();
+      mbar_arrive(&p_ready[t]);
+    }
+    if (ok && nb > 0) {
+      if (!gf_wait(&pv_done[t], (nb - 1) & 1)) { if (lane == 0) ft_set_status(status, FT_K_GQA, 9, 0); ok = false; }
+    }
+    if (ok && nb > 0) {
+      tc_fence_after();
+      const size_t row = (size_t)(tl.x + t * tok + tk);
+      if (A.M.sink != nullptr && live) l += ex2(A.M.sink[head] * LOG2E - m_used * scale_log2);
+      float k = A.M.out_scale / l;
+      if (A.M.gate_kind == GATE_HEAD && live) k *= sigmoid_fast(reinterpret_cast<const float*>(A.M.gate)[row * A.M.ldg + head]);
+      __nv_bfloat16* dst = out + row * ldo + (size_t)head * A.D.v16;
+      const __nv_bfloat16* gate = reinterpret_cast<const __nv_bfloat16*>(A.M.gate) + row * A.M.ldg + (size_t)head * A.D.v16;
+      const bool gated = A.M.gate_kind == GATE_ELEMENT;
+      // rows outside the tile only skip the loads and stores: the warp-wide TMEM loads stay in code that all lanes run together
+#pragma unroll 1
+      for (int c = 0; c < nv * 2; c++) {
+        uint32_t ov[32];
+        __syncwarp();
+        tmem_ld_32x32b_x32(tO + lane_off + t * nv * 64 + c * 32, ov);
+        tmem_ld_wait();
+#pragma unroll
+        for (int c8 = 0; c8 < 4; c8++) {
+          if (live && c * 32 + c8 * 8 < A.D.v16) {
+            float e[8];
+#pragma unroll
+            for (int i = 0; i < 8; i++) e[i] = __uint_as_float(ov[8 * c8 + i]) * k;
+            if (gated) {
+              float gv[8];
+              load8(gate + c * 32 + c8 * 8, gv);
+#pragma unroll
+              for (int i = 0; i < 8; i++) e[i] *= sigmoid_fast(gv[i]);
+            }
+            store8(dst + c * 32 + c8 * 8, e);
+          }
+        }
+        __syncwarp();
+      }
+    }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tS, TMEM);
+  }
+}
+
+constexpr int SMEM_MAX = 232448;
+int flash_smem(int NT, int nq, int nv) { return NT * nq * GF_QB + 2 * (nq + nv) * GF_KB + NT * GF_PB + 256 + 1024; }
+
+bool make_dims(GqaDims& D, int H, int G, int d, int dv, int rot) {
+  if (G < 1 || H < G || H % G || H > 65535 || d < 1 || dv < 1 || rot < 0 || rot > d || (rot & 1)) return false;
+  D = GqaDims{H, G, d, dv, (d + 15) & ~15, (dv + 15) & ~15, rot, 0};
+  D.row = G * (D.d16 + D.v16);
+  return true;
+}
+MaskGate make_mask(float scale, int window, const float* sink, const void* gate, int64_t ldg, int kind, float out_scale) {
+  return MaskGate{scale, window > 0 ? window : 0x3fffffff, sink, gate, ldg, kind, out_scale};
+}
+
+template <int NT, int NQ, int NV>
+int launch_flash(const CUtensorMap (&m)[3], const int* tiles, int ntiles, const int* bt, const FlashArgs& A, void* out, int64_t ldo, int smem, cudaStream_t st) {
+  static bool done[64] = {};
+  int dev = 0;
+  FT_CUDA_TRY(cudaGetDevice(&dev));
+  if (dev < 64 && !done[dev]) {
+    FT_CUDA_TRY(cudaFuncSetAttribute(gqa_flash_kernel<NT, NQ, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX));
+    done[dev] = true;
+  }
+  gqa_flash_kernel<NT, NQ, NV><<<dim3(ntiles, A.D.G), 64 + 128 * NT, smem, st>>>(m[0], m[1], m[2], reinterpret_cast<const int4*>(tiles), bt, A, (__nv_bfloat16*)out, ldo,
+                                                                                 ft_status_ptr());
+  return (int)cudaGetLastError();
+}
+
+template <int NP>
+int launch_decode(dim3 grid, int smem, cudaStream_t st, const void* q, const void* cache, const int* bt, int mb, const int* lens, const GqaDims& D, const MaskGate& M,
+                  int tiles, float* ws, int* counters, void* out, int64_t ldo) {
+  static bool done[64] = {};
+  int dev = 0;
+  FT_CUDA_TRY(cudaGetDevice(&dev));
+  if (dev < 64 && !done[dev]) {
+    FT_CUDA_TRY(cudaFuncSetAttribute(gqa_decode_kernel<NP>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX - 8192));
+    done[dev] = true;
+  }
+  return (int)ft_launch_pdl(gqa_decode_kernel<NP>, grid, dim3(256), (size_t)smem, st, (const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, bt, mb, lens, D, M, tiles, ws,
+                            counters, (__nv_bfloat16*)out, ldo);
+}
+
+}  // namespace
+
+// Projection rows qkv [rows][ld] (bf16, or f32 with is_f32): H query heads, G key heads (d padded to d16 = a multiple of 16 columns each), G value heads (dv
+// padded to v16). Norms queries and keys (RMS over each head, or with whole != 0 over all query and all key heads; wq, wk f32 in the same padding, one head long or
+// all heads long), turns the first `rot` dimensions of each (pairs of neighbouring columns, tables cos / sin f32 [position][rot / 2]), leaves the queries in
+// place and writes keys and values to cache row slots[r] (= page * 16 + offset): [G x d16 | G x v16]. With lambda (one f32 on the device) the values become
+// (1 - lambda) v + lambda vfirst (rows of G * v16, pitch ldf).
+FT_EXPORT int ft_gqa_prep(void* qkv, int64_t ld, int rows, int H, int G, int d, int dv, int rot, int whole, const float* wq, const float* wk, float eps, const int* positions,
+                          const float* cos_t, const float* sin_t, const int* slots, void* cache, const void* vfirst, int64_t ldf, const float* lambda, int is_f32,
+                          cudaStream_t st) {
+  PrepArgs A{};
+  if (rows < 1 || !make_dims(A.D, H, G, d, dv, rot) || (ld & 7) || ld < (int64_t)(H + G) * A.D.d16 + G * A.D.v16 || (lambda && (!vfirst || (ldf & 7)))) return FT_ERR_ARG;
+  A.wq = wq; A.wk = wk; A.eps = eps; A.positions = positions; A.cos_t = cos_t; A.sin_t = sin_t; A.slots = slots;
+#define FT_GP(T, W) gqa_prep_kernel<T, W><<<rows, PREP_T, 0, st>>>((T*)qkv, ld, A, (T*)cache, (const T*)vfirst, ldf, lambda)
+  if (is_f32) { if (whole) FT_GP(float, true); else FT_GP(float, false); }
+  else { if (whole) FT_GP(__nv_bfloat16, true); else FT_GP(__nv_bfloat16, false); }
+#undef FT_GP
+  return (int)cudaGetLastError();
+}
+
+// Plain attention over cached rows: q [rows][ldq] as left by ft_gqa_prep; row r of sequence seq_of[r] sees the last `window` (0: all) of the positions
+// 0..positions[r]; sink f32 [H] or null; gate_kind 0: none, 1: rows of H * v16 pre-activations in the data type (pitch ldg), 2: f32 rows of H; out [rows][ldo], heads of
+// v16, times out_scale. Value sizes up to 1024.
+FT_EXPORT int ft_gqa_rows(const void* q, int64_t ldq, const void* cache, const int* block_table, int max_blocks, const int* seq_of, const int* positions, int rows, int H, int G,
+                          int d, int dv, float scale, int window, const float* sink, const void* gate, int64_t ldg, int gate_kind, float out_scale, void* out, int64_t ldo,
+                          int is_f32, cudaStream_t st) {
+  GqaDims D;
+  if (rows < 1 || !make_dims(D, H, G, d, dv, 0) || (gate_kind && !gate)) return FT_ERR_ARG;
+  if (D.v16 > 128 * ROWS_MAX_COLS || D.d16 > 8192) return FT_ERR_TOO_LARGE;
+  const MaskGate M = make_mask(scale, window, sink, gate, ldg, gate_kind, out_scale);
+  const dim3 grid(rows, H);
+  if (is_f32) gqa_rows_kernel<float><<<grid, 128, D.d16 * 4, st>>>((const float*)q, ldq, (const float*)cache, block_table, max_blocks, seq_of, positions, D, M, (float*)out, ldo);
+  else gqa_rows_kernel<__nv_bfloat16><<<grid, 128, D.d16 * 4, st>>>((const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)cache, block_table, max_blocks, seq_of, positions, D, M,
+                                                                   (__nv_bfloat16*)out, ldo);
+  return (int)cudaGetLastError();
+}
+
+// ft_gqa_prep for one token of B <= 16 sequences, from split-K planes of the projection (columns as there; gate pre-activations from column gate_col on, kind as in
+// ft_gqa_rows): queries q bf16 [B][H][d16], cache row of each sequence's current position, sigmoid of the gate (f32 [B][H * v16] or [B][H]). vf_out (f32
+// [B][G * v16]) keeps the values; vf_in and lambda mix such values in. Head sizes up to 512.
+FT_EXPORT int ft_gqa_decode_prep(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int B, int H, int G, int d, int dv, int rot, int whole, const float* wq,
+                                 const float* wk, float eps, const int* positions, const float* cos_t, const float* sin_t, const int* block_table, int max_blocks,
+                                 int gate_col, int gate_kind, float* gate, float* vf_out, const float* vf_in, const float* lambda, void* q, void* cache, cudaStream_t st) {
+  DecPrepArgs A{};
+  GqaDims& D = A.P.D;
+  if (B < 1 || B > DEC_TOK || splits < 1 || !make_dims(D, H, G, d, dv, rot) || (ldp & 3) || (plane_stride & 3) || (gate_col & 3) || (gate_kind && !gate) ||
+      (lambda && !vf_in))
+    return FT_ERR_ARG;
+  if (D.d16 > 128 * DP_MAXC) return FT_ERR_TOO_LARGE;
+  A.P.wq = wq; A.P.wk = wk; A.P.eps = eps; A.P.positions = positions; A.P.cos_t = cos_t; A.P.sin_t = sin_t;
+  A.planes = planes; A.splits = splits; A.ldp = ldp; A.pstride = (size_t)plane_stride; A.block_table = block_table; A.max_blocks = max_blocks;
+  A.gate_col = gate_col; A.gate_kind = gate_kind; A.gate = gate; A.vf_out = vf_out; A.vf_in = vf_in; A.lambda = lambda;
+  const int gate_cols = gate_kind == GATE_ELEMENT ? H * D.v16 : gate_kind == GATE_HEAD ? H : 0;
+  const int units = H + 2 * G + (gate_cols + 127) / 128;
+  int ctas = (units + DP_WARPS - 1) / DP_WARPS;
+  if (!whole)
+    return (int)ft_launch_pdl(gqa_decode_prep_kernel<false>, dim3(ctas, B), dim3(DP_WARPS * 32), 0, st, A, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
+  int cl = 1;
+  while (cl < 8 && cl < ctas) cl *= 2;
+  ctas = cl;
+  const size_t smem = (size_t)((H + G + ctas * DP_WARPS - 1) / (ctas * DP_WARPS)) * DP_WARPS * D.d16 * 4;
+  if (smem > (size_t)SMEM_MAX - 1024) return FT_ERR_TOO_LARGE;
+  if (smem > 48 * 1024) FT_CUDA_TRY(cudaFuncSetAttribute(gqa_decode_prep_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX - 1024));
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(ctas, B);
+  cfg.blockDim = dim3(DP_WARPS * 32);
+  cfg.dynamicSmemBytes = smem;
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = ctas;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = ft_pdl_enabled() ? 2 : 1;
+  return (int)cudaLaunchKernelEx(&cfg, gqa_decode_prep_kernel<true>, A, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
+}
+
+// Attention of one token per sequence over its visible cached rows (seq_lens[b] rows, the newest included, or the last `window` of them); q and gate as written by
+// ft_gqa_decode_prep. ws: f32 [B][G * ceil(H / G / 16)][nsplit][16][v16 + 4], 16-byte aligned; counters: int [B][G * ceil(H / G / 16)], zero before the first
+// launch (the kernel leaves them zero). nsplit <= 64; value sizes up to 512. out: bf16 [B][ldo], heads of v16.
+FT_EXPORT int ft_gqa_decode(const void* q, const void* cache, const int* block_table, int max_blocks, const int* seq_lens, int B, int H, int G, int d, int dv, float scale,
+                            int window, const float* sink, const float* gate, int gate_kind, float out_scale, int nsplit, float* ws, int* counters, void* out, int64_t ldo,
+                            cudaStream_t st) {
+  GqaDims D;
+  if (B < 1 || nsplit < 1 || nsplit > GD_MAX_SPLIT || !make_dims(D, H, G, d, dv, 0) || (reinterpret_cast<uintptr_t>(ws) & 15) || (ldo & 3) || (gate_kind && !gate)) return FT_ERR_ARG;
+  const MaskGate M = make_mask(scale, window, sink, gate, 0, gate_kind, out_scale);
+  const int smem = gd_smem(D.d16, D.v16), np = (D.v16 / 16 + 7) / 8, tiles = (H / G + GD_HT - 1) / GD_HT;
+  if (smem > SMEM_MAX - 8192 || np > 4) return FT_ERR_TOO_LARGE;
+  const dim3 grid(nsplit, G * tiles, B);
+#define FT_GD(N) return launch_decode<N>(grid, smem, st, q, cache, block_table, max_blocks, seq_lens, D, M, tiles, ws, counters, out, ldo)
+  if (np <= 1) FT_GD(1);
+  if (np <= 2) FT_GD(2);
+  FT_GD(4);
+#undef FT_GD
+}
+
+// Whether ft_gqa_decode_prep and ft_gqa_decode take these sizes.
+FT_EXPORT int ft_gqa_decode_fits(int H, int G, int d, int dv) {
+  GqaDims D;
+  return make_dims(D, H, G, d, dv, 0) && D.d16 <= 128 * DP_MAXC && D.v16 <= 512 && gd_smem(D.d16, D.v16) <= SMEM_MAX - 8192 &&
+         (size_t)((H + G + 63) / 64) * DP_WARPS * D.d16 * 4 <= (size_t)SMEM_MAX - 1024;
+}
+
+// Sub-tiles (of 128 / (H / G) tokens each) per tile of ft_gqa_flash: 1 or 2; 0 when these sizes do not fit the kernel (use ft_gqa_rows).
+FT_EXPORT int ft_gqa_flash_subtiles(int H, int G, int d, int dv) {
+  GqaDims D;
+  if (!make_dims(D, H, G, d, dv, 0) || H / G > GF_BM) return 0;
+  const int nq = (d + 63) / 64, nv = (dv + 63) / 64;
+  if (nq <= 2 && nv == 1) return 1;                    // two CTAs of one sub-tile per SM
+  if (nv <= 2 && flash_smem(2, nq, nv) <= SMEM_MAX) return 2;
+  if (nv <= 4 && flash_smem(1, nq, nv) <= SMEM_MAX) return 1;
+  return 0;
+}
+
+// Attention of a ragged batch of prompts or portions: q bf16 [q_rows][ldq] as left by ft_gqa_prep; keys and values from the cache's pages [pages][16][row] (those
+// of the new tokens included). tiles: int4 per tile {first query row, tokens (<= subtiles * (128 / (H / G))), position of the first token, row of block_table}.
+// Mask, sink, gate and output as in ft_gqa_rows. Leading dimensions are multiples of 8.
+FT_EXPORT int ft_gqa_flash(const void* q, int64_t ldq, int q_rows, const void* cache, int pages, const int* block_table, int max_blocks, const int* tiles, int ntiles, int H,
+                           int G, int d, int dv, float scale, int window, const float* sink, const void* gate, int64_t ldg, int gate_kind, float out_scale, void* out,
+                           int64_t ldo, cudaStream_t st) {
+  FlashArgs A{};
+  GqaDims& D = A.D;
+  if (q_rows < 1 || pages < 1 || ntiles < 1 || !make_dims(D, H, G, d, dv, 0) || (ldq & 7) || (ldo & 7) || (gate_kind && !gate) || (gate_kind == GATE_ELEMENT && (ldg & 7)))
+    return FT_ERR_ARG;
+  const int nt = ft_gqa_flash_subtiles(H, G, d, dv);
+  if (nt == 0) return FT_ERR_TOO_LARGE;
+  int dev = 0;
+  FT_CUDA_TRY(cudaGetDevice(&dev));
+  FT_CUDA_TRY(ft_bind_context(dev));
+  A.M = make_mask(scale, window, sink, gate, ldg, gate_kind, out_scale);
+  A.R = H / G;
+  A.tok = GF_BM / A.R;
+  A.nq = (d + 63) / 64;
+  A.nv = (dv + 63) / 64;
+  A.max_blocks = max_blocks;
+  CUtensorMap m[3];
+  const __nv_bfloat16* cp = (const __nv_bfloat16*)cache;
+  const uint64_t krow = (uint64_t)D.row * 2, slots = (uint64_t)pages * KV_BLOCK;
+  int r = ft_make_tmap_3d(&m[0], q, 2, true, D.d16, H, q_rows, (uint64_t)D.d16 * 2, (uint64_t)ldq * 2, 64, A.R, A.tok, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!r) r = ft_make_tmap_3d(&m[1], cp, 2, true, D.d16, G, slots, (uint64_t)D.d16 * 2, krow, 64, 1, KV_BLOCK, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!r) r = ft_make_tmap_3d(&m[2], cp + (size_t)G * D.d16, 2, true, D.v16, G, slots, (uint64_t)D.v16 * 2, krow, 64, 1, KV_BLOCK, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (r) return r;
+  const int smem = flash_smem(nt, A.nq, A.nv);
+#define FT_GF(T, Q, V) return launch_flash<T, Q, V>(m, tiles, ntiles, block_table, A, out, ldo, smem, st)
+  if (nt == 2) {
+    if (A.nq == 2 && A.nv == 2) FT_GF(2, 2, 2);
+    FT_GF(2, 0, 0);
+  }
+  if (A.nq == 1 && A.nv == 1) FT_GF(1, 1, 1);
+  if (A.nq == 2 && A.nv == 1) FT_GF(1, 2, 1);
+  FT_GF(1, 0, 0);
+#undef FT_GF
+}

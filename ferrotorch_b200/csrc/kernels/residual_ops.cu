@@ -1,0 +1,290 @@
+// One f32 residual per token with the norm on the sublayer's output, and the activation of a gated feed-forward.
+//
+//   ft_residual_embed    x = scale * table[id];  h = x in the operand type
+//   ft_residual_update   y = sum of the sublayer's f32 planes;  x += y / rms(y) * w;  h = x, or x / rms(x) * w_last ahead of the output projection
+//   ft_gated_act         act(gate) * up of interleaved gate / up columns, from a 16-bit or f32 matrix or from split-K planes
+//
+// ft_residual_update takes one row per cluster of CTAs: one CTA where there are rows enough to fill the GPU, up to eight (sums of squares meet in
+// distributed shared memory) for the few rows of a decode step, whose planes are then read by eight SMs instead of one. Everything a row needs stays in
+// registers between its two norms. Compiled without fast-math.
+#include <cooperative_groups.h>
+
+#include "common.cuh"
+#include "host_common.h"
+
+namespace {
+
+template <typename H> FT_DEVICE void put4(H* dst, float4 v);
+template <> FT_DEVICE void put4<float>(float* dst, float4 v) { *reinterpret_cast<float4*>(dst) = v; }
+template <> FT_DEVICE void put4<__nv_bfloat16>(__nv_bfloat16* dst, float4 v) {
+  __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  uint2 pk;
+  pk.x = *reinterpret_cast<uint32_t*>(&a);
+  pk.y = *reinterpret_cast<uint32_t*>(&b);
+  *reinterpret_cast<uint2*>(dst) = pk;
+}
+template <typename H> FT_DEVICE float4 get4(const H* src);
+template <> FT_DEVICE float4 get4<float>(const float* src) { return *reinterpret_cast<const float4*>(src); }
+template <> FT_DEVICE float4 get4<__nv_bfloat16>(const __nv_bfloat16* src) {
+  const uint2 r = *reinterpret_cast<const uint2*>(src);
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+FT_DEVICE float sq4(float4 v) { return v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w; }
+// elements past the row's width: padding of the buffers, of unknown content
+FT_DEVICE float4 keep4(float4 v, int c, int W) {
+  if (c + 1 > W) v.x = 0.f;
+  if (c + 2 > W) v.y = 0.f;
+  if (c + 3 > W) v.z = 0.f;
+  if (c + 4 > W) v.w = 0.f;
+  return v;
+}
+
+template <typename H>
+__global__ void __launch_bounds__(256) residual_embed_kernel(const int64_t* __restrict__ ids, const H* __restrict__ table, int64_t ld_table, int64_t vocab, float scale,
+                                                             float* __restrict__ x, int64_t ldx, H* __restrict__ h, int64_t ldh, int rows, int W) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int c = (blockIdx.x * 256 + threadIdx.x) * 4;
+  if (c >= W) return;
+  for (int r = blockIdx.y; r < rows; r += gridDim.y) {
+    const int64_t id = ids[r];
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (id >= 0 && id < vocab) v = keep4(get4(table + (size_t)id * ld_table + c), c, W);
+    v = make_float4(v.x * scale, v.y * scale, v.z * scale, v.w * scale);
+    *reinterpret_cast<float4*>(x + (size_t)r * ldx + c) = v;
+    put4(h + (size_t)r * ldh + c, v);
+  }
+}
+
+constexpr int UPD_THREADS = 256;
+// NV: float4 columns per thread
+template <int NV, typename H>
+__global__ void __launch_bounds__(UPD_THREADS) residual_update_kernel(float* __restrict__ x, int64_t ldx, const float* __restrict__ y, int planes, size_t pstride, int64_t ldy,
+                                                                      const float* __restrict__ w, const float* __restrict__ w_last, float eps, H* __restrict__ h,
+                                                                      int64_t ldh, int ncta, int W, int cols, int store_x) {
+  namespace cg = cooperative_groups;
+  __shared__ float red[32];
+  __shared__ float cta_ss[2];
+  cg::cluster_group cluster = cg::this_cluster();
+  const int row = blockIdx.x / ncta, c0 = blockIdx.x % ncta * cols, cend = min(W, c0 + cols);
+  float4 wv[NV];                                    // weights do not depend on the predecessor
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    wv[i] = c < cend ? *reinterpret_cast<const float4*>(w + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+  }
+  pdl_wait();
+  pdl_launch_dependents();
+  auto row_sum = [&](float ss, int slot) -> float {
+    ss = block_sum(ss, red);
+    if (ncta == 1) return ss;
+    if (threadIdx.x == 0) cta_ss[slot] = ss;
+    cluster.sync();
+    float t = 0.f;
+    for (int r = 0; r < ncta; r++) t += *cluster.map_shared_rank(&cta_ss[slot], r);
+    return t;
+  };
+  const float* yr = y + (size_t)row * ldy;
+  float* xr = x + (size_t)row * ldx;
+  float4 v[NV], xv[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    v[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < cend) {
+      xv[i] = *reinterpret_cast<const float4*>(xr + c);
+      int p = 0;
+      for (; p + 4 <= planes; p += 4) {
+        float4 t[4];
+#pragma unroll
+        for (int j = 0; j < 4; j++) t[j] = __ldcg(reinterpret_cast<const float4*>(yr + (p + j) * pstride + c));
+        v[i].x += (t[0].x + t[1].x) + (t[2].x + t[3].x);
+        v[i].y += (t[0].y + t[1].y) + (t[2].y + t[3].y);
+        v[i].z += (t[0].z + t[1].z) + (t[2].z + t[3].z);
+        v[i].w += (t[0].w + t[1].w) + (t[2].w + t[3].w);
+      }
+      for (; p < planes; p++) {
+        const float4 t = __ldcg(reinterpret_cast<const float4*>(yr + p * pstride + c));
+        v[i].x += t.x; v[i].y += t.y; v[i].z += t.z; v[i].w += t.w;
+      }
+      v[i] = keep4(v[i], c, W);
+      ss += sq4(v[i]);
+    }
+  }
+  const float rstd = 1.f / sqrtf(row_sum(ss, 0) / (float)W + eps);
+  float s2 = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    xv[i] = make_float4(xv[i].x + v[i].x * rstd * wv[i].x, xv[i].y + v[i].y * rstd * wv[i].y, xv[i].z + v[i].z * rstd * wv[i].z, xv[i].w + v[i].w * rstd * wv[i].w);
+    if (c < cend) {
+      xv[i] = keep4(xv[i], c, W);
+      if (store_x) *reinterpret_cast<float4*>(xr + c) = xv[i];
+      if (w_last == nullptr) put4(h + (size_t)row * ldh + c, xv[i]);
+      s2 += sq4(xv[i]);
+    }
+  }
+  if (w_last != nullptr) {
+    const float r2 = 1.f / sqrtf(row_sum(s2, 1) / (float)W + eps);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      if (c < cend) {
+        const float4 l = *reinterpret_cast<const float4*>(w_last + c);
+        put4(h + (size_t)row * ldh + c, make_float4(xv[i].x * r2 * l.x, xv[i].y * r2 * l.y, xv[i].z * r2 * l.z, xv[i].w * r2 * l.w));
+      }
+    }
+  }
+  if (ncta > 1) cluster.sync();                     // nobody leaves while a partner may still read its shared memory
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// gated activation
+// ------------------------------------------------------------------------------------------------------------
+enum { ACT_GELU_TANH = 0, ACT_SILU = 1 };
+FT_DEVICE float gate_act(float z, int kind) {
+  if (kind == ACT_SILU) return z / (1.f + __expf(-z));
+  // 0.5 (1 + tanh(u)) = 1 / (1 + exp(-2u))
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return z / (1.f + __expf(-2.f * u));
+}
+FT_DEVICE float gate_act_exact(float z, int kind) {
+  if (kind == ACT_SILU) return z / (1.f + expf(-z));
+  return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
+}
+template <bool EXACT> FT_DEVICE float4 gated4(float4 g, float4 u, int kind) {
+  if constexpr (EXACT) return make_float4(gate_act_exact(g.x, kind) * u.x, gate_act_exact(g.y, kind) * u.y, gate_act_exact(g.z, kind) * u.z, gate_act_exact(g.w, kind) * u.w);
+  else return make_float4(gate_act(g.x, kind) * u.x, gate_act(g.y, kind) * u.y, gate_act(g.z, kind) * u.z, gate_act(g.w, kind) * u.w);
+}
+FT_DEVICE float4 unpack4(uint2 r) {
+  const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&r.y));
+  return make_float4(a.x, a.y, b.x, b.y);
+}
+
+// columns come in blocks of eight gates and the eight ups of the same neurons; a thread takes one block (bf16: two 16-byte loads, one 16-byte store)
+template <typename T>
+__global__ void __launch_bounds__(256) gated_act_kernel(const T* __restrict__ gu, int64_t ld, int rows, int blocks, int kind, T* __restrict__ out, int64_t ldo) {
+  const int b = blockIdx.x * blockDim.x + threadIdx.x;
+  if (b >= blocks) return;
+  constexpr int RU = sizeof(T) == 2 ? 4 : 1;
+  for (int r0 = blockIdx.y * RU; r0 < rows; r0 += gridDim.y * RU) {
+    if constexpr (sizeof(T) == 2) {
+      uint4 g[RU], u[RU];
+#pragma unroll
+      for (int i = 0; i < RU; i++) {
+        const uint4* s = reinterpret_cast<const uint4*>(gu + (size_t)min(r0 + i, rows - 1) * ld + b * 16);
+        g[i] = s[0];
+        u[i] = s[1];
+      }
+#pragma unroll
+      for (int i = 0; i < RU; i++) {
+        const float4 a = gated4<false>(unpack4(make_uint2(g[i].x, g[i].y)), unpack4(make_uint2(u[i].x, u[i].y)), kind);
+        const float4 c = gated4<false>(unpack4(make_uint2(g[i].z, g[i].w)), unpack4(make_uint2(u[i].z, u[i].w)), kind);
+        const float e[8] = {a.x, a.y, a.z, a.w, c.x, c.y, c.z, c.w};
+        if (r0 + i < rows) *reinterpret_cast<bf16x8*>(out + (size_t)(r0 + i) * ldo + b * 8) = float_to_bf16x8(e);
+      }
+    } else {
+      const float* s = gu + (size_t)r0 * ld + b * 16;
+#pragma unroll
+      for (int i = 0; i < 8; i += 4)
+        *reinterpret_cast<float4*>(out + (size_t)r0 * ldo + b * 8 + i) = gated4<true>(*reinterpret_cast<const float4*>(s + i), *reinterpret_cast<const float4*>(s + 8 + i), kind);
+    }
+  }
+}
+
+__global__ void __launch_bounds__(128) gated_act_planes_kernel(const float* __restrict__ p, int splits, int64_t ldp, size_t pstride, int rows, int quads, int kind,
+                                                               __nv_bfloat16* __restrict__ out, int64_t ldo) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int i = blockIdx.x * 128 + threadIdx.x;
+  if (i >= rows * quads) return;
+  const int r = i / quads, q = i % quads;                       // four neurons
+  const float* s = p + (size_t)r * ldp + (q >> 1) * 16 + (q & 1) * 4;
+  float4 g = make_float4(0.f, 0.f, 0.f, 0.f), u = g;
+#pragma unroll 4
+  for (int k = 0; k < splits; k++) {
+    const float4 a = __ldcg(reinterpret_cast<const float4*>(s + k * pstride)), b = __ldcg(reinterpret_cast<const float4*>(s + k * pstride + 8));
+    g.x += a.x; g.y += a.y; g.z += a.z; g.w += a.w;
+    u.x += b.x; u.y += b.y; u.z += b.z; u.w += b.w;
+  }
+  put4(out + (size_t)r * ldo + q * 4, gated4<false>(g, u, kind));
+}
+
+template <int NV, typename H>
+int launch_update(int ncta, int rows, cudaStream_t st, float* x, int64_t ldx, const float* y, int planes, int64_t pstride, int64_t ldy, const float* w, const float* w_last,
+                  float eps, H* h, int64_t ldh, int W, int cols, int store) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(ncta * rows);
+  cfg.blockDim = dim3(UPD_THREADS);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = ncta;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = ft_pdl_enabled() ? 2 : 1;
+  return (int)cudaLaunchKernelEx(&cfg, residual_update_kernel<NV, H>, x, ldx, y, planes, (size_t)pstride, ldy, w, w_last, eps, h, ldh, ncta, W, cols, store);
+}
+
+template <typename H>
+int dispatch_update(float* x, int64_t ldx, const float* y, int planes, int64_t pstride, int64_t ldy, const float* w, const float* w_last, float eps, void* h, int64_t ldh,
+                    int rows, int W, int store, cudaStream_t st) {
+  // rows alone fill the GPU, or a row is spread over up to eight SMs (at least 256 columns each)
+  int ncta = 1;
+  while (ncta < 8 && (rows * ncta < 148 && W > 256 * ncta * 2)) ncta *= 2;
+  while (ncta < 8 && (W + ncta - 1) / ncta > UPD_THREADS * 4 * 8) ncta *= 2;
+  const int cols = ((W + ncta - 1) / ncta + 3) & ~3;
+  const int nv = (cols + UPD_THREADS * 4 - 1) / (UPD_THREADS * 4);
+  if (nv > 8) return FT_ERR_TOO_LARGE;
+#define FT_RU(N) return launch_update<N, H>(ncta, rows, st, x, ldx, y, planes, pstride, ldy, w, w_last, eps, (H*)h, ldh, W, cols, store)
+  if (nv <= 1) FT_RU(1);
+  if (nv <= 2) FT_RU(2);
+  if (nv <= 4) FT_RU(4);
+  FT_RU(8);
+#undef FT_RU
+}
+
+}  // namespace
+
+// x [rows][ldx] f32 = scale * table[ids[r]] (zeros for ids outside [0, vocab)), h [rows][ldh] the same in the table's type (bf16, or f32 with is_f32).
+// Leading dimensions are multiples of four.
+FT_EXPORT int ft_residual_embed(const int64_t* ids, const void* table, int64_t ld_table, int64_t vocab, float scale, float* x, int64_t ldx, void* h, int64_t ldh,
+                                int is_f32, int rows, int W, cudaStream_t st) {
+  if (rows < 1 || W < 1 || (ld_table & 3) || (ldx & 3) || (ldh & 3)) return FT_ERR_ARG;
+  const dim3 grid((W + 1023) / 1024, rows < 2048 ? rows : 2048);
+  if (is_f32) return (int)ft_launch_pdl(residual_embed_kernel<float>, grid, dim3(256), 0, st, ids, (const float*)table, ld_table, vocab, scale, x, ldx, (float*)h, ldh, rows, W);
+  return (int)ft_launch_pdl(residual_embed_kernel<__nv_bfloat16>, grid, dim3(256), 0, st, ids, (const __nv_bfloat16*)table, ld_table, vocab, scale, x, ldx, (__nv_bfloat16*)h,
+                            ldh, rows, W);
+}
+
+// y = sum of `planes` f32 planes [row][ldy]; x += y / sqrt(mean(y^2) + eps) * w; h = x, or with w_last x / sqrt(mean(x^2) + eps) * w_last, bf16 (f32 with
+// is_f32). w, w_last: f32, readable up to W rounded up to a multiple of four. x is left alone when store_x is 0. Widths up to 65536.
+FT_EXPORT int ft_residual_update(float* x, int64_t ldx, const float* y, int planes, int64_t plane_stride, int64_t ldy, const float* w, const float* w_last, float eps,
+                                 void* h, int64_t ldh, int is_f32, int rows, int W, int store_x, cudaStream_t st) {
+  if (rows < 1 || W < 1 || planes < 1 || (ldx & 3) || (ldy & 3) || (ldh & 3) || (plane_stride & 3)) return FT_ERR_ARG;
+  if (is_f32) return dispatch_update<float>(x, ldx, y, planes, plane_stride, ldy, w, w_last, eps, h, ldh, rows, W, store_x, st);
+  return dispatch_update<__nv_bfloat16>(x, ldx, y, planes, plane_stride, ldy, w, w_last, eps, h, ldh, rows, W, store_x, st);
+}
+
+// out[r][f] = act(gate) * up for f < fp (a multiple of 8) from columns in blocks of eight gates and eight ups; kind 0: gelu (tanh form), 1: silu.
+FT_EXPORT int ft_gated_act(const void* gu, int64_t ld, int rows, int fp, int kind, void* out, int64_t ldo, int is_f32, cudaStream_t st) {
+  if (rows < 1 || fp < 8 || (fp & 7) || (ld & 7) || (ldo & 7) || kind < 0 || kind > 1) return FT_ERR_ARG;
+  const int blocks = fp / 8, threads = blocks >= 256 ? 256 : (blocks + 31) & ~31, ru = is_f32 ? 1 : 4;
+  const int gx = (blocks + threads - 1) / threads, want = (rows + ru - 1) / ru, cap = 148 * 16 / gx + 1;
+  const dim3 grid(gx, want < cap ? want : cap);
+  if (is_f32) gated_act_kernel<float><<<grid, threads, 0, st>>>((const float*)gu, ld, rows, blocks, kind, (float*)out, ldo);
+  else gated_act_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>((const __nv_bfloat16*)gu, ld, rows, blocks, kind, (__nv_bfloat16*)out, ldo);
+  return (int)cudaGetLastError();
+}
+
+// The same from split-K planes [split][row][ldp] (f32) to bf16 rows.
+FT_EXPORT int ft_gated_act_planes(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int rows, int fp, int kind, void* out, int64_t ldo, cudaStream_t st) {
+  if (rows < 1 || splits < 1 || fp < 8 || (fp & 7) || (ldp & 3) || (plane_stride & 3) || (ldo & 3) || kind < 0 || kind > 1) return FT_ERR_ARG;
+  const int quads = fp / 4;
+  return (int)ft_launch_pdl(gated_act_planes_kernel, dim3((rows * quads + 127) / 128), dim3(128), 0, st, planes, splits, ldp, (size_t)plane_stride, rows, quads, kind,
+                            (__nv_bfloat16*)out, ldo);
+}

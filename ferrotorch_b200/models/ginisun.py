@@ -21,11 +21,12 @@ from typing import Dict, List, Optional, Tuple
 import torch
 
 from .. import _lib
-from ..errors import InvalidArgument, ShapeMismatch
+from ..errors import InvalidArgument
 from ..ops.latent_attention import (LatentDecodeBuffers, LatentDims, LatentWeights, latent_attention_decode, latent_attention_rows, rotary_pair_tables)
 from ..ops.moe import ExpertStack, MoeSmallBuffers, MoeWeights, linear_rows, moe_rows, moe_small
 from ..ops.streams import DynamicTanhWeights, HyperWeights, SublayerOutput, hyper_embed, hyper_update, round_up
 from .llama_infer import PAD_ROWS, _SplitKGemm
+from .registry import checked_weights
 
 EXPERT_SLOPE = 1.702          # g * sigmoid(1.702 g): fixed by the design
 MAX_STREAMS = 16
@@ -238,19 +239,7 @@ class GinisunModel:
     # -- weights ---------------------------------------------------------------
     def _load(self, weights) -> None:
         cfg, dev, dt = self.cfg, self.device, self.dtype
-        shapes = cfg.tensor_shapes()
-        missing = [k for k in shapes if k not in weights]
-        if missing:
-            raise InvalidArgument(f"Ginisun: missing weights: {', '.join(missing[:8])}{' ...' if len(missing) > 8 else ''}")
-        extra = [k for k in weights.keys() if k not in shapes]
-        if extra:
-            raise InvalidArgument(f"Ginisun: weights that the configuration does not have: {', '.join(extra[:8])}{' ...' if len(extra) > 8 else ''}")
-
-        def get(name):
-            t = weights[name]
-            if tuple(t.shape) != shapes[name]:
-                raise ShapeMismatch(f"{name}: {tuple(t.shape)} vs {shapes[name]}")
-            return t.to(dev)
+        get = checked_weights("Ginisun", cfg.tensor_shapes(), weights, dev)
 
         def norm(name):
             return DynamicTanhWeights.from_tensors(get(name + ".alpha"), get(name), get(name + ".b"), dev)

@@ -12,7 +12,7 @@ from typing import Callable, Dict, List
 
 import torch
 
-from ..errors import InvalidArgument
+from ..errors import InvalidArgument, ShapeMismatch
 
 
 @dataclass
@@ -59,6 +59,23 @@ def load_checkpoint_weights(directory) -> Dict[str, torch.Tensor]:
     return load_safetensors_sharded(idx) if idx.exists() else load_safetensors(d / "model.safetensors")
 
 
+def checked_weights(name: str, shapes: Dict[str, tuple], weights, device, optional=()):
+    """``get(tensor name)`` over ``weights`` (anything with ``[]``, ``in`` and ``keys``) after checking that it has the tensors of ``shapes`` and no others; a tensor of the
+    wrong shape is refused when it is asked for. ``optional`` names may be absent, or present without an entry in ``shapes``."""
+    missing = [k for k in shapes if k not in weights and k not in optional]
+    extra = [k for k in weights.keys() if k not in shapes and k not in optional]
+    for text, names in (("missing weights", missing), ("weights that the configuration does not have", extra)):
+        if names:
+            raise InvalidArgument(f"{name}: {text}: {', '.join(names[:8])}{' ...' if len(names) > 8 else ''}")
+
+    def get(key: str) -> torch.Tensor:
+        t = weights[key]
+        if tuple(t.shape) != tuple(shapes[key]):
+            raise ShapeMismatch(f"{key}: {tuple(t.shape)} vs {tuple(shapes[key])}")
+        return t.to(device)
+    return get
+
+
 def load_engine(directory, device="cuda", dtype: torch.dtype = torch.bfloat16, max_tokens: int = 4096):
     arch, cfg = load_model_config(directory)
     return arch.engine(cfg, load_checkpoint_weights(directory), device, dtype, max_tokens)
@@ -75,6 +92,17 @@ def _ginisun_engine(cfg, weights, device, dtype, max_tokens):
     return ServingEngine(GinisunModel(cfg, weights, device, dtype), max_tokens=max_tokens)
 
 
+def _pufevik_config(d: dict):
+    from .pufevik import PufevikConfig
+    return PufevikConfig.from_dict(d)
+
+
+def _pufevik_engine(cfg, weights, device, dtype, max_tokens):
+    from .pufevik import PufevikModel
+    from .serving import ServingEngine
+    return ServingEngine(PufevikModel(cfg, weights, device, dtype), max_tokens=max_tokens)
+
+
 def _llama_config(d: dict):
     from .llama import LlamaConfig
     return LlamaConfig.from_hf(d)
@@ -89,4 +117,5 @@ def _llama_engine(cfg, weights, device, dtype, max_tokens):
 
 
 register_architecture(Architecture("Ginisun", _ginisun_config, _ginisun_engine))
+register_architecture(Architecture("Pufevik", _pufevik_config, _pufevik_engine))
 register_architecture(Architecture("LlamaForCausalLM", _llama_config, _llama_engine, ("llama",)))

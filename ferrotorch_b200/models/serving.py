@@ -1,10 +1,11 @@
-"""Serving engine for decoder models with a paged row cache: ragged batches of prompts, portions of prompts and single tokens through one step
+"""Serving engine for decoder models with a paged row cache and recurrent state slots: ragged batches of prompts, portions of prompts and single tokens through one step
 function, a captured decode step, a small continuous-batching scheduler, and an adapter that gives the sampling functions of ``llama_gen`` (greedy,
 nucleus, beam, speculative, streaming) the cached-model interface they expect.
 
 A model plugs in with
 
 * ``vocab``, ``dtype``, ``device``, ``cache_rows`` (row length per layer),
+* optionally ``state_sizes`` (f32 values of recurrent state per sequence and layer, 0 for none),
 * ``prepare(max_positions)``,
 * ``forward_rows(batch, cache) -> logits of batch.want``,
 * ``decode_supported()``, ``decode_begin(max_batch, max_tokens)`` and ``decode(state, batch_size, cache) -> logits`` (capturable: it reads everything that
@@ -23,11 +24,13 @@ import torch
 
 from .. import _lib
 from ..errors import InvalidArgument
-from ..nn.extras import PagedRowCache, PagePool
+from ..nn.extras import PagedRowCache, PagePool, StateSlots
 from .llama_gen import GenerationConfig, sample_next
 
 PAGE = 16
 DECODE_ROWS = 16
+MEMORY_CHUNK = 64                    # tokens that a recurrent layer takes at once
+SEGMENT_MIN, SEGMENT_CTAS = 256, 296
 
 
 @dataclass
@@ -38,9 +41,21 @@ class StepEntry:
     want: Sequence[int] = ()
 
 
+@dataclass
+class MemoryPlan:
+    """How recurrent layers go over the new tokens of a batch. ``segments`` ``[n, 8]``: first row, rows, state slot, sequence, flags (1 the only segment, 2 the last, 4 the
+    sequence starts), scratch state; ``inner``: those that are not last (``None`` if there are none); ``chains`` ``[sequences, 4]``: first scratch state, segments, slot,
+    whether the sequence starts; ``scratch``: number of scratch states."""
+    segments: torch.Tensor
+    inner: Optional[torch.Tensor]
+    chains: torch.Tensor
+    sequences: int
+    scratch: int
+
+
 class RowBatch:
     """Device tables of a ragged batch: one row per new token (``ids``, ``positions``, cache ``slots``, ``seq_of``), the page table of its sequences, and the
-    dense context layout that prompt attention uses (``ctx_rows`` of the new tokens, ``past_slots`` -> ``past_rows`` of the cached ones)."""
+    dense context layout that prompt attention over gathered rows uses (``ctx_rows`` of the new tokens, ``past_slots`` -> ``past_rows`` of the cached ones)."""
 
     def __init__(self, entries: Sequence[StepEntry], cache: PagedRowCache, device, max_blocks: int):
         self.device = device
@@ -69,7 +84,10 @@ class RowBatch:
         self.past_slots, self.past_rows = (ps, pr) if m else (None, None)
         self.block_table = cache.block_table([e.id for e in entries], max_blocks).to(device)
         self.want = torch.tensor(want, dtype=torch.int64).to(device) if want else None
+        self._state_slots = [cache.states.slot[e.id] for e in entries] if cache.states is not None else []
         self._tiles: Dict[int, torch.Tensor] = {}
+        self._query_tiles: Dict[int, torch.Tensor] = {}
+        self._plans: Dict[int, MemoryPlan] = {}
 
     def tiles_for(self, dims) -> Optional[torch.Tensor]:
         """Query tiles ``[tiles, 4]`` (first row, rows, first position, first context row), longest context first; ``None`` when the layer's sizes do not fit
@@ -83,24 +101,59 @@ class RowBatch:
             self._tiles[size] = torch.tensor(t, dtype=torch.int32).to(self.device)
         return self._tiles[size]
 
+    def query_tiles(self, size: int) -> torch.Tensor:
+        """Query tiles of up to ``size`` tokens for attention over the pages: ``[tiles, 4]`` (first row, tokens, first position, row of ``block_table``), longest
+        context first."""
+        if size not in self._query_tiles:
+            t = [(r0 + m, min(size, n - m), start + m, i) for i, (r0, n, start, _) in enumerate(self._spans) for m in range(0, n, size)]
+            t.sort(key=lambda x: -(x[1] + x[2]))
+            self._query_tiles[size] = torch.tensor(t, dtype=torch.int32).to(self.device)
+        return self._query_tiles[size]
+
+    def memory_plan(self, ctas: int) -> MemoryPlan:
+        """Segments of the new tokens for recurrent layers whose walk takes ``ctas`` CTAs per segment: as many as fill the GPU, none shorter than ``SEGMENT_MIN`` tokens.
+        ``ctas`` 0: one segment per sequence."""
+        if ctas not in self._plans:
+            segs, inner, chains = [], [], []
+            per_seq = max(1, SEGMENT_CTAS // (ctas * len(self._spans))) if ctas else 1
+            scratch = 0
+            for i, (r0, n, start, _) in enumerate(self._spans):
+                size = -(-n // min(per_seq, max(1, n // SEGMENT_MIN)) // MEMORY_CHUNK) * MEMORY_CHUNK if ctas else n
+                count, slot, fresh = -(-n // size), self._state_slots[i], int(start == 0)
+                base = scratch if count > 1 else 0
+                for j in range(count):
+                    flags = (count == 1) * 1 + (j + 1 == count) * 2 + fresh * 4
+                    row = (r0 + j * size, min(size, n - j * size), slot, i, flags, base + j, 0, 0)
+                    segs.append(row)
+                    if j + 1 < count:
+                        inner.append(row)
+                chains.append((base, count, slot, fresh))
+                scratch += count if count > 1 else 0
+            packed = torch.tensor([x for r in segs + inner for x in r] + [x for r in chains for x in r], dtype=torch.int32).to(self.device)
+            a, b, c = torch.split(packed, [8 * len(segs), 8 * len(inner), 4 * len(chains)])
+            self._plans[ctas] = MemoryPlan(a.view(-1, 8), b.view(-1, 8) if inner else None, c.view(-1, 4), len(chains), scratch)
+        return self._plans[ctas]
+
 
 class DecodeState:
     """Device inputs of the captured decode step; a step advances them, so consecutive greedy steps need nothing from the host."""
 
     def __init__(self, device, max_blocks: int):
         self.tokens = torch.zeros(DECODE_ROWS, device=device, dtype=torch.int64)
-        self._ints = torch.zeros(2 * DECODE_ROWS + DECODE_ROWS * max_blocks, device=device, dtype=torch.int32)
-        self.positions, self.seq_lens = self._ints[:DECODE_ROWS], self._ints[DECODE_ROWS: 2 * DECODE_ROWS]
-        self.block_table = self._ints[2 * DECODE_ROWS:].view(DECODE_ROWS, max_blocks)
+        self._ints = torch.zeros(3 * DECODE_ROWS + DECODE_ROWS * max_blocks, device=device, dtype=torch.int32)
+        self.positions, self.seq_lens, self.slots = self._ints[: 3 * DECODE_ROWS].view(3, DECODE_ROWS)
+        self.block_table = self._ints[3 * DECODE_ROWS:].view(DECODE_ROWS, max_blocks)
         self.picked = torch.zeros(DECODE_ROWS, device=device, dtype=torch.int64)
 
-    def load(self, tokens: Sequence[int], positions: Sequence[int], block_table: torch.Tensor) -> None:
+    def load(self, tokens: Sequence[int], positions: Sequence[int], block_table: torch.Tensor, slots: Optional[Sequence[int]] = None) -> None:
         B = len(tokens)
-        host = torch.zeros(2 * DECODE_ROWS, dtype=torch.int32)
-        host[:B] = torch.tensor(list(positions), dtype=torch.int32)
-        host[DECODE_ROWS: DECODE_ROWS + B] = host[:B] + 1
+        host = torch.zeros(3, DECODE_ROWS, dtype=torch.int32)
+        host[0, :B] = torch.tensor(list(positions), dtype=torch.int32)
+        host[1, :B] = host[0, :B] + 1
+        if slots is not None:
+            host[2, :B] = torch.tensor(list(slots), dtype=torch.int32)
         used = block_table.reshape(-1)
-        self._ints[: 2 * DECODE_ROWS + used.numel()].copy_(torch.cat([host, used]))
+        self._ints[: 3 * DECODE_ROWS + used.numel()].copy_(torch.cat([host.reshape(-1), used]))
         self.tokens[:B].copy_(torch.tensor(list(tokens), dtype=torch.int64))
 
 
@@ -116,7 +169,10 @@ class ServingEngine:
         self.max_blocks = -(-max_tokens // PAGE)
         # a sequence wastes at most one page beyond its tokens
         self.pool = PagePool(self.max_blocks + max_sequences, PAGE)
-        self.cache = PagedRowCache(self.pool, model.cache_rows, self.device, model.dtype)
+        sizes = getattr(model, "state_sizes", ())
+        self.states = StateSlots(max_sequences, sizes, self.device) if any(sizes) else None
+        self.cache = PagedRowCache(self.pool, model.cache_rows, self.device, model.dtype, self.states)
+        self._fed: Dict[object, List[int]] = {}               # tokens of live sequences, kept where a state can only be rebuilt from them
         model.prepare(self.max_blocks * PAGE)
         self.use_graph = use_graph
         self.graphs: Dict[int, Tuple[torch.cuda.CUDAGraph, torch.Tensor]] = {}
@@ -135,6 +191,24 @@ class ServingEngine:
     def release(self, seq_id) -> None:
         """Gives back what a finished sequence holds."""
         self.cache.free_sequence(seq_id)
+        self._fed.pop(seq_id, None)
+
+    def fork(self, src, dst) -> None:
+        """A new sequence ``dst`` that continues from where ``src`` is: pages are shared until one of them writes, recurrent state is copied."""
+        self.cache.fork(src, dst)
+        if src in self._fed:
+            self._fed[dst] = list(self._fed[src])
+
+    def truncate(self, seq_id, n: int) -> None:
+        """Forgets every token from position ``n`` on. Recurrent state cannot step back: its remaining tokens are run again."""
+        if self.states is None or not 0 < n < self.length(seq_id):
+            self.cache.truncate(seq_id, n)
+            if seq_id in self._fed:
+                del self._fed[seq_id][n:]
+            return
+        tokens = self._fed.pop(seq_id)[:n]
+        self.cache.truncate(seq_id, 0)
+        self.step([StepEntry(seq_id, tokens)])
 
     # -- steps -----------------------------------------------------------------
     def _admit(self, entries: Sequence[StepEntry]) -> None:
@@ -157,6 +231,8 @@ class ServingEngine:
             need += self.cache.pages_for(e.id, total)
         if need > self.pool.num_free():
             raise InvalidArgument(f"step: {need} more cache pages needed, {self.pool.num_free()} free")
+        if self.states is not None and sum(e.id not in self for e in entries) > self.states.num_free():
+            raise InvalidArgument(f"step: more new sequences than free state slots ({self.states.num_free()})")
         for e in entries:
             if e.id not in self:
                 self.cache.add_sequence(e.id)
@@ -179,18 +255,24 @@ class ServingEngine:
                 out = self.model.forward_rows(batch, self.cache, taps)
             for e in entries:
                 self.cache.lengths[e.id] += len(e.tokens)
+                if self.states is not None:
+                    self._fed.setdefault(e.id, []).extend(int(t) for t in e.tokens)
         for s in end:
             self.release(s)
         return out
 
     def _decode(self, entries: Sequence[StepEntry]) -> Optional[torch.Tensor]:
         B = len(entries)
-        self.state.load([e.tokens[0] for e in entries], [self.cache.lengths[e.id] for e in entries], self.cache.block_table([e.id for e in entries], self.max_blocks))
+        self._load_state([e.id for e in entries], [e.tokens[0] for e in entries])
         logits = self._decode_launch(B)
         rows = [i for i, e in enumerate(entries) for _ in e.want]
         if not rows:
             return None
         return logits[:B].clone() if rows == list(range(B)) else logits[torch.tensor(rows, device=self.device)]
+
+    def _load_state(self, ids: Sequence, tokens: Sequence[int]) -> None:
+        slots = None if self.states is None else [self.states.slot[s] for s in ids]
+        self.state.load(tokens, [self.cache.lengths[s] for s in ids], self.cache.block_table(ids, self.max_blocks), slots)
 
     def _decode_body(self, B: int) -> torch.Tensor:
         """One decode step of the first ``B`` rows of the state. Its kernels are launched as programmatic dependents (each is scheduled while its
@@ -213,6 +295,8 @@ class ServingEngine:
         if B not in self.graphs:
             s = self.state
             saved = [t.clone() for t in (s.tokens, s._ints)]
+            if self.states is not None:
+                s.slots.fill_(self.states.spare)                # the first run below must not advance anybody's state
             side = torch.cuda.Stream(self.device)
             side.wait_stream(torch.cuda.current_stream())
             with torch.cuda.stream(side):                       # lazy initialisation outside the capture; its cache write is simply redone
@@ -239,14 +323,17 @@ class ServingEngine:
         for s in seq_ids:
             self.cache.reserve(s, self.cache.lengths[s] + steps)
         B = len(seq_ids)
-        self.state.load(tokens, [self.cache.lengths[s] for s in seq_ids], self.cache.block_table(seq_ids, self.max_blocks))
+        self._load_state(seq_ids, tokens)
         out = torch.empty(steps, B, device=self.device, dtype=torch.int64)
         for i in range(steps):
             self._decode_launch(B)
             out[i].copy_(self.state.picked[:B])
-        for s in seq_ids:
+        rows = out.t().tolist()
+        for s, t, row in zip(seq_ids, tokens, rows):
             self.cache.lengths[s] += steps
-        return out.t().tolist()
+            if self.states is not None:
+                self._fed[s].extend([int(t), *row[:-1]])
+        return rows
 
     # -- whole requests --------------------------------------------------------
     def generate(self, prompts: Sequence[Sequence[int]], config: Optional[GenerationConfig] = None, streamer: Optional[Callable[[int, int], None]] = None) -> List[List[int]]:
@@ -418,12 +505,12 @@ class EngineCache:
 
     def truncate(self, n: int) -> None:
         for s in self.ids:
-            self._engine.cache.truncate(s, n)
+            self._engine.truncate(s, n)
 
     def _replace(self, sources: List[object]) -> None:
         new = self._new_ids(len(sources))
         for d, s in zip(new, sources):
-            self._engine.cache.fork(s, d)
+            self._engine.fork(s, d)
         for s in self.ids:
             self._engine.release(s)
             self._held.remove(s)

@@ -5,7 +5,7 @@ from .layers import *  # noqa: F401,F403
 from .layers import (Linear, LazyLinear, LoRALinear, SqueezeExcitation, RMSNorm, LayerNorm, Embedding, RoPEConvention, RoPEScaling,
                      RotaryPositionEmbedding, SwiGLU, KVCache, MultiheadAttention, CrossEntropyLoss, repeat_kv, reshape_to_heads,
                      transpose_heads_to_2d, standard_attention, flash_attention, attention_backend, PaddingMode, RNNNonlinearity, EmbeddingBagMode)
-from .extras import (KVPage, PagePool, PagedKVCache, PagedRowCache, PagedAttentionManager, BlockMask, flex_attention, causal_score_mod, alibi_score_mod,
+from .extras import (KVPage, PagePool, PagedKVCache, PagedRowCache, StateSlots, PagedAttentionManager, BlockMask, flex_attention, causal_score_mod, alibi_score_mod,
                      relative_position_score_mod, NonLinearity, init, clip_grad_norm_, clip_grad_value_, PackedSequence,
                      pack_padded_sequence, pad_packed_sequence, interpolate, grid_sample, affine_grid, functional_pad_1d,
                      functional_pad_2d, functional_pad_3d, ObserverType, QatConfig, FakeQuantize, QuantizedModel, QatModel, prepare_qat, InterpolateMode,

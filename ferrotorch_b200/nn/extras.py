@@ -115,13 +115,41 @@ class PagedKVCache:
         return t.to(self.k.device)
 
 
+class StateSlots:
+    """Recurrent state of fixed size per sequence: ``[slots + 1, size]`` f32 for every layer that has one (``None`` for the others). A sequence owns one slot; what it
+    finds there at its first token is void. The last slot is spare: a run whose result is thrown away may write to it."""
+
+    def __init__(self, slots: int, sizes: Sequence[int], device="cpu"):
+        self.data = [torch.zeros(slots + 1, n, device=device) if n else None for n in sizes]
+        self.spare = slots
+        self.free: List[int] = list(range(slots - 1, -1, -1))
+        self.slot: Dict[object, int] = {}
+
+    def open(self, seq_id) -> None:
+        if not self.free:
+            raise InvalidArgument("no free state slot")
+        self.slot[seq_id] = self.free.pop()
+
+    def close(self, seq_id) -> None:
+        if seq_id in self.slot:
+            self.free.append(self.slot.pop(seq_id))
+
+    def copy(self, src, dst) -> None:
+        for d in self.data:
+            if d is not None:
+                d[self.slot[dst]].copy_(d[self.slot[src]])
+
+    def num_free(self) -> int:
+        return len(self.free)
+
+
 class PagedRowCache:
     """Paged storage of one row per token and layer, ``[num_pages, page_size, row]`` per layer with its own row length, behind one page table per
-    sequence that all layers share: for mixers that cache a single vector per token (latent attention). Pages come from a :class:`PagePool`; a
-    shared page is copied before it is written (:meth:`fork`)."""
+    sequence that all layers share: for mixers that cache a single vector per token (latent attention) or all keys and values of a token side by side. Pages
+    come from a :class:`PagePool`; a shared page is copied before it is written (:meth:`fork`). ``states`` holds the recurrent state of the same sequences."""
 
-    def __init__(self, pool: PagePool, row_sizes: Sequence[int], device="cpu", dtype=torch.float32):
-        self.pool = pool
+    def __init__(self, pool: PagePool, row_sizes: Sequence[int], device="cpu", dtype=torch.float32, states: Optional[StateSlots] = None):
+        self.pool, self.states = pool, states
         n, ps = len(pool.pages), pool.page_size
         self.rows = [torch.zeros(n, ps, r, device=device, dtype=dtype) for r in row_sizes]
         self.tables: Dict[object, List[int]] = {}
@@ -130,9 +158,13 @@ class PagedRowCache:
     def add_sequence(self, seq_id) -> None:
         if seq_id in self.tables:
             raise InvalidArgument(f"sequence {seq_id!r} is already in the cache")
+        if self.states is not None:
+            self.states.open(seq_id)
         self.tables[seq_id], self.lengths[seq_id] = [], 0
 
     def free_sequence(self, seq_id) -> None:
+        if self.states is not None:
+            self.states.close(seq_id)
         for p in self.tables.pop(seq_id, []):
             self.pool.release(p)
         self.lengths.pop(seq_id, None)
@@ -160,7 +192,10 @@ class PagedRowCache:
         return [t[p // ps] * ps + p % ps for p in range(start, start + count)]
 
     def truncate(self, seq_id, n: int) -> None:
-        """Forgets every token from position ``n`` on; pages that hold none of the rest go back to the pool."""
+        """Forgets every token from position ``n`` on; pages that hold none of the rest go back to the pool. A recurrent state cannot forget the last tokens alone:
+        with ``states``, ``n`` is 0 or the present length."""
+        if self.states is not None and 0 < n < self.lengths[seq_id]:
+            raise InvalidArgument("a recurrent state cannot be cut back; truncate to 0 and feed the tokens again")
         table, ps = self.tables[seq_id], self.pool.page_size
         while len(table) > -(-n // ps):
             self.pool.release(table.pop())
@@ -169,6 +204,8 @@ class PagedRowCache:
     def fork(self, src, dst) -> None:
         self.add_sequence(dst)
         self.tables[dst], self.lengths[dst] = list(self.tables[src]), self.lengths[src]
+        if self.states is not None:
+            self.states.copy(src, dst)
         for p in self.tables[dst]:
             self.pool.retain(p)
 

@@ -1,0 +1,142 @@
+"""Grouped-query attention over a paged row cache on the kernels of ``csrc/kernels/gqa_attn.cu``: own key and value sizes, RMS norms on queries and keys (per head or
+over the whole projection), rotary positions on the first dimensions, an optional sliding window, an optional sink per head, values optionally mixed with an
+earlier layer's, an output gate (per element or per head) and a scale.
+
+Prompts of any ragged batch run a tcgen05 flash kernel that reads keys and values from the pages; a decode step streams the visible rows once for all heads of a
+group. f32 data takes a plain kernel.
+"""
+from __future__ import annotations
+
+from dataclasses import dataclass
+from typing import Optional
+
+import torch
+
+from .. import _lib
+from .streams import padded_vector, round_up
+
+GATE_NONE, GATE_ELEMENT, GATE_HEAD = 0, 1, 2
+SMALL_TOKENS = 16
+GROUP_ROWS = 128                     # query rows (tokens x heads of a group) of a flash sub-tile
+MAX_SPLITS = 64
+
+
+@dataclass(frozen=True)
+class GqaDims:
+    """Sizes and constants of one attention layer. ``window`` 0: every earlier position is visible. Head sizes are padded to multiples of 16: projection rows
+    ``heads x d16 | kv_heads x d16 | kv_heads x v16``, cache rows ``kv_heads x d16 | kv_heads x v16``."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    rot_dims: int
+    scale: float
+    eps: float
+    window: int = 0
+    whole_norm: bool = False
+    gate: int = GATE_NONE
+    out_scale: float = 1.0
+
+    @property
+    def d16(self): return round_up(self.dim, 16)
+    @property
+    def v16(self): return round_up(self.vdim, 16)
+    @property
+    def k_col(self): return self.heads * self.d16
+    @property
+    def v_col(self): return (self.heads + self.kv_heads) * self.d16
+    @property
+    def qkv_cols(self): return self.v_col + self.kv_heads * self.v16
+    @property
+    def out_cols(self): return self.heads * self.v16
+    @property
+    def row(self): return self.kv_heads * (self.d16 + self.v16)
+
+    def flash_tile(self) -> int:
+        """Tokens per tile of the flash kernel, 0 when these sizes do not fit it."""
+        return _lib.kernels().ft_gqa_flash_subtiles(self.heads, self.kv_heads, self.dim, self.vdim) * (GROUP_ROWS // (self.heads // self.kv_heads))
+
+    def decode_supported(self) -> bool:
+        return bool(_lib.kernels().ft_gqa_decode_fits(self.heads, self.kv_heads, self.dim, self.vdim))
+
+
+def pack_head_rows(w: torch.Tensor, heads: int, size: int, device, dtype) -> torch.Tensor:
+    """``[heads * size, k]`` -> ``[heads * padded size, k]`` with zero rows behind every head."""
+    out = torch.zeros(heads, round_up(size, 16), w.shape[1], device=device, dtype=dtype)
+    out[:, :size] = w.to(device, dtype).reshape(heads, size, -1)
+    return out.flatten(0, 1)
+
+
+def pack_head_columns(w: torch.Tensor, heads: int, size: int, device, dtype) -> torch.Tensor:
+    """``[n, heads * size]`` -> ``[n, heads * padded size]``."""
+    out = torch.zeros(w.shape[0], heads, round_up(size, 16), device=device, dtype=dtype)
+    out[:, :, :size] = w.to(device, dtype).reshape(-1, heads, size)
+    return out.flatten(1)
+
+
+def pack_head_vector(v: torch.Tensor, heads: int, size: int, device) -> torch.Tensor:
+    """f32 vector ``[heads * size]`` in the padding of the heads."""
+    return pack_head_columns(v.reshape(1, -1), heads, size, device, torch.float32)[0].contiguous()
+
+
+@dataclass
+class GqaWeights:
+    """Vectors of an attention layer (f32 on the device): query and key norm weights, ``sink`` ``[heads]``, ``mix`` (the weight of an earlier layer's values)."""
+    dims: GqaDims
+    q_norm: torch.Tensor
+    k_norm: torch.Tensor
+    sink: Optional[torch.Tensor] = None
+    mix: Optional[torch.Tensor] = None
+
+    @staticmethod
+    def pack(dims: GqaDims, q_norm, k_norm, device, sink=None, mix=None) -> "GqaWeights":
+        hq, hk = (dims.heads, dims.kv_heads) if dims.whole_norm else (1, 1)
+        return GqaWeights(dims, pack_head_vector(q_norm, hq, dims.dim, device), pack_head_vector(k_norm, hk, dims.dim, device),
+                          None if sink is None else padded_vector(sink, device), None if mix is None else mix.reshape(1).to(device, torch.float32))
+
+
+def gqa_attention_rows(qkv: torch.Tensor, w: GqaWeights, batch, cache: torch.Tensor, cos: torch.Tensor, sin: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor,
+                       first_values: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Attention of a ragged batch of new tokens into ``out`` ``[rows, out_cols]``. ``qkv``: projection rows (their queries are normed and turned in place);
+    ``gate``: pre-activations ``[rows, out_cols]`` in the data type or ``[rows, heads]`` f32; ``first_values`` ``[rows, kv_heads * v16]``: mixed in with
+    ``w.mix``. ``batch`` holds the tables of :class:`~ferrotorch_b200.models.serving.RowBatch`, ``cache`` is this layer's page storage."""
+    D, T, S = w.dims, qkv.shape[0], _lib.S()
+    f32 = qkv.dtype == torch.float32
+    _lib.call("ft_gqa_prep", qkv, qkv.stride(0), T, D.heads, D.kv_heads, D.dim, D.vdim, D.rot_dims, int(D.whole_norm), w.q_norm, w.k_norm, D.eps, batch.positions, cos, sin,
+              batch.slots, cache, first_values, 0 if first_values is None else first_values.stride(0), None if first_values is None else w.mix, int(f32), S)
+    bt = batch.block_table
+    tail = (D.heads, D.kv_heads, D.dim, D.vdim, D.scale, D.window, w.sink, gate, 0 if gate is None else gate.stride(0), D.gate, D.out_scale, out, out.stride(0))
+    tile = 0 if f32 else D.flash_tile()
+    if tile:
+        tiles = batch.query_tiles(tile)
+        _lib.call("ft_gqa_flash", qkv, qkv.stride(0), T, cache, cache.shape[0], bt, bt.shape[1], tiles, tiles.shape[0], *tail, S)
+    else:
+        _lib.call("ft_gqa_rows", qkv, qkv.stride(0), cache, bt, bt.shape[1], batch.seq_of, batch.positions, T, *tail, int(f32), S)
+    return out
+
+
+class GqaDecodeBuffers:
+    """Scratch of the decode kernels for one layer size (shared by layers of the same size, which run one after another)."""
+
+    def __init__(self, dims: GqaDims, max_batch: int, max_tokens: int, device, splits: Optional[int] = None):
+        D = dims
+        groups = D.kv_heads * -(-(D.heads // D.kv_heads) // 16)
+        span = min(max_tokens, D.window or max_tokens)
+        # by batch size: two CTAs per SM, at least one 64-row chunk per split at the longest visible range
+        self.splits = [splits or max(1, min(MAX_SPLITS, 296 // (b * groups), -(-span // 64))) for b in range(1, max_batch + 1)]
+        self.q = torch.zeros(SMALL_TOKENS, D.heads, D.d16, device=device, dtype=torch.bfloat16)
+        self.gate = torch.zeros(SMALL_TOKENS, D.out_cols if D.gate == GATE_ELEMENT else D.heads, device=device)
+        self.ws = torch.zeros(max(b * n for b, n in enumerate(self.splits, 1)) * groups * 16 * (D.v16 + 4), device=device)
+        self.counters = torch.zeros(SMALL_TOKENS * groups, device=device, dtype=torch.int32)
+
+
+def gqa_attention_decode(planes: torch.Tensor, splits: int, w: GqaWeights, b: GqaDecodeBuffers, state, cache: torch.Tensor, cos, sin, B: int, gate_col: int, out: torch.Tensor,
+                         keep_values: Optional[torch.Tensor] = None, first_values: Optional[torch.Tensor] = None) -> None:
+    """One token per sequence from the split-K planes of the projection (columns ``qkv_cols`` from 0 on, the gate's pre-activations at ``gate_col``) into ``out``
+    ``[16, out_cols]``. ``keep_values`` (f32 ``[16, kv_heads * v16]``) receives the values, ``first_values`` such values are mixed in."""
+    D, S = w.dims, _lib.S()
+    bt, mb = state.block_table, state.block_table.shape[1]
+    _lib.call("ft_gqa_decode_prep", planes, splits, planes.stride(1), planes.stride(0), B, D.heads, D.kv_heads, D.dim, D.vdim, D.rot_dims, int(D.whole_norm), w.q_norm, w.k_norm,
+              D.eps, state.positions, cos, sin, bt, mb, gate_col, D.gate, b.gate, keep_values, first_values, None if first_values is None else w.mix, b.q, cache, S)
+    _lib.call("ft_gqa_decode", b.q, cache, bt, mb, state.seq_lens, B, D.heads, D.kv_heads, D.dim, D.vdim, D.scale, D.window, w.sink, b.gate, D.gate, D.out_scale, b.splits[B - 1],
+              b.ws, b.counters, out, out.stride(0), S)
