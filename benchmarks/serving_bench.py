@@ -1,5 +1,5 @@
-"""Prefill and decode throughput of the serving models on layers of realistic size with random weights: the Ginisun decoder beside a Llama decoder of the
-same width and the same number of feed-forward neurons per token. Run through ``bench.py --serving``.
+"""Prefill and decode throughput of the serving models on layers of realistic size with random weights: the Ginisun and Pufevik decoders beside a Llama decoder
+of the same width and the same number of feed-forward neurons per token (Pufevik also has its attention sizes; its layers alternate between the two kinds). Run through ``bench.py --serving``.
 
 Every kernel class is also timed (CUDA events around its launches, L2 flushed by the step's own traffic) against its roofline, the slower of algorithmic
 bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate. Times of single launches below ~5 us are dominated by launch overhead.
@@ -15,6 +15,7 @@ import torch
 from ferrotorch_b200 import _lib
 from ferrotorch_b200.models import GenerationConfig, LlamaConfig
 from ferrotorch_b200.models.ginisun import GinisunConfig, GinisunModel, RandomGinisunWeights
+from ferrotorch_b200.models.pufevik import PufevikConfig, PufevikModel, RandomPufevikWeights
 from ferrotorch_b200.models.llama_infer import LlamaTPEngine, TPContext
 from ferrotorch_b200.models.serving import ServingEngine, StepEntry
 
@@ -22,6 +23,11 @@ SIZES = {
     "1k": dict(width=1024, heads=8, dim=64, rot_dim=32, vdim=64, kv_rank=256, experts=16, top=2, ff=1024, shared_ff=1024),
     "2k": dict(width=2048, heads=16, dim=128, rot_dim=64, vdim=128, kv_rank=512, experts=64, top=6, ff=1408, shared_ff=2816),
     "4k": dict(width=4096, heads=32, dim=128, rot_dim=64, vdim=128, kv_rank=512, experts=32, top=4, ff=2048, shared_ff=4096),
+}
+PUFEVIK = {                          # matrix memory beside the attention, window of its layers
+    "1k": dict(memory_heads=4, memory_dim=128, memory_vdim=256, window=1024),
+    "2k": dict(memory_heads=4, memory_dim=256, memory_vdim=512, window=1024),
+    "4k": dict(memory_heads=8, memory_dim=256, memory_vdim=512, window=1024),
 }
 VOCAB = 32768
 
@@ -158,6 +164,90 @@ def run_ginisun(size, layers, batch, prompt, ctx, steps, kernels=True):
             "decode_kernels": dtable}
 
 
+def run_pufevik(size, layers, batch, prompt, ctx, steps, kernels=True):
+    """Layers alternate: attention and matrix memory side by side, full attention."""
+    bw, fl, _ = peaks()
+    s, W = SIZES[size], SIZES[size]["width"]
+    H, F = W // 128, s["top"] * s["ff"] + s["shared_ff"]
+    G = max(1, H // 4)
+    cfg = PufevikConfig.pattern(("pa" * layers)[:layers], VOCAB, W, F, H, G, 128, 128, **PUFEVIK[size])
+    eng = ServingEngine(PufevikModel(cfg, RandomPufevikWeights(cfg)), max_tokens=max(batch * (ctx + steps * 4 + 64), prompt + 64), max_sequences=batch + 1)
+    g = torch.Generator().manual_seed(1)
+    ids = torch.randint(0, VOCAB, (prompt,), generator=g).tolist()
+    from ferrotorch_b200.models.serving import RowBatch
+    entry = [StepEntry("p", ids, [prompt - 1])]
+    eng._admit(entry)
+    rb = RowBatch(entry, eng.cache, eng.device, eng.max_blocks)
+    device_prefill = lambda: eng.model.forward_rows(rb, eng.cache)          # the device part: tables of the batch are built once
+    pre_ms = timed(device_prefill)
+    par, att = eng.model.subs[0].mixer, eng.model.subs[2].mixer
+    D, M = par.attn.dims, par.memory.dims
+    T, win = prompt, D.window
+    table = dtable = None
+    def g_(n, k, out=2, m=T): return (2 * (m * k + n * k) + out * m * n, 2 * m * n * k)
+    na, np_, n_gates = att.proj.shape[0], par.main, par.proj.shape[0] - par.main
+    if kernels:
+        names = {(np_, W): "projection gemm (two mixers)", (na, W): "projection gemm (attention)", (n_gates, W): "gate gemm", (W, par.out_cols): "output gemm (two mixers)",
+                 (W, att.out_cols): "output gemm (attention)", (2 * F, W): "gate/up gemm", (W, F): "down gemm"}
+        classify = _by_shape(names)
+        seen = win * T - win * (win - 1) // 2 if win < T else T * (T + 1) // 2            # keys that the window's queries see
+        qkv = D.qkv_cols
+        roofs = {"projection gemm (two mixers)": g_(np_, W), "projection gemm (attention)": g_(na, W), "gate gemm": g_(n_gates, W, 4), "output gemm (two mixers)": g_(W, par.out_cols, 4),
+                 "output gemm (attention)": g_(W, att.out_cols, 4), "gate/up gemm": g_(2 * F, W), "down gemm": g_(W, F, 4),
+                 "flash (window)": (2 * T * (qkv + D.out_cols), 4 * H * seen * 128), "flash (full)": (2 * T * (qkv + 2 * D.out_cols), H * T * T * 256),
+                 "ft_gqa_prep": (2 * T * (2 * qkv), 0), "ft_gated_act": (6 * T * F, 0), "ft_residual_update": (14 * T * W, 0),
+                 # inner: keys and values in; outputs: queries, keys, values in, f32 outputs out; finish: those, gates in, bf16 out. Products of a chunk of 64
+                 "memory walk (states)": (2 * T * M.heads * (M.d16 + M.v16), 2 * T * M.heads * M.d16 * M.v16),
+                 "memory walk (outputs)": (T * M.heads * (4 * M.d16 + 6 * M.v16), 2 * T * M.heads * (2 * M.d16 * M.v16 + 32 * (M.d16 + M.v16))),
+                 "ft_mm_finish": (T * M.heads * M.v16 * 8, 0)}
+        def label(fn, raw):
+            if fn == "ft_gqa_flash":
+                return "flash (window)" if raw[14] else "flash (full)"
+            if fn == "ft_mm_walk":
+                return "memory walk (outputs)" if raw[17] else "memory walk (states)"
+            return classify(fn, raw)
+        table = kernel_table(device_prefill, label, roofs, bw, fl)
+    eng.release("p")
+    seqs = [f"s{i}" for i in range(batch)]
+    for q in seqs:
+        eng.step([StepEntry(q, torch.randint(0, VOCAB, (ctx,), generator=g).tolist(), [])])
+    eng.decode_greedy(seqs, [1] * batch, 4)
+    best = []
+    for _ in range(3):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        eng.decode_greedy(seqs, [1] * batch, steps)
+        e1.record()
+        torch.cuda.synchronize()
+        best.append(e0.elapsed_time(e1) / steps)
+    dec_ms = statistics.median(best)
+    if kernels:
+        for q in seqs:
+            eng.cache.reserve(q, eng.cache.lengths[q] + 1)
+        eng._load_state(seqs, [1 + i for i in range(batch)])
+        positions, lens, tokens = eng.state.positions.clone(), eng.state.seq_lens.clone(), eng.state.tokens.clone()
+        def one():
+            eng.state.positions.copy_(positions); eng.state.seq_lens.copy_(lens); eng.state.tokens.copy_(tokens)
+            eng.model.decode(eng.state, batch, eng.cache)
+        one()
+        L = eng.cache.lengths[seqs[0]] + 1
+        names = {(par.proj.shape[0], W): "projection gemm (two mixers)", (na, W): "projection gemm (attention)", (W, par.out_cols): "output gemm (two mixers)",
+                 (W, att.out_cols): "output gemm (attention)", (2 * F, W): "gate/up gemm", (W, F): "down gemm", (VOCAB, W): "head gemm"}
+        classify = _by_shape(names)
+        roofs = {"projection gemm (two mixers)": (2 * par.proj.shape[0] * W, 0), "projection gemm (attention)": (2 * na * W, 0), "output gemm (two mixers)": (2 * W * par.out_cols, 0),
+                 "output gemm (attention)": (2 * W * att.out_cols, 0), "gate/up gemm": (4 * F * W, 0), "down gemm": (2 * F * W, 0), "head gemm": (2 * VOCAB * W, 0),
+                 "attention (window)": (2 * batch * min(L, win) * D.row, 0), "attention (full)": (2 * batch * L * D.row, 0), "ft_mm_decode": (2 * batch * M.state_size * 4, 0)}
+        def label_d(fn, raw):
+            if fn == "ft_gqa_decode":
+                return "attention (window)" if raw[11] else "attention (full)"
+            return classify(fn, raw)
+        dtable = kernel_table(one, label_d, roofs, bw, fl)
+    eng.check()
+    return {"prefill_ms": round(pre_ms, 3), "prefill_tokens_per_s": round(prompt / pre_ms * 1e3), "decode_ms_per_step": round(dec_ms, 4),
+            "decode_tokens_per_s": round(batch / dec_ms * 1e3), "prefill_kernels": table, "decode_kernels": dtable}
+
+
 def run_llama(size, layers, batch, prompt, ctx, steps, kernels=True):
     bw, fl, _ = peaks()
     s = SIZES[size]
@@ -210,13 +300,15 @@ def run_llama(size, layers, batch, prompt, ctx, steps, kernels=True):
             "decode_tokens_per_s": round(batch / dec_ms * 1e3), "prefill_kernels": table, "decode_kernels": dtable}
 
 
-def main(sizes="1k,2k,4k", layers=4, batch=8, prompt=4096, ctx=2048, steps=64, kernels=True) -> int:
+def main(sizes="1k,2k,4k", layers=4, batch=8, prompt=4096, ctx=2048, steps=64, kernels=True, models="") -> int:
     torch.cuda.set_device(0)
     _, _, of = peaks()
     res = {}
     for size in sizes.split(","):
         res[size] = {}
-        for name, run in (("ginisun", run_ginisun), ("llama", run_llama)):
+        for name, run in (("ginisun", run_ginisun), ("pufevik", run_pufevik), ("llama", run_llama)):
+            if models and name not in models.split(","):
+                continue
             res[size][name] = run(size, layers, batch, prompt, ctx, steps, kernels)
             torch.cuda.empty_cache()
     print(json.dumps({"bench": "serving", "layers": layers, "decode_batch": batch, "prompt": prompt, "context": ctx, "dtype": "bf16", "peaks": of,

@@ -158,3 +158,54 @@ def greedy(cfg, weights, prompt, new):
     for _ in range(new):
         seq.append(int(np.argmax(forward(cfg, weights, seq)[-1])))
     return seq[len(prompt):]
+
+
+def bf16(a):
+    """Values rounded to bf16."""
+    u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
+    return (((u.astype(np.uint64) + 0x7FFF + ((u >> 16) & 1)) >> 16) << 16).astype(np.uint32).view(np.float32).reshape(np.shape(a))
+
+
+def random_model(seed, kinds="pa", vocab=90, width=56, ff=72, heads=4, kv_heads=2, dim=16, vdim=24, rot=8, base=10000.0, scale=None, v_mix=True, window=20, mem_heads=3,
+                 mem_dim=16, mem_vdim=16, cap=6.0, left_scale=0.7, right_scale=0.6, sink=1.5, emb_scale=3.0, eps=1e-5, overrides=None):
+    """A configuration with one layer per letter of ``kinds`` (``p``: two mixers side by side, ``a``: full attention) and random weights rounded to bf16.
+    ``overrides[i]`` replaces keyword values for layer i; ``ff=0`` leaves the feed-forward out."""
+    rng = np.random.default_rng(seed)
+
+    def mat(o, i, s=1.0):
+        return bf16(rng.standard_normal((o, i)) * s / math.sqrt(i))
+
+    def vec(n, mean=1.0, s=0.2):
+        return bf16(mean + s * rng.standard_normal(n))
+    W, layers = {"embed": bf16(rng.standard_normal((vocab, width)) / emb_scale)}, []
+    for i, kind in enumerate(kinds):
+        o = dict(ff=ff, heads=heads, kv_heads=kv_heads, dim=dim, vdim=vdim, rot=rot, base=base, scale=scale, v_mix=v_mix, window=window, mem_heads=mem_heads, mem_dim=mem_dim,
+                 mem_vdim=mem_vdim, cap=cap, left_scale=left_scale, right_scale=right_scale, sink=sink)
+        o.update((overrides or {}).get(i, {}))
+        p, H, G, d, dv = f"l{i}.", o["heads"], o["kv_heads"], o["dim"], o["vdim"]
+        att = dict(heads=H, kv_heads=G, dim=d, vdim=dv, rot=dict(base=o["base"], dims=o["rot"]), scale=o["scale"] if o["scale"] is not None else d ** -0.5)
+
+        def attention(q, whole, gate_rows):
+            W.update({q + "q": mat(H * d, width), q + "k": mat(G * d, width), q + "v": mat(G * dv, width), q + "g": mat(gate_rows, width), q + "o": mat(width, H * dv),
+                      q + "q.norm": vec(H * d if whole else d, 1.4), q + "k.norm": vec(G * d if whole else d, 1.4)})
+        if kind == "a":
+            attention(p + "mix.", False, H * dv)
+            mixer = dict(att, v_mix=o["v_mix"])
+            if o["v_mix"]:
+                W[p + "mix.vmix"] = bf16(np.float32(0.3 + 0.4 * rng.random()))
+        else:
+            attention(p + "mix.left.", True, H)
+            W[p + "mix.left.sink"] = bf16(o["sink"] * rng.standard_normal(H))
+            mh, md, mv, q = o["mem_heads"], o["mem_dim"], o["mem_vdim"], p + "mix.right."
+            W.update({q + "q": mat(mh * md, width), q + "k": mat(mh * md, width), q + "v": mat(mh * mv, width), q + "g": mat(mh * mv, width), q + "o": mat(width, mh * mv),
+                      q + "norm": vec(mh * mv), q + "i": mat(mh, width, 2.0), q + "f": mat(mh, width, 2.0), q + "i.b": vec(mh, -1.0, 1.0), q + "f.b": vec(mh, 3.0, 2.0)})
+            mixer = dict(left=dict(att, mask=dict(size=o["window"])), right=dict(heads=mh, dim=md, vdim=mv, gate_cap=o["cap"]), left_scale=o["left_scale"],
+                         right_scale=o["right_scale"])
+        W[p + "norm1"] = vec(width)
+        mlp = None
+        if o["ff"]:
+            mlp = dict(kind="dense", ff=o["ff"])
+            W.update({p + "norm2": vec(width), p + "mlp.gate": mat(o["ff"], width, 1.5), p + "mlp.up": mat(o["ff"], width), p + "mlp.down": mat(width, o["ff"])})
+        layers.append(dict(type="attention" if kind == "a" else "parallel", mixer=mixer, mlp=mlp))
+    W["final.norm"], W["head"] = vec(width), mat(vocab, width, 2.0)
+    return dict(architecture="Pufevik", vocab=vocab, width=width, norm=dict(eps=eps), embedding=dict(scale=emb_scale), layers=layers), W
