@@ -11,8 +11,8 @@
 //   m_t = F_t + R_t,   weight of key s at t: e^(u_s - R_t),   weight of the state before the stretch: e^(m_in - R_t)
 // so nothing but differences of nearby numbers is exponentiated, and every exponent is at most zero.
 //
-//   ft_mm_walk     prompts (bf16): a CTA walks a segment of a sequence in chunks of 64 tokens with 64 value columns of one head's state in registers. Long
-//                  sequences are cut into segments that walk at the same time: a first pass collects every segment's own contribution,
+//   ft_mm_walk     prompts (bf16, tcgen05): a CTA walks a segment of a sequence in chunks of 128 tokens with 128 value columns of one head's state in registers.
+//                  Long sequences are cut into segments that walk at the same time: a first pass collects every segment's own contribution,
 //                  ft_mm_merge chains them into the state ahead of each segment, a second pass produces the outputs. f32 quantities (weighted values, state, weights
 //                  of the keys) meet the 16-bit tensor cores as sums of two bf16 numbers.
 //   ft_mm_rows     one token after another, any sizes, f32 or bf16 data (the 32-bit path)
@@ -120,23 +120,33 @@ __global__ void __launch_bounds__(256) mm_rows_kernel(MemIO io, MemDims D) {
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// chunk walk: grid (segments, H, ceil(v16 / 64)), 256 threads
+// chunk walk (tcgen05): grid (segments, H, ceil(v16 / 128)), 256 threads. A chunk is 128 tokens; a CTA keeps 128 value columns of the state, transposed: thread
+// (row v, half) holds S[half of the key dimensions][v] in registers, and as bf16 high and low parts in TMEM, where they are an operand of the tensor cores.
+//
+//   scores [t][s]  = Q K^T                                                          (Q, K from shared memory)
+//   O1 [v][t]      = S^T Q^T      (S^T from TMEM, high + low)                       the past, scaled per token when it is read
+//   O2 [v][t]      = V^T P^T      (P = masked, weighted scores, high + low)         the chunk itself
+//   dS [v][d]      = (w V)^T K    (w V: values times their weight in the next state, high + low);  S <- decay S + dS in f32
+//
+// The steps of a chunk depend on one another, so one thread issues everything and all threads do the work in between. Shared memory: Q (reused for w V) | K | V | P;
+// of P's second 64 columns only the lower rows exist. TMEM: [scores, then O2 | O1], later dS over both | S^T high | S^T low.
 // ------------------------------------------------------------------------------------------------------------
-constexpr int MW_C = 64, MW_V = 64, MW_VP = MW_V * 2 + 16;      // chunk, value columns, pitch of 64-column bf16 rows in bytes
+constexpr int MW_C = 128, MW_V = 128, MW_BLK = MW_C * 128;      // chunk, value columns, bytes of a 64-column block of 128 rows
+constexpr uint32_t FT_K_MEMORY = 11;
 
-FT_DEVICE void cp_async16z(uint32_t dst, const void* src, bool live) {       // 16 bytes, or zeros
-  const int n = live ? 16 : 0;
-  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(n) : "memory");
+FT_DEVICE float ex2(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
 }
-FT_DEVICE void ldmatrix_x4(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-FT_DEVICE void ldmatrix_x4_trans(uint32_t (&r)[4], uint32_t addr) {
-  asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-FT_DEVICE void mma_16816(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-  asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-               : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+FT_DEVICE float exp_fast(float x) { return ex2(x * 1.4426950408889634f); }
+FT_DEVICE bool mw_wait(uint64_t* bar, uint32_t parity) {
+  if (mbar_try_wait(bar, parity)) return true;
+  const uint64_t t0 = globaltimer_ns();
+  for (uint32_t i = 1;; i++) {
+    if (mbar_try_wait(bar, parity)) return true;
+    if ((i & 0xff) == 0 && globaltimer_ns() - t0 > 2000000000ull) return false;
+  }
 }
 // two neighbouring f32 values as bf16 high parts and bf16 remainders (16 mantissa bits together)
 FT_DEVICE void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
@@ -146,119 +156,142 @@ FT_DEVICE void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
   hi = *reinterpret_cast<const uint32_t*>(&h);
   lo = *reinterpret_cast<const uint32_t*>(&l);
 }
-__host__ __device__ inline int mw_pitch(int d16) { return d16 * 2 + 16; }
-inline int mw_smem(int d16, bool out) {
-  const int rows = MW_C * MW_VP;
-  return MW_C * mw_pitch(d16) * (out ? 2 : 1) + rows * (out ? 5 : 3) + (out ? 2 * d16 * MW_VP : 0) + (8 * MW_C + d16) * 4;
+// 16-byte chunk c of row r in a block of 128-byte rows, as TMA and the tensor cores place it
+FT_DEVICE uint32_t sw128(int r, int c) { return (uint32_t)(r * 128 + ((c ^ (r & 7)) << 4)); }
+
+__host__ __device__ constexpr int mw_q_bytes(int nq) { return (nq < 4 ? 4 : nq) * MW_BLK; }      // at least the four blocks of w V
+__host__ __device__ constexpr int mw_smem(int nq, bool out) {
+  return mw_q_bytes(nq) + nq * MW_BLK + 2 * MW_BLK + (out ? 3 * MW_BLK : 0) + (8 * MW_C + 64 * nq) * 4 + 64 + 1024;
 }
 
-// MT: 16-row tiles of the state per warp (d16 <= 128 MT). OUT: outputs from the state ahead of the segment; else: the segment's own contribution, into
-// scratch state [scratch index + 1], with m relative to an empty past and the sum of the forget gates beside it.
-template <int MT, bool OUT>
-__global__ void __launch_bounds__(256, 1) mm_walk_kernel(MemIO io, MemDims D, float* __restrict__ scratch) {
-  extern __shared__ __align__(128) uint8_t smem[];
-  const int pd = mw_pitch(D.d16);
-  uint8_t* p = smem;
-  uint8_t* sK = p;              p += MW_C * pd;
-  uint8_t* sV = p;              p += MW_C * MW_VP;
-  uint8_t* sWh = p;             p += MW_C * MW_VP;      // values times their weight in the state, high and low parts
-  uint8_t* sWl = p;             p += MW_C * MW_VP;
-  uint8_t* sQ = p;              p += OUT ? MW_C * pd : 0;
-  uint8_t* sPh = p;             p += OUT ? MW_C * MW_VP : 0;      // weights of the keys
-  uint8_t* sPl = p;             p += OUT ? MW_C * MW_VP : 0;
-  uint8_t* sSh = p;             p += OUT ? D.d16 * MW_VP : 0;     // state ahead of the chunk
-  uint8_t* sSl = p;             p += OUT ? D.d16 * MW_VP : 0;
-  float* u = reinterpret_cast<float*>(p);     // [64] i - F
-  float* R = u + MW_C;                        // [64] running maximum of u and m_in
-  float* Fs = R + MW_C;                       // [64] running sum of f
-  float* w = Fs + MW_C;                       // [64] weight in the next state
-  float* rs = w + MW_C;                       // [2][64] row sums of the key weights
-  float* nq = rs + 2 * MW_C;                  // [64] n . q
-  float* n = nq + 2 * MW_C;                   // [d16]
+// NQ: 64-column blocks of the key size. OUT: outputs from the state ahead of the segment; else: the segment's own contribution, into scratch state [scratch index + 1],
+// with m relative to an empty past and the sum of the forget gates beside it.
+template <int NQ, bool OUT>
+__global__ void __launch_bounds__(256, 1) mm_walk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                                                         MemIO io, MemDims D, float* __restrict__ scratch, uint32_t* status) {
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t* sQ = smem;                                    // [NQ] blocks; later w V: high (two blocks), low (two blocks)
+  uint8_t* sK = sQ + mw_q_bytes(NQ);                     // [NQ]
+  uint8_t* sV = sK + NQ * MW_BLK;                        // [2]
+  uint8_t* sP = sV + 2 * MW_BLK;                         // high: block of columns 0..63, half block of columns 64..127; low: the same
+  constexpr int P_LOW = MW_BLK + MW_BLK / 2;
+  float* u = reinterpret_cast<float*>(sP + (OUT ? 3 * MW_BLK : 0));      // [128] i - F
+  float* R = u + MW_C;                                   // [128] running maximum of u and m_in
+  float* w = R + MW_C;                                   // [128] weight in the next state
+  float* ein = w + MW_C;                                 // [128] weight of the past, times the queries' scale
+  float* inv = ein + MW_C;                               // [128] e^(-m), then 1 / denominator
+  float* nq = inv + MW_C;                                // [128] n . q
+  float* rs = nq + MW_C;                                 // [2][128] sums of the key weights
+  float* n = rs + 2 * MW_C;                              // [64 NQ]
+  uint64_t* bars = reinterpret_cast<uint64_t*>(n + 64 * NQ);             // loads, scores, O1, O2, dS
+  uint64_t *b_load = bars, *b_s = bars + 1, *b_o1 = bars + 2, *b_o2 = bars + 3, *b_ds = bars + 4;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
+  float* f_sum = reinterpret_cast<float*>(tmem_slot + 1);                // [1] sum of the chunk's forget gates
+
   const int* sg = io.segs + (size_t)blockIdx.x * SEG_INTS;
   const int row0 = sg[0], rows = sg[1], flags = sg[4], hd = blockIdx.y, v0 = blockIdx.z * MW_V;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t2 = (lane & 3) * 2;
-  const int rt = warp & 3, ch = warp >> 2, mtiles = D.d16 / 16, ksteps = D.d16 / 16;
-  const float scale = rsqrtf((float)D.d);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = (warp & 3) * 32 + lane, half = warp >> 2;
   const bool zero = !OUT || ((flags & SEG_ONLY) && (flags & SEG_ZERO));
   float* slot = io.slots + (size_t)sg[2] * io.slot_stride + hd * D.head();
   const float* in = (flags & SEG_ONLY) ? slot : scratch + (size_t)sg[5] * D.H * D.head() + hd * D.head();
   const size_t n_at = (size_t)D.d16 * D.v16;
-  const __nv_bfloat16* x = reinterpret_cast<const __nv_bfloat16*>(io.x);
+  const float scale = rsqrtf((float)D.d);
+  const int ksteps = D.d16 / 16;
 
-  float S[MT][8][4];
+  if (tid == 0) {
+    for (int i = 0; i < 5; i++) mbar_init(&bars[i], 1);
+    mbar_fence_init();
+    tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
+  }
+  if (warp == 1) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
+  for (int i = tid; i < 64 * NQ; i += 256) n[i] = zero || i >= D.d16 ? 0.f : in[n_at + i];
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tX = *tmem_slot, tA = tX + 256;
+  const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
+
+  auto load_chunk = [&](int c0) {                        // one thread
+    mbar_expect_tx(b_load, ((OUT ? NQ : 0) + NQ + 2) * MW_BLK);
+    for (int c = 0; c < NQ; c++) {
+      if (OUT) tma_load_3d(sQ + c * MW_BLK, &tmQ, b_load, c * 64, hd, row0 + c0);
+      tma_load_3d(sK + c * MW_BLK, &tmK, b_load, c * 64, hd, row0 + c0);
+    }
+    for (int c = 0; c < 2; c++) tma_load_3d(sV + c * MW_BLK, &tmV, b_load, v0 + c * 64, hd, row0 + c0);
+  };
+  if (tid == 0) load_chunk(0);
+
+  float S[NQ * 32];                                      // S[half * 32 NQ + i][v0 + row]
 #pragma unroll
-  for (int a = 0; a < MT; a++)
+  for (int i = 0; i < NQ * 32; i++) {
+    const int d = half * NQ * 32 + i;
+    S[i] = !zero && d < D.d16 && v0 + row < D.v16 ? in[(size_t)d * D.v16 + v0 + row] : 0.f;
+  }
+  auto publish = [&]() {                                 // state registers -> TMEM, as the operand of the next chunk's outputs
 #pragma unroll
-    for (int b = 0; b < 8; b++)
+    for (int i = 0; i < NQ; i++) {
+      uint32_t h[16], l[16];
 #pragma unroll
-      for (int e = 0; e < 2; e++) {
-        const int r = (warp * MT + a) * 16 + g + 8 * e, c = v0 + b * 8 + t2;
-        float2 v = make_float2(0.f, 0.f);
-        if (!zero && r < D.d16 && c < D.v16) v = *reinterpret_cast<const float2*>(in + (size_t)r * D.v16 + c);
-        S[a][b][2 * e] = v.x;
-        S[a][b][2 * e + 1] = v.y;
-      }
-  for (int i = tid; i < D.d16; i += 256) n[i] = zero ? 0.f : in[n_at + i];
+      for (int e = 0; e < 16; e++) split2(S[i * 32 + 2 * e], S[i * 32 + 2 * e + 1], h[e], l[e]);
+      tmem_st_32x32b_x16(tA + lanes + half * NQ * 16 + i * 16, h);
+      tmem_st_32x32b_x16(tA + 128 + lanes + half * NQ * 16 + i * 16, l);
+    }
+    tmem_st_wait();
+  };
+  if (OUT) publish();
   float m_in = OUT ? (zero ? 0.f : in[n_at + D.d16 + ((flags & SEG_ONLY) ? 0 : 2)]) : -INFINITY, f_total = 0.f;
-  auto publish = [&]() {                      // state registers -> shared memory, as the operand of the next chunk's outputs
+
+  float gi[4], gf[4];                                    // raw gates of this lane's tokens of the next chunk (warp 0)
+  auto fetch_gates = [&](int c0) {
 #pragma unroll
-    for (int a = 0; a < MT; a++)
-#pragma unroll
-      for (int b = 0; b < 8; b++)
-#pragma unroll
-        for (int e = 0; e < 2; e++) {
-          const int r = (warp * MT + a) * 16 + g + 8 * e;
-          if (r < D.d16) {
-            uint32_t h, l;
-            split2(S[a][b][2 * e], S[a][b][2 * e + 1], h, l);
-            *reinterpret_cast<uint32_t*>(sSh + r * MW_VP + (b * 8 + t2) * 2) = h;
-            *reinterpret_cast<uint32_t*>(sSl + r * MW_VP + (b * 8 + t2) * 2) = l;
-          }
-        }
-  };
-  auto load_chunk = [&](int c0, int cnt) {
-    const int kv = D.d16 / 8;
-    for (int i = tid; i < MW_C * kv; i += 256) {
-      const int r = i / kv, v = i % kv;
-      const bool live = r < cnt;
-      const __nv_bfloat16* xr = x + (size_t)(row0 + c0 + (live ? r : 0)) * io.ld + v * 8;
-      cp_async16z(smem_u32(sK + r * pd + v * 16), xr + (D.H + hd) * D.d16, live);
-      if (OUT) cp_async16z(smem_u32(sQ + r * pd + v * 16), xr + hd * D.d16, live);
-    }
-    for (int i = tid; i < MW_C * 8; i += 256) {
-      const int r = i >> 3, v = i & 7;
-      const bool live = r < cnt && v0 + v * 8 < D.v16;
-      cp_async16z(smem_u32(sV + r * MW_VP + v * 16), x + (size_t)(row0 + c0 + (live ? r : 0)) * io.ld + 2 * D.H * D.d16 + hd * D.v16 + (live ? v0 + v * 8 : 0), live);
-    }
-    asm volatile("cp.async.commit_group;" ::: "memory");
-  };
-  bool have_state = !zero;
-  if (OUT && have_state) publish();
-  load_chunk(0, min(MW_C, rows));
-  for (int c0 = 0; c0 < rows; c0 += MW_C) {
-    const int cnt = min(MW_C, rows - c0);
-    if (warp == 0) {                          // gates of two neighbouring tokens per lane, running sum and running maximum
-      float f[2], ig[2];
-#pragma unroll
-      for (int e = 0; e < 2; e++) {
-        const int t = lane * 2 + e;
-        f[e] = 0.f;
-        ig[e] = -INFINITY;
-        if (t < cnt) {
-          const float* gr = io.gates + (size_t)(row0 + c0 + t) * io.ldg;
-          ig[e] = soft_cap(gr[hd] + io.bi[hd], D.cap);
-          f[e] = log_sigmoid(soft_cap(gr[D.h8 + hd] + io.bf[hd], D.cap));
-        }
+    for (int e = 0; e < 4; e++) {
+      const int t = c0 + lane * 4 + e;
+      if (t < rows) {
+        const float* gr = io.gates + (size_t)(row0 + t) * io.ldg;
+        gi[e] = gr[hd];
+        gf[e] = gr[D.h8 + hd];
       }
-      float s = f[0] + f[1];
+    }
+  };
+  const float bias_i = io.bi[hd], bias_f = io.bf[hd];
+  if (warp == 0) fetch_gates(0);
+  const uint32_t idesc_s = make_idesc_f16(128, 128, 1, 0, 0), idesc_o2 = make_idesc_f16(128, 128, 1, 1, 0), idesc_o2h = make_idesc_f16(128, 64, 1, 1, 0),
+                 idesc_ds = make_idesc_f16(128, NQ * 64, 1, 1, 1);
+  // K-major operands (rows of 64-column blocks), and the same memory with the contiguous dimension as M or N
+  const uint64_t q_k = make_smem_desc(smem_u32(sQ), 16, 1024, FT_SWZ_128B), k_k = make_smem_desc(smem_u32(sK), 16, 1024, FT_SWZ_128B),
+                 p_k = make_smem_desc(smem_u32(sP), 16, 1024, FT_SWZ_128B), k_mn = make_smem_desc(smem_u32(sK), MW_BLK, 1024, FT_SWZ_128B),
+                 v_mn = make_smem_desc(smem_u32(sV), MW_BLK, 1024, FT_SWZ_128B), w_mn = make_smem_desc(smem_u32(sQ), MW_BLK, 1024, FT_SWZ_128B);
+  bool ok = true;
+  auto fail = [&](uint32_t site) { ft_set_status(status, FT_K_MEMORY, site, blockIdx.x); return false; };
+
+  int c0 = 0;
+  for (int ch = 0; c0 < rows && ok; ch++, c0 += MW_C) {
+    const int cnt = min(MW_C, rows - c0), par = ch & 1;
+    if (warp == 0) {                                     // running sum and running maximum of the gates, four neighbouring tokens a lane
+      float F[4], uu[4];
+      float s = 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const bool live = lane * 4 + e < cnt;
+        s += live ? log_sigmoid(soft_cap(gf[e] + bias_f, D.cap)) : 0.f;
+        F[e] = s;
+        uu[e] = live ? soft_cap(gi[e] + bias_i, D.cap) : -INFINITY;
+      }
+      float tot = s;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
-        const float y = __shfl_up_sync(0xffffffffu, s, o);
-        if (lane >= o) s += y;
+        const float y = __shfl_up_sync(0xffffffffu, tot, o);
+        if (lane >= o) tot += y;
       }
-      const float F0 = s - f[1], F1 = s, u0 = ig[0] - F0, u1 = ig[1] - F1;
-      float mx = fmaxf(u0, u1);
+      const float ahead = tot - s;
+      float mx = -INFINITY;
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        F[e] += ahead;
+        uu[e] -= F[e];
+        mx = fmaxf(mx, uu[e]);
+      }
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const float y = __shfl_up_sync(0xffffffffu, mx, o);
@@ -266,202 +299,222 @@ __global__ void __launch_bounds__(256, 1) mm_walk_kernel(MemIO io, MemDims D, fl
       }
       float before = __shfl_up_sync(0xffffffffu, mx, 1);
       before = fmaxf(lane == 0 ? -INFINITY : before, m_in);
-      const float R0 = fmaxf(before, u0), R1 = fmaxf(R0, u1), Rl = __shfl_sync(0xffffffffu, R1, 31);
-      const int t = lane * 2;
-      u[t] = u0; u[t + 1] = u1;
-      R[t] = R0; R[t + 1] = R1;
-      Fs[t] = F0; Fs[t + 1] = F1;
-      w[t] = __expf(u0 - Rl); w[t + 1] = __expf(u1 - Rl);
+      const float last = fmaxf(__shfl_sync(0xffffffffu, mx, 31), m_in);
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const int t = lane * 4 + e;
+        before = fmaxf(before, uu[e]);
+        u[t] = uu[e];
+        R[t] = before;
+        w[t] = exp_fast(uu[e] - last);
+        ein[t] = exp_fast(m_in - before) * scale;
+        inv[t] = exp_fast(-(F[e] + before));
+      }
+      if (lane == 31) *f_sum = F[3];
+      if (c0 + MW_C < rows) fetch_gates(c0 + MW_C);
     }
-    asm volatile("cp.async.wait_group 0;" ::: "memory");
-    __syncthreads();
-    const float R_last = R[MW_C - 1], decay = __expf(m_in - R_last);
-    // weighted values
-    for (int i = tid; i < MW_C * MW_V / 2; i += 256) {
-      const int t = i >> 5, c = (i & 31) * 4;
-      const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sV + t * MW_VP + c));
-      uint32_t h, l;
-      split2(v.x * w[t], v.y * w[t], h, l);
-      *reinterpret_cast<uint32_t*>(sWh + t * MW_VP + c) = h;
-      *reinterpret_cast<uint32_t*>(sWl + t * MW_VP + c) = l;
-    }
+    tc_fence_before();
+    ok = __syncthreads_and(ok);                          // (1) gates visible; the state's TMEM stores are done
+    tc_fence_after();
+    if (ok && !mw_wait(b_load, par)) ok = fail(1);
     if constexpr (OUT) {
-      // weights of the keys: rows 16 rt, tokens 32 ch
-      float s[4][4];
-#pragma unroll
-      for (int b = 0; b < 4; b++) s[b][0] = s[b][1] = s[b][2] = s[b][3] = 0.f;
-      if (ch * 32 <= rt * 16 + 15) {
-        const uint32_t qa = smem_u32(sQ) + (rt * 16 + (lane & 15)) * pd + (lane >> 4) * 16;
-        const uint32_t ka = smem_u32(sK) + (ch * 32 + (lane & 7) + ((lane >> 4) << 3)) * pd + ((lane >> 3) & 1) * 16;
-        for (int ks = 0; ks < ksteps; ks++) {
-          uint32_t a[4], b0[4], b1[4];
-          ldmatrix_x4(a, qa + ks * 32);
-          ldmatrix_x4(b0, ka + ks * 32);
-          ldmatrix_x4(b1, ka + 16 * pd + ks * 32);
-          mma_16816(s[0], a, b0[0], b0[1]);
-          mma_16816(s[1], a, b0[2], b0[3]);
-          mma_16816(s[2], a, b1[0], b1[1]);
-          mma_16816(s[3], a, b1[2], b1[3]);
+      if (tid == 0 && ok) {
+#pragma unroll 1
+        for (int k = 0; k < ksteps; k++) umma_f16_ss(tX, q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, k_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, idesc_s, k != 0);
+        umma_commit(b_s);
+#pragma unroll 1
+        for (int k = 0; k < ksteps; k++) {
+          const uint64_t b = q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2;
+          umma_f16_ts(tX + 128, tA + k * 8, b, idesc_s, k != 0);
+          umma_f16_ts(tX + 128, tA + 128 + k * 8, b, idesc_s, 1);
         }
+        umma_commit(b_o1);
       }
-#pragma unroll
-      for (int e = 0; e < 2; e++) {
-        const int r = rt * 16 + g + 8 * e;
-        const float Rr = R[r];
-        float sum = 0.f;
-#pragma unroll
-        for (int b = 0; b < 4; b++) {
-          const int c = ch * 32 + b * 8 + t2;
-          const float p0 = c <= r ? s[b][2 * e] * scale * __expf(u[c] - Rr) : 0.f, p1 = c + 1 <= r ? s[b][2 * e + 1] * scale * __expf(u[c + 1] - Rr) : 0.f;
-          sum += p0 + p1;
-          uint32_t h, l;
-          split2(p0, p1, h, l);
-          *reinterpret_cast<uint32_t*>(sPh + r * MW_VP + c * 2) = h;
-          *reinterpret_cast<uint32_t*>(sPl + r * MW_VP + c * 2) = l;
-        }
-        sum += __shfl_xor_sync(0xffffffffu, sum, 1);
-        sum += __shfl_xor_sync(0xffffffffu, sum, 2);
-        if ((lane & 3) == 0) rs[ch * MW_C + r] = sum;
-      }
-      // n . q: four threads per token
-      {
-        const int t = tid >> 2;
+      __syncwarp();
+      {                                                  // n . q: two threads per token
+        const int t = tid >> 1;
         float a = 0.f;
-        if (have_state)
-          for (int v = tid & 3; v < D.d16 / 8; v += 4) {
-            float q8[8];
-            bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sQ + t * pd + v * 16), q8);
+#pragma unroll 4
+        for (int j = tid & 1; j < NQ * 8; j += 2) {
+          float q8[8];
+          bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sQ + (j >> 3) * MW_BLK + sw128(t, j & 7)), q8);
 #pragma unroll
-            for (int e = 0; e < 8; e++) a += q8[e] * n[v * 8 + e];
-          }
-        a += __shfl_xor_sync(0xffffffffu, a, 1);
-        a += __shfl_xor_sync(0xffffffffu, a, 2);
-        if ((tid & 3) == 0) nq[t] = a;
-      }
-    }
-    __syncthreads();
-    if constexpr (OUT) {
-      // outputs: rows 16 rt, value columns 32 ch
-      float o[4][4];
-#pragma unroll
-      for (int b = 0; b < 4; b++) o[b][0] = o[b][1] = o[b][2] = o[b][3] = 0.f;
-      const uint32_t bofs = ((lane & 7) + (((lane >> 3) & 1) << 3)) * MW_VP + (ch * 32 + (lane >> 4) * 8) * 2;
-      const int r0 = rt * 16 + g;
-      const float e0 = __expf(m_in - R[r0]) * scale, e1 = __expf(m_in - R[r0 + 8]) * scale;
-      if (have_state) {
-        const uint32_t qa = smem_u32(sQ) + (rt * 16 + (lane & 15)) * pd + (lane >> 4) * 16;
-        const uint32_t sh = smem_u32(sSh) + bofs, sl = smem_u32(sSl) + bofs;
-        for (int ks = 0; ks < ksteps; ks++) {
-          uint32_t a[4];
-          ldmatrix_x4(a, qa + ks * 32);
-#pragma unroll
-          for (int b = 0; b < 2; b++) {
-            uint32_t h[4], l[4];
-            ldmatrix_x4_trans(h, sh + ks * 16 * MW_VP + b * 32);
-            ldmatrix_x4_trans(l, sl + ks * 16 * MW_VP + b * 32);
-            mma_16816(o[2 * b], a, h[0], h[1]);
-            mma_16816(o[2 * b + 1], a, h[2], h[3]);
-            mma_16816(o[2 * b], a, l[0], l[1]);
-            mma_16816(o[2 * b + 1], a, l[2], l[3]);
-          }
+          for (int e = 0; e < 8; e++) a += q8[e] * n[j * 8 + e];
         }
-#pragma unroll
-        for (int b = 0; b < 4; b++) { o[b][0] *= e0; o[b][1] *= e0; o[b][2] *= e1; o[b][3] *= e1; }
+        a += __shfl_xor_sync(0xffffffffu, a, 1);
+        if ((tid & 1) == 0) nq[t] = a;
       }
-      const uint32_t pofs = (rt * 16 + (lane & 15)) * MW_VP + (lane >> 4) * 16;
-      for (int kt = 0; kt <= rt; kt++) {
-        uint32_t ah[4], al[4];
-        ldmatrix_x4(ah, smem_u32(sPh) + pofs + kt * 32);
-        ldmatrix_x4(al, smem_u32(sPl) + pofs + kt * 32);
+      if (ok && !mw_wait(b_s, par)) ok = fail(2);
+      tc_fence_after();
+      if (half == 0 || row >= 64) {                      // weights of the keys: thread (token row, half of the keys); the upper right quarter is masked whole
+        const float Rt = R[row];
+        float sum = 0.f;
+        uint8_t* dst = half == 0 ? sP : sP + MW_BLK;
+        const int pr = half == 0 ? row : row - 64;
 #pragma unroll
         for (int b = 0; b < 2; b++) {
-          uint32_t v[4];
-          ldmatrix_x4_trans(v, smem_u32(sV) + bofs + kt * 16 * MW_VP + b * 32);
-          mma_16816(o[2 * b], ah, v[0], v[1]);
-          mma_16816(o[2 * b + 1], ah, v[2], v[3]);
-          mma_16816(o[2 * b], al, v[0], v[1]);
-          mma_16816(o[2 * b + 1], al, v[2], v[3]);
-        }
-      }
+          uint32_t sv[32];
+          __syncwarp();
+          tmem_ld_32x32b_x32(tX + lanes + half * 64 + b * 32, sv);
+          tmem_ld_wait();
 #pragma unroll
-      for (int e = 0; e < 2; e++) {
-        const int r = r0 + 8 * e;
-        const float dot = nq[r] * (e ? e1 : e0) + rs[r] + rs[MW_C + r];
-        const float inv = 1.f / (fmaxf(fabsf(dot), __expf(-(Fs[r] + R[r]))) + DEN_EPS);
-        float* dst = io.o + (size_t)(row0 + c0 + r) * D.H * D.v16 + hd * D.v16;
+          for (int c8 = 0; c8 < 4; c8++) {
+            uint32_t h[4], l[4];
 #pragma unroll
-        for (int b = 0; b < 4; b++) {
-          const int c = v0 + ch * 32 + b * 8 + t2;
-          if (r < cnt && c < D.v16) *reinterpret_cast<float2*>(dst + c) = make_float2(o[b][2 * e] * inv, o[b][2 * e + 1] * inv);
-        }
-      }
-    }
-    // the state after the chunk
-    if (warp * MT < mtiles) {
-#pragma unroll
-      for (int a = 0; a < MT; a++)
-#pragma unroll
-        for (int b = 0; b < 8; b++)
-#pragma unroll
-          for (int e = 0; e < 4; e++) S[a][b][e] *= decay;
-      const uint32_t bofs = ((lane & 7) + (((lane >> 3) & 1) << 3)) * MW_VP + (lane >> 4) * 16;
-      for (int kt = 0; kt < MW_C / 16; kt++) {
-        uint32_t a[MT][4];
-#pragma unroll
-        for (int i = 0; i < MT; i++) {
-          const int m0 = min(warp * MT + i, mtiles - 1) * 16;
-          ldmatrix_x4_trans(a[i], smem_u32(sK) + (kt * 16 + ((lane >> 4) << 3) + (lane & 7)) * pd + (m0 + ((lane >> 3) & 1) * 8) * 2);
-        }
-#pragma unroll
-        for (int b = 0; b < 4; b++) {
-          uint32_t h[4], l[4];
-          ldmatrix_x4_trans(h, smem_u32(sWh) + bofs + kt * 16 * MW_VP + b * 32);
-          ldmatrix_x4_trans(l, smem_u32(sWl) + bofs + kt * 16 * MW_VP + b * 32);
-#pragma unroll
-          for (int i = 0; i < MT; i++) {
-            mma_16816(S[i][2 * b], a[i], h[0], h[1]);
-            mma_16816(S[i][2 * b + 1], a[i], h[2], h[3]);
-            mma_16816(S[i][2 * b], a[i], l[0], l[1]);
-            mma_16816(S[i][2 * b + 1], a[i], l[2], l[3]);
+            for (int e = 0; e < 4; e++) {
+              const int s = half * 64 + b * 32 + c8 * 8 + 2 * e;
+              const float2 us = *reinterpret_cast<const float2*>(u + s);
+              const float p0 = s <= row ? __uint_as_float(sv[c8 * 8 + 2 * e]) * scale * exp_fast(us.x - Rt) : 0.f;
+              const float p1 = s + 1 <= row ? __uint_as_float(sv[c8 * 8 + 2 * e + 1]) * scale * exp_fast(us.y - Rt) : 0.f;
+              sum += p0 + p1;
+              split2(p0, p1, h[e], l[e]);
+            }
+            const uint32_t at = sw128(pr, b * 4 + c8);
+            *reinterpret_cast<uint4*>(dst + at) = make_uint4(h[0], h[1], h[2], h[3]);
+            *reinterpret_cast<uint4*>(dst + P_LOW + at) = make_uint4(l[0], l[1], l[2], l[3]);
           }
         }
+        rs[half * MW_C + row] = sum;
+      } else {
+        rs[half * MW_C + row] = 0.f;
+      }
+      fence_proxy_async_smem();
+      tc_fence_before();
+      ok = __syncthreads_and(ok);                        // (2) P complete, scores read
+      tc_fence_after();
+      if (tid == 0 && ok) {
+#pragma unroll 1
+        for (int part = 0; part < 2; part++) {           // high, low
+          const uint64_t p = p_k + part * (P_LOW / 16);
+          for (int k = 0; k < 4; k++) umma_f16_ss(tX, v_mn + k * 128, p + k * 2, idesc_o2, (part | k) != 0);
+          for (int k = 0; k < 4; k++) umma_f16_ss(tX + 64, v_mn + (k + 4) * 128, p + MW_BLK / 16 + k * 2, idesc_o2h, 1);
+        }
+        umma_commit(b_o2);
+      }
+      __syncwarp();
+      if (tid < MW_C) {
+        const float dot = nq[tid] * ein[tid] + rs[tid] + rs[MW_C + tid];
+        inv[tid] = 1.f / (fmaxf(fabsf(dot), inv[tid]) + DEN_EPS);
+      }
+      if (ok && !mw_wait(b_o1, par)) ok = fail(3);       // the queries are consumed
+    }
+    // values times their weight in the next state, over the queries
+    for (int i = tid; i < 2 * MW_C * 8; i += 256) {
+      const int r = (i >> 3) & (MW_C - 1);
+      const uint32_t at = (i >> 10) * MW_BLK + sw128(r, i & 7);
+      const float k = w[r];
+      float v8[8];
+      bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sV + at), v8);
+      uint32_t h[4], l[4];
+#pragma unroll
+      for (int e = 0; e < 4; e++) split2(v8[2 * e] * k, v8[2 * e + 1] * k, h[e], l[e]);
+      *reinterpret_cast<uint4*>(sQ + at) = make_uint4(h[0], h[1], h[2], h[3]);
+      *reinterpret_cast<uint4*>(sQ + 2 * MW_BLK + at) = make_uint4(l[0], l[1], l[2], l[3]);
+    }
+    const float r_last = R[MW_C - 1], decay = exp_fast(m_in - r_last), f_chunk = *f_sum;
+    if constexpr (OUT) {
+      __syncthreads();                                   // (3) denominators
+      if (ok && !mw_wait(b_o2, par)) ok = fail(4);
+      tc_fence_after();
+      float* dst = io.o + (size_t)(row0 + c0) * D.H * D.v16 + hd * D.v16 + v0 + row;
+      const bool live = v0 + row < D.v16;
+#pragma unroll 1
+      for (int b = 0; b < 4; b++) {                      // thread (value row, half of the tokens), sixteen tokens at a time
+        const int t0 = half * 64 + b * 16;
+        uint32_t o1[16], o2[16];
+        __syncwarp();
+        tmem_ld_32x32b_x16(tX + 128 + lanes + t0, o1);
+        tmem_ld_32x32b_x16(tX + lanes + t0, o2);
+        tmem_ld_wait();
+#pragma unroll
+        for (int e = 0; e < 16; e++) {
+          const int t = t0 + e;
+          if (live && t < cnt) dst[(size_t)t * D.H * D.v16] = (__uint_as_float(o1[e]) * ein[t] + __uint_as_float(o2[e])) * inv[t];
+        }
       }
     }
-    for (int i = tid; i < D.d16; i += 256) {
-      float a = 0.f;
-#pragma unroll 8
-      for (int t = 0; t < MW_C; t++) a += w[t] * __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(sK + t * pd + i * 2));
-      n[i] = n[i] * decay + a;                // read by the next chunk only: the barrier below and the one after its loads lie in between
+    fence_proxy_async_smem();
+    tc_fence_before();
+    ok = __syncthreads_and(ok);                          // (4) w V complete, outputs read
+    tc_fence_after();
+    if (tid == 0 && ok) {
+#pragma unroll 1
+      for (int k = 0; k < 8; k++) {
+        umma_f16_ss(tX, w_mn + k * 128, k_mn + k * 128, idesc_ds, k != 0);
+        umma_f16_ss(tX, w_mn + 2 * (MW_BLK / 16) + k * 128, k_mn + k * 128, idesc_ds, 1);
+      }
+      umma_commit(b_ds);
     }
-    const float f_last = Fs[MW_C - 1];
-    m_in = f_last + R_last;
-    f_total += f_last;
-    have_state = true;
-    __syncthreads();
-    if (c0 + MW_C < rows) {
-      load_chunk(c0 + MW_C, min(MW_C, rows - c0 - MW_C));
-      if (OUT) publish();
+    __syncwarp();
+    {                                                    // n <- decay n + sum_t w_t k_t: a lane takes eight columns of every eighth token
+      const int tg = lane >> 2;
+      for (int j = warp * 4 + (lane & 3); j < NQ * 8; j += 32) {
+        float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+        for (int i = 0; i < MW_C / 8; i++) {
+          const int t = i * 8 + tg;
+          float k8[8];
+          bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sK + (j >> 3) * MW_BLK + sw128(t, j & 7)), k8);
+          const float wt = w[t];
+#pragma unroll
+          for (int e = 0; e < 8; e++) a[e] += wt * k8[e];
+        }
+#pragma unroll
+        for (int e = 0; e < 8; e++) {
+          a[e] += __shfl_xor_sync(0xffffffffu, a[e], 4);
+          a[e] += __shfl_xor_sync(0xffffffffu, a[e], 8);
+          a[e] += __shfl_xor_sync(0xffffffffu, a[e], 16);
+        }
+        if (tg == 0) {
+#pragma unroll
+          for (int e = 0; e < 8; e++) n[j * 8 + e] = n[j * 8 + e] * decay + a[e];
+        }
+      }
+    }
+    if (ok && !mw_wait(b_ds, par)) ok = fail(5);
+    ok = __syncthreads_and(ok);                          // (5) everybody is done with the chunk's shared memory
+    if (!ok) break;
+    if (tid == 0 && c0 + MW_C < rows) load_chunk(c0 + MW_C);
+    __syncwarp();
+    tc_fence_after();
+#pragma unroll
+    for (int i = 0; i < NQ; i++) {
+      uint32_t x[32];
+      tmem_ld_32x32b_x32(tX + lanes + half * NQ * 32 + i * 32, x);
+      tmem_ld_wait();
+#pragma unroll
+      for (int e = 0; e < 32; e++) S[i * 32 + e] = S[i * 32 + e] * decay + __uint_as_float(x[e]);
+    }
+    if (OUT && c0 + MW_C < rows) publish();
+    m_in = f_chunk + r_last;
+    f_total += f_chunk;
+  }
+  if (!ok)
+    for (int i = 0; i < 64; i++) __nanosleep(1000);      // copies in flight land before the shared memory goes away
+  if (ok && (!OUT || (flags & SEG_LAST))) {
+    float* dst = OUT ? slot : scratch + (size_t)(sg[5] + 1) * D.H * D.head() + hd * D.head();
+    if (v0 + row < D.v16) {
+#pragma unroll
+      for (int i = 0; i < NQ * 32; i++) {
+        const int d = half * NQ * 32 + i;
+        if (d < D.d16) dst[(size_t)d * D.v16 + v0 + row] = S[i];
+      }
+    }
+    if (blockIdx.z == 0) {
+      // a slot's n may still be unread by the other CTAs of this head: it moves there later
+      float* nd = OUT ? io.nm + ((size_t)sg[3] * D.H + hd) * (D.d16 + 4) : dst + n_at;
+      for (int i = tid; i < D.d16; i += 256) nd[i] = n[i];
+      if (tid == 0) {
+        nd[D.d16] = m_in;
+        nd[D.d16 + 1] = f_total;
+      }
     }
   }
-  if (OUT && !(flags & SEG_LAST)) return;
-  float* dst = OUT ? slot : scratch + (size_t)(sg[5] + 1) * D.H * D.head() + hd * D.head();
-#pragma unroll
-  for (int a = 0; a < MT; a++)
-#pragma unroll
-    for (int b = 0; b < 8; b++)
-#pragma unroll
-      for (int e = 0; e < 2; e++) {
-        const int r = (warp * MT + a) * 16 + g + 8 * e, c = v0 + b * 8 + t2;
-        if (r < D.d16 && c < D.v16) *reinterpret_cast<float2*>(dst + (size_t)r * D.v16 + c) = make_float2(S[a][b][2 * e], S[a][b][2 * e + 1]);
-      }
-  if (blockIdx.z == 0) {
-    // a slot's n may still be unread by the other CTAs of this head: it moves there later
-    float* nd = OUT ? io.nm + ((size_t)sg[3] * D.H + hd) * (D.d16 + 4) : dst + n_at;
-    for (int i = tid; i < D.d16; i += 256) nd[i] = n[i];
-    if (tid == 0) {
-      nd[D.d16] = m_in;
-      nd[D.d16 + 1] = f_total;
-    }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 1) {
+    tc_fence_after();
+    tmem_dealloc(tX, 512);
   }
 }
 
@@ -687,16 +740,16 @@ bool make_dims(MemDims& D, int H, int d, int dv, float cap) {
 constexpr int SMEM_MAX = 232448;
 int rows_smem(int d16) { return (d16 * MR_COLS + 3 * d16 + 8 * 32 + 32) * 4; }
 
-template <int MT, bool OUT>
-int launch_walk(dim3 grid, cudaStream_t st, const MemIO& io, const MemDims& D, float* scratch) {
+template <int NQ, bool OUT>
+int launch_walk(const CUtensorMap (&m)[3], dim3 grid, cudaStream_t st, const MemIO& io, const MemDims& D, float* scratch) {
   static bool done[64] = {};
   int dev = 0;
   FT_CUDA_TRY(cudaGetDevice(&dev));
   if (dev < 64 && !done[dev]) {
-    FT_CUDA_TRY(cudaFuncSetAttribute(mm_walk_kernel<MT, OUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX));
+    FT_CUDA_TRY(cudaFuncSetAttribute(mm_walk_kernel<NQ, OUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, mw_smem(NQ, OUT)));
     done[dev] = true;
   }
-  mm_walk_kernel<MT, OUT><<<grid, 256, mw_smem(D.d16, OUT), st>>>(io, D, scratch);
+  mm_walk_kernel<NQ, OUT><<<grid, 256, mw_smem(NQ, OUT), st>>>(m[0], m[1], m[2], io, D, scratch, ft_status_ptr());
   return (int)cudaGetLastError();
 }
 
@@ -721,24 +774,35 @@ int launch_decode(int ctas, int B, cudaStream_t st, const MemDecode& A, const Me
 }  // namespace
 
 // Whether ft_mm_walk takes these head sizes.
-FT_EXPORT int ft_mm_walk_fits(int d, int dv) {
-  const int d16 = (d + 15) & ~15;
-  return d >= 1 && dv >= 1 && d16 <= 256 && mw_smem(d16, true) <= SMEM_MAX;
-}
+FT_EXPORT int ft_mm_walk_fits(int d, int dv) { return d >= 1 && dv >= 1 && d <= 256; }
 
 // Prompt stretches of a ragged batch in bf16. x [rows][ld]: queries H x d16 | keys H x d16 | values H x v16 (16-byte aligned, ld a multiple of 8); gates f32 [rows][ldg]: input
 // gates, at column h8 = H rounded up to 8 forget gates; biases f32 [H]. segs int[nsegs][8] {first row, rows, slot, sequence, flags, scratch state, 0, 0}, flags 1: the only segment
 // of its stretch (its state comes from the slot), 2: last, 4: the sequence starts (zero state). out = 0: contributions of the segments into scratch states [scratch state + 1] (f32 [H][d16 v16 + d16 + 4]
 // each); out = 1: outputs o f32 [rows][H * v16], last segments leave S in their slot (f32 slots of slot_stride) and n, m in nm f32 [sequence][H][d16 + 4].
-FT_EXPORT int ft_mm_walk(const void* x, int64_t ld, const float* gates, int64_t ldg, const float* bias_i, const float* bias_f, float cap, const int* segs, int nsegs, int H, int d,
+FT_EXPORT int ft_mm_walk(const void* x, int64_t ld, int rows, const float* gates, int64_t ldg, const float* bias_i, const float* bias_f, float cap, const int* segs, int nsegs, int H, int d,
                          int dv, float* slots, int64_t slot_stride, float* scratch, float* nm, float* o, int out, cudaStream_t st) {
   MemDims D;
-  if (nsegs < 1 || !make_dims(D, H, d, dv, cap) || (ld & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (!out && !scratch) || (out && (!o || !nm))) return FT_ERR_ARG;
+  if (nsegs < 1 || rows < 1 || !make_dims(D, H, d, dv, cap) || (ld & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (!out && !scratch) || (out && (!o || !nm))) return FT_ERR_ARG;
   if (!ft_mm_walk_fits(d, dv)) return FT_ERR_TOO_LARGE;
   const MemIO io{x, ld, gates, ldg, bias_i, bias_f, segs, slots, (size_t)slot_stride, nm, o};
   const dim3 grid(nsegs, H, (D.v16 + MW_V - 1) / MW_V);
-  if (D.d16 <= 128) return out ? launch_walk<1, true>(grid, st, io, D, scratch) : launch_walk<1, false>(grid, st, io, D, scratch);
-  return out ? launch_walk<2, true>(grid, st, io, D, scratch) : launch_walk<2, false>(grid, st, io, D, scratch);
+  int dev = 0;
+  FT_CUDA_TRY(cudaGetDevice(&dev));
+  FT_CUDA_TRY(ft_bind_context(dev));
+  CUtensorMap m[3];
+  const __nv_bfloat16* xp = (const __nv_bfloat16*)x;
+  const uint64_t dp = (uint64_t)D.d16 * 2, vp = (uint64_t)D.v16 * 2, lp = (uint64_t)ld * 2;
+  int r = ft_make_tmap_3d(&m[0], xp, 2, true, D.d16, H, rows, dp, lp, 64, 1, MW_C, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!r) r = ft_make_tmap_3d(&m[1], xp + (size_t)H * D.d16, 2, true, D.d16, H, rows, dp, lp, 64, 1, MW_C, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!r) r = ft_make_tmap_3d(&m[2], xp + (size_t)2 * H * D.d16, 2, true, D.v16, H, rows, vp, lp, 64, 1, MW_C, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (r) return r;
+#define FT_MW(N) return out ? launch_walk<N, true>(m, grid, st, io, D, scratch) : launch_walk<N, false>(m, grid, st, io, D, scratch)
+  if (D.d16 <= 64) FT_MW(1);
+  if (D.d16 <= 128) FT_MW(2);
+  if (D.d16 <= 192) FT_MW(3);
+  FT_MW(4);
+#undef FT_MW
 }
 
 // seqs int4[nseq] {scratch state of the first segment, segments, slot, 1 if the sequence starts}: turns the contributions left by ft_mm_walk into the states ahead of

@@ -29,8 +29,8 @@ from .llama_gen import GenerationConfig, sample_next
 
 PAGE = 16
 DECODE_ROWS = 16
-MEMORY_CHUNK = 64                    # tokens that a recurrent layer takes at once
-SEGMENT_MIN, SEGMENT_CTAS = 256, 296
+MEMORY_CHUNK = 128                   # tokens that a recurrent layer takes at once
+SEGMENT_MIN, SEGMENT_CTAS = 256, 148
 
 
 @dataclass

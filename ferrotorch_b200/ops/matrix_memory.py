@@ -1,7 +1,7 @@
 """Matrix memory (the mLSTM cell of xLSTM) on the kernels of ``csrc/kernels/matrix_memory.cu``: per head an f32 matrix and vector that decay and take in outer products
 under log-domain gates with a soft limit, a normalised read-out, a norm per head, an output gate and a scale.
 
-Prompts walk chunks of 64 tokens on the tensor cores, long ones in several segments at the same time; a decode step reads and writes the state once. f32 data and
+Prompts walk chunks of 128 tokens on the tensor cores, long ones in several segments at the same time; a decode step reads and writes the state once. f32 data and
 sizes beyond the walk kernel go token by token.
 """
 from __future__ import annotations
@@ -15,7 +15,7 @@ from .. import _lib
 from .gqa_attention import pack_head_vector
 from .streams import padded_vector, round_up
 
-VALUE_SLICE = 64                     # value columns per CTA of the walk kernel
+VALUE_SLICE = 128                    # value columns per CTA of the walk kernel
 MAX_DECODE_SIZE = 1024
 
 
@@ -76,7 +76,8 @@ def matrix_memory_rows(x: torch.Tensor, gates: torch.Tensor, w: MemoryWeights, b
     plan = batch.memory_plan(D.heads * -(-D.v16 // VALUE_SLICE) if walk else 0)
     o = torch.empty(T, D.out_cols, device=x.device, dtype=torch.float32)
     nm = torch.empty(plan.sequences, D.heads * (D.d16 + 4), device=x.device, dtype=torch.float32)
-    head = (x, x.stride(0), gates, gates.stride(0), w.bias_i, w.bias_f, D.cap)
+    vectors = (gates, gates.stride(0), w.bias_i, w.bias_f, D.cap)
+    head = (x, x.stride(0), T, *vectors)
     if walk:
         scratch = torch.empty(plan.scratch * D.state_size, device=x.device, dtype=torch.float32) if plan.scratch else None
         if plan.scratch:
@@ -84,7 +85,7 @@ def matrix_memory_rows(x: torch.Tensor, gates: torch.Tensor, w: MemoryWeights, b
             _lib.call("ft_mm_merge", plan.chains, plan.sequences, D.heads, D.dim, D.vdim, states, states.stride(0), scratch, S)
         _lib.call("ft_mm_walk", *head, plan.segments, plan.segments.shape[0], D.heads, D.dim, D.vdim, states, states.stride(0), scratch, nm, o, 1, S)
     else:
-        _lib.call("ft_mm_rows", *head, plan.segments, plan.segments.shape[0], D.heads, D.dim, D.vdim, states, states.stride(0), nm, o, int(f32), S)
+        _lib.call("ft_mm_rows", x, x.stride(0), *vectors, plan.segments, plan.segments.shape[0], D.heads, D.dim, D.vdim, states, states.stride(0), nm, o, int(f32), S)
     gate = x[:, D.gate_col:]
     _lib.call("ft_mm_finish", o, T, gate, gate.stride(0), w.norm, D.eps, D.out_scale, out, out.stride(0), D.heads, D.dim, D.vdim, plan.chains, plan.sequences, nm, states,
               states.stride(0), int(f32), S)
