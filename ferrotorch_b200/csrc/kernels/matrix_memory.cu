@@ -13,8 +13,8 @@
 //
 //   ft_mm_walk     prompts (bf16, tcgen05): a CTA walks a segment of a sequence in chunks of 128 tokens with 128 value columns of one head's state in registers.
 //                  Long sequences are cut into segments that walk at the same time: a first pass collects every segment's own contribution,
-//                  ft_mm_merge chains them into the state ahead of each segment, a second pass produces the outputs. f32 quantities (weighted values, state, weights
-//                  of the keys) meet the 16-bit tensor cores as sums of two bf16 numbers.
+//                  ft_mm_merge chains them into the state ahead of each segment, a second pass produces the outputs. What enters the states meets the
+//                  16-bit tensor cores as sums of two bf16 numbers.
 //   ft_mm_rows     one token after another, any sizes, f32 or bf16 data (the 32-bit path)
 //   ft_mm_finish   norm, gate, scale of the outputs; moves n and m of the finished stretch into the slots
 //   ft_mm_decode   one token per sequence from split-K planes: the state is read and written once; the CTAs of a head form a cluster
@@ -41,6 +41,10 @@ template <typename T> FT_DEVICE float one(T v);
 template <> FT_DEVICE float one<float>(float v) { return v; }
 template <> FT_DEVICE float one<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
 
+template <typename T> FT_DEVICE T to(float v);
+template <> FT_DEVICE float to<float>(float v) { return v; }
+template <> FT_DEVICE __nv_bfloat16 to<__nv_bfloat16>(float v) { return __float2bfloat16(v); }
+
 // A segment of a sequence's new tokens: {first row, rows, state slot, sequence, flags, scratch state}
 constexpr int SEG_INTS = 8, SEG_ONLY = 1, SEG_LAST = 2, SEG_ZERO = 4;      // ONLY: state from the slot, not from scratch; ZERO: the sequence starts, its slot's content is void
 struct MemIO {
@@ -53,7 +57,7 @@ struct MemIO {
   float* slots;                      // [slot][slot_stride]
   size_t slot_stride;
   float* nm;                         // [sequence][H][d16 + 4]: n and m after the stretch
-  float* o;                          // [rows][H * v16] f32
+  void* o;                           // [rows][H * v16] in the data type
 };
 
 // ------------------------------------------------------------------------------------------------------------
@@ -106,7 +110,7 @@ __global__ void __launch_bounds__(256) mm_rows_kernel(MemIO io, MemDims D) {
       float a = 0.f;
 #pragma unroll
       for (int g = 0; g < 8; g++) a += red[g * 32 + c];
-      if (col < D.v16) io.o[(size_t)(row0 + t) * D.H * D.v16 + hd * D.v16 + col] = a / (fmaxf(fabsf(nq), expf(-m)) + DEN_EPS);
+      if (col < D.v16) reinterpret_cast<T*>(io.o)[(size_t)(row0 + t) * D.H * D.v16 + hd * D.v16 + col] = to<T>(a / (fmaxf(fabsf(nq), expf(-m)) + DEN_EPS));
     }
     __syncthreads();
   }
@@ -120,18 +124,27 @@ __global__ void __launch_bounds__(256) mm_rows_kernel(MemIO io, MemDims D) {
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// chunk walk (tcgen05): grid (segments, H, ceil(v16 / 128)), 256 threads. A chunk is 128 tokens; a CTA keeps 128 value columns of the state, transposed: thread
-// (row v, half) holds S[half of the key dimensions][v] in registers, and as bf16 high and low parts in TMEM, where they are an operand of the tensor cores.
+// chunk walk (tcgen05): grid (segments, H, ceil(v16 / 128)), 384 threads. A chunk is 128 tokens; a CTA keeps 128 value columns of the state, transposed: thread
+// (row v, half) of the first eight warps holds S[half of the key dimensions][v] in f32 registers, and as bf16 in TMEM, where it is an operand of the tensor cores.
 //
 //   scores [t][s]  = Q K^T                                                          (Q, K from shared memory)
-//   O1 [v][t]      = S^T Q^T      (S^T from TMEM, high + low)                       the past, scaled per token when it is read
-//   O2 [v][t]      = V^T P^T      (P = masked, weighted scores, high + low)         the chunk itself
+//   O1 [v][t]      = S^T Q^T      (S^T from TMEM)                                   the past, scaled per token when it is read
+//   nq [t]         = Q n          (n: high + low part)
+//   O2 [v][t]      = V^T P^T      (P = masked, weighted scores)                     the chunk itself
 //   dS [v][d]      = (w V)^T K    (w V: values times their weight in the next state, high + low);  S <- decay S + dS in f32
+//   dn [d]         = K^T w        (w: high + low);                                                 n <- decay n + dn in f32
 //
-// The steps of a chunk depend on one another, so one thread issues everything and all threads do the work in between. Shared memory: Q (reused for w V) | K | V | P;
-// of P's second 64 columns only the lower rows exist. TMEM: [scores, then O2 | O1], later dS over both | S^T high | S^T low.
+// What enters the state (w V, w) and the normaliser meets the 16-bit tensor cores as sums of two bf16 numbers, so that states are exact to 16 mantissa bits per
+// addend; the read-out takes P and S in bf16, as attention takes its weights.
+//
+// Warps 0..7: weights of the keys, outputs, state. Warp 8: issues copies and products. Warps 9..11: w V; warp 9 also the gates of the next chunk. Named barriers separate
+// the steps of a chunk, which depend on one another. Shared memory: Q (then w V) | K | V | P (of its second 64 columns only the lower rows exist) | n and w as
+// operands. TMEM: [scores, then O2 | O1], later dS over both | S^T | nq | dn.
 // ------------------------------------------------------------------------------------------------------------
 constexpr int MW_C = 128, MW_V = 128, MW_BLK = MW_C * 128;      // chunk, value columns, bytes of a 64-column block of 128 rows
+constexpr int MW_THREADS = 384, MW_GATES = 5 * MW_C + 4;        // floats of one chunk's gate arrays
+constexpr int MW_VEC = 16 * 128;                                // bytes of a 64-column block of a 16-row operand (rows: high, low, zeros)
+constexpr int MW_REGS = 168, MW_REGS_STATE = 208, MW_REGS_HELP = 88;
 constexpr uint32_t FT_K_MEMORY = 11;
 
 FT_DEVICE float ex2(float x) {
@@ -148,135 +161,121 @@ FT_DEVICE bool mw_wait(uint64_t* bar, uint32_t parity) {
     if ((i & 0xff) == 0 && globaltimer_ns() - t0 > 2000000000ull) return false;
   }
 }
+FT_DEVICE void bar_named(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+template <int N> FT_DEVICE void reg_inc() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(N)); }
+template <int N> FT_DEVICE void reg_dec() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(N)); }
 // two neighbouring f32 values as bf16 high parts and bf16 remainders (16 mantissa bits together)
-FT_DEVICE void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+FT_DEVICE uint32_t pack2(float a, float b) {
   const __nv_bfloat162 h = __floats2bfloat162_rn(a, b);
-  const float2 f = __bfloat1622float2(h);
-  const __nv_bfloat162 l = __floats2bfloat162_rn(a - f.x, b - f.y);
-  hi = *reinterpret_cast<const uint32_t*>(&h);
-  lo = *reinterpret_cast<const uint32_t*>(&l);
+  return *reinterpret_cast<const uint32_t*>(&h);
+}
+FT_DEVICE void split2(float a, float b, uint32_t& hi, uint32_t& lo) {
+  hi = pack2(a, b);
+  lo = pack2(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
 }
 // 16-byte chunk c of row r in a block of 128-byte rows, as TMA and the tensor cores place it
 FT_DEVICE uint32_t sw128(int r, int c) { return (uint32_t)(r * 128 + ((c ^ (r & 7)) << 4)); }
+// element i of a 16-row operand: high part in row 0, remainder in row 1
+FT_DEVICE void put_vec(uint8_t* base, int i, float v) {
+  uint8_t* b = base + (i >> 6) * MW_VEC;
+  const int e = i & 63;
+  const __nv_bfloat16 h = __float2bfloat16(v);
+  *reinterpret_cast<__nv_bfloat16*>(b + sw128(0, e >> 3) + (e & 7) * 2) = h;
+  *reinterpret_cast<__nv_bfloat16*>(b + sw128(1, e >> 3) + (e & 7) * 2) = __float2bfloat16(v - __bfloat162float(h));
+}
 
-__host__ __device__ constexpr int mw_q_bytes(int nq) { return (nq < 4 ? 4 : nq) * MW_BLK; }      // at least the four blocks of w V
 __host__ __device__ constexpr int mw_smem(int nq, bool out) {
-  return mw_q_bytes(nq) + nq * MW_BLK + 2 * MW_BLK + (out ? 3 * MW_BLK : 0) + (8 * MW_C + 64 * nq) * 4 + 64 + 1024;
+  return 4 * MW_BLK + nq * MW_BLK + 2 * MW_BLK + (out ? MW_BLK + MW_BLK / 2 : 0) + (nq + 4) * MW_VEC + (2 * MW_GATES + 2 * MW_C) * 4 + 64 + 1024;
 }
 
 // NQ: 64-column blocks of the key size. OUT: outputs from the state ahead of the segment; else: the segment's own contribution, into scratch state [scratch index + 1],
 // with m relative to an empty past and the sum of the forget gates beside it.
 template <int NQ, bool OUT>
-__global__ void __launch_bounds__(256, 1) mm_walk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
-                                                         MemIO io, MemDims D, float* __restrict__ scratch, uint32_t* status) {
+__global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV,
+                                                                MemIO io, MemDims D, float* __restrict__ scratch, uint32_t* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint8_t* sQ = smem;                                    // [NQ] blocks; later w V: high (two blocks), low (two blocks)
-  uint8_t* sK = sQ + mw_q_bytes(NQ);                     // [NQ]
+  uint8_t* sQ = smem;                                    // four blocks: queries [NQ]; later w V: high (two blocks), low (two blocks)
+  uint8_t* sK = sQ + 4 * MW_BLK;                         // [NQ]
   uint8_t* sV = sK + NQ * MW_BLK;                        // [2]
-  uint8_t* sP = sV + 2 * MW_BLK;                         // high: block of columns 0..63, half block of columns 64..127; low: the same
-  constexpr int P_LOW = MW_BLK + MW_BLK / 2;
-  float* u = reinterpret_cast<float*>(sP + (OUT ? 3 * MW_BLK : 0));      // [128] i - F
-  float* R = u + MW_C;                                   // [128] running maximum of u and m_in
-  float* w = R + MW_C;                                   // [128] weight in the next state
-  float* ein = w + MW_C;                                 // [128] weight of the past, times the queries' scale
-  float* inv = ein + MW_C;                               // [128] e^(-m), then 1 / denominator
-  float* nq = inv + MW_C;                                // [128] n . q
-  float* rs = nq + MW_C;                                 // [2][128] sums of the key weights
-  float* n = rs + 2 * MW_C;                              // [64 NQ]
-  uint64_t* bars = reinterpret_cast<uint64_t*>(n + 64 * NQ);             // loads, scores, O1, O2, dS
+  uint8_t* sP = sV + 2 * MW_BLK;                         // block of columns 0..63, half block of columns 64..127
+  uint8_t* sN = sP + (OUT ? MW_BLK + MW_BLK / 2 : 0);    // [NQ] n as an operand
+  uint8_t* sW = sN + NQ * MW_VEC;                        // [2][2] w as an operand, two chunks in turn
+  // per chunk, two in turn: [128] u = i - F | running maximum R of u and m_in | weight in the next state | weight of the past times the queries' scale | e^(-m), then
+  // 1 / denominator | sum of the forget gates
+  float* gate_sets = reinterpret_cast<float*>(sW + 4 * MW_VEC);
+  float* rs = gate_sets + 2 * MW_GATES;                  // [2][128] sums of the key weights
+  uint64_t* bars = reinterpret_cast<uint64_t*>(rs + 2 * MW_C);
   uint64_t *b_load = bars, *b_s = bars + 1, *b_o1 = bars + 2, *b_o2 = bars + 3, *b_ds = bars + 4;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
-  float* f_sum = reinterpret_cast<float*>(tmem_slot + 1);                // [1] sum of the chunk's forget gates
+  volatile int* failed = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int* sg = io.segs + (size_t)blockIdx.x * SEG_INTS;
   const int row0 = sg[0], rows = sg[1], flags = sg[4], hd = blockIdx.y, v0 = blockIdx.z * MW_V;
-  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, row = (warp & 3) * 32 + lane, half = warp >> 2;
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const bool zero = !OUT || ((flags & SEG_ONLY) && (flags & SEG_ZERO));
   float* slot = io.slots + (size_t)sg[2] * io.slot_stride + hd * D.head();
   const float* in = (flags & SEG_ONLY) ? slot : scratch + (size_t)sg[5] * D.H * D.head() + hd * D.head();
   const size_t n_at = (size_t)D.d16 * D.v16;
-  const float scale = rsqrtf((float)D.d);
-  const int ksteps = D.d16 / 16;
 
   if (tid == 0) {
     for (int i = 0; i < 5; i++) mbar_init(&bars[i], 1);
     mbar_fence_init();
+    *failed = 0;
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
   }
-  if (warp == 1) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
-  for (int i = tid; i < 64 * NQ; i += 256) n[i] = zero || i >= D.d16 ? 0.f : in[n_at + i];
+  if (warp == 8) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
+  for (int i = tid; i < (NQ + 4) * MW_VEC / 16; i += MW_THREADS) reinterpret_cast<uint4*>(sN)[i] = make_uint4(0, 0, 0, 0);
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tX = *tmem_slot, tA = tX + 256;
-  const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
-
-  auto load_chunk = [&](int c0) {                        // one thread
-    mbar_expect_tx(b_load, ((OUT ? NQ : 0) + NQ + 2) * MW_BLK);
-    for (int c = 0; c < NQ; c++) {
-      if (OUT) tma_load_3d(sQ + c * MW_BLK, &tmQ, b_load, c * 64, hd, row0 + c0);
-      tma_load_3d(sK + c * MW_BLK, &tmK, b_load, c * 64, hd, row0 + c0);
-    }
-    for (int c = 0; c < 2; c++) tma_load_3d(sV + c * MW_BLK, &tmV, b_load, v0 + c * 64, hd, row0 + c0);
-  };
-  if (tid == 0) load_chunk(0);
-
-  float S[NQ * 32];                                      // S[half * 32 NQ + i][v0 + row]
-#pragma unroll
-  for (int i = 0; i < NQ * 32; i++) {
-    const int d = half * NQ * 32 + i;
-    S[i] = !zero && d < D.d16 && v0 + row < D.v16 ? in[(size_t)d * D.v16 + v0 + row] : 0.f;
-  }
-  auto publish = [&]() {                                 // state registers -> TMEM, as the operand of the next chunk's outputs
-#pragma unroll
-    for (int i = 0; i < NQ; i++) {
-      uint32_t h[16], l[16];
-#pragma unroll
-      for (int e = 0; e < 16; e++) split2(S[i * 32 + 2 * e], S[i * 32 + 2 * e + 1], h[e], l[e]);
-      tmem_st_32x32b_x16(tA + lanes + half * NQ * 16 + i * 16, h);
-      tmem_st_32x32b_x16(tA + 128 + lanes + half * NQ * 16 + i * 16, l);
-    }
-    tmem_st_wait();
-  };
-  if (OUT) publish();
-  float m_in = OUT ? (zero ? 0.f : in[n_at + D.d16 + ((flags & SEG_ONLY) ? 0 : 2)]) : -INFINITY, f_total = 0.f;
-
-  float gi[4], gf[4];                                    // raw gates of this lane's tokens of the next chunk (warp 0)
-  auto fetch_gates = [&](int c0) {
-#pragma unroll
-    for (int e = 0; e < 4; e++) {
-      const int t = c0 + lane * 4 + e;
-      if (t < rows) {
-        const float* gr = io.gates + (size_t)(row0 + t) * io.ldg;
-        gi[e] = gr[hd];
-        gf[e] = gr[D.h8 + hd];
-      }
-    }
-  };
-  const float bias_i = io.bi[hd], bias_f = io.bf[hd];
-  if (warp == 0) fetch_gates(0);
-  const uint32_t idesc_s = make_idesc_f16(128, 128, 1, 0, 0), idesc_o2 = make_idesc_f16(128, 128, 1, 1, 0), idesc_o2h = make_idesc_f16(128, 64, 1, 1, 0),
-                 idesc_ds = make_idesc_f16(128, NQ * 64, 1, 1, 1);
-  // K-major operands (rows of 64-column blocks), and the same memory with the contiguous dimension as M or N
-  const uint64_t q_k = make_smem_desc(smem_u32(sQ), 16, 1024, FT_SWZ_128B), k_k = make_smem_desc(smem_u32(sK), 16, 1024, FT_SWZ_128B),
-                 p_k = make_smem_desc(smem_u32(sP), 16, 1024, FT_SWZ_128B), k_mn = make_smem_desc(smem_u32(sK), MW_BLK, 1024, FT_SWZ_128B),
-                 v_mn = make_smem_desc(smem_u32(sV), MW_BLK, 1024, FT_SWZ_128B), w_mn = make_smem_desc(smem_u32(sQ), MW_BLK, 1024, FT_SWZ_128B);
+  const uint32_t tX = *tmem_slot, tA = tX + 256, tNq = tX + 384, tDn = tX + 400;
+  float m_in = OUT ? (zero ? 0.f : in[n_at + D.d16 + ((flags & SEG_ONLY) ? 0 : 2)]) : -INFINITY;
   bool ok = true;
-  auto fail = [&](uint32_t site) { ft_set_status(status, FT_K_MEMORY, site, blockIdx.x); return false; };
+  // a wait that ran out: everybody keeps to the barriers and leaves at the next chunk
+  auto wait = [&](uint64_t* bar, int par, uint32_t site) {
+    if (ok && !mw_wait(bar, par)) {
+      ft_set_status(status, FT_K_MEMORY, site, blockIdx.x);
+      *failed = 1;
+      ok = false;
+    }
+  };
+  // values times their weight in the next state, over the queries: 16-byte pieces first, first + step, ...
+  auto weigh_values = [&](const float* w, int first, int step) {
+#pragma unroll 2
+    for (int i = first; i < 2 * MW_C * 8; i += step) {
+      const int r = (i >> 3) & (MW_C - 1);
+      const uint32_t at = (i >> 10) * MW_BLK + sw128(r, i & 7);
+      const float k = w[r];
+      float v8[8];
+      bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sV + at), v8);
+      uint32_t h[4], l[4];
+#pragma unroll
+      for (int e = 0; e < 4; e++) split2(v8[2 * e] * k, v8[2 * e + 1] * k, h[e], l[e]);
+      *reinterpret_cast<uint4*>(sQ + at) = make_uint4(h[0], h[1], h[2], h[3]);
+      *reinterpret_cast<uint4*>(sQ + 2 * MW_BLK + at) = make_uint4(l[0], l[1], l[2], l[3]);
+    }
+  };
+  enum { BAR_CHUNK = 1, BAR_P, BAR_DEN, BAR_STATE };
 
-  int c0 = 0;
-  for (int ch = 0; c0 < rows && ok; ch++, c0 += MW_C) {
-    const int cnt = min(MW_C, rows - c0), par = ch & 1;
-    if (warp == 0) {                                     // running sum and running maximum of the gates, four neighbouring tokens a lane
-      float F[4], uu[4];
-      float s = 0.f;
+  if (warp >= 8) {
+    if constexpr (NQ > 2) reg_dec<MW_REGS_HELP>();
+    // gates of a chunk (one warp), four neighbouring tokens a lane: running sum of the forget gates, running maximum
+    const float bias_i = io.bi[hd], bias_f = io.bf[hd], scale = rsqrtf((float)D.d);
+    auto make_gates = [&](int c0, float m, int set) {
+      float* g = gate_sets + set * MW_GATES;
+      const int cnt = min(MW_C, rows - c0);
+      float F[4], uu[4], s = 0.f;
 #pragma unroll
       for (int e = 0; e < 4; e++) {
-        const bool live = lane * 4 + e < cnt;
-        s += live ? log_sigmoid(soft_cap(gf[e] + bias_f, D.cap)) : 0.f;
+        const int t = lane * 4 + e;
+        uu[e] = -INFINITY;
+        if (t < cnt) {
+          const float* gr = io.gates + (size_t)(row0 + c0 + t) * io.ldg;
+          uu[e] = soft_cap(gr[hd] + bias_i, D.cap);
+          s += log_sigmoid(soft_cap(gr[D.h8 + hd] + bias_f, D.cap));
+        }
         F[e] = s;
-        uu[e] = live ? soft_cap(gi[e] + bias_i, D.cap) : -INFINITY;
       }
       float tot = s;
 #pragma unroll
@@ -298,221 +297,264 @@ __global__ void __launch_bounds__(256, 1) mm_walk_kernel(const __grid_constant__
         if (lane >= o) mx = fmaxf(mx, y);
       }
       float before = __shfl_up_sync(0xffffffffu, mx, 1);
-      before = fmaxf(lane == 0 ? -INFINITY : before, m_in);
-      const float last = fmaxf(__shfl_sync(0xffffffffu, mx, 31), m_in);
+      before = fmaxf(lane == 0 ? -INFINITY : before, m);
+      const float last = fmaxf(__shfl_sync(0xffffffffu, mx, 31), m);
 #pragma unroll
       for (int e = 0; e < 4; e++) {
         const int t = lane * 4 + e;
         before = fmaxf(before, uu[e]);
-        u[t] = uu[e];
-        R[t] = before;
-        w[t] = exp_fast(uu[e] - last);
-        ein[t] = exp_fast(m_in - before) * scale;
-        inv[t] = exp_fast(-(F[e] + before));
+        const float wt = exp_fast(uu[e] - last);
+        g[t] = uu[e];
+        g[MW_C + t] = before;
+        g[2 * MW_C + t] = wt;
+        g[3 * MW_C + t] = exp_fast(m - before) * scale;
+        g[4 * MW_C + t] = exp_fast(-(F[e] + before));
+        put_vec(sW + set * 2 * MW_VEC, t, wt);
       }
-      if (lane == 31) *f_sum = F[3];
-      if (c0 + MW_C < rows) fetch_gates(c0 + MW_C);
-    }
-    tc_fence_before();
-    ok = __syncthreads_and(ok);                          // (1) gates visible; the state's TMEM stores are done
-    tc_fence_after();
-    if (ok && !mw_wait(b_load, par)) ok = fail(1);
-    if constexpr (OUT) {
-      if (tid == 0 && ok) {
-#pragma unroll 1
-        for (int k = 0; k < ksteps; k++) umma_f16_ss(tX, q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, k_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, idesc_s, k != 0);
-        umma_commit(b_s);
-#pragma unroll 1
-        for (int k = 0; k < ksteps; k++) {
-          const uint64_t b = q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2;
-          umma_f16_ts(tX + 128, tA + k * 8, b, idesc_s, k != 0);
-          umma_f16_ts(tX + 128, tA + 128 + k * 8, b, idesc_s, 1);
-        }
-        umma_commit(b_o1);
+      if (lane == 31) g[5 * MW_C] = F[3];
+      fence_proxy_async_smem();
+    };
+    auto load_chunk = [&](int c0) {                      // one thread
+      mbar_expect_tx(b_load, ((OUT ? NQ : 0) + NQ + 2) * MW_BLK);
+      for (int c = 0; c < NQ; c++) {
+        if (OUT) tma_load_3d(sQ + c * MW_BLK, &tmQ, b_load, c * 64, hd, row0 + c0);
+        tma_load_3d(sK + c * MW_BLK, &tmK, b_load, c * 64, hd, row0 + c0);
       }
-      __syncwarp();
-      {                                                  // n . q: two threads per token
-        const int t = tid >> 1;
-        float a = 0.f;
-#pragma unroll 4
-        for (int j = tid & 1; j < NQ * 8; j += 2) {
-          float q8[8];
-          bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sQ + (j >> 3) * MW_BLK + sw128(t, j & 7)), q8);
-#pragma unroll
-          for (int e = 0; e < 8; e++) a += q8[e] * n[j * 8 + e];
-        }
-        a += __shfl_xor_sync(0xffffffffu, a, 1);
-        if ((tid & 1) == 0) nq[t] = a;
-      }
-      if (ok && !mw_wait(b_s, par)) ok = fail(2);
+      for (int c = 0; c < 2; c++) tma_load_3d(sV + c * MW_BLK, &tmV, b_load, v0 + c * 64, hd, row0 + c0);
+    };
+    if (warp == 8 && lane == 0) load_chunk(0);
+    if (warp == 9) make_gates(0, m_in, 0);
+    const uint32_t idesc_s = make_idesc_f16(128, 128, 1, 0, 0), idesc_n = make_idesc_f16(128, 16, 1, 0, 0), idesc_o2 = make_idesc_f16(128, 128, 1, 1, 0),
+                   idesc_o2h = make_idesc_f16(128, 64, 1, 1, 0), idesc_ds = make_idesc_f16(128, NQ * 64, 1, 1, 1), idesc_dn = make_idesc_f16(128, 16, 1, 1, 0);
+    // K-major operands (rows of 64-column blocks), and the same memory with the contiguous dimension as M or N
+    const uint64_t q_k = make_smem_desc(smem_u32(sQ), 16, 1024, FT_SWZ_128B), k_k = make_smem_desc(smem_u32(sK), 16, 1024, FT_SWZ_128B),
+                   p_k = make_smem_desc(smem_u32(sP), 16, 1024, FT_SWZ_128B), n_k = make_smem_desc(smem_u32(sN), 16, 1024, FT_SWZ_128B),
+                   k_mn = make_smem_desc(smem_u32(sK), MW_BLK, 1024, FT_SWZ_128B), v_mn = make_smem_desc(smem_u32(sV), MW_BLK, 1024, FT_SWZ_128B),
+                   w_mn = make_smem_desc(smem_u32(sQ), MW_BLK, 1024, FT_SWZ_128B);
+    int c0 = 0;
+    for (int ch = 0; c0 < rows; ch++, c0 += MW_C) {
+      const int par = ch & 1;
+      const float* g = gate_sets + par * MW_GATES;
+      bar_named(BAR_CHUNK, MW_THREADS);                  // gates, state and normaliser are in place
+      if (*failed) break;
       tc_fence_after();
-      if (half == 0 || row >= 64) {                      // weights of the keys: thread (token row, half of the keys); the upper right quarter is masked whole
-        const float Rt = R[row];
-        float sum = 0.f;
-        uint8_t* dst = half == 0 ? sP : sP + MW_BLK;
-        const int pr = half == 0 ? row : row - 64;
+      wait(b_load, par, 1);
+      if constexpr (OUT) {
+        if (warp == 8) {
+          if (lane == 0 && ok) {
 #pragma unroll
-        for (int b = 0; b < 2; b++) {
-          uint32_t sv[32];
-          __syncwarp();
-          tmem_ld_32x32b_x32(tX + lanes + half * 64 + b * 32, sv);
-          tmem_ld_wait();
+            for (int k = 0; k < NQ * 4; k++) umma_f16_ss(tX, q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, k_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, idesc_s, k != 0);
+            umma_commit(b_s);
 #pragma unroll
-          for (int c8 = 0; c8 < 4; c8++) {
-            uint32_t h[4], l[4];
-#pragma unroll
-            for (int e = 0; e < 4; e++) {
-              const int s = half * 64 + b * 32 + c8 * 8 + 2 * e;
-              const float2 us = *reinterpret_cast<const float2*>(u + s);
-              const float p0 = s <= row ? __uint_as_float(sv[c8 * 8 + 2 * e]) * scale * exp_fast(us.x - Rt) : 0.f;
-              const float p1 = s + 1 <= row ? __uint_as_float(sv[c8 * 8 + 2 * e + 1]) * scale * exp_fast(us.y - Rt) : 0.f;
-              sum += p0 + p1;
-              split2(p0, p1, h[e], l[e]);
+            for (int k = 0; k < NQ * 4; k++) {
+              const uint64_t q = q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2;
+              umma_f16_ss(tNq, q, n_k + (k >> 2) * (MW_VEC / 16) + (k & 3) * 2, idesc_n, k != 0);
+              umma_f16_ts(tX + 128, tA + k * 8, q, idesc_s, k != 0);
             }
-            const uint32_t at = sw128(pr, b * 4 + c8);
-            *reinterpret_cast<uint4*>(dst + at) = make_uint4(h[0], h[1], h[2], h[3]);
-            *reinterpret_cast<uint4*>(dst + P_LOW + at) = make_uint4(l[0], l[1], l[2], l[3]);
+            umma_commit(b_o1);
+          }
+          __syncwarp();
+          bar_named(BAR_P, 288);                         // P complete, scores read
+          tc_fence_after();
+          if (lane == 0 && ok) {
+#pragma unroll
+            for (int k = 0; k < 4; k++) umma_f16_ss(tX, v_mn + k * 128, p_k + k * 2, idesc_o2, k != 0);
+#pragma unroll
+            for (int k = 0; k < 4; k++) umma_f16_ss(tX + 64, v_mn + (k + 4) * 128, p_k + MW_BLK / 16 + k * 2, idesc_o2h, 1);
+            umma_commit(b_o2);
+          }
+          __syncwarp();
+        } else {
+          wait(b_o1, par, 3);                            // the queries are consumed
+          weigh_values(g + 2 * MW_C, tid - 288, 96);
+          fence_proxy_async_smem();
+        }
+      }
+      bar_named(BAR_STATE, MW_THREADS);                  // w V complete, outputs read
+      tc_fence_after();
+      if (warp == 8) {
+        if (lane == 0 && ok) {
+          const uint64_t w_k = make_smem_desc(smem_u32(sW + par * 2 * MW_VEC), 16, 1024, FT_SWZ_128B);
+#pragma unroll
+          for (int k = 0; k < 8; k++) {
+            umma_f16_ss(tX, w_mn + k * 128, k_mn + k * 128, idesc_ds, k != 0);
+            umma_f16_ss(tX, w_mn + 2 * (MW_BLK / 16) + k * 128, k_mn + k * 128, idesc_ds, 1);
+          }
+#pragma unroll
+          for (int i = 0; i < (NQ + 1) / 2; i++)
+#pragma unroll
+            for (int k = 0; k < 8; k++) umma_f16_ss(tDn + i * 16, k_mn + i * 2 * (MW_BLK / 16) + k * 128, w_k + (k >> 2) * (MW_VEC / 16) + (k & 3) * 2, idesc_dn, k != 0);
+          umma_commit(b_ds);
+        }
+        __syncwarp();
+        wait(b_ds, par, 5);
+        if (lane == 0 && ok && c0 + MW_C < rows) load_chunk(c0 + MW_C);
+        __syncwarp();
+      }
+      m_in = g[5 * MW_C] + g[2 * MW_C - 1];              // sum of the forget gates + last running maximum
+      if (warp == 9 && c0 + MW_C < rows) make_gates(c0 + MW_C, m_in, par ^ 1);
+    }
+  } else {
+    if constexpr (NQ > 2) reg_inc<MW_REGS_STATE>();
+    const int row = (warp & 3) * 32 + lane, half = warp >> 2, nd = half * 128 + row;      // nd: the element of n that this thread keeps
+    const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
+    const float scale = rsqrtf((float)D.d);
+    float S[NQ * 32];                                    // S[half * 32 NQ + i][v0 + row]
+#pragma unroll
+    for (int i = 0; i < NQ * 32; i++) {
+      const int d = half * NQ * 32 + i;
+      S[i] = !zero && d < D.d16 && v0 + row < D.v16 ? in[(size_t)d * D.v16 + v0 + row] : 0.f;
+    }
+    float n = !zero && nd < D.d16 ? in[n_at + nd] : 0.f, f_total = 0.f;
+    auto publish = [&]() {                               // state and normaliser as operands of the next chunk's outputs
+#pragma unroll
+      for (int i = 0; i < NQ; i++) {
+        uint32_t h[16];
+#pragma unroll
+        for (int e = 0; e < 16; e++) h[e] = pack2(S[i * 32 + 2 * e], S[i * 32 + 2 * e + 1]);
+        tmem_st_32x32b_x16(tA + lanes + half * NQ * 16 + i * 16, h);
+      }
+      if (nd < NQ * 64) put_vec(sN, nd, n);
+      fence_proxy_async_smem();
+      tmem_st_wait();
+    };
+    if (OUT) publish();
+    int c0 = 0;
+    for (int ch = 0; c0 < rows; ch++, c0 += MW_C) {
+      const int cnt = min(MW_C, rows - c0), par = ch & 1;
+      float* u = gate_sets + par * MW_GATES;
+      const float *R = u + MW_C, *ein = u + 3 * MW_C;
+      float* inv = u + 4 * MW_C;
+      tc_fence_before();
+      bar_named(BAR_CHUNK, MW_THREADS);
+      if (*failed) break;
+      tc_fence_after();
+      if constexpr (OUT) {
+        wait(b_s, par, 2);
+        tc_fence_after();
+        float sum = 0.f;
+        if (half == 0 || row >= 64) {                    // weights of the keys: thread (token row, half of the keys); the upper right quarter is masked whole
+          const float Rt = R[row];
+          uint8_t* dst = half == 0 ? sP : sP + MW_BLK;
+          const int pr = half == 0 ? row : row - 64;
+#pragma unroll
+          for (int b = 0; b < 2; b++) {
+            uint32_t sv[32];
+            __syncwarp();
+            tmem_ld_32x32b_x32(tX + lanes + half * 64 + b * 32, sv);
+            tmem_ld_wait();
+#pragma unroll
+            for (int c8 = 0; c8 < 4; c8++) {
+              uint32_t h[4];
+#pragma unroll
+              for (int e = 0; e < 4; e++) {
+                const int s = half * 64 + b * 32 + c8 * 8 + 2 * e;
+                const float2 us = *reinterpret_cast<const float2*>(u + s);
+                const float p0 = s <= row ? __uint_as_float(sv[c8 * 8 + 2 * e]) * scale * exp_fast(us.x - Rt) : 0.f;
+                const float p1 = s + 1 <= row ? __uint_as_float(sv[c8 * 8 + 2 * e + 1]) * scale * exp_fast(us.y - Rt) : 0.f;
+                sum += p0 + p1;
+                h[e] = pack2(p0, p1);
+              }
+              *reinterpret_cast<uint4*>(dst + sw128(pr, b * 4 + c8)) = make_uint4(h[0], h[1], h[2], h[3]);
+            }
           }
         }
         rs[half * MW_C + row] = sum;
-      } else {
-        rs[half * MW_C + row] = 0.f;
-      }
-      fence_proxy_async_smem();
-      tc_fence_before();
-      ok = __syncthreads_and(ok);                        // (2) P complete, scores read
-      tc_fence_after();
-      if (tid == 0 && ok) {
-#pragma unroll 1
-        for (int part = 0; part < 2; part++) {           // high, low
-          const uint64_t p = p_k + part * (P_LOW / 16);
-          for (int k = 0; k < 4; k++) umma_f16_ss(tX, v_mn + k * 128, p + k * 2, idesc_o2, (part | k) != 0);
-          for (int k = 0; k < 4; k++) umma_f16_ss(tX + 64, v_mn + (k + 4) * 128, p + MW_BLK / 16 + k * 2, idesc_o2h, 1);
+        fence_proxy_async_smem();
+        tc_fence_before();
+        bar_named(BAR_P, 288);                           // P complete, scores read
+        tc_fence_after();
+        wait(b_o1, par, 3);
+        tc_fence_after();
+        if (half == 0) {                                 // denominators: thread = token
+          uint32_t x[16];
+          __syncwarp();
+          tmem_ld_32x32b_x16(tNq + lanes, x);
+          tmem_ld_wait();
+          const float dot = (__uint_as_float(x[0]) + __uint_as_float(x[1])) * ein[row] + sum + rs[MW_C + row];
+          inv[row] = 1.f / (fmaxf(fabsf(dot), inv[row]) + DEN_EPS);
         }
-        umma_commit(b_o2);
-      }
-      __syncwarp();
-      if (tid < MW_C) {
-        const float dot = nq[tid] * ein[tid] + rs[tid] + rs[MW_C + tid];
-        inv[tid] = 1.f / (fmaxf(fabsf(dot), inv[tid]) + DEN_EPS);
-      }
-      if (ok && !mw_wait(b_o1, par)) ok = fail(3);       // the queries are consumed
-    }
-    // values times their weight in the next state, over the queries
-    for (int i = tid; i < 2 * MW_C * 8; i += 256) {
-      const int r = (i >> 3) & (MW_C - 1);
-      const uint32_t at = (i >> 10) * MW_BLK + sw128(r, i & 7);
-      const float k = w[r];
-      float v8[8];
-      bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sV + at), v8);
-      uint32_t h[4], l[4];
+        bar_named(BAR_DEN, 256);
+        wait(b_o2, par, 4);
+        tc_fence_after();
+        // outputs: thread (value row, half of the tokens); neighbouring lanes trade every second token, so that each stores pairs of columns
+        const int odd = lane & 1, col = v0 + (row & ~1);
+        const size_t pitch = (size_t)D.H * D.v16;
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(io.o) + (size_t)(row0 + c0 + half * 64 + odd) * pitch + hd * D.v16 + col;
+        const int left = col < D.v16 ? cnt - half * 64 - odd : 0;        // tokens of this thread that exist, every second one counted twice
 #pragma unroll
-      for (int e = 0; e < 4; e++) split2(v8[2 * e] * k, v8[2 * e + 1] * k, h[e], l[e]);
-      *reinterpret_cast<uint4*>(sQ + at) = make_uint4(h[0], h[1], h[2], h[3]);
-      *reinterpret_cast<uint4*>(sQ + 2 * MW_BLK + at) = make_uint4(l[0], l[1], l[2], l[3]);
-    }
-    const float r_last = R[MW_C - 1], decay = exp_fast(m_in - r_last), f_chunk = *f_sum;
-    if constexpr (OUT) {
-      __syncthreads();                                   // (3) denominators
-      if (ok && !mw_wait(b_o2, par)) ok = fail(4);
+        for (int b = 0; b < 4; b++) {
+          const int t0 = half * 64 + b * 16;
+          uint32_t o1[16], o2[16];
+          __syncwarp();
+          tmem_ld_32x32b_x16(tX + 128 + lanes + t0, o1);
+          tmem_ld_32x32b_x16(tX + lanes + t0, o2);
+          tmem_ld_wait();
+#pragma unroll
+          for (int e = 0; e < 16; e += 2) {
+            const float2 en = *reinterpret_cast<const float2*>(ein + t0 + e), iv = *reinterpret_cast<const float2*>(inv + t0 + e);
+            const float x = (__uint_as_float(o1[e]) * en.x + __uint_as_float(o2[e])) * iv.x, y = (__uint_as_float(o1[e + 1]) * en.y + __uint_as_float(o2[e + 1])) * iv.y;
+            const float got = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
+            if (b * 16 + e < left) *reinterpret_cast<uint32_t*>(dst) = odd ? pack2(got, y) : pack2(x, got);
+            dst += 2 * pitch;
+          }
+        }
+      } else {
+        wait(b_load, par, 1);
+        weigh_values(u + 2 * MW_C, tid, 256);
+        fence_proxy_async_smem();
+      }
+      const float r_last = R[MW_C - 1], f_chunk = u[5 * MW_C], decay = exp_fast(m_in - r_last);
+      tc_fence_before();
+      bar_named(BAR_STATE, MW_THREADS);
       tc_fence_after();
-      float* dst = io.o + (size_t)(row0 + c0) * D.H * D.v16 + hd * D.v16 + v0 + row;
-      const bool live = v0 + row < D.v16;
-#pragma unroll 1
-      for (int b = 0; b < 4; b++) {                      // thread (value row, half of the tokens), sixteen tokens at a time
-        const int t0 = half * 64 + b * 16;
-        uint32_t o1[16], o2[16];
+      m_in = f_chunk + r_last;
+      f_total += f_chunk;
+      wait(b_ds, par, 5);
+      tc_fence_after();
+#pragma unroll
+      for (int i = 0; i < NQ; i++) {
+        uint32_t x[32];
         __syncwarp();
-        tmem_ld_32x32b_x16(tX + 128 + lanes + t0, o1);
-        tmem_ld_32x32b_x16(tX + lanes + t0, o2);
+        tmem_ld_32x32b_x32(tX + lanes + half * NQ * 32 + i * 32, x);
         tmem_ld_wait();
 #pragma unroll
-        for (int e = 0; e < 16; e++) {
-          const int t = t0 + e;
-          if (live && t < cnt) dst[(size_t)t * D.H * D.v16] = (__uint_as_float(o1[e]) * ein[t] + __uint_as_float(o2[e])) * inv[t];
+        for (int e = 0; e < 32; e++) S[i * 32 + e] = S[i * 32 + e] * decay + __uint_as_float(x[e]);
+      }
+      if (NQ > 2 || half == 0) {
+        uint32_t x[16];
+        __syncwarp();
+        tmem_ld_32x32b_x16(tDn + lanes + half * 16, x);
+        tmem_ld_wait();
+        n = n * decay + (__uint_as_float(x[0]) + __uint_as_float(x[1]));
+      }
+      if (OUT && c0 + MW_C < rows) publish();
+    }
+    if (ok && !*failed && (!OUT || (flags & SEG_LAST))) {
+      float* dst = OUT ? slot : scratch + (size_t)(sg[5] + 1) * D.H * D.head() + hd * D.head();
+      if (v0 + row < D.v16) {
+#pragma unroll
+        for (int i = 0; i < NQ * 32; i++) {
+          const int d = half * NQ * 32 + i;
+          if (d < D.d16) dst[(size_t)d * D.v16 + v0 + row] = S[i];
+        }
+      }
+      if (blockIdx.z == 0) {
+        // a slot's n may still be unread by the other CTAs of this head: it moves there later
+        float* to = OUT ? io.nm + ((size_t)sg[3] * D.H + hd) * (D.d16 + 4) : dst + n_at;
+        if (nd < D.d16) to[nd] = n;
+        if (tid == 0) {
+          to[D.d16] = m_in;
+          to[D.d16 + 1] = f_total;
         }
       }
     }
-    fence_proxy_async_smem();
-    tc_fence_before();
-    ok = __syncthreads_and(ok);                          // (4) w V complete, outputs read
-    tc_fence_after();
-    if (tid == 0 && ok) {
-#pragma unroll 1
-      for (int k = 0; k < 8; k++) {
-        umma_f16_ss(tX, w_mn + k * 128, k_mn + k * 128, idesc_ds, k != 0);
-        umma_f16_ss(tX, w_mn + 2 * (MW_BLK / 16) + k * 128, k_mn + k * 128, idesc_ds, 1);
-      }
-      umma_commit(b_ds);
-    }
-    __syncwarp();
-    {                                                    // n <- decay n + sum_t w_t k_t: a lane takes eight columns of every eighth token
-      const int tg = lane >> 2;
-      for (int j = warp * 4 + (lane & 3); j < NQ * 8; j += 32) {
-        float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-#pragma unroll 4
-        for (int i = 0; i < MW_C / 8; i++) {
-          const int t = i * 8 + tg;
-          float k8[8];
-          bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sK + (j >> 3) * MW_BLK + sw128(t, j & 7)), k8);
-          const float wt = w[t];
-#pragma unroll
-          for (int e = 0; e < 8; e++) a[e] += wt * k8[e];
-        }
-#pragma unroll
-        for (int e = 0; e < 8; e++) {
-          a[e] += __shfl_xor_sync(0xffffffffu, a[e], 4);
-          a[e] += __shfl_xor_sync(0xffffffffu, a[e], 8);
-          a[e] += __shfl_xor_sync(0xffffffffu, a[e], 16);
-        }
-        if (tg == 0) {
-#pragma unroll
-          for (int e = 0; e < 8; e++) n[j * 8 + e] = n[j * 8 + e] * decay + a[e];
-        }
-      }
-    }
-    if (ok && !mw_wait(b_ds, par)) ok = fail(5);
-    ok = __syncthreads_and(ok);                          // (5) everybody is done with the chunk's shared memory
-    if (!ok) break;
-    if (tid == 0 && c0 + MW_C < rows) load_chunk(c0 + MW_C);
-    __syncwarp();
-    tc_fence_after();
-#pragma unroll
-    for (int i = 0; i < NQ; i++) {
-      uint32_t x[32];
-      tmem_ld_32x32b_x32(tX + lanes + half * NQ * 32 + i * 32, x);
-      tmem_ld_wait();
-#pragma unroll
-      for (int e = 0; e < 32; e++) S[i * 32 + e] = S[i * 32 + e] * decay + __uint_as_float(x[e]);
-    }
-    if (OUT && c0 + MW_C < rows) publish();
-    m_in = f_chunk + r_last;
-    f_total += f_chunk;
   }
-  if (!ok)
+  if (*failed)
     for (int i = 0; i < 64; i++) __nanosleep(1000);      // copies in flight land before the shared memory goes away
-  if (ok && (!OUT || (flags & SEG_LAST))) {
-    float* dst = OUT ? slot : scratch + (size_t)(sg[5] + 1) * D.H * D.head() + hd * D.head();
-    if (v0 + row < D.v16) {
-#pragma unroll
-      for (int i = 0; i < NQ * 32; i++) {
-        const int d = half * NQ * 32 + i;
-        if (d < D.d16) dst[(size_t)d * D.v16 + v0 + row] = S[i];
-      }
-    }
-    if (blockIdx.z == 0) {
-      // a slot's n may still be unread by the other CTAs of this head: it moves there later
-      float* nd = OUT ? io.nm + ((size_t)sg[3] * D.H + hd) * (D.d16 + 4) : dst + n_at;
-      for (int i = tid; i < D.d16; i += 256) nd[i] = n[i];
-      if (tid == 0) {
-        nd[D.d16] = m_in;
-        nd[D.d16 + 1] = f_total;
-      }
-    }
-  }
   tc_fence_before();
   __syncthreads();
-  if (warp == 1) {
+  if (warp == 8) {
     tc_fence_after();
     tmem_dealloc(tX, 512);
   }
@@ -555,55 +597,72 @@ __global__ void __launch_bounds__(256) mm_merge_kernel(const int4* __restrict__ 
   }
 }
 
-// rows: warp per head. CTAs past the rows move n and m of one sequence into its slot.
+// a warp per (row, head), eight columns a lane. CTAs past the rows move n and m of one sequence into its slot.
+template <typename T> FT_DEVICE void load8(const T* p, float (&v)[8]);
+template <> FT_DEVICE void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> FT_DEVICE void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) { bf16x8_to_float(*reinterpret_cast<const bf16x8*>(p), v); }
+template <typename T> FT_DEVICE void store8(T* p, const float (&v)[8]);
+template <> FT_DEVICE void store8<float>(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <> FT_DEVICE void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) { *reinterpret_cast<bf16x8*>(p) = float_to_bf16x8(v); }
+
+constexpr int FIN_WARPS = 8;
 template <typename T>
-__global__ void __launch_bounds__(128) mm_finish_kernel(const float* __restrict__ o, int rows, const T* __restrict__ gate, int64_t ldg, const float* __restrict__ norm, float eps,
-                                                        float out_scale, T* __restrict__ out, int64_t ldo, MemDims D, const int4* __restrict__ seqs,
-                                                        const float* __restrict__ nm, float* __restrict__ slots, size_t slot_stride) {
-  if ((int)blockIdx.x >= rows) {
-    const int s = blockIdx.x - rows;
+__global__ void __launch_bounds__(FIN_WARPS * 32) mm_finish_kernel(const T* __restrict__ o, int rows, int ctas, const T* __restrict__ gate, int64_t ldg, const float* __restrict__ norm,
+                                                                   float eps, float out_scale, T* __restrict__ out, int64_t ldo, MemDims D, const int4* __restrict__ seqs,
+                                                                   const float* __restrict__ nm, float* __restrict__ slots, size_t slot_stride) {
+  if ((int)blockIdx.x >= ctas) {
+    const int s = blockIdx.x - ctas;
     float* dst = slots + (size_t)seqs[s].z * slot_stride;
-    for (int i = threadIdx.x; i < D.H * (D.d16 + 1); i += 128) {
+    for (int i = threadIdx.x; i < D.H * (D.d16 + 1); i += FIN_WARPS * 32) {
       const int hd = i / (D.d16 + 1), e = i % (D.d16 + 1);
       dst[hd * D.head() + (size_t)D.d16 * D.v16 + e] = nm[((size_t)s * D.H + hd) * (D.d16 + 4) + e];
     }
     return;
   }
-  const int r = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  for (int hd = warp; hd < D.H; hd += 4) {
-    const float* src = o + (size_t)r * D.H * D.v16 + hd * D.v16;
-    float ss = 0.f;
-    for (int c = lane * 4; c < D.v16; c += 128) {
-      const float4 v = *reinterpret_cast<const float4*>(src + c);
-      ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
-    }
-    const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)D.dv + eps) * out_scale;
-    for (int c = lane * 4; c < D.v16; c += 128) {
-      const float4 v = *reinterpret_cast<const float4*>(src + c), w = *reinterpret_cast<const float4*>(norm + hd * D.v16 + c);
-      const float x[4] = {v.x * w.x, v.y * w.y, v.z * w.z, v.w * w.w};
-      const T* gr = gate + (size_t)r * ldg + hd * D.v16 + c;
-      T* dst = out + (size_t)r * ldo + hd * D.v16 + c;
-      float y[4];
-      if constexpr (sizeof(T) == 4) {
-        const float4 gv = *reinterpret_cast<const float4*>(gr);
-        y[0] = gv.x; y[1] = gv.y; y[2] = gv.z; y[3] = gv.w;
-      } else {
-        const uint2 raw = *reinterpret_cast<const uint2*>(gr);
-        const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
-        y[0] = a.x; y[1] = a.y; y[2] = b.x; y[3] = b.y;
-      }
+  const int unit = blockIdx.x * FIN_WARPS + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (unit >= rows * D.H) return;
+  const int r = unit / D.H, hd = unit % D.H;
+  const T* src = o + (size_t)unit * D.v16;
+  const T* gr = gate + (size_t)r * ldg + hd * D.v16;
+  constexpr int KEEP = 2;                                  // vectors of a lane that stay in registers (heads of up to 512 columns)
+  float x[KEEP][8], ss = 0.f;
 #pragma unroll
-      for (int e = 0; e < 4; e++) y[e] = x[e] * rstd * (sizeof(T) == 4 ? sigmoid_exact(y[e]) : 1.f / (1.f + __expf(-y[e])));
-      if constexpr (sizeof(T) == 4) {
-        *reinterpret_cast<float4*>(dst) = make_float4(y[0], y[1], y[2], y[3]);
-      } else {
-        __nv_bfloat162 a = __floats2bfloat162_rn(y[0], y[1]), b = __floats2bfloat162_rn(y[2], y[3]);
-        uint2 pk;
-        pk.x = *reinterpret_cast<uint32_t*>(&a);
-        pk.y = *reinterpret_cast<uint32_t*>(&b);
-        *reinterpret_cast<uint2*>(dst) = pk;
-      }
+  for (int i = 0; i < KEEP; i++) {
+    const int c = lane * 8 + i * 256;
+    if (c < D.v16) {
+      load8(src + c, x[i]);
+#pragma unroll
+      for (int e = 0; e < 8; e++) ss += x[i][e] * x[i][e];
     }
+  }
+  for (int c = lane * 8 + KEEP * 256; c < D.v16; c += 256) {
+    float y[8];
+    load8(src + c, y);
+#pragma unroll
+    for (int e = 0; e < 8; e++) ss += y[e] * y[e];
+  }
+  const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)D.dv + eps) * out_scale;
+  auto finish = [&](int c, float (&v)[8]) {
+    float g[8], w[8];
+    load8(gr + c, g);
+    load8(norm + hd * D.v16 + c, w);
+#pragma unroll
+    for (int e = 0; e < 8; e++) v[e] = v[e] * rstd * w[e] * (sizeof(T) == 4 ? sigmoid_exact(g[e]) : 1.f / (1.f + __expf(-g[e])));
+    store8(out + (size_t)r * ldo + hd * D.v16 + c, v);
+  };
+#pragma unroll
+  for (int i = 0; i < KEEP; i++)
+    if (lane * 8 + i * 256 < D.v16) finish(lane * 8 + i * 256, x[i]);
+  for (int c = lane * 8 + KEEP * 256; c < D.v16; c += 256) {
+    float y[8];
+    load8(src + c, y);
+    finish(c, y);
   }
 }
 
@@ -746,10 +805,15 @@ int launch_walk(const CUtensorMap (&m)[3], dim3 grid, cudaStream_t st, const Mem
   int dev = 0;
   FT_CUDA_TRY(cudaGetDevice(&dev));
   if (dev < 64 && !done[dev]) {
+    // the warps trade registers (NQ > 2) out of what the block was launched with
+    cudaFuncAttributes fa;
+    FT_CUDA_TRY(cudaFuncGetAttributes(&fa, mm_walk_kernel<NQ, OUT>));
+    static_assert(MW_REGS_STATE * 256 + MW_REGS_HELP * 128 <= MW_REGS * MW_THREADS, "register split");
+    if (NQ > 2 && fa.numRegs < MW_REGS) return FT_ERR_ARG;
     FT_CUDA_TRY(cudaFuncSetAttribute(mm_walk_kernel<NQ, OUT>, cudaFuncAttributeMaxDynamicSharedMemorySize, mw_smem(NQ, OUT)));
     done[dev] = true;
   }
-  mm_walk_kernel<NQ, OUT><<<grid, 256, mw_smem(NQ, OUT), st>>>(m[0], m[1], m[2], io, D, scratch, ft_status_ptr());
+  mm_walk_kernel<NQ, OUT><<<grid, MW_THREADS, mw_smem(NQ, OUT), st>>>(m[0], m[1], m[2], io, D, scratch, ft_status_ptr());
   return (int)cudaGetLastError();
 }
 
@@ -779,9 +843,9 @@ FT_EXPORT int ft_mm_walk_fits(int d, int dv) { return d >= 1 && dv >= 1 && d <= 
 // Prompt stretches of a ragged batch in bf16. x [rows][ld]: queries H x d16 | keys H x d16 | values H x v16 (16-byte aligned, ld a multiple of 8); gates f32 [rows][ldg]: input
 // gates, at column h8 = H rounded up to 8 forget gates; biases f32 [H]. segs int[nsegs][8] {first row, rows, slot, sequence, flags, scratch state, 0, 0}, flags 1: the only segment
 // of its stretch (its state comes from the slot), 2: last, 4: the sequence starts (zero state). out = 0: contributions of the segments into scratch states [scratch state + 1] (f32 [H][d16 v16 + d16 + 4]
-// each); out = 1: outputs o f32 [rows][H * v16], last segments leave S in their slot (f32 slots of slot_stride) and n, m in nm f32 [sequence][H][d16 + 4].
+// each); out = 1: outputs o bf16 [rows][H * v16], last segments leave S in their slot (f32 slots of slot_stride) and n, m in nm f32 [sequence][H][d16 + 4].
 FT_EXPORT int ft_mm_walk(const void* x, int64_t ld, int rows, const float* gates, int64_t ldg, const float* bias_i, const float* bias_f, float cap, const int* segs, int nsegs, int H, int d,
-                         int dv, float* slots, int64_t slot_stride, float* scratch, float* nm, float* o, int out, cudaStream_t st) {
+                         int dv, float* slots, int64_t slot_stride, float* scratch, float* nm, void* o, int out, cudaStream_t st) {
   MemDims D;
   if (nsegs < 1 || rows < 1 || !make_dims(D, H, d, dv, cap) || (ld & 7) || (reinterpret_cast<uintptr_t>(x) & 15) || (!out && !scratch) || (out && (!o || !nm))) return FT_ERR_ARG;
   if (!ft_mm_walk_fits(d, dv)) return FT_ERR_TOO_LARGE;
@@ -816,7 +880,7 @@ FT_EXPORT int ft_mm_merge(const int* seqs, int nseq, int H, int d, int dv, const
 
 // The same stretches token by token, bf16 or f32 (is_f32), one segment per sequence (flags 3, or 7 where the sequence starts). Key sizes up to 1600.
 FT_EXPORT int ft_mm_rows(const void* x, int64_t ld, const float* gates, int64_t ldg, const float* bias_i, const float* bias_f, float cap, const int* segs, int nsegs, int H, int d,
-                         int dv, float* slots, int64_t slot_stride, float* nm, float* o, int is_f32, cudaStream_t st) {
+                         int dv, float* slots, int64_t slot_stride, float* nm, void* o, int is_f32, cudaStream_t st) {
   MemDims D;
   if (nsegs < 1 || nsegs > 65535 || !make_dims(D, H, d, dv, cap)) return FT_ERR_ARG;
   const int smem = rows_smem(D.d16);
@@ -833,16 +897,18 @@ FT_EXPORT int ft_mm_rows(const void* x, int64_t ld, const float* gates, int64_t 
   return (int)cudaGetLastError();
 }
 
-// out [rows][ldo] (heads of v16) = o / rms(o of the head) * norm (f32 [H * v16]) * sigmoid(gate [rows][ldg]) * out_scale; moves n and m of every sequence of seqs (as for
+// out [rows][ldo] (heads of v16; o, gate and out in one type) = o / rms(o of the head) * norm (f32 [H * v16]) * sigmoid(gate [rows][ldg]) * out_scale; moves n and m of every sequence of seqs (as for
 // ft_mm_merge) from nm into its slot.
-FT_EXPORT int ft_mm_finish(const float* o, int rows, const void* gate, int64_t ldg, const float* norm, float eps, float out_scale, void* out, int64_t ldo, int H, int d, int dv,
+FT_EXPORT int ft_mm_finish(const void* o, int rows, const void* gate, int64_t ldg, const float* norm, float eps, float out_scale, void* out, int64_t ldo, int H, int d, int dv,
                            const int* seqs, int nseq, const float* nm, float* slots, int64_t slot_stride, int is_f32, cudaStream_t st) {
   MemDims D;
-  if (rows < 1 || nseq < 1 || !make_dims(D, H, d, dv, 1.f) || (ldg & 3) || (ldo & 3)) return FT_ERR_ARG;
+  if (rows < 1 || nseq < 1 || !make_dims(D, H, d, dv, 1.f) || (ldg & 7) || (ldo & 7)) return FT_ERR_ARG;
   const int4* sq = reinterpret_cast<const int4*>(seqs);
-  if (is_f32) mm_finish_kernel<float><<<rows + nseq, 128, 0, st>>>(o, rows, (const float*)gate, ldg, norm, eps, out_scale, (float*)out, ldo, D, sq, nm, slots, (size_t)slot_stride);
-  else mm_finish_kernel<__nv_bfloat16><<<rows + nseq, 128, 0, st>>>(o, rows, (const __nv_bfloat16*)gate, ldg, norm, eps, out_scale, (__nv_bfloat16*)out, ldo, D, sq, nm, slots,
-                                                                   (size_t)slot_stride);
+  const int ctas = (int)(((int64_t)rows * H + FIN_WARPS - 1) / FIN_WARPS);
+#define FT_FIN(T) mm_finish_kernel<T><<<ctas + nseq, FIN_WARPS * 32, 0, st>>>((const T*)o, rows, ctas, (const T*)gate, ldg, norm, eps, out_scale, (T*)out, ldo, D, sq, nm, slots, \
+                                                                              (size_t)slot_stride)
+  if (is_f32) FT_FIN(float); else FT_FIN(__nv_bfloat16);
+#undef FT_FIN
   return (int)cudaGetLastError();
 }
 

@@ -74,7 +74,7 @@ def matrix_memory_rows(x: torch.Tensor, gates: torch.Tensor, w: MemoryWeights, b
     f32 = x.dtype == torch.float32
     walk = not f32 and D.walk_supported() if walk is None else walk
     plan = batch.memory_plan(D.heads * -(-D.v16 // VALUE_SLICE) if walk else 0)
-    o = torch.empty(T, D.out_cols, device=x.device, dtype=torch.float32)
+    o = torch.empty(T, D.out_cols, device=x.device, dtype=x.dtype)
     nm = torch.empty(plan.sequences, D.heads * (D.d16 + 4), device=x.device, dtype=torch.float32)
     vectors = (gates, gates.stride(0), w.bias_i, w.bias_f, D.cap)
     head = (x, x.stride(0), T, *vectors)

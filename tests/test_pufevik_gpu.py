@@ -426,7 +426,7 @@ def test_matrix_memory_of_prompts_and_portions(D, form):
             got[s].append(out[at: at + hi - lo])
             at += hi - lo
     for s in P:
-        assert rel(torch.cat(got[s]), want[s][0].reshape(len(want[s][0]), -1)) < (2e-5 if form == "f32" else 1e-2), s
+        assert rel(torch.cat(got[s]), want[s][0].reshape(len(want[s][0]), -1)) < (2e-5 if form == "f32" else 2e-2), s
         assert state_error(rig.state(s), want[s][1]) < (5e-6 if form != "walk" else 5e-5), s
 
 
@@ -443,8 +443,8 @@ def test_long_prompts_walk_in_segments(D):
     rig.cache.reserve("p", 1900)
     batch = RowBatch([StepEntry("p", [0] * 600)], rig.cache, torch.device("cuda"), 130)
     assert batch.memory_plan(D.heads * -(-D.v16 // 128)).scratch > 1
-    assert rel(torch.cat([a, b[70:]]), want.reshape(1300, -1)) < 1e-2 and state_error(rig.state("p"), last) < 5e-5
-    assert rel(b[:70], rig.reference(Q)[0].reshape(70, -1)) < 1e-2
+    assert rel(torch.cat([a, b[70:]]), want.reshape(1300, -1)) < 2e-2 and state_error(rig.state("p"), last) < 5e-5
+    assert rel(b[:70], rig.reference(Q)[0].reshape(70, -1)) < 2e-2
 
 
 @pytest.mark.parametrize("bias,scale", [((6.0, -6.0), 4.0), ((-6.0, 8.0), 1.0), ((0.0, 0.0), 30.0)])
@@ -457,7 +457,7 @@ def test_gates_at_their_limits(bias, scale, form):
     want, last = rig.reference(P)
     rig.cache.add_sequence("s")
     got = torch.cat([rig.decode({"s": (P, t)}) for t in range(150)]) if form == "decode" else rig.step({"s": (P, 0, 150)})
-    assert rel(got, want.reshape(150, -1)) < (5e-4 if form == "f32" else 1e-2) and state_error(rig.state("s"), last) < 1e-4
+    assert rel(got, want.reshape(150, -1)) < (5e-4 if form == "f32" else 2e-2) and state_error(rig.state("s"), last) < 1e-4
 
 
 @pytest.mark.parametrize("D", MEMORIES + [MemoryDims(1, 400, 300, 6.0, 1e-6), MemoryDims(1, 32, 600, 6.0, 1e-6)], ids=lambda d: f"{d.heads}-{d.dim}-{d.vdim}")
