@@ -132,17 +132,17 @@ __global__ void __launch_bounds__(256) mm_rows_kernel(MemIO io, MemDims D) {
 //   nq [t]         = Q n          (n: high + low part)
 //   O2 [v][t]      = V^T P^T      (P = masked, weighted scores)                     the chunk itself
 //   dS [v][d]      = (w V)^T K    (w V: values times their weight in the next state, high + low);  S <- decay S + dS in f32
-//   dn [d]         = K^T w        (w: high + low);                                                 n <- decay n + dn in f32
+//   n <- decay n + sum_t w_t k_t  on the FMA pipes, under dS
 //
-// What enters the state (w V, w) and the normaliser meets the 16-bit tensor cores as sums of two bf16 numbers, so that states are exact to 16 mantissa bits per
+// What enters the state (w V) and the normaliser meet the 16-bit tensor cores as sums of two bf16 numbers, so that states are exact to 16 mantissa bits per
 // addend; the read-out takes P and S in bf16, as attention takes its weights.
 //
 // Warps 0..7: weights of the keys, outputs, state. Warp 8: issues copies and products. Warps 9..11: w V; warp 9 also the gates of the next chunk. Named barriers separate
-// the steps of a chunk, which depend on one another. Shared memory: Q (then w V) | K | V | P (of its second 64 columns only the lower rows exist) | n and w as
-// operands. TMEM: [scores, then O2 | O1], later dS over both | S^T | nq | dn.
+// the steps of a chunk, which depend on one another. Shared memory: Q (then w V) | K | V | P (of its second 64 columns only the lower rows exist) | n as an
+// operand. TMEM: [scores, then O2 | O1], later dS over both | S^T | nq.
 // ------------------------------------------------------------------------------------------------------------
 constexpr int MW_C = 128, MW_V = 128, MW_BLK = MW_C * 128;      // chunk, value columns, bytes of a 64-column block of 128 rows
-constexpr int MW_THREADS = 384, MW_GATES = 5 * MW_C + 4;        // floats of one chunk's gate arrays
+constexpr int MW_THREADS = 384, MW_GATES = 6 * MW_C + 8;        // floats of one chunk's gate arrays
 constexpr int MW_VEC = 16 * 128;                                // bytes of a 64-column block of a 16-row operand (rows: high, low, zeros)
 constexpr int MW_REGS = 168, MW_REGS_STATE = 208, MW_REGS_HELP = 88;
 constexpr uint32_t FT_K_MEMORY = 11;
@@ -185,7 +185,7 @@ FT_DEVICE void put_vec(uint8_t* base, int i, float v) {
 }
 
 __host__ __device__ constexpr int mw_smem(int nq, bool out) {
-  return 4 * MW_BLK + nq * MW_BLK + 2 * MW_BLK + (out ? MW_BLK + MW_BLK / 2 : 0) + (nq + 4) * MW_VEC + (2 * MW_GATES + 2 * MW_C) * 4 + 64 + 1024;
+  return 4 * MW_BLK + nq * MW_BLK + 2 * MW_BLK + (out ? MW_BLK + MW_BLK / 2 : 0) + nq * MW_VEC + (2 * MW_GATES + 4 * MW_C + 64 * nq) * 4 + 64 + 1024;
 }
 
 // NQ: 64-column blocks of the key size. OUT: outputs from the state ahead of the segment; else: the segment's own contribution, into scratch state [scratch index + 1],
@@ -200,12 +200,13 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
   uint8_t* sV = sK + NQ * MW_BLK;                        // [2]
   uint8_t* sP = sV + 2 * MW_BLK;                         // block of columns 0..63, half block of columns 64..127
   uint8_t* sN = sP + (OUT ? MW_BLK + MW_BLK / 2 : 0);    // [NQ] n as an operand
-  uint8_t* sW = sN + NQ * MW_VEC;                        // [2][2] w as an operand, two chunks in turn
   // per chunk, two in turn: [128] u = i - F | running maximum R of u and m_in | weight in the next state | weight of the past times the queries' scale | e^(-m), then
-  // 1 / denominator | sum of the forget gates
-  float* gate_sets = reinterpret_cast<float*>(sW + 4 * MW_VEC);
+  // 1 / denominator | e^(u - largest u of its 32 tokens) | those four maxima | sum of the forget gates
+  float* gate_sets = reinterpret_cast<float*>(sN + NQ * MW_VEC);
   float* rs = gate_sets + 2 * MW_GATES;                  // [2][128] sums of the key weights
-  uint64_t* bars = reinterpret_cast<uint64_t*>(rs + 2 * MW_C);
+  float* raw = rs + 2 * MW_C;                            // [2][128] log gates of the next chunk
+  float* nf = raw + 2 * MW_C;                            // [64 NQ] n
+  uint64_t* bars = reinterpret_cast<uint64_t*>(nf + 64 * NQ);
   uint64_t *b_load = bars, *b_s = bars + 1, *b_o1 = bars + 2, *b_o2 = bars + 3, *b_ds = bars + 4;
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 5);
   volatile int* failed = reinterpret_cast<volatile int*>(tmem_slot + 1);
@@ -225,11 +226,12 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
     tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV);
   }
   if (warp == 8) { tmem_alloc(tmem_slot, 512); tmem_relinquish(); }
-  for (int i = tid; i < (NQ + 4) * MW_VEC / 16; i += MW_THREADS) reinterpret_cast<uint4*>(sN)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < NQ * MW_VEC / 16; i += MW_THREADS) reinterpret_cast<uint4*>(sN)[i] = make_uint4(0, 0, 0, 0);
+  for (int i = tid; i < 64 * NQ; i += MW_THREADS) nf[i] = zero || i >= D.d16 ? 0.f : in[n_at + i];
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tX = *tmem_slot, tA = tX + 256, tNq = tX + 384, tDn = tX + 400;
+  const uint32_t tX = *tmem_slot, tA = tX + 256, tNq = tX + 384;
   float m_in = OUT ? (zero ? 0.f : in[n_at + D.d16 + ((flags & SEG_ONLY) ? 0 : 2)]) : -INFINITY;
   bool ok = true;
   // a wait that ran out: everybody keeps to the barriers and leaves at the next chunk
@@ -256,26 +258,33 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
       *reinterpret_cast<uint4*>(sQ + 2 * MW_BLK + at) = make_uint4(l[0], l[1], l[2], l[3]);
     }
   };
-  enum { BAR_CHUNK = 1, BAR_P, BAR_DEN, BAR_STATE };
+  enum { BAR_CHUNK = 1, BAR_P, BAR_DEN, BAR_STATE, BAR_N, BAR_GATES };
 
   if (warp >= 8) {
     if constexpr (NQ > 2) reg_dec<MW_REGS_HELP>();
     // gates of a chunk (one warp), four neighbouring tokens a lane: running sum of the forget gates, running maximum
     const float bias_i = io.bi[hd], bias_f = io.bf[hd], scale = rsqrtf((float)D.d);
-    auto make_gates = [&](int c0, float m, int set) {
+    auto fetch_gates = [&](int c0) {                     // warps 9..11
+      for (int i = tid - 288; i < MW_C; i += 96) {
+        const int t = c0 + i;
+        float ig = -INFINITY, fg = 0.f;
+        if (t < rows) {
+          const float* gr = io.gates + (size_t)(row0 + t) * io.ldg;
+          ig = soft_cap(gr[hd] + bias_i, D.cap);
+          fg = log_sigmoid(soft_cap(gr[D.h8 + hd] + bias_f, D.cap));
+        }
+        raw[i] = ig;
+        raw[MW_C + i] = fg;
+      }
+    };
+    auto make_gates = [&](float m, int set) {
       float* g = gate_sets + set * MW_GATES;
-      const int cnt = min(MW_C, rows - c0);
       float F[4], uu[4], s = 0.f;
 #pragma unroll
       for (int e = 0; e < 4; e++) {
-        const int t = lane * 4 + e;
-        uu[e] = -INFINITY;
-        if (t < cnt) {
-          const float* gr = io.gates + (size_t)(row0 + c0 + t) * io.ldg;
-          uu[e] = soft_cap(gr[hd] + bias_i, D.cap);
-          s += log_sigmoid(soft_cap(gr[D.h8 + hd] + bias_f, D.cap));
-        }
+        s += raw[MW_C + lane * 4 + e];
         F[e] = s;
+        uu[e] = raw[lane * 4 + e];
       }
       float tot = s;
 #pragma unroll
@@ -291,6 +300,10 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
         uu[e] -= F[e];
         mx = fmaxf(mx, uu[e]);
       }
+      float top = mx;                                    // of the 32 tokens that eight lanes hold
+#pragma unroll
+      for (int o = 1; o < 8; o <<= 1) top = fmaxf(top, __shfl_xor_sync(0xffffffffu, top, o));
+      if ((lane & 7) == 0) g[6 * MW_C + (lane >> 3)] = top;
 #pragma unroll
       for (int o = 1; o < 32; o <<= 1) {
         const float y = __shfl_up_sync(0xffffffffu, mx, o);
@@ -303,16 +316,14 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
       for (int e = 0; e < 4; e++) {
         const int t = lane * 4 + e;
         before = fmaxf(before, uu[e]);
-        const float wt = exp_fast(uu[e] - last);
         g[t] = uu[e];
         g[MW_C + t] = before;
-        g[2 * MW_C + t] = wt;
+        g[2 * MW_C + t] = exp_fast(uu[e] - last);
         g[3 * MW_C + t] = exp_fast(m - before) * scale;
         g[4 * MW_C + t] = exp_fast(-(F[e] + before));
-        put_vec(sW + set * 2 * MW_VEC, t, wt);
+        g[5 * MW_C + t] = top == -INFINITY ? 0.f : exp_fast(uu[e] - top);
       }
-      if (lane == 31) g[5 * MW_C] = F[3];
-      fence_proxy_async_smem();
+      if (lane == 31) g[6 * MW_C + 4] = F[3];
     };
     auto load_chunk = [&](int c0) {                      // one thread
       mbar_expect_tx(b_load, ((OUT ? NQ : 0) + NQ + 2) * MW_BLK);
@@ -323,14 +334,20 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
       for (int c = 0; c < 2; c++) tma_load_3d(sV + c * MW_BLK, &tmV, b_load, v0 + c * 64, hd, row0 + c0);
     };
     if (warp == 8 && lane == 0) load_chunk(0);
-    if (warp == 9) make_gates(0, m_in, 0);
+    if (warp > 8) {
+      fetch_gates(0);
+      bar_named(BAR_GATES, 96);
+      if (warp == 9) make_gates(m_in, 0);
+    }
     const uint32_t idesc_s = make_idesc_f16(128, 128, 1, 0, 0), idesc_n = make_idesc_f16(128, 16, 1, 0, 0), idesc_o2 = make_idesc_f16(128, 128, 1, 1, 0),
-                   idesc_o2h = make_idesc_f16(128, 64, 1, 1, 0), idesc_ds = make_idesc_f16(128, NQ * 64, 1, 1, 1), idesc_dn = make_idesc_f16(128, 16, 1, 1, 0);
-    // K-major operands (rows of 64-column blocks), and the same memory with the contiguous dimension as M or N
-    const uint64_t q_k = make_smem_desc(smem_u32(sQ), 16, 1024, FT_SWZ_128B), k_k = make_smem_desc(smem_u32(sK), 16, 1024, FT_SWZ_128B),
-                   p_k = make_smem_desc(smem_u32(sP), 16, 1024, FT_SWZ_128B), n_k = make_smem_desc(smem_u32(sN), 16, 1024, FT_SWZ_128B),
-                   k_mn = make_smem_desc(smem_u32(sK), MW_BLK, 1024, FT_SWZ_128B), v_mn = make_smem_desc(smem_u32(sV), MW_BLK, 1024, FT_SWZ_128B),
-                   w_mn = make_smem_desc(smem_u32(sQ), MW_BLK, 1024, FT_SWZ_128B);
+                   idesc_o2h = make_idesc_f16(128, 64, 1, 1, 0), idesc_ds = make_idesc_f16(128, NQ * 64, 1, 1, 1);
+    // all descriptors share their upper half (1024 bytes between groups of eight rows, 128-byte swizzle); the lower half counts 16-byte units from the operand's start.
+    // K-major operands are rows of 64-column blocks, "mn" is the same memory with the contiguous dimension as M or N
+    auto desc = [](uint32_t low) -> uint64_t { return ((uint64_t)((1024 >> 4) | (1u << 14) | (FT_SWZ_128B << 29)) << 32) | low; };
+    auto low_k = [](const uint8_t* p) -> uint32_t { return (smem_u32(p) >> 4) | (1u << 16); };
+    auto low_mn = [](const uint8_t* p) -> uint32_t { return (smem_u32(p) >> 4) | ((uint32_t)(MW_BLK >> 4) << 16); };
+    const uint32_t q_k = low_k(sQ), k_k = low_k(sK), p_k = low_k(sP), n_k = low_k(sN), k_mn = low_mn(sK), v_mn = low_mn(sV), w_mn = low_mn(sQ);
+    auto block = [](int k) -> uint32_t { return (k >> 2) * (MW_BLK / 16) + (k & 3) * 2; };      // 16 columns number k of a K-major operand
     int c0 = 0;
     for (int ch = 0; c0 < rows; ch++, c0 += MW_C) {
       const int par = ch & 1;
@@ -338,18 +355,18 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
       bar_named(BAR_CHUNK, MW_THREADS);                  // gates, state and normaliser are in place
       if (*failed) break;
       tc_fence_after();
+      if (warp > 8 && c0 + MW_C < rows) fetch_gates(c0 + MW_C);
       wait(b_load, par, 1);
       if constexpr (OUT) {
         if (warp == 8) {
           if (lane == 0 && ok) {
 #pragma unroll
-            for (int k = 0; k < NQ * 4; k++) umma_f16_ss(tX, q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, k_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2, idesc_s, k != 0);
+            for (int k = 0; k < NQ * 4; k++) umma_f16_ss(tX, desc(q_k + block(k)), desc(k_k + block(k)), idesc_s, k != 0);
             umma_commit(b_s);
 #pragma unroll
             for (int k = 0; k < NQ * 4; k++) {
-              const uint64_t q = q_k + (k >> 2) * (MW_BLK / 16) + (k & 3) * 2;
-              umma_f16_ss(tNq, q, n_k + (k >> 2) * (MW_VEC / 16) + (k & 3) * 2, idesc_n, k != 0);
-              umma_f16_ts(tX + 128, tA + k * 8, q, idesc_s, k != 0);
+              umma_f16_ts(tX + 128, tA + k * 8, desc(q_k + block(k)), idesc_s, k != 0);
+              umma_f16_ss(tNq, desc(q_k + block(k)), desc(n_k + (k >> 2) * (MW_VEC / 16) + (k & 3) * 2), idesc_n, k != 0);
             }
             umma_commit(b_o1);
           }
@@ -358,9 +375,9 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
           tc_fence_after();
           if (lane == 0 && ok) {
 #pragma unroll
-            for (int k = 0; k < 4; k++) umma_f16_ss(tX, v_mn + k * 128, p_k + k * 2, idesc_o2, k != 0);
+            for (int k = 0; k < 4; k++) umma_f16_ss(tX, desc(v_mn + k * 128), desc(p_k + k * 2), idesc_o2, k != 0);
 #pragma unroll
-            for (int k = 0; k < 4; k++) umma_f16_ss(tX + 64, v_mn + (k + 4) * 128, p_k + MW_BLK / 16 + k * 2, idesc_o2h, 1);
+            for (int k = 0; k < 4; k++) umma_f16_ss(tX + 64, desc(v_mn + (k + 4) * 128), desc(p_k + MW_BLK / 16 + k * 2), idesc_o2h, 1);
             umma_commit(b_o2);
           }
           __syncwarp();
@@ -374,29 +391,25 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
       tc_fence_after();
       if (warp == 8) {
         if (lane == 0 && ok) {
-          const uint64_t w_k = make_smem_desc(smem_u32(sW + par * 2 * MW_VEC), 16, 1024, FT_SWZ_128B);
 #pragma unroll
           for (int k = 0; k < 8; k++) {
-            umma_f16_ss(tX, w_mn + k * 128, k_mn + k * 128, idesc_ds, k != 0);
-            umma_f16_ss(tX, w_mn + 2 * (MW_BLK / 16) + k * 128, k_mn + k * 128, idesc_ds, 1);
+            umma_f16_ss(tX, desc(w_mn + k * 128), desc(k_mn + k * 128), idesc_ds, k != 0);
+            umma_f16_ss(tX, desc(w_mn + 2 * (MW_BLK / 16) + k * 128), desc(k_mn + k * 128), idesc_ds, 1);
           }
-#pragma unroll
-          for (int i = 0; i < (NQ + 1) / 2; i++)
-#pragma unroll
-            for (int k = 0; k < 8; k++) umma_f16_ss(tDn + i * 16, k_mn + i * 2 * (MW_BLK / 16) + k * 128, w_k + (k >> 2) * (MW_VEC / 16) + (k & 3) * 2, idesc_dn, k != 0);
           umma_commit(b_ds);
         }
         __syncwarp();
+        bar_named(BAR_N, 288);                           // n is done with the keys
         wait(b_ds, par, 5);
         if (lane == 0 && ok && c0 + MW_C < rows) load_chunk(c0 + MW_C);
         __syncwarp();
       }
-      m_in = g[5 * MW_C] + g[2 * MW_C - 1];              // sum of the forget gates + last running maximum
-      if (warp == 9 && c0 + MW_C < rows) make_gates(c0 + MW_C, m_in, par ^ 1);
+      m_in = g[6 * MW_C + 4] + g[2 * MW_C - 1];              // sum of the forget gates + last running maximum
+      if (warp == 9 && c0 + MW_C < rows) make_gates(m_in, par ^ 1);
     }
   } else {
     if constexpr (NQ > 2) reg_inc<MW_REGS_STATE>();
-    const int row = (warp & 3) * 32 + lane, half = warp >> 2, nd = half * 128 + row;      // nd: the element of n that this thread keeps
+    const int row = (warp & 3) * 32 + lane, half = warp >> 2;
     const uint32_t lanes = (uint32_t)((warp & 3) * 32) << 16;
     const float scale = rsqrtf((float)D.d);
     float S[NQ * 32];                                    // S[half * 32 NQ + i][v0 + row]
@@ -405,7 +418,7 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
       const int d = half * NQ * 32 + i;
       S[i] = !zero && d < D.d16 && v0 + row < D.v16 ? in[(size_t)d * D.v16 + v0 + row] : 0.f;
     }
-    float n = !zero && nd < D.d16 ? in[n_at + nd] : 0.f, f_total = 0.f;
+    float f_total = 0.f;
     auto publish = [&]() {                               // state and normaliser as operands of the next chunk's outputs
 #pragma unroll
       for (int i = 0; i < NQ; i++) {
@@ -414,11 +427,13 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
         for (int e = 0; e < 16; e++) h[e] = pack2(S[i * 32 + 2 * e], S[i * 32 + 2 * e + 1]);
         tmem_st_32x32b_x16(tA + lanes + half * NQ * 16 + i * 16, h);
       }
-      if (nd < NQ * 64) put_vec(sN, nd, n);
-      fence_proxy_async_smem();
       tmem_st_wait();
     };
-    if (OUT) publish();
+    if (OUT) {
+      publish();
+      if (tid < NQ * 64) put_vec(sN, tid, nf[tid]);
+      fence_proxy_async_smem();
+    }
     int c0 = 0;
     for (int ch = 0; c0 < rows; ch++, c0 += MW_C) {
       const int cnt = min(MW_C, rows - c0), par = ch & 1;
@@ -439,23 +454,50 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
           const int pr = half == 0 ? row : row - 64;
 #pragma unroll
           for (int b = 0; b < 2; b++) {
+            const int kb = half * 2 + b, s0 = kb * 32;   // 32 keys: all ahead of this warp's tokens, around them, or behind
+            if (kb > (warp & 3)) {
+#pragma unroll
+              for (int c8 = 0; c8 < 4; c8++) *reinterpret_cast<uint4*>(dst + sw128(pr, b * 4 + c8)) = make_uint4(0, 0, 0, 0);
+              continue;
+            }
             uint32_t sv[32];
             __syncwarp();
-            tmem_ld_32x32b_x32(tX + lanes + half * 64 + b * 32, sv);
+            tmem_ld_32x32b_x32(tX + lanes + s0, sv);
             tmem_ld_wait();
+            if (kb < (warp & 3)) {                       // e^(u - R) = e^(u - top) e^(top - R), both at most one
+              const float k = scale * exp_fast(u[6 * MW_C + kb] - Rt);
 #pragma unroll
-            for (int c8 = 0; c8 < 4; c8++) {
-              uint32_t h[4];
+              for (int c8 = 0; c8 < 4; c8++) {
+                uint32_t h[4];
 #pragma unroll
-              for (int e = 0; e < 4; e++) {
-                const int s = half * 64 + b * 32 + c8 * 8 + 2 * e;
-                const float2 us = *reinterpret_cast<const float2*>(u + s);
-                const float p0 = s <= row ? __uint_as_float(sv[c8 * 8 + 2 * e]) * scale * exp_fast(us.x - Rt) : 0.f;
-                const float p1 = s + 1 <= row ? __uint_as_float(sv[c8 * 8 + 2 * e + 1]) * scale * exp_fast(us.y - Rt) : 0.f;
-                sum += p0 + p1;
-                h[e] = pack2(p0, p1);
+                for (int e = 0; e < 8; e += 4) {
+                  const float4 eu = *reinterpret_cast<const float4*>(u + 5 * MW_C + s0 + c8 * 8 + e);
+                  const float p0 = __uint_as_float(sv[c8 * 8 + e]) * (eu.x * k), p1 = __uint_as_float(sv[c8 * 8 + e + 1]) * (eu.y * k);
+                  const float p2 = __uint_as_float(sv[c8 * 8 + e + 2]) * (eu.z * k), p3 = __uint_as_float(sv[c8 * 8 + e + 3]) * (eu.w * k);
+                  sum += (p0 + p1) + (p2 + p3);
+                  h[e / 2] = pack2(p0, p1);
+                  h[e / 2 + 1] = pack2(p2, p3);
+                }
+                *reinterpret_cast<uint4*>(dst + sw128(pr, b * 4 + c8)) = make_uint4(h[0], h[1], h[2], h[3]);
               }
-              *reinterpret_cast<uint4*>(dst + sw128(pr, b * 4 + c8)) = make_uint4(h[0], h[1], h[2], h[3]);
+            } else {
+#pragma unroll
+              for (int c8 = 0; c8 < 4; c8++) {
+                uint32_t h[4];
+#pragma unroll
+                for (int e = 0; e < 8; e += 4) {
+                  const int i = c8 * 8 + e;                // key, counted from the warp's first token; this thread's is `lane`
+                  const float4 us = *reinterpret_cast<const float4*>(u + s0 + i);
+                  const float p0 = i <= lane ? __uint_as_float(sv[i]) * (scale * exp_fast(us.x - Rt)) : 0.f;
+                  const float p1 = i + 1 <= lane ? __uint_as_float(sv[i + 1]) * (scale * exp_fast(us.y - Rt)) : 0.f;
+                  const float p2 = i + 2 <= lane ? __uint_as_float(sv[i + 2]) * (scale * exp_fast(us.z - Rt)) : 0.f;
+                  const float p3 = i + 3 <= lane ? __uint_as_float(sv[i + 3]) * (scale * exp_fast(us.w - Rt)) : 0.f;
+                  sum += (p0 + p1) + (p2 + p3);
+                  h[e / 2] = pack2(p0, p1);
+                  h[e / 2 + 1] = pack2(p2, p3);
+                }
+                *reinterpret_cast<uint4*>(dst + sw128(pr, b * 4 + c8)) = make_uint4(h[0], h[1], h[2], h[3]);
+              }
             }
           }
         }
@@ -477,26 +519,36 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
         bar_named(BAR_DEN, 256);
         wait(b_o2, par, 4);
         tc_fence_after();
-        // outputs: thread (value row, half of the tokens); neighbouring lanes trade every second token, so that each stores pairs of columns
-        const int odd = lane & 1, col = v0 + (row & ~1);
+        // outputs: thread (value row, half of the tokens); four neighbouring lanes turn four tokens around, so that each stores four columns of one token
+        const int b0 = lane & 1, b1 = (lane >> 1) & 1, mine = lane & 3, col = v0 + (row & ~3);
         const size_t pitch = (size_t)D.H * D.v16;
-        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(io.o) + (size_t)(row0 + c0 + half * 64 + odd) * pitch + hd * D.v16 + col;
-        const int left = col < D.v16 ? cnt - half * 64 - odd : 0;        // tokens of this thread that exist, every second one counted twice
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(io.o) + (size_t)(row0 + c0 + half * 64 + mine) * pitch + hd * D.v16 + col;
+        const int left = col < D.v16 ? cnt - half * 64 - mine : 0;       // tokens of this thread's that exist, every fourth one counted as four
+        uint32_t o1[2][16], o2[2][16];
+        auto fetch = [&](int b) {
+          tmem_ld_32x32b_x16(tX + 128 + lanes + half * 64 + b * 16, o1[b & 1]);
+          tmem_ld_32x32b_x16(tX + lanes + half * 64 + b * 16, o2[b & 1]);
+        };
+        __syncwarp();
+        fetch(0);
 #pragma unroll
         for (int b = 0; b < 4; b++) {
           const int t0 = half * 64 + b * 16;
-          uint32_t o1[16], o2[16];
-          __syncwarp();
-          tmem_ld_32x32b_x16(tX + 128 + lanes + t0, o1);
-          tmem_ld_32x32b_x16(tX + lanes + t0, o2);
           tmem_ld_wait();
+          __syncwarp();
+          if (b < 3) fetch(b + 1);
+          const uint32_t (&p1)[16] = o1[b & 1];
+          const uint32_t (&p2)[16] = o2[b & 1];
 #pragma unroll
-          for (int e = 0; e < 16; e += 2) {
-            const float2 en = *reinterpret_cast<const float2*>(ein + t0 + e), iv = *reinterpret_cast<const float2*>(inv + t0 + e);
-            const float x = (__uint_as_float(o1[e]) * en.x + __uint_as_float(o2[e])) * iv.x, y = (__uint_as_float(o1[e + 1]) * en.y + __uint_as_float(o2[e + 1])) * iv.y;
-            const float got = __shfl_xor_sync(0xffffffffu, odd ? x : y, 1);
-            if (b * 16 + e < left) *reinterpret_cast<uint32_t*>(dst) = odd ? pack2(got, y) : pack2(x, got);
-            dst += 2 * pitch;
+          for (int e = 0; e < 16; e += 4) {
+            const float4 en = *reinterpret_cast<const float4*>(ein + t0 + e), iv = *reinterpret_cast<const float4*>(inv + t0 + e);
+            const float a = (__uint_as_float(p1[e]) * en.x + __uint_as_float(p2[e])) * iv.x, bb = (__uint_as_float(p1[e + 1]) * en.y + __uint_as_float(p2[e + 1])) * iv.y;
+            const float c = (__uint_as_float(p1[e + 2]) * en.z + __uint_as_float(p2[e + 2])) * iv.z, d = (__uint_as_float(p1[e + 3]) * en.w + __uint_as_float(p2[e + 3])) * iv.w;
+            const float g0 = __shfl_xor_sync(0xffffffffu, b0 ? a : bb, 1), g1 = __shfl_xor_sync(0xffffffffu, b0 ? c : d, 1);
+            const uint32_t lo = b0 ? pack2(g0, bb) : pack2(a, g0), hi = b0 ? pack2(g1, d) : pack2(c, g1);      // columns of the lane pair: token b0, token 2 + b0
+            const uint32_t got = __shfl_xor_sync(0xffffffffu, b1 ? lo : hi, 2);
+            if (b * 16 + e < left) *reinterpret_cast<uint2*>(dst) = b1 ? make_uint2(got, hi) : make_uint2(lo, got);
+            dst += 4 * pitch;
           }
         }
       } else {
@@ -504,12 +556,44 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
         weigh_values(u + 2 * MW_C, tid, 256);
         fence_proxy_async_smem();
       }
-      const float r_last = R[MW_C - 1], f_chunk = u[5 * MW_C], decay = exp_fast(m_in - r_last);
+      const float r_last = R[MW_C - 1], f_chunk = u[6 * MW_C + 4], decay = exp_fast(m_in - r_last);
       tc_fence_before();
       bar_named(BAR_STATE, MW_THREADS);
       tc_fence_after();
       m_in = f_chunk + r_last;
       f_total += f_chunk;
+      {                                                  // n: a lane takes eight columns of every eighth token
+        const int tg = lane >> 2;
+        const float* w = u + 2 * MW_C;
+        for (int j = warp * 4 + (lane & 3); j < NQ * 8; j += 32) {
+          float a[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
+#pragma unroll 4
+          for (int i = 0; i < MW_C / 8; i++) {
+            const int t = i * 8 + tg;
+            float k8[8];
+            bf16x8_to_float(*reinterpret_cast<const bf16x8*>(sK + (j >> 3) * MW_BLK + sw128(t, j & 7)), k8);
+            const float wt = w[t];
+#pragma unroll
+            for (int e = 0; e < 8; e++) a[e] += wt * k8[e];
+          }
+#pragma unroll
+          for (int e = 0; e < 8; e++) {
+            a[e] += __shfl_xor_sync(0xffffffffu, a[e], 4);
+            a[e] += __shfl_xor_sync(0xffffffffu, a[e], 8);
+            a[e] += __shfl_xor_sync(0xffffffffu, a[e], 16);
+          }
+          if (tg == 0) {
+#pragma unroll
+            for (int e = 0; e < 8; e++) {
+              const float v = nf[j * 8 + e] * decay + a[e];
+              nf[j * 8 + e] = v;
+              if (OUT) put_vec(sN, j * 8 + e, v);        // the products that read the old one are done
+            }
+          }
+        }
+        fence_proxy_async_smem();
+      }
+      bar_named(BAR_N, 288);                             // K may be overwritten from here on
       wait(b_ds, par, 5);
       tc_fence_after();
 #pragma unroll
@@ -520,13 +604,6 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
         tmem_ld_wait();
 #pragma unroll
         for (int e = 0; e < 32; e++) S[i * 32 + e] = S[i * 32 + e] * decay + __uint_as_float(x[e]);
-      }
-      if (NQ > 2 || half == 0) {
-        uint32_t x[16];
-        __syncwarp();
-        tmem_ld_32x32b_x16(tDn + lanes + half * 16, x);
-        tmem_ld_wait();
-        n = n * decay + (__uint_as_float(x[0]) + __uint_as_float(x[1]));
       }
       if (OUT && c0 + MW_C < rows) publish();
     }
@@ -542,7 +619,7 @@ __global__ void __launch_bounds__(MW_THREADS, 1) mm_walk_kernel(const __grid_con
       if (blockIdx.z == 0) {
         // a slot's n may still be unread by the other CTAs of this head: it moves there later
         float* to = OUT ? io.nm + ((size_t)sg[3] * D.H + hd) * (D.d16 + 4) : dst + n_at;
-        if (nd < D.d16) to[nd] = n;
+        for (int i = tid; i < D.d16; i += 256) to[i] = nf[i];
         if (tid == 0) {
           to[D.d16] = m_in;
           to[D.d16 + 1] = f_total;
