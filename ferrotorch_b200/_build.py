@@ -42,6 +42,9 @@ PRECISE_MATH = {"elementwise.cu", "reduce_index.cu", "nn_ops.cu", "stream_ops.cu
 CXX_FLAGS = ["-O3", "-fno-math-errno", "-fno-trapping-math", "-ffp-contract=off", "-std=c++20", "-fPIC", "-fvisibility=hidden", "-pthread", "-I", str(CSRC / "include"), "-I", str(CSRC / "runtime")]
 
 
+KERNEL_LINK = [NVCC, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-cudart", "static", "-Xcompiler", "-fPIC", "-Xlinker", "--exclude-libs,ALL"]
+
+
 def _newest_header_mtime(dirs) -> float:
     m = 0.0
     for d in dirs:
@@ -98,9 +101,15 @@ def runtime_sources():
 
 def build_kernels(verbose=False, ptxas_info=False):
     extra = ["-Xptxas", "-v"] if ptxas_info else []
-    link = [NVCC, "-shared", "-gencode", "arch=compute_100a,code=sm_100a", "-cudart", "static", "-Xcompiler", "-fPIC", "-Xlinker", "--exclude-libs,ALL"]
-    return _build_lib("libft_kernels.so", kernel_sources(), NVCC, NVCC_FLAGS, link, [CSRC / "kernels", CSRC / "include"],
+    return _build_lib("libft_kernels.so", kernel_sources(), NVCC, NVCC_FLAGS, KERNEL_LINK, [CSRC / "kernels", CSRC / "include"],
                       verbose or ptxas_info, extra)
+
+
+def build_kernels_part(name: str, stems):
+    """``libft_kernels_<name>.so``: the launchers of the named sources only (their objects are shared with the full library)."""
+    OUT.mkdir(parents=True, exist_ok=True)
+    sources = [CSRC / "kernels" / f"{s}.cu" for s in sorted({*stems, "host_common"})]
+    return _build_lib(f"libft_kernels_{name}.so", sources, NVCC, NVCC_FLAGS, KERNEL_LINK, [CSRC / "kernels", CSRC / "include"], False)
 
 
 def build_runtime(verbose=False):

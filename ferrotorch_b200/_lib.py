@@ -44,12 +44,38 @@ def _load(name: str):
     return ctypes.CDLL(str(path), mode=ctypes.RTLD_LOCAL)
 
 
+_part = None          # (name, sources) that suffice for this process, see prefer_part
+_on_part = False
+
+
+def prefer_part(name: str, sources) -> None:
+    """In a checkout without a built kernel library, compile and load the launchers of ``sources`` alone (file stems): what one architecture needs. A built full
+    library is used as ever, and a launcher outside the part brings the full one in."""
+    global _part
+    if _kernels is None:
+        _part = (name, tuple(sources))
+
+
 def kernels():
-    global _kernels
+    global _kernels, _on_part
     if _kernels is None:
         with _lock:
             if _kernels is None:
-                _kernels = _load("libft_kernels.so")
+                if _part and not (_DIR / "libft_kernels.so").exists() and os.environ.get("FT_NO_AUTOBUILD") != "1":
+                    from . import _build
+                    _kernels, _on_part = ctypes.CDLL(str(_build.build_kernels_part(*_part)), mode=ctypes.RTLD_LOCAL), True
+                else:
+                    _kernels = _load("libft_kernels.so")
+    return _kernels
+
+
+def _full_kernels():
+    """Leaves a partial library for the full one."""
+    global _kernels, _on_part
+    with _lock:
+        if _on_part:
+            _kernels, _on_part = _load("libft_kernels.so"), False
+            _bound.clear()
     return _kernels
 
 
@@ -116,7 +142,8 @@ def register_sigs(sigs: dict) -> None:
 def _fn(fn_name: str):
     f = _bound.get(fn_name)
     if f is None:
-        f = getattr(kernels(), fn_name)
+        lib = kernels()
+        f = getattr(lib if not _on_part or hasattr(lib, fn_name) else _full_kernels(), fn_name)
         if not _SIGS:
             _parse_sigs()
         sig = _SIGS.get(fn_name)

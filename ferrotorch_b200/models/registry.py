@@ -12,16 +12,19 @@ from typing import Callable, Dict, List
 
 import torch
 
+from .. import _lib
 from ..errors import InvalidArgument, ShapeMismatch
 
 
 @dataclass
 class Architecture:
-    """``config(dict)`` parses ``config.json``; ``engine(config, weights, device, dtype, max_tokens)`` builds the engine."""
+    """``config(dict)`` parses ``config.json``; ``engine(config, weights, device, dtype, max_tokens)`` builds the engine; ``kernels`` names the kernel sources that
+    serve it (all that has to be compiled where nothing is built yet; empty: all of them)."""
     name: str
     config: Callable[[dict], object]
     engine: Callable[..., object]
     aliases: tuple = ()
+    kernels: tuple = ()
 
 
 _ARCHITECTURES: Dict[str, Architecture] = {}
@@ -78,6 +81,8 @@ def checked_weights(name: str, shapes: Dict[str, tuple], weights, device, option
 
 def load_engine(directory, device="cuda", dtype: torch.dtype = torch.bfloat16, max_tokens: int = 4096):
     arch, cfg = load_model_config(directory)
+    if arch.kernels:
+        _lib.prefer_part(arch.name.lower(), arch.kernels)
     return arch.engine(cfg, load_checkpoint_weights(directory), device, dtype, max_tokens)
 
 
@@ -116,6 +121,7 @@ def _llama_engine(cfg, weights, device, dtype, max_tokens):
     return CachedModelEngine(CachedLlama(cfg, {k: v.to(device, dtype) for k, v in weights.items()}), cfg.vocab_size, device)
 
 
-register_architecture(Architecture("Ginisun", _ginisun_config, _ginisun_engine))
-register_architecture(Architecture("Pufevik", _pufevik_config, _pufevik_engine))
+PRODUCTS = ("gemm_tcgen05", "gemm_2sm", "gemm_simt", "fsdp_gather", "decode")      # matrix products and their split-K forms
+register_architecture(Architecture("Ginisun", _ginisun_config, _ginisun_engine, kernels=(*PRODUCTS, "stream_ops", "moe", "latent_attn")))
+register_architecture(Architecture("Pufevik", _pufevik_config, _pufevik_engine, kernels=(*PRODUCTS, "gqa_attn", "matrix_memory", "residual_ops")))
 register_architecture(Architecture("LlamaForCausalLM", _llama_config, _llama_engine, ("llama",)))

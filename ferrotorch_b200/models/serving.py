@@ -115,10 +115,11 @@ class RowBatch:
         ``ctas`` 0: one segment per sequence."""
         if ctas not in self._plans:
             segs, inner, chains = [], [], []
-            per_seq = max(1, SEGMENT_CTAS // (ctas * len(self._spans))) if ctas else 1
+            # an equal share of all new tokens per segment, as many segments as the GPU takes at once
+            share = max(SEGMENT_MIN, -(-self.rows // max(1, SEGMENT_CTAS // ctas) // MEMORY_CHUNK) * MEMORY_CHUNK) if ctas else 0
             scratch = 0
             for i, (r0, n, start, _) in enumerate(self._spans):
-                size = -(-n // min(per_seq, max(1, n // SEGMENT_MIN)) // MEMORY_CHUNK) * MEMORY_CHUNK if ctas else n
+                size = share or n
                 count, slot, fresh = -(-n // size), self._state_slots[i], int(start == 0)
                 base = scratch if count > 1 else 0
                 for j in range(count):
