@@ -669,8 +669,9 @@ gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 9 + 4 * NT);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  const int4 tl = tiles[blockIdx.x];                // first query row, tokens, position of the first token, sequence
-  const int g = blockIdx.y, tok = A.tok, window = A.M.window;
+  // the groups of a tile next to one another: tiles come longest first, so the CTAs do too
+  const int4 tl = tiles[blockIdx.x / A.D.G];        // first query row, tokens, position of the first token, sequence
+  const int g = blockIdx.x % A.D.G, tok = A.tok, window = A.M.window;
   // key blocks [j0, j0 + nblk[t]) of every sub-tile; the start is the window of the tile's first token
   const int j0 = (tl.z - window >= 0 ? tl.z - window + 1 : 0) / GF_BN;
   int nblk[NT], nmax = 0;
@@ -930,7 +931,7 @@ int launch_flash(const CUtensorMap (&m)[3], const int* tiles, int ntiles, const 
     FT_CUDA_TRY(cudaFuncSetAttribute(gqa_flash_kernel<NT, NQ, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX));
     done[dev] = true;
   }
-  gqa_flash_kernel<NT, NQ, NV><<<dim3(ntiles, A.D.G), 64 + 128 * NT, smem, st>>>(m[0], m[1], m[2], reinterpret_cast<const int4*>(tiles), bt, A, (__nv_bfloat16*)out, ldo,
+  gqa_flash_kernel<NT, NQ, NV><<<ntiles * A.D.G, 64 + 128 * NT, smem, st>>>(m[0], m[1], m[2], reinterpret_cast<const int4*>(tiles), bt, A, (__nv_bfloat16*)out, ldo,
                                                                                  ft_status_ptr());
   return (int)cudaGetLastError();
 }
