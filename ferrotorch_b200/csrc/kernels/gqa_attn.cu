@@ -642,15 +642,20 @@ struct FlashArgs {
   int R, tok;                      // query heads per key / value head, tokens per sub-tile
   int nq, nv;                      // 64-column blocks of key and value sizes
   int max_blocks;
+  int slack;                       // bytes of shared memory left for alignment
 };
+
+// two CTAs of one sub-tile per SM: their halves of tensor memory hold scores and up to two value blocks
+constexpr bool gf_pair(int NT, int NV) { return NT == 1 && NV > 0 && NV <= 2; }
 
 // NQ, NV: column blocks at compile time (the issuing thread's descriptors then are constants added to a base), or 0 to read them from A.
 template <int NT, int NQ, int NV>
-__global__ void __launch_bounds__(64 + 128 * NT, (NT == 1 && NV == 1) ? 2 : 1)
+__global__ void __launch_bounds__(64 + 128 * NT, gf_pair(NT, NV) ? 2 : 1)
 gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, const int4* __restrict__ tiles,
                  const int* __restrict__ block_table, FlashArgs A, __nv_bfloat16* __restrict__ out, int64_t ldo, uint32_t* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  if ((int)(smem - smem_raw) > A.slack) { ft_set_status(status, FT_K_GQA, 10, 0); return; }      // dynamic shared memory starts at a multiple of 1024 here
   const int nq = NQ > 0 ? NQ : A.nq, nv = NV > 0 ? NV : A.nv;
   const int k_bytes = nq * GF_KB, v_bytes = nv * GF_KB;
   uint8_t* sQ = smem;                               // [NT][nq]
@@ -688,7 +693,7 @@ gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     mbar_fence_init();
   }
   if (warp == 0 && lane == 0) { tma_prefetch_desc(&tmQ); tma_prefetch_desc(&tmK); tma_prefetch_desc(&tmV); }
-  constexpr uint32_t TMEM = (NT == 1 && NV == 1) ? 256 : 512;       // small heads leave room for a second CTA
+  constexpr uint32_t TMEM = gf_pair(NT, NV) ? 256 : 512;
   if (warp == 1) { tmem_alloc(tmem_slot, TMEM); tmem_relinquish(); }
   tc_fence_before();
   __syncthreads();
@@ -910,7 +915,8 @@ gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
 }
 
 constexpr int SMEM_MAX = 232448;
-int flash_smem(int NT, int nq, int nv) { return NT * nq * GF_QB + 2 * (nq + nv) * GF_KB + NT * GF_PB + 256 + 1024; }
+int flash_slack(int NT, int nq, int nv) { return NT == 1 && nq == 2 && nv == 2 ? 640 : 1024; }      // two CTAs of the largest pair fit an SM to within this
+int flash_smem(int NT, int nq, int nv) { return NT * nq * GF_QB + 2 * (nq + nv) * GF_KB + NT * GF_PB + 64 + 64 * NT + flash_slack(NT, nq, nv); }
 
 bool make_dims(GqaDims& D, int H, int G, int d, int dv, int rot) {
   if (G < 1 || H < G || H % G || H > 65535 || d < 1 || dv < 1 || rot < 0 || rot > d || (rot & 1)) return false;
@@ -1060,7 +1066,7 @@ FT_EXPORT int ft_gqa_flash_subtiles(int H, int G, int d, int dv) {
   GqaDims D;
   if (!make_dims(D, H, G, d, dv, 0) || H / G > GF_BM) return 0;
   const int nq = (d + 63) / 64, nv = (dv + 63) / 64;
-  if (nq <= 2 && nv == 1) return 1;                    // two CTAs of one sub-tile per SM
+  if (nq <= 2 && nv <= 2) return 1;                    // two CTAs of one sub-tile per SM
   if (nv <= 2 && flash_smem(2, nq, nv) <= SMEM_MAX) return 2;
   if (nv <= 4 && flash_smem(1, nq, nv) <= SMEM_MAX) return 1;
   return 0;
@@ -1095,13 +1101,13 @@ FT_EXPORT int ft_gqa_flash(const void* q, int64_t ldq, int q_rows, const void* c
   if (!r) r = ft_make_tmap_3d(&m[2], cp + (size_t)G * D.d16, 2, true, D.v16, G, slots, (uint64_t)D.v16 * 2, krow, 64, 1, KV_BLOCK, CU_TENSOR_MAP_SWIZZLE_128B);
   if (r) return r;
   const int smem = flash_smem(nt, A.nq, A.nv);
+  A.slack = flash_slack(nt, A.nq, A.nv);
 #define FT_GF(T, Q, V) return launch_flash<T, Q, V>(m, tiles, ntiles, block_table, A, out, ldo, smem, st)
-  if (nt == 2) {
-    if (A.nq == 2 && A.nv == 2) FT_GF(2, 2, 2);
-    FT_GF(2, 0, 0);
-  }
+  if (nt == 2) FT_GF(2, 0, 0);
   if (A.nq == 1 && A.nv == 1) FT_GF(1, 1, 1);
   if (A.nq == 2 && A.nv == 1) FT_GF(1, 2, 1);
+  if (A.nq == 1 && A.nv == 2) FT_GF(1, 1, 2);
+  if (A.nq == 2 && A.nv == 2) FT_GF(1, 2, 2);
   FT_GF(1, 0, 0);
 #undef FT_GF
 }
