@@ -1,8 +1,9 @@
-// Matrix memory (the mLSTM cell of xLSTM, Beck et al. 2024): per head a d x dv matrix S and a vector n that decay by a forget gate and take in k v^T and k with an
-// input gate, both gates in the log domain against a running maximum m that starts at zero:
+// Matrix memory (the mLSTM cell of Beck et al., "xLSTM: Extended Long Short-Term Memory", 2024). A head remembers a d x dv matrix S, a vector n of size d and a level m,
+// all zero ahead of the first token; S and n are kept divided by e^m. A token with log forget gate f, log input gate i, query q (scaled), key k and value v does
 //
-//   m_t = max(f_t + m_(t-1), i_t);   S_t = e^(f_t + m_(t-1) - m_t) S_(t-1) + e^(i_t - m_t) k_t v_t^T;   n_t alike with k_t
-//   o_t = S_t^T q_t / (max(|n_t . q_t|, e^(-m_t)) + 1e-6)
+//   level   m'   = larger of m + f and i           keep = e^(m + f - m'),  take = e^(i - m')
+//   memory  S'   = keep S + take k v^T             n'   = keep n + take k
+//   output  S'^T q divided by (1e-6 + larger of |n' . q| and e^(-m'))
 //
 // followed by an RMS norm of every head's output, a weight, a sigmoid gate and a scale. States live in f32, one slot per sequence: [heads][d16 x v16 | n (d16) |
 // m, 3 spare], head sizes padded to multiples of 16 with zeros.
