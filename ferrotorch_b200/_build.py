@@ -36,7 +36,8 @@ NVCC_FLAGS = [
     "-I", str(CSRC / "kernels"), "-I", str(CSRC / "include"),
 ]
 # bandwidth-bound generic kernels keep IEEE-accurate transcendentals (they are compared against f32 / f64 references at tight tolerances)
-PRECISE_MATH = {"elementwise.cu", "reduce_index.cu", "nn_ops.cu", "stream_ops.cu", "moe.cu", "latent_attn.cu", "residual_ops.cu", "gqa_attn.cu", "matrix_memory.cu"}
+PRECISE_MATH = {"elementwise.cu", "reduce_index.cu", "nn_ops.cu", "stream_ops.cu", "moe.cu", "latent_attn.cu", "residual_ops.cu", "gqa_attn.cu", "matrix_memory.cu",
+                "state_space.cu"}
 # no errno / trap bookkeeping for the math builtins (lets the Box-Muller and Philox loops vectorise); no FMA contraction, so the random streams are
 # the same on every x86-64 machine whatever instruction set the vector path picks
 CXX_FLAGS = ["-O3", "-fno-math-errno", "-fno-trapping-math", "-ffp-contract=off", "-std=c++20", "-fPIC", "-fvisibility=hidden", "-pthread", "-I", str(CSRC / "include"), "-I", str(CSRC / "runtime")]

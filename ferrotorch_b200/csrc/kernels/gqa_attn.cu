@@ -1,6 +1,7 @@
-// Grouped-query attention with per-head key and value sizes, over a paged row cache: rotary positions on the first dimensions of a head (neighbouring pairs),
-// RMS norms on queries and keys (per head, or over the whole projection), an optional sliding window, softmax with an optional sink per head, values
-// optionally mixed with those of an earlier layer, and an output gate (per element or per head) with a scale.
+// Grouped-query attention with per-head key and value sizes, over a paged row cache: rotary positions on the first dimensions of a head (neighbouring pairs, or the
+// two halves of the rotated part), RMS norms on queries and keys (per head, over the whole projection, or none), an optional sliding window beside which the first
+// tokens of a sequence may stay visible, softmax with an optional sink per head, values optionally mixed with those of an earlier layer, and an output gate (per
+// element or per head) with a scale.
 //
 // Head sizes are padded to multiples of 16 (zeros): d16, v16. A token's cache row is [G keys of d16 | G values of v16]; pages hold 16 rows.
 //
@@ -34,6 +35,7 @@ struct GqaDims {
   int row;                           // cache row: G * (d16 + v16)
 };
 enum { GATE_NONE = 0, GATE_ELEMENT = 1, GATE_HEAD = 2 };
+enum { NORM_HEAD = 0, NORM_WHOLE = 1, NORM_NONE = 2 };
 
 // eight consecutive elements
 template <typename T> FT_DEVICE void load8(const T* p, float (&v)[8]);
@@ -51,14 +53,17 @@ template <> FT_DEVICE void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (
 template <typename T> FT_DEVICE float one(T v);
 template <> FT_DEVICE float one<float>(float v) { return v; }
 template <> FT_DEVICE float one<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+FT_DEVICE void put1(float* p, float v) { *p = v; }
+FT_DEVICE void put1(__nv_bfloat16* p, float v) { *p = __float2bfloat16(v); }
 
 // ------------------------------------------------------------------------------------------------------------
 // prompt rows: one CTA per row; a thread holds eight neighbouring columns (four rotation pairs) of a head. WHOLE: one norm over all heads.
 // ------------------------------------------------------------------------------------------------------------
 struct PrepArgs {
   GqaDims D;
-  const float *wq, *wk;              // per head: [d16]; whole: [heads * d16]
+  const float *wq, *wk;              // per head: [d16]; whole: [heads * d16]; null: no norm
   float eps;
+  int halves;                        // dimension i turns with i + rot / 2, not 2 i with 2 i + 1
   const int* positions;
   const float *cos_t, *sin_t;
   const int* slots;
@@ -75,11 +80,13 @@ __global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, i
   T* dst = cache + (size_t)A.slots[r] * D.row;
   const float* ct = A.cos_t + (size_t)pos * half;
   const float* st = A.sin_t + (size_t)pos * half;
+  const bool normed = WHOLE || A.wq != nullptr;
+  auto weights = [&](int head) -> const float* { return (head < D.H ? A.wq : A.wk) + (WHOLE ? (head < D.H ? head : head - D.H) * D.d16 : 0); };
   auto finish = [&](int head, int vi, bool is_q, const float (&x)[8], float rstd) {       // norm weight, rotation, store
-    const float* w = (is_q ? A.wq : A.wk) + (WHOLE ? (is_q ? head : head - D.H) * D.d16 : 0) + vi * 8;
+    const float* w = normed ? weights(head) + vi * 8 : nullptr;
     float v[8];
 #pragma unroll
-    for (int e = 0; e < 8; e++) v[e] = x[e] * rstd * w[e];
+    for (int e = 0; e < 8; e++) v[e] = normed ? x[e] * rstd * w[e] : x[e];
 #pragma unroll
     for (int e = 0; e < 4; e++) {
       const int p = vi * 4 + e;
@@ -90,6 +97,46 @@ __global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, i
       }
     }
     store8(is_q ? row + head * D.d16 + vi * 8 : dst + (head - D.H) * D.d16 + vi * 8, v);
+  };
+  // the same for pairs (i, i + half): a lane takes both of a pair, so nothing is read after it was overwritten
+  auto finish_halves = [&](int head, int l, int lanes, float rstd) {
+    const bool is_q = head < D.H;
+    const T* src = row + head * D.d16;
+    T* to = is_q ? row + head * D.d16 : dst + (head - D.H) * D.d16;
+    const float* w = normed ? weights(head) : nullptr;
+    if ((half & 7) == 0) {
+      for (int vi = l; vi < half / 8; vi += lanes) {
+        float a[8], b[8];
+        load8(src + vi * 8, a);
+        load8(src + half + vi * 8, b);
+#pragma unroll
+        for (int e = 0; e < 8; e++) {
+          const int p = vi * 8 + e;
+          const float c = ct[p], s = st[p], u = normed ? a[e] * rstd * w[p] : a[e], v = normed ? b[e] * rstd * w[half + p] : b[e];
+          a[e] = u * c - v * s;
+          b[e] = v * c + u * s;
+        }
+        store8(to + vi * 8, a);
+        store8(to + half + vi * 8, b);
+      }
+      if (is_q && !normed) return;                   // the rest stays as it is
+      for (int vi = D.rot / 8 + l; vi < hv; vi += lanes) {
+        float a[8];
+        load8(src + vi * 8, a);
+        if (normed)
+#pragma unroll
+          for (int e = 0; e < 8; e++) a[e] = a[e] * rstd * w[vi * 8 + e];
+        store8(to + vi * 8, a);
+      }
+    } else {
+      auto at = [&](int c) { return normed ? one(src[c]) * rstd * w[c] : one(src[c]); };
+      for (int p = l; p < half; p += lanes) {
+        const float c = ct[p], s = st[p], u = at(p), v = at(half + p);
+        put1(to + p, u * c - v * s);
+        put1(to + half + p, v * c + u * s);
+      }
+      for (int c = D.rot + l; c < D.d16; c += lanes) put1(to + c, at(c));
+    }
   };
   if constexpr (WHOLE) {
     float sq = 0.f, sk = 0.f, x[8];
@@ -103,9 +150,13 @@ __global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, i
     sq = block_sum(sq, red);
     sk = block_sum(sk, red);
     const float rq = 1.f / sqrtf(sq / (float)(D.H * D.d) + A.eps), rk = 1.f / sqrtf(sk / (float)(D.G * D.d) + A.eps);
-    for (int i = threadIdx.x; i < nq + nk; i += PREP_T) {
-      load8(row + i * 8, x);
-      finish(i / hv, i % hv, i < nq, x, i < nq ? rq : rk);
+    if (A.halves) {
+      for (int head = threadIdx.x >> 5; head < D.H + D.G; head += PREP_T / 32) finish_halves(head, threadIdx.x & 31, 32, head < D.H ? rq : rk);
+    } else {
+      for (int i = threadIdx.x; i < nq + nk; i += PREP_T) {
+        load8(row + i * 8, x);
+        finish(i / hv, i % hv, i < nq, x, i < nq ? rq : rk);
+      }
     }
   } else {
     int lanes = 1;                                   // lanes of a head: a power of two that covers its columns, at most a warp
@@ -115,7 +166,7 @@ __global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, i
       const int head = h0 + threadIdx.x / lanes;
       const bool live = head < D.H + D.G;
       float x[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f}, s = 0.f;
-      if (live)
+      if (live && (normed || !A.halves))
         for (int vi = l; vi < hv; vi += lanes) {
           load8(row + head * D.d16 + vi * 8, x);
 #pragma unroll
@@ -123,7 +174,8 @@ __global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, i
         }
       for (int o = lanes / 2; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
       const float rstd = 1.f / sqrtf(s / (float)D.d + A.eps);
-      if (live)
+      if (live && A.halves) finish_halves(head, l, lanes, rstd);
+      if (live && !A.halves)
         for (int vi = l; vi < hv; vi += lanes) {
           if (hv > lanes) load8(row + head * D.d16 + vi * 8, x);       // a single vector per lane is still in registers
           finish(head, vi, head < D.H, x, rstd);
@@ -150,6 +202,7 @@ __global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, i
 struct MaskGate {
   float scale;
   int window;                        // keys a position sees, itself included (INT_MAX: all)
+  int keep;                          // and the first keys of the sequence
   const float* sink;                 // [H] or null
   const void* gate;                  // per element: rows of H * v16 in the data type; per head: f32 rows of H (pre-activation)
   int64_t ldg;
@@ -165,6 +218,7 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const T* __restrict__ q, 
   __shared__ float sp[ROWS_CHUNK];
   const int r = blockIdx.x, hd = blockIdx.y, g = hd / (D.H / D.G), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int len = positions[r] + 1, first = M.window < len ? len - M.window : 0;
+  const int kept = min(M.keep, first), gap = first - kept, total = len - gap;        // visible keys in order: 0..kept, first..len
   const int* bt = block_table + (size_t)seq_of[r] * max_blocks;
   for (int i = threadIdx.x; i < D.d16; i += 128) sq[i] = one(q[(size_t)r * ldq + hd * D.d16 + i]);
   float o[ROWS_MAX_COLS];
@@ -173,10 +227,10 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const T* __restrict__ q, 
   float m = -INFINITY, l = 0.f;
   if (M.sink) { m = M.sink[hd]; l = 1.f; }           // the sink is a score without a value
   __syncthreads();
-  for (int t0 = first; t0 < len; t0 += ROWS_CHUNK) {
-    const int cnt = min(ROWS_CHUNK, len - t0);
+  for (int t0 = 0; t0 < total; t0 += ROWS_CHUNK) {
+    const int cnt = min(ROWS_CHUNK, total - t0);
     for (int k = warp; k < cnt; k += 4) {
-      const int t = t0 + k;
+      const int t = t0 + k < kept ? t0 + k : t0 + k + gap;
       const T* kr = cache + ((size_t)bt[t / KV_BLOCK] * KV_BLOCK + t % KV_BLOCK) * D.row + g * D.d16;
       float a = 0.f;
       for (int i = lane; i < D.d16; i += 32) a += sq[i] * one(kr[i]);
@@ -191,7 +245,7 @@ __global__ void __launch_bounds__(128) gqa_rows_kernel(const T* __restrict__ q, 
 #pragma unroll
     for (int i = 0; i < ROWS_MAX_COLS; i++) o[i] *= alpha;
     for (int k = 0; k < cnt; k++) {
-      const int t = t0 + k;
+      const int t = t0 + k < kept ? t0 + k : t0 + k + gap;
       const T* vr = cache + ((size_t)bt[t / KV_BLOCK] * KV_BLOCK + t % KV_BLOCK) * D.row + D.G * D.d16 + g * D.v16;
       const float p = expf(sp[k] - mx);
       l += p;
@@ -263,7 +317,7 @@ FT_DEVICE void put_bf16x4(__nv_bfloat16* p, float4 v) {
 template <bool WHOLE>
 __global__ void __launch_bounds__(DP_WARPS * 32) gqa_decode_prep_kernel(DecPrepArgs A, __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache) {
   namespace cg = cooperative_groups;
-  extern __shared__ __align__(16) float held[];      // WHOLE: plane sums of this CTA's query and key heads, [local unit][d16]
+  extern __shared__ __align__(16) float held[];      // plane sums of query and key heads: WHOLE [local unit][d16], else (halves) [warp][d16]
   __shared__ float red[32];
   __shared__ float cta_ss[2];
   pdl_wait();
@@ -276,21 +330,39 @@ __global__ void __launch_bounds__(DP_WARPS * 32) gqa_decode_prep_kernel(DecPrepA
   __nv_bfloat16* dst = blk < 0 ? nullptr : cache + ((size_t)blk * KV_BLOCK + pos % KV_BLOCK) * D.row;
   const float* ct = A.P.cos_t + (size_t)pos * half;
   const float* st = A.P.sin_t + (size_t)pos * half;
-  auto finish = [&](int u, int c, float4 v, float rstd) {
+  const bool normed = WHOLE || A.P.wq != nullptr;
+  auto finish = [&](int u, int c, float4 v, float rstd, const float* sums) {       // sums: this head's plane sums (read for pairs of halves only)
     const bool is_q = u < D.H;
-    const float* wp = (is_q ? A.P.wq : A.P.wk) + (WHOLE ? (is_q ? u : u - D.H) * D.d16 : 0) + c;
-    const float4 w = *reinterpret_cast<const float4*>(wp);
-    v = make_float4(v.x * rstd * w.x, v.y * rstd * w.y, v.z * rstd * w.z, v.w * rstd * w.w);
-    const int p = c / 2;
-    if (p < half) {
-      const float cc = ct[p], ss = st[p], a = v.x;
-      v.x = a * cc - v.y * ss;
-      v.y = v.y * cc + a * ss;
+    const float* wh = normed ? (is_q ? A.P.wq : A.P.wk) + (WHOLE ? (is_q ? u : u - D.H) * D.d16 : 0) : nullptr;
+    if (normed) {
+      const float4 w = *reinterpret_cast<const float4*>(wh + c);
+      v = make_float4(v.x * rstd * w.x, v.y * rstd * w.y, v.z * rstd * w.z, v.w * rstd * w.w);
     }
-    if (p + 1 < half) {
-      const float cc = ct[p + 1], ss = st[p + 1], a = v.z;
-      v.z = a * cc - v.w * ss;
-      v.w = v.w * cc + a * ss;
+    const int p = c / 2;
+    if (A.P.halves) {
+      float e[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int i = 0; i < 4; i++) {
+        const int d = c + i;
+        if (d < D.rot) {
+          const bool low = d < half;
+          const int o = low ? d + half : d - half;
+          const float other = normed ? sums[o] * rstd * wh[o] : sums[o], cc = ct[low ? d : o], ss = st[low ? d : o];
+          e[i] = low ? e[i] * cc - other * ss : e[i] * cc + other * ss;
+        }
+      }
+      v = make_float4(e[0], e[1], e[2], e[3]);
+    } else {
+      if (p < half) {
+        const float cc = ct[p], ss = st[p], a = v.x;
+        v.x = a * cc - v.y * ss;
+        v.y = v.y * cc + a * ss;
+      }
+      if (p + 1 < half) {
+        const float cc = ct[p + 1], ss = st[p + 1], a = v.z;
+        v.z = a * cc - v.w * ss;
+        v.w = v.w * cc + a * ss;
+      }
     }
     if (is_q) put_bf16x4(q + ((size_t)b * D.H + u) * D.d16 + c, v);
     else if (dst) put_bf16x4(dst + (u - D.H) * D.d16 + c, v);
@@ -307,15 +379,18 @@ __global__ void __launch_bounds__(DP_WARPS * 32) gqa_decode_prep_kernel(DecPrepA
         v[i] = plane_sum4(src + (size_t)u * D.d16 + c, A.splits, A.pstride);
         ss += v[i].x * v[i].x + v[i].y * v[i].y + v[i].z * v[i].z + v[i].w * v[i].w;
         if constexpr (WHOLE) *reinterpret_cast<float4*>(held + local * D.d16 + c) = v[i];
+        else if (A.P.halves) *reinterpret_cast<float4*>(held + warp * D.d16 + c) = v[i];
       }
     }
     if constexpr (WHOLE) {
       if (u < D.H) ssq += ss; else ssk += ss;
     } else {
       const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)D.d + A.P.eps);
+      __syncwarp();
 #pragma unroll
       for (int i = 0; i < DP_MAXC; i++)
-        if (lane * 4 + i * 128 < D.d16) finish(u, lane * 4 + i * 128, v[i], rstd);
+        if (lane * 4 + i * 128 < D.d16) finish(u, lane * 4 + i * 128, v[i], rstd, held + warp * D.d16);
+      __syncwarp();
     }
   }
   if constexpr (WHOLE) {
@@ -365,7 +440,7 @@ __global__ void __launch_bounds__(DP_WARPS * 32) gqa_decode_prep_kernel(DecPrepA
     const float rq = 1.f / sqrtf(tq / (float)(D.H * D.d) + A.P.eps), rk = 1.f / sqrtf(tk / (float)(D.G * D.d) + A.P.eps);
     local = warp;
     for (int v = u0; v < heads; v += stride, local += DP_WARPS)
-      for (int c = lane * 4; c < D.d16; c += 128) finish(v, c, *reinterpret_cast<const float4*>(held + local * D.d16 + c), v < D.H ? rq : rk);
+      for (int c = lane * 4; c < D.d16; c += 128) finish(v, c, *reinterpret_cast<const float4*>(held + local * D.d16 + c), v < D.H ? rq : rk, held + local * D.d16);
     cluster.sync();                                  // nobody leaves while a partner may still read its shared memory
   }
 }
@@ -413,8 +488,9 @@ __global__ void __launch_bounds__(256) gqa_decode_kernel(const __nv_bfloat16* __
   const int R = D.H / D.G, h0 = g * R + tile * GD_HT, nh = min(GD_HT, R - tile * GD_HT);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, t2 = (lane & 3) * 2;
   const int len = seq_lens[b], first = M.window < len ? len - M.window : 0;
-  const int per = ((len - first + nsplit - 1) / nsplit + 15) & ~15;
-  const int t0 = first + split * per, t1 = min(len, t0 + per);
+  const int kept = min(M.keep, first), gap = first - kept, total = len - gap;        // visible rows in order: 0..kept, first..len
+  const int per = ((total + nsplit - 1) / nsplit + 15) & ~15;
+  const int t0 = split * per, t1 = min(total, t0 + per);
   const int nchunks = t1 > t0 ? (t1 - t0 + GD_CHUNK - 1) / GD_CHUNK : 0;
   const int wrow = D.v16 + 4;
   float* base = ws + ((size_t)b * gridDim.y + blockIdx.y) * nsplit * GD_HT * wrow;
@@ -428,7 +504,7 @@ __global__ void __launch_bounds__(256) gqa_decode_kernel(const __nv_bfloat16* __
     const int c0 = t0 + c * GD_CHUNK, cnt = min(GD_CHUNK, t1 - c0);
     const uint32_t dst = sK + stage * GD_CHUNK * pitch;
     for (int r = warp; r < cnt; r += 8) {
-      const int t = c0 + r;
+      const int t = c0 + r < kept ? c0 + r : c0 + r + gap;
       const __nv_bfloat16* src = cache + ((size_t)__ldg(bt + t / KV_BLOCK) * KV_BLOCK + t % KV_BLOCK) * D.row;
       for (int i = lane; i < vecs; i += 32)
         cp_async16(dst + r * pitch + i * 16, i < kvecs ? src + g * D.d16 + i * 8 : src + D.G * D.d16 + g * D.v16 + (i - kvecs) * 8);
@@ -676,14 +752,15 @@ gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   // the groups of a tile next to one another: tiles come longest first, so the CTAs do too
   const int4 tl = tiles[blockIdx.x / A.D.G];        // first query row, tokens, position of the first token, sequence
-  const int g = blockIdx.x % A.D.G, tok = A.tok, window = A.M.window;
-  // key blocks [j0, j0 + nblk[t]) of every sub-tile; the start is the window of the tile's first token
-  const int j0 = (tl.z - window >= 0 ? tl.z - window + 1 : 0) / GF_BN;
+  const int g = blockIdx.x % A.D.G, tok = A.tok, window = A.M.window, keep = A.M.keep;
+  // every sub-tile goes over the jk blocks of the kept first keys, then over those from j0 on, where the window of the tile's first token starts
+  const int j0 = (tl.z - window >= 0 ? tl.z - window + 1 : 0) / GF_BN, jk = min((keep + GF_BN - 1) / GF_BN, j0);
+  auto block_at = [&](int j) { return j < jk ? j : j - jk + j0; };
   int nblk[NT], nmax = 0;
 #pragma unroll
   for (int t = 0; t < NT; t++) {
     const int n = min(tok, tl.y - t * tok);
-    nblk[t] = n > 0 ? (tl.z + t * tok + n + GF_BN - 1) / GF_BN - j0 : 0;
+    nblk[t] = n > 0 ? (tl.z + t * tok + n + GF_BN - 1) / GF_BN - j0 + jk : 0;
     nmax = max(nmax, nblk[t]);
   }
   if (threadIdx.x == 0) {
@@ -713,7 +790,7 @@ gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
     const int* bt = block_table + (size_t)tl.w * A.max_blocks;
     const int pg = lane & 3, cb = lane >> 2;        // this lane's page of a key block, and its first column block
     auto page_row = [&](int j) -> int {             // first row of that page in the cache, out of bounds past the sequence's pages
-      const int p = (j0 + j) * 4 + pg;
+      const int p = block_at(j) * 4 + pg;
       const int blk = p < A.max_blocks ? __ldg(bt + p) : -1;
       return blk * KV_BLOCK;                        // -1: a negative coordinate, read as zeros
     };
@@ -813,11 +890,11 @@ gqa_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant_
       tmem_ld_32x32b_x32(tS + lane_off + t * 2 * GF_BN + (j & 1) * GF_BN, sv);
       tmem_ld_32x32b_x32(tS + lane_off + t * 2 * GF_BN + (j & 1) * GF_BN + 32, sv + 32);
       tmem_ld_wait();
-      const int kv0 = (j0 + j) * GF_BN;
-      if (kv0 + GF_BN - 1 > lo_pos || kv0 <= hi_pos - window) {   // the diagonal or the window's edge can cross this block
+      const int kv0 = block_at(j) * GF_BN;
+      if (kv0 + GF_BN - 1 > lo_pos || (kv0 <= hi_pos - window && kv0 + GF_BN > keep)) {   // the diagonal or an edge of the visible keys can cross this block
 #pragma unroll
         for (int c = 0; c < 64; c++)
-          if (kv0 + c > qpos || kv0 + c <= wlow) sv[c] = __float_as_uint(-INFINITY);
+          if (kv0 + c > qpos || (kv0 + c <= wlow && kv0 + c >= keep)) sv[c] = __float_as_uint(-INFINITY);
       }
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
 #pragma unroll
@@ -924,8 +1001,8 @@ bool make_dims(GqaDims& D, int H, int G, int d, int dv, int rot) {
   D.row = G * (D.d16 + D.v16);
   return true;
 }
-MaskGate make_mask(float scale, int window, const float* sink, const void* gate, int64_t ldg, int kind, float out_scale) {
-  return MaskGate{scale, window > 0 ? window : 0x3fffffff, sink, gate, ldg, kind, out_scale};
+MaskGate make_mask(float scale, int window, int keep, const float* sink, const void* gate, int64_t ldg, int kind, float out_scale) {
+  return MaskGate{scale, window > 0 ? window : 0x3fffffff, keep, sink, gate, ldg, kind, out_scale};
 }
 
 template <int NT, int NQ, int NV>
@@ -959,16 +1036,20 @@ int launch_decode(dim3 grid, int smem, cudaStream_t st, const void* q, const voi
 }  // namespace
 
 // Projection rows qkv [rows][ld] (bf16, or f32 with is_f32): H query heads, G key heads (d padded to d16 = a multiple of 16 columns each), G value heads (dv
-// padded to v16). Norms queries and keys (RMS over each head, or with whole != 0 over all query and all key heads; wq, wk f32 in the same padding, one head long or
-// all heads long), turns the first `rot` dimensions of each (pairs of neighbouring columns, tables cos / sin f32 [position][rot / 2]), leaves the queries in
-// place and writes keys and values to cache row slots[r] (= page * 16 + offset): [G x d16 | G x v16]. With lambda (one f32 on the device) the values become
+// padded to v16). Norms queries and keys (norm 0: RMS over each head, 1: over all query and all key heads; wq, wk f32 in the same padding, one head long or
+// all heads long; 2: no norm), turns the first `rot` dimensions of each (pairs of neighbouring columns, or with halves != 0 column i with i + rot / 2; tables cos / sin f32
+// [position][rot / 2]), leaves the queries in place and writes keys and values to cache row slots[r] (= page * 16 + offset): [G x d16 | G x v16]. With lambda (one f32 on the device) the values become
 // (1 - lambda) v + lambda vfirst (rows of G * v16, pitch ldf).
-FT_EXPORT int ft_gqa_prep(void* qkv, int64_t ld, int rows, int H, int G, int d, int dv, int rot, int whole, const float* wq, const float* wk, float eps, const int* positions,
-                          const float* cos_t, const float* sin_t, const int* slots, void* cache, const void* vfirst, int64_t ldf, const float* lambda, int is_f32,
+FT_EXPORT int ft_gqa_prep(void* qkv, int64_t ld, int rows, int H, int G, int d, int dv, int rot, int norm, int halves, const float* wq, const float* wk, float eps,
+                          const int* positions, const float* cos_t, const float* sin_t, const int* slots, void* cache, const void* vfirst, int64_t ldf, const float* lambda, int is_f32,
                           cudaStream_t st) {
   PrepArgs A{};
-  if (rows < 1 || !make_dims(A.D, H, G, d, dv, rot) || (ld & 7) || ld < (int64_t)(H + G) * A.D.d16 + G * A.D.v16 || (lambda && (!vfirst || (ldf & 7)))) return FT_ERR_ARG;
-  A.wq = wq; A.wk = wk; A.eps = eps; A.positions = positions; A.cos_t = cos_t; A.sin_t = sin_t; A.slots = slots;
+  if (rows < 1 || !make_dims(A.D, H, G, d, dv, rot) || (ld & 7) || ld < (int64_t)(H + G) * A.D.d16 + G * A.D.v16 || (lambda && (!vfirst || (ldf & 7))) ||
+      norm < NORM_HEAD || norm > NORM_NONE || (norm != NORM_NONE && !(wq && wk)))
+    return FT_ERR_ARG;
+  const bool whole = norm == NORM_WHOLE;
+  A.halves = halves;
+  A.wq = norm == NORM_NONE ? nullptr : wq; A.wk = wk; A.eps = eps; A.positions = positions; A.cos_t = cos_t; A.sin_t = sin_t; A.slots = slots;
 #define FT_GP(T, W) gqa_prep_kernel<T, W><<<rows, PREP_T, 0, st>>>((T*)qkv, ld, A, (T*)cache, (const T*)vfirst, ldf, lambda)
   if (is_f32) { if (whole) FT_GP(float, true); else FT_GP(float, false); }
   else { if (whole) FT_GP(__nv_bfloat16, true); else FT_GP(__nv_bfloat16, false); }
@@ -977,15 +1058,15 @@ FT_EXPORT int ft_gqa_prep(void* qkv, int64_t ld, int rows, int H, int G, int d, 
 }
 
 // Plain attention over cached rows: q [rows][ldq] as left by ft_gqa_prep; row r of sequence seq_of[r] sees the last `window` (0: all) of the positions
-// 0..positions[r]; sink f32 [H] or null; gate_kind 0: none, 1: rows of H * v16 pre-activations in the data type (pitch ldg), 2: f32 rows of H; out [rows][ldo], heads of
+// 0..positions[r] and the first `keep` of them; sink f32 [H] or null; gate_kind 0: none, 1: rows of H * v16 pre-activations in the data type (pitch ldg), 2: f32 rows of H; out [rows][ldo], heads of
 // v16, times out_scale. Value sizes up to 1024.
 FT_EXPORT int ft_gqa_rows(const void* q, int64_t ldq, const void* cache, const int* block_table, int max_blocks, const int* seq_of, const int* positions, int rows, int H, int G,
-                          int d, int dv, float scale, int window, const float* sink, const void* gate, int64_t ldg, int gate_kind, float out_scale, void* out, int64_t ldo,
-                          int is_f32, cudaStream_t st) {
+                          int d, int dv, float scale, int window, int keep, const float* sink, const void* gate, int64_t ldg, int gate_kind, float out_scale, void* out,
+                          int64_t ldo, int is_f32, cudaStream_t st) {
   GqaDims D;
-  if (rows < 1 || !make_dims(D, H, G, d, dv, 0) || (gate_kind && !gate)) return FT_ERR_ARG;
+  if (rows < 1 || keep < 0 || !make_dims(D, H, G, d, dv, 0) || (gate_kind && !gate)) return FT_ERR_ARG;
   if (D.v16 > 128 * ROWS_MAX_COLS || D.d16 > 8192) return FT_ERR_TOO_LARGE;
-  const MaskGate M = make_mask(scale, window, sink, gate, ldg, gate_kind, out_scale);
+  const MaskGate M = make_mask(scale, window, keep, sink, gate, ldg, gate_kind, out_scale);
   const dim3 grid(rows, H);
   if (is_f32) gqa_rows_kernel<float><<<grid, 128, D.d16 * 4, st>>>((const float*)q, ldq, (const float*)cache, block_table, max_blocks, seq_of, positions, D, M, (float*)out, ldo);
   else gqa_rows_kernel<__nv_bfloat16><<<grid, 128, D.d16 * 4, st>>>((const __nv_bfloat16*)q, ldq, (const __nv_bfloat16*)cache, block_table, max_blocks, seq_of, positions, D, M,
@@ -996,23 +1077,24 @@ FT_EXPORT int ft_gqa_rows(const void* q, int64_t ldq, const void* cache, const i
 // ft_gqa_prep for one token of B <= 16 sequences, from split-K planes of the projection (columns as there; gate pre-activations from column gate_col on, kind as in
 // ft_gqa_rows): queries q bf16 [B][H][d16], cache row of each sequence's current position, sigmoid of the gate (f32 [B][H * v16] or [B][H]). vf_out (f32
 // [B][G * v16]) keeps the values; vf_in and lambda mix such values in. Head sizes up to 512.
-FT_EXPORT int ft_gqa_decode_prep(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int B, int H, int G, int d, int dv, int rot, int whole, const float* wq,
-                                 const float* wk, float eps, const int* positions, const float* cos_t, const float* sin_t, const int* block_table, int max_blocks,
+FT_EXPORT int ft_gqa_decode_prep(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int B, int H, int G, int d, int dv, int rot, int norm, int halves,
+                                 const float* wq, const float* wk, float eps, const int* positions, const float* cos_t, const float* sin_t, const int* block_table, int max_blocks,
                                  int gate_col, int gate_kind, float* gate, float* vf_out, const float* vf_in, const float* lambda, void* q, void* cache, cudaStream_t st) {
   DecPrepArgs A{};
   GqaDims& D = A.P.D;
   if (B < 1 || B > DEC_TOK || splits < 1 || !make_dims(D, H, G, d, dv, rot) || (ldp & 3) || (plane_stride & 3) || (gate_col & 3) || (gate_kind && !gate) ||
-      (lambda && !vf_in))
+      (lambda && !vf_in) || norm < NORM_HEAD || norm > NORM_NONE || (norm != NORM_NONE && !(wq && wk)))
     return FT_ERR_ARG;
   if (D.d16 > 128 * DP_MAXC) return FT_ERR_TOO_LARGE;
-  A.P.wq = wq; A.P.wk = wk; A.P.eps = eps; A.P.positions = positions; A.P.cos_t = cos_t; A.P.sin_t = sin_t;
+  A.P.halves = halves;
+  A.P.wq = norm == NORM_NONE ? nullptr : wq; A.P.wk = wk; A.P.eps = eps; A.P.positions = positions; A.P.cos_t = cos_t; A.P.sin_t = sin_t;
   A.planes = planes; A.splits = splits; A.ldp = ldp; A.pstride = (size_t)plane_stride; A.block_table = block_table; A.max_blocks = max_blocks;
   A.gate_col = gate_col; A.gate_kind = gate_kind; A.gate = gate; A.vf_out = vf_out; A.vf_in = vf_in; A.lambda = lambda;
   const int gate_cols = gate_kind == GATE_ELEMENT ? H * D.v16 : gate_kind == GATE_HEAD ? H : 0;
   const int units = H + 2 * G + (gate_cols + 127) / 128;
   int ctas = (units + DP_WARPS - 1) / DP_WARPS;
-  if (!whole)
-    return (int)ft_launch_pdl(gqa_decode_prep_kernel<false>, dim3(ctas, B), dim3(DP_WARPS * 32), 0, st, A, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
+  if (norm != NORM_WHOLE)
+    return (int)ft_launch_pdl(gqa_decode_prep_kernel<false>, dim3(ctas, B), dim3(DP_WARPS * 32), halves ? (size_t)DP_WARPS * D.d16 * 4 : 0, st, A, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
   int cl = 1;
   while (cl < 8 && cl < ctas) cl *= 2;
   ctas = cl;
@@ -1035,15 +1117,15 @@ FT_EXPORT int ft_gqa_decode_prep(const float* planes, int splits, int64_t ldp, i
   return (int)cudaLaunchKernelEx(&cfg, gqa_decode_prep_kernel<true>, A, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
 }
 
-// Attention of one token per sequence over its visible cached rows (seq_lens[b] rows, the newest included, or the last `window` of them); q and gate as written by
+// Attention of one token per sequence over its visible cached rows (seq_lens[b] rows, the newest included, or the last `window` and the first `keep` of them); q and gate as written by
 // ft_gqa_decode_prep. ws: f32 [B][G * ceil(H / G / 16)][nsplit][16][v16 + 4], 16-byte aligned; counters: int [B][G * ceil(H / G / 16)], zero before the first
 // launch (the kernel leaves them zero). nsplit <= 64; value sizes up to 512. out: bf16 [B][ldo], heads of v16.
 FT_EXPORT int ft_gqa_decode(const void* q, const void* cache, const int* block_table, int max_blocks, const int* seq_lens, int B, int H, int G, int d, int dv, float scale,
-                            int window, const float* sink, const float* gate, int gate_kind, float out_scale, int nsplit, float* ws, int* counters, void* out, int64_t ldo,
-                            cudaStream_t st) {
+                            int window, int keep, const float* sink, const float* gate, int gate_kind, float out_scale, int nsplit, float* ws, int* counters, void* out,
+                            int64_t ldo, cudaStream_t st) {
   GqaDims D;
-  if (B < 1 || nsplit < 1 || nsplit > GD_MAX_SPLIT || !make_dims(D, H, G, d, dv, 0) || (reinterpret_cast<uintptr_t>(ws) & 15) || (ldo & 3) || (gate_kind && !gate)) return FT_ERR_ARG;
-  const MaskGate M = make_mask(scale, window, sink, gate, 0, gate_kind, out_scale);
+  if (B < 1 || keep < 0 || nsplit < 1 || nsplit > GD_MAX_SPLIT || !make_dims(D, H, G, d, dv, 0) || (reinterpret_cast<uintptr_t>(ws) & 15) || (ldo & 3) || (gate_kind && !gate)) return FT_ERR_ARG;
+  const MaskGate M = make_mask(scale, window, keep, sink, gate, 0, gate_kind, out_scale);
   const int smem = gd_smem(D.d16, D.v16), np = (D.v16 / 16 + 7) / 8, tiles = (H / G + GD_HT - 1) / GD_HT;
   if (smem > SMEM_MAX - 8192 || np > 4) return FT_ERR_TOO_LARGE;
   const dim3 grid(nsplit, G * tiles, B);
@@ -1076,18 +1158,18 @@ FT_EXPORT int ft_gqa_flash_subtiles(int H, int G, int d, int dv) {
 // of the new tokens included). tiles: int4 per tile {first query row, tokens (<= subtiles * (128 / (H / G))), position of the first token, row of block_table}.
 // Mask, sink, gate and output as in ft_gqa_rows. Leading dimensions are multiples of 8.
 FT_EXPORT int ft_gqa_flash(const void* q, int64_t ldq, int q_rows, const void* cache, int pages, const int* block_table, int max_blocks, const int* tiles, int ntiles, int H,
-                           int G, int d, int dv, float scale, int window, const float* sink, const void* gate, int64_t ldg, int gate_kind, float out_scale, void* out,
-                           int64_t ldo, cudaStream_t st) {
+                           int G, int d, int dv, float scale, int window, int keep, const float* sink, const void* gate, int64_t ldg, int gate_kind, float out_scale,
+                           void* out, int64_t ldo, cudaStream_t st) {
   FlashArgs A{};
   GqaDims& D = A.D;
-  if (q_rows < 1 || pages < 1 || ntiles < 1 || !make_dims(D, H, G, d, dv, 0) || (ldq & 7) || (ldo & 7) || (gate_kind && !gate) || (gate_kind == GATE_ELEMENT && (ldg & 7)))
+  if (q_rows < 1 || pages < 1 || ntiles < 1 || keep < 0 || !make_dims(D, H, G, d, dv, 0) || (ldq & 7) || (ldo & 7) || (gate_kind && !gate) || (gate_kind == GATE_ELEMENT && (ldg & 7)))
     return FT_ERR_ARG;
   const int nt = ft_gqa_flash_subtiles(H, G, d, dv);
   if (nt == 0) return FT_ERR_TOO_LARGE;
   int dev = 0;
   FT_CUDA_TRY(cudaGetDevice(&dev));
   FT_CUDA_TRY(ft_bind_context(dev));
-  A.M = make_mask(scale, window, sink, gate, ldg, gate_kind, out_scale);
+  A.M = make_mask(scale, window, keep, sink, gate, ldg, gate_kind, out_scale);
   A.R = H / G;
   A.tok = GF_BM / A.R;
   A.nq = (d + 63) / 64;

@@ -1,6 +1,7 @@
 // Latent attention: keys and values are linear images of one small vector per token (the latent c, RMS-normalised) plus one rotated key part shared by
 // all heads, so a token's cache row is [c | k_rot] whatever the number of heads. Rows are padded: c to a multiple of 16 elements (`r16`), k_rot to a
-// multiple of 16 (`row` = r16 + padded rot), zeros in the padding. Pages hold 16 rows.
+// multiple of 16 (`row` = r16 + padded rot), zeros in the padding. Pages hold 16 rows. The rotated part may be absent (rot = 0), queries may come through a
+// normalised latent of their own, and a layer may read the latent that an earlier layer cached.
 //
 //   score(q, j) = scale (q_plain . W_uk c_j + q_rot . k_rot_j) = scale (W_uk^T q_plain | q_rot) . (c_j | k_rot_j)
 //   out         = W_uv sum_j p_j c_j
@@ -8,6 +9,7 @@
 //   ft_latent_prep          projection rows of a prompt -> rotated queries (in place), normalised latent and rotated key -> cache page (+ dense row)
 //   ft_latent_ctx_gather    cached rows of earlier portions -> dense rows
 //   ft_latent_flash         prompts: per-head keys / values expanded from the latent by a GEMM; tcgen05 flash attention over ragged sequences
+//   ft_latent_decode_norms  split-K planes of a query latent and a latent -> both normalised, one for the query expansion, one into the cache page
 //   ft_latent_decode_prep   split-K planes of one token per sequence -> absorbed queries W_uk^T q_plain, rotations, norm, cache write (one launch)
 //   ft_latent_decode        one query token per sequence over the cached rows, all heads of a tile share every loaded row (mma.sync), split over the
 //                           sequence; ft_latent_combine merges the splits
@@ -32,9 +34,11 @@ FT_DEVICE float ex2(float x) {
   return y;
 }
 
-// Column layout of a projection row: heads of [plain padded to d8 | rot padded to dr8], then the latent (rank padded to rank8), then the shared rot part.
+// Column layout of a projection row: heads of [plain padded to d8 | rot padded to dr8] (or, with q_rank, the query latent padded to a multiple of 8), then the latent
+// (rank padded to rank8), then the shared rot part.
 struct LatentDims {
   int H, d, dr, rank;
+  int q_rank, q_cols;
   int d8, dr8, rank8, r16, row;      // padded sizes; row = cache row length
 };
 
@@ -51,20 +55,34 @@ template <> FT_DEVICE void store2<__nv_bfloat16>(__nv_bfloat16* p, float a, floa
 template <typename T>
 __global__ void __launch_bounds__(128) latent_prep_kernel(T* __restrict__ qkv, int64_t ld, LatentDims D, const float* __restrict__ w, float eps,
                                                           const int* __restrict__ positions, const float* __restrict__ cos_t, const float* __restrict__ sin_t,
-                                                          const int* __restrict__ slots, const int* __restrict__ ctx_rows, T* __restrict__ cache, T* __restrict__ ctx) {
+                                                          const int* __restrict__ slots, const int* __restrict__ ctx_rows, T* __restrict__ cache, T* __restrict__ ctx,
+                                                          const float* __restrict__ wq) {
   __shared__ float red[32];
   const int r = blockIdx.x, half = D.dr / 2, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int pos = positions[r];
   T* row = qkv + (size_t)r * ld;
   const float* ct = cos_t + (size_t)pos * half;
   const float* st = sin_t + (size_t)pos * half;
-  const T* lat = row + D.H * (D.d8 + D.dr8);
+  const T* lat = row + D.q_cols;
   float ss = 0.f;
+  if (D.q_rank) {                                    // the query latent, in place
+    for (int i = threadIdx.x * 2; i < D.q_rank; i += 256) {
+      const float2 v = load2(row + i);
+      ss += v.x * v.x + (i + 1 < D.q_rank ? v.y * v.y : 0.f);
+    }
+    const float rq = 1.f / sqrtf(block_sum(ss, red) / (float)D.q_rank + eps);
+    for (int i = threadIdx.x * 2; i < D.q_rank; i += 256) {
+      const float2 v = load2(row + i);
+      store2(row + i, v.x * rq * wq[i], i + 1 < D.q_rank ? v.y * rq * wq[i + 1] : 0.f);
+    }
+    if (cache == nullptr) return;                    // keys and values from an earlier layer's latent
+    ss = 0.f;
+  }
   for (int i = threadIdx.x * 2; i < D.rank; i += 256) {
     const float2 v = load2(lat + i);
     ss += v.x * v.x + (i + 1 < D.rank ? v.y * v.y : 0.f);
   }
-  for (int p = lane; p < half; p += 32) {
+  for (int p = lane; p < half && !D.q_rank; p += 32) {
     const float c = ct[p], s = st[p];
 #pragma unroll 4
     for (int hd = warp; hd < D.H; hd += 4) {
@@ -268,6 +286,37 @@ __global__ void __launch_bounds__(PREP_THREADS) latent_decode_prep_kernel(const 
     }
     *reinterpret_cast<__nv_bfloat162*>(dst + D.r16 + 2 * p) = __floats2bfloat162_rn(a, bb);
   }
+}
+
+// grid (B, 1 or 2): y = 0 the query latent of a token, y = 1 its cached latent
+__global__ void __launch_bounds__(PREP_THREADS) latent_decode_norms_kernel(const float* __restrict__ planes, int splits, int64_t ldp, size_t pstride, LatentDims D,
+                                                                           const float* __restrict__ wq, const float* __restrict__ w, float eps,
+                                                                           const int* __restrict__ positions, const int* __restrict__ block_table, int max_blocks,
+                                                                           __nv_bfloat16* __restrict__ cq, int64_t ldq, __nv_bfloat16* __restrict__ cache) {
+  pdl_wait();
+  pdl_launch_dependents();
+  extern __shared__ __align__(16) uint8_t prep_smem[];
+  __shared__ float red[32];
+  float* v = reinterpret_cast<float*>(prep_smem);
+  const int b = blockIdx.x;
+  const bool is_q = blockIdx.y == 0;
+  const int n = is_q ? D.q_rank : D.rank;
+  const size_t base = (size_t)b * ldp + (is_q ? 0 : D.q_cols);
+  float ss = 0.f;
+  for (int i = threadIdx.x; i < n; i += PREP_THREADS) {
+    const float x = plane_sum(planes, splits, pstride, base + i);
+    v[i] = x;
+    ss += x * x;
+  }
+  const float rstd = 1.f / sqrtf(block_sum(ss, red) / (float)n + eps);
+  if (is_q) {
+    for (int i = threadIdx.x; i < n; i += PREP_THREADS) cq[(size_t)b * ldq + i] = __float2bfloat16(v[i] * rstd * wq[i]);
+    return;
+  }
+  const int pos = positions[b], blk = block_table[(size_t)b * max_blocks + pos / KV_BLOCK];
+  if (blk < 0) return;
+  __nv_bfloat16* dst = cache + ((size_t)blk * KV_BLOCK + pos % KV_BLOCK) * D.row;
+  for (int i = threadIdx.x; i < D.r16; i += PREP_THREADS) dst[i] = __float2bfloat16(i < n ? v[i] * rstd * w[i] : 0.f);
 }
 
 // ------------------------------------------------------------------------------------------------------------
@@ -808,7 +857,7 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
   }
 }
 
-LatentDims make_dims(int H, int d, int dr, int rank) {
+LatentDims make_dims(int H, int d, int dr, int rank, int q_rank = 0) {
   LatentDims D;
   D.H = H; D.d = d; D.dr = dr; D.rank = rank;
   D.d8 = (d + 7) & ~7;
@@ -816,9 +865,11 @@ LatentDims make_dims(int H, int d, int dr, int rank) {
   D.rank8 = (rank + 7) & ~7;
   D.r16 = (rank + 15) & ~15;
   D.row = D.r16 + ((dr + 15) & ~15);
+  D.q_rank = q_rank;
+  D.q_cols = q_rank ? (q_rank + 7) & ~7 : H * (D.d8 + D.dr8);
   return D;
 }
-bool dims_ok(int H, int d, int dr, int rank) { return H >= 1 && d >= 1 && dr >= 2 && (dr & 1) == 0 && rank >= 1; }
+bool dims_ok(int H, int d, int dr, int rank) { return H >= 1 && d >= 1 && dr >= 0 && (dr & 1) == 0 && rank >= 1; }
 int flash_smem(int NT, int nq, int nv) { return NT * nq * LF_QB + 2 * (nq + nv) * LF_KB + NT * LF_PB + 256 + 1024; }
 constexpr int SMEM_MAX = 232448;
 
@@ -851,15 +902,16 @@ int launch_decode(dim3 grid, int smem, cudaStream_t st, const void* q, const voi
 // Projection rows qkv [rows][ld] (bf16, or f32 with is_f32): heads of [plain | rot] (each padded to 8 columns), latent (padded to 8), shared rot part.
 // Rotates the queries' rot parts in place (pairs of neighbouring columns, tables cos/sin f32 [position][dr / 2]), normalises the latent (w f32[rank])
 // and rotates the shared key part into cache row slots[r] (= page * 16 + offset) and, when ctx is given, dense row ctx_rows[r]. Cache rows have
-// 16-padded latent + 16-padded rot elements.
-FT_EXPORT int ft_latent_prep(void* qkv, int64_t ld, int rows, int H, int d, int dr, int rank, const float* w, float eps, const int* positions, const float* cos_t,
-                             const float* sin_t, const int* slots, const int* ctx_rows, void* cache, void* ctx, int is_f32, cudaStream_t st) {
-  if (rows < 1 || !dims_ok(H, d, dr, rank) || (ctx && !ctx_rows)) return FT_ERR_ARG;
-  const LatentDims D = make_dims(H, d, dr, rank);
-  if (ld < (int64_t)H * (D.d8 + D.dr8) + D.rank8 + dr || (ld & 7)) return FT_ERR_ARG;
-  if (is_f32) latent_prep_kernel<float><<<rows, 128, 0, st>>>((float*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (float*)cache, (float*)ctx);
+// 16-padded latent + 16-padded rot elements. q_rank > 0 (with dr = 0): the heads' columns hold the query latent instead (padded to 8), which is normalised in place
+// with wq (f32[q_rank]); cache may then be null, for rows without a latent of their own.
+FT_EXPORT int ft_latent_prep(void* qkv, int64_t ld, int rows, int H, int d, int dr, int rank, int q_rank, const float* wq, const float* w, float eps, const int* positions,
+                             const float* cos_t, const float* sin_t, const int* slots, const int* ctx_rows, void* cache, void* ctx, int is_f32, cudaStream_t st) {
+  if (rows < 1 || !dims_ok(H, d, dr, rank) || q_rank < 0 || (ctx && !ctx_rows) || (q_rank ? dr != 0 || !wq : !cache)) return FT_ERR_ARG;
+  const LatentDims D = make_dims(H, d, dr, rank, q_rank);
+  if (ld < (int64_t)D.q_cols + (cache ? D.rank8 + dr : 0) || (ld & 7)) return FT_ERR_ARG;
+  if (is_f32) latent_prep_kernel<float><<<rows, 128, 0, st>>>((float*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (float*)cache, (float*)ctx, wq);
   else latent_prep_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>((__nv_bfloat16*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (__nv_bfloat16*)cache,
-                                                               (__nv_bfloat16*)ctx);
+                                                               (__nv_bfloat16*)ctx, wq);
   return (int)cudaGetLastError();
 }
 
@@ -884,8 +936,19 @@ FT_EXPORT int ft_latent_rows(const void* q, const void* cache, const int* block_
   return (int)cudaGetLastError();
 }
 
+// Decode step of B <= 16 sequences whose queries come through a latent, from split-K planes [query latent padded to 8 | latent padded to 8]: the normalised query
+// latent (bf16 [B][ldq]) and, unless cache is null, the cache row of every sequence's current position. Latents of up to 12288.
+FT_EXPORT int ft_latent_decode_norms(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int B, int q_rank, int rank, const float* wq, const float* w, float eps,
+                                     const int* positions, const int* block_table, int max_blocks, void* cq, int64_t ldq, void* cache, cudaStream_t st) {
+  if (B < 1 || B > DEC_TOK || splits < 1 || q_rank < 1 || rank < 1 || ldq < q_rank) return FT_ERR_ARG;
+  const size_t smem = sizeof(float) * (size_t)(q_rank > rank ? q_rank : rank);
+  if (smem > 48 * 1024) return FT_ERR_TOO_LARGE;
+  return (int)ft_launch_pdl(latent_decode_norms_kernel, dim3(B, cache ? 2 : 1), dim3(PREP_THREADS), smem, st, planes, splits, ldp, (size_t)plane_stride,
+                            make_dims(1, 1, 0, rank, q_rank), wq, w, eps, positions, block_table, max_blocks, (__nv_bfloat16*)cq, ldq, (__nv_bfloat16*)cache);
+}
+
 // Decode step of B <= 16 sequences, from the split-K planes of the fused query / latent projection (column layout as in ft_latent_prep): absorbed and
-// rotated queries q [B][H][row] bf16, cache row of every sequence's current position. wuk: bf16 [H * d8][ldw], ldw >= rank padded to 16, zeros past rank.
+// rotated queries q [B][H][row] bf16, cache row of every sequence's current position (cache null: the planes hold queries alone). wuk: bf16 [H * d8][ldw], ldw >= rank padded to 16, zeros past rank.
 FT_EXPORT int ft_latent_decode_prep(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int B, int H, int d, int dr, int rank, const void* wuk,
                                     int64_t ldw, const float* w, float eps, const int* positions, const float* cos_t, const float* sin_t, const int* block_table,
                                     int max_blocks, void* q, void* cache, cudaStream_t st) {
@@ -896,7 +959,7 @@ FT_EXPORT int ft_latent_decode_prep(const float* planes, int splits, int64_t ldp
   const size_t absorb = (size_t)d * (ABS_COLS * 2 + DEC_TOK * 4), norm = sizeof(float) * (size_t)rank;
   const size_t smem = absorb > norm ? absorb : norm;
   if (smem > 48 * 1024) return FT_ERR_TOO_LARGE;
-  return (int)ft_launch_pdl(latent_decode_prep_kernel, dim3(H * slices + B), dim3(PREP_THREADS), smem, st, planes, splits, ldp, (size_t)plane_stride, D, B,
+  return (int)ft_launch_pdl(latent_decode_prep_kernel, dim3(H * slices + (cache ? B : 0)), dim3(PREP_THREADS), smem, st, planes, splits, ldp, (size_t)plane_stride, D, B,
                             (const __nv_bfloat16*)wuk, ldw, w, eps, positions, cos_t, sin_t, block_table, max_blocks, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
 }
 
@@ -934,7 +997,7 @@ FT_EXPORT int ft_latent_combine(const float* ws, int B, int H, int rank, int nsp
 // Query rows of one tile of ft_latent_flash for these head sizes: 256 or 128; 0 when the sizes do not fit the kernel (use ft_latent_rows).
 FT_EXPORT int ft_latent_flash_tile(int d, int dr, int dv) {
   const int nq = (d + 63) / 64 + (dr + 63) / 64, nv = (dv + 63) / 64;
-  if (nq == 2 && nv == 1) return 128;                  // two CTAs of one tile per SM
+  if (nq <= 2 && nv == 1) return 128;                  // two CTAs of one tile per SM
   if (nv <= 2 && flash_smem(2, nq, nv) <= SMEM_MAX) return 256;
   if (nv <= 4 && flash_smem(1, nq, nv) <= SMEM_MAX) return 128;
   return 0;
@@ -943,10 +1006,10 @@ FT_EXPORT int ft_latent_flash_tile(int d, int dr, int dv) {
 // Causal attention over ragged sequences. q: [q_rows][ldq] with heads of [d padded to 8 | dr padded to 8]; kv: [ctx_rows][ldkv] with H heads of keys (d
 // padded to 8), then H heads of values (dv padded to 8); kr: rotated key part, [ctx_rows][ldkr]; out: [q_rows][ldo], heads of dv padded to 8. tiles: int4
 // per tile {first query row, rows (<= the tile size), position of the first row, first context row of its sequence}: the row at position p sees context
-// rows 0..p of its sequence. All bf16, leading dimensions multiples of 8.
+// rows 0..p of its sequence. dr may be 0 (kr is not read then). All bf16, leading dimensions multiples of 8.
 FT_EXPORT int ft_latent_flash(const void* q, int64_t ldq, int q_rows, const void* kv, int64_t ldkv, const void* kr, int64_t ldkr, int ctx_rows, const int* tiles, int ntiles,
                               int H, int d, int dr, int dv, float scale, void* out, int64_t ldo, cudaStream_t st) {
-  if (q_rows < 1 || ctx_rows < 1 || ntiles < 1 || H < 1 || H > 65535 || d < 1 || dr < 1 || dv < 1 || (ldq & 7) || (ldkv & 7) || (ldkr & 7) || (ldo & 7)) return FT_ERR_ARG;
+  if (q_rows < 1 || ctx_rows < 1 || ntiles < 1 || H < 1 || H > 65535 || d < 1 || dr < 0 || dv < 1 || (ldq & 7) || (ldkv & 7) || (ldkr & 7) || (ldo & 7)) return FT_ERR_ARG;
   const int tile = ft_latent_flash_tile(d, dr, dv);
   if (tile == 0) return FT_ERR_TOO_LARGE;
   int dev = 0;
@@ -957,11 +1020,12 @@ FT_EXPORT int ft_latent_flash(const void* q, int64_t ldq, int q_rows, const void
   CUtensorMap m[5];
   const __nv_bfloat16 *qp = (const __nv_bfloat16*)q, *kp = (const __nv_bfloat16*)kv;
   int r = ft_make_tmap_3d(&m[0], qp, 2, true, d, H, q_rows, hq, (uint64_t)ldq * 2, 64, 1, LF_BM, CU_TENSOR_MAP_SWIZZLE_128B);
-  if (!r) r = ft_make_tmap_3d(&m[1], qp + d8, 2, true, dr, H, q_rows, hq, (uint64_t)ldq * 2, 64, 1, LF_BM, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!r && dr) r = ft_make_tmap_3d(&m[1], qp + d8, 2, true, dr, H, q_rows, hq, (uint64_t)ldq * 2, 64, 1, LF_BM, CU_TENSOR_MAP_SWIZZLE_128B);
   if (!r) r = ft_make_tmap_3d(&m[2], kp, 2, true, d, H, ctx_rows, (uint64_t)d8 * 2, (uint64_t)ldkv * 2, 64, 1, LF_BN, CU_TENSOR_MAP_SWIZZLE_128B);
-  if (!r) r = ft_make_tmap_2d(&m[3], kr, 2, true, dr, ctx_rows, (uint64_t)ldkr * 2, 64, LF_BN, CU_TENSOR_MAP_SWIZZLE_128B);
+  if (!r && dr) r = ft_make_tmap_2d(&m[3], kr, 2, true, dr, ctx_rows, (uint64_t)ldkr * 2, 64, LF_BN, CU_TENSOR_MAP_SWIZZLE_128B);
   if (!r) r = ft_make_tmap_3d(&m[4], kp + (size_t)H * d8, 2, true, dv, H, ctx_rows, (uint64_t)dv8 * 2, (uint64_t)ldkv * 2, 64, 1, LF_BN, CU_TENSOR_MAP_SWIZZLE_128B);
   if (r) return r;
+  if (!dr) { m[1] = m[0]; m[3] = m[2]; }               // named by the kernel, never read
   const FlashDims F{d, dr, dv, (d + 63) / 64, (dr + 63) / 64, (dv + 63) / 64, dv8};
   const int nq = F.nn + F.nr;
   const int smem = flash_smem(tile / 128, nq, F.nv);
@@ -972,6 +1036,7 @@ FT_EXPORT int ft_latent_flash(const void* q, int64_t ldq, int q_rows, const void
     if (nq == 3 && F.nv == 2) FT_LF(2, 3, 2);
     FT_LF(2, 0, 0);
   }
+  if (nq == 1 && F.nv == 1) FT_LF(1, 1, 1);
   if (nq == 2 && F.nv == 1) FT_LF(1, 2, 1);
   FT_LF(1, 0, 0);
 #undef FT_LF

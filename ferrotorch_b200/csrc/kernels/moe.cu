@@ -1,7 +1,9 @@
-// Mixture of experts: sigmoid router with the top experts per token, experts of the clamped gated form
-//   g = min(W_gate x, limit),  u = clamp(W_up x, -limit, limit),  expert(x) = W_down (g sigmoid(slope g) (u + 1)),
-// every chosen expert applied to score * x. The projections are linear, so W (score x) = score (W x): the score multiplies the f32 accumulators and
-// no scaled copy of the tokens is made (or rounded).
+// Mixture of experts: sigmoid router with the top experts per token, and experts of two forms.
+//   clamped   g = min(W_gate x, limit),  u = clamp(W_up x, -limit, limit),  expert(x) = W_down (g sigmoid(slope g) (u + 1)), applied to score * x: the
+//             projections are linear, so W (score x) = score (W x), and the score multiplies the f32 accumulators: no scaled copy of the tokens is made (or rounded)
+//   silu      expert(x) = score W_down (g sigmoid(g) u): the score multiplies the activation, in f32, ahead of the down projection
+// The router takes the largest logits, or (RouteRule) the largest sums of sigmoid and a per-expert correction, among the experts of the best groups, with weights that
+// are normed to a given sum.
 //
 // Weights: gate and up rows are interleaved in blocks of eight (eight gate rows, then the eight up rows of the same neurons), so that a warp's 16
 // weight rows -- and a thread's accumulators -- hold a neuron's gate and up together, and the tiles of the grouped GEMM hold both as well.
@@ -34,6 +36,11 @@ FT_DEVICE float gated_clamped_fast(float g, float u, float limit, float slope) {
   u = fminf(fmaxf(u, -limit), limit);
   return __fdividef(g * (u + 1.f), 1.f + __expf(-slope * g));
 }
+enum { EXPERT_CLAMPED = 0, EXPERT_SILU = 1 };
+template <bool FAST> FT_DEVICE float expert_act(int kind, float k, float g, float u, float limit, float slope) {
+  if (kind == EXPERT_SILU) return FAST ? k * u * (g / (1.f + __expf(-g))) : k * u * (g * sigmoid_f(g));
+  return FAST ? gated_clamped_fast(k * g, k * u, limit, slope) : gated_clamped(k * g, k * u, limit, slope);
+}
 
 // whole warp: (value, index) of the largest logit that comes after (pv, pi) in the order "value descending, index ascending"
 FT_DEVICE void next_best(const float* z, int E, float pv, int pi, float& bv, int& bi) {
@@ -52,27 +59,92 @@ FT_DEVICE void next_best(const float* z, int E, float pv, int pi, float& bv, int
   }
 }
 
-// one warp per token
-__global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__ logits, int64_t ld, int T, int E, int top, int* __restrict__ expert,
-                                                       float* __restrict__ score, int* __restrict__ pos, int* __restrict__ count) {
-  const int tok = blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (tok >= T) return;
-  const float* z = logits + (size_t)tok * ld;
+// How a router with a correction chooses: experts by sigmoid(logit) + correction, within the `keep` groups (of neighbours) whose two best experts have the largest sum
+// (groups 0: all experts); the weights are the chosen sigmoids divided by their sum, times scale. correction null: by logit, weights are the sigmoids.
+struct RouteRule {
+  const float* correction;
+  int groups, keep;
+  float scale;
+};
+constexpr float WEIGHT_SUM_EPS = 1e-20f;
+constexpr int MAX_GROUPS = 256;
+
+// whole warp: ch[e] = choice score of expert e, minus infinity outside the best groups. gs: [groups] scratch
+FT_DEVICE void choice_scores(const float* z, float* ch, int E, const RouteRule& rule, float* gs) {
+  const int lane = threadIdx.x & 31;
+  for (int e = lane; e < E; e += 32) ch[e] = sigmoid_f(__ldcg(z + e)) + rule.correction[e];
+  __syncwarp();
+  if (rule.groups == 0) return;
+  const int size = E / rule.groups;
+  for (int g = lane; g < rule.groups; g += 32) {
+    float a = -INFINITY, b = -INFINITY;              // the two largest
+    for (int i = 0; i < size; i++) {
+      const float v = ch[g * size + i];
+      b = fmaxf(b, fminf(a, v));
+      a = fmaxf(a, v);
+    }
+    gs[g] = size > 1 ? a + b : a;
+  }
+  __syncwarp();
   float pv = INFINITY;
   int pi = -1;
+  for (int k = 0; k < rule.keep; k++) {              // the last group that stays, in the order "score descending, index ascending"
+    float v;
+    int g;
+    next_best(gs, rule.groups, pv, pi, v, g);
+    pv = v;
+    pi = g;
+  }
+  for (int e = lane; e < E; e += 32) {
+    const int g = e / size;
+    if (gs[g] < pv || (gs[g] == pv && g > pi)) ch[e] = -INFINITY;
+  }
+  __syncwarp();
+}
+// whole warp: the `top` best of ch in order, take(slot, expert, sigmoid of its logit) on every lane; a ruled router's normed weights follow, lane j with take(-1 - j, 0, weight)
+template <typename Take>
+FT_DEVICE void choose(const float* z, const float* ch, int E, int top, const RouteRule& rule, Take take) {
+  float pv = INFINITY, sum = 0.f;
+  int pi = -1;
+  const bool ruled = rule.correction != nullptr;
+  float mine = 0.f;                                  // lane j keeps the weight of slot j (of a ruled router: top <= 32)
   for (int j = 0; j < top; j++) {
     float v;
     int e;
-    next_best(z, E, pv, pi, v, e);
+    next_best(ch, E, pv, pi, v, e);
     if (e >= E) e = j;                               // only with NaN logits
-    if ((threadIdx.x & 31) == 0) {
-      expert[(size_t)tok * top + j] = e;
-      score[(size_t)tok * top + j] = sigmoid_f(v);
-      pos[(size_t)tok * top + j] = atomicAdd(&count[e], 1);
-    }
+    const float s = sigmoid_f(ruled ? __ldcg(z + e) : v);
+    sum += s;
+    if ((threadIdx.x & 31) == j) mine = s;
+    take(j, e, s);
     pv = v;
     pi = e;
   }
+  if (ruled) {
+    const float k = rule.scale / (sum + WEIGHT_SUM_EPS);
+    if ((int)(threadIdx.x & 31) < top) take(-1 - (int)(threadIdx.x & 31), 0, mine * k);
+  }
+}
+
+// one warp per token; dynamic shared memory (ruled routers): [8][E + groups]
+__global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__ logits, int64_t ld, int T, int E, int top, RouteRule rule, int* __restrict__ expert,
+                                                       float* __restrict__ score, int* __restrict__ pos, int* __restrict__ count) {
+  extern __shared__ float choice_sh[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, tok = blockIdx.x * 8 + warp;
+  if (tok >= T) return;
+  const float* z = logits + (size_t)tok * ld;
+  float* ch = choice_sh + (size_t)warp * (E + rule.groups);
+  if (rule.correction) choice_scores(z, ch, E, rule, ch + E);
+  const size_t at = (size_t)tok * top;
+  choose(z, rule.correction ? ch : z, E, top, rule, [&](int j, int e, float s) {
+    if (j < 0) {                                     // final weights, a lane each
+      score[at - 1 - j] = s;
+    } else if (lane == 0) {
+      expert[at + j] = e;
+      if (!rule.correction) score[at + j] = s;
+      pos[at + j] = atomicAdd(&count[e], 1);
+    }
+  });
 }
 
 // one CTA: segment starts (multiples of SEG), group of every SEG-row tile (-1: unused), number of rows in use; count is zeroed for the next launch
@@ -125,7 +197,7 @@ __global__ void __launch_bounds__(128) moe_gather_kernel(const uint4* __restrict
 // gate and the up half of a block (16 bytes each, a warp reads 512 contiguous bytes) and swap halves, so each ends up with four neurons.
 template <typename T>
 __global__ void __launch_bounds__(256) moe_act_kernel(const T* __restrict__ gu, int64_t ld_gu, const float* __restrict__ row_score, const int* __restrict__ rows_used,
-                                                      int rows, int fp, float limit, float slope, T* __restrict__ act, int64_t ld_act) {
+                                                      int rows, int fp, int kind, float limit, float slope, T* __restrict__ act, int64_t ld_act) {
   const int n = rows_used ? min(rows, *rows_used) : rows;
   const int unit = blockIdx.x * blockDim.x + threadIdx.x, units = fp / 4;
   if constexpr (sizeof(T) == 2) {
@@ -151,8 +223,8 @@ __global__ void __launch_bounds__(256) moe_act_kernel(const T* __restrict__ gu, 
         const float2 ga = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g0)), gb = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g1));
         const float2 ua = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u0)), ub = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u1));
         const float k = sc[i];
-        __nv_bfloat162 o0 = __floats2bfloat162_rn(gated_clamped_fast(k * ga.x, k * ua.x, limit, slope), gated_clamped_fast(k * ga.y, k * ua.y, limit, slope));
-        __nv_bfloat162 o1 = __floats2bfloat162_rn(gated_clamped_fast(k * gb.x, k * ub.x, limit, slope), gated_clamped_fast(k * gb.y, k * ub.y, limit, slope));
+        __nv_bfloat162 o0 = __floats2bfloat162_rn(expert_act<true>(kind, k, ga.x, ua.x, limit, slope), expert_act<true>(kind, k, ga.y, ua.y, limit, slope));
+        __nv_bfloat162 o1 = __floats2bfloat162_rn(expert_act<true>(kind, k, gb.x, ub.x, limit, slope), expert_act<true>(kind, k, gb.y, ub.y, limit, slope));
         uint2 pk;
         pk.x = *reinterpret_cast<uint32_t*>(&o0);
         pk.y = *reinterpret_cast<uint32_t*>(&o1);
@@ -165,7 +237,7 @@ __global__ void __launch_bounds__(256) moe_act_kernel(const T* __restrict__ gu, 
       const float s = row_score ? row_score[r] : 1.f;
       const T* src = gu + (size_t)r * ld_gu + (unit / 2) * 16 + (unit % 2) * 4;
 #pragma unroll
-      for (int e = 0; e < 4; e++) act[(size_t)r * ld_act + unit * 4 + e] = gated_clamped(s * src[e], s * src[8 + e], limit, slope);
+      for (int e = 0; e < 4; e++) act[(size_t)r * ld_act + unit * 4 + e] = expert_act<false>(kind, s, src[e], src[8 + e], limit, slope);
     }
   }
 }
@@ -186,13 +258,15 @@ struct SmallRoute {
 
 constexpr int ROUTE_LOGITS = 8192;   // logits of the choosing CTA that fit its shared memory
 
-// grid E: one CTA per expert computes its logit for every token; the last CTA chooses and builds the lists
+// grid E: one CTA per expert computes its logit for every token; the last CTA chooses and builds the lists. logits: [16][E], and [16][E] more of scratch behind them
 __global__ void __launch_bounds__(128) moe_route_small_kernel(const __nv_bfloat16* __restrict__ h, int64_t ldh, const __nv_bfloat16* __restrict__ router, int64_t ldr,
-                                                              int B, int W, int E, int top, float* __restrict__ logits, int* __restrict__ counter, SmallRoute R) {
+                                                              int B, int W, int E, int top, RouteRule rule, float* __restrict__ logits, int* __restrict__ counter,
+                                                              SmallRoute R) {
   pdl_wait();
   pdl_launch_dependents();
   __shared__ float part[4][SMALL_TOK];
   __shared__ float zs[ROUTE_LOGITS];
+  __shared__ float gs[4][MAX_GROUPS];
   __shared__ int chosen[SMALL_TOK * MAX_TOP];
   __shared__ int is_last;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, e = blockIdx.x;
@@ -233,23 +307,22 @@ __global__ void __launch_bounds__(128) moe_route_small_kernel(const __nv_bfloat1
   if (!is_last) return;
   __threadfence();
   const bool staged = B * E <= ROUTE_LOGITS;
-  if (staged) {
+  if (staged && !rule.correction) {
     for (int i = threadIdx.x; i < B * E; i += 128) zs[i] = __ldcg(logits + i);
     __syncthreads();
   }
   for (int b = warp; b < B; b += 4) {
-    const float* z = staged ? zs + (size_t)b * E : logits + (size_t)b * E;
-    float pv = INFINITY;
-    int pi = -1;
-    for (int j = 0; j < top; j++) {
-      float v;
-      int c;
-      next_best(z, E, pv, pi, v, c);
-      if (c >= E) c = j;
-      if (lane == 0) { chosen[b * top + j] = c; R.score[b * top + j] = sigmoid_f(v); }
-      pv = v;
-      pi = c;
-    }
+    const float* z = logits + (size_t)b * E;
+    float* ch = staged ? zs + (size_t)b * E : logits + (size_t)SMALL_TOK * E + (size_t)b * E;
+    if (rule.correction) choice_scores(z, ch, E, rule, gs[warp]);
+    choose(z, rule.correction || staged ? ch : z, E, top, rule, [&](int j, int c, float s) {
+      if (j < 0) {
+        R.score[b * top - 1 - j] = s;
+      } else if (lane == 0) {
+        chosen[b * top + j] = c;
+        if (!rule.correction) R.score[b * top + j] = s;
+      }
+    });
   }
   __syncthreads();
   // active experts in ascending order; thread t of a round looks at expert e0 + t
@@ -299,7 +372,7 @@ struct GateUpWork {
   int B, W, tok0;
   SmallRoute R;
   ExpertSet ex, sh;
-  int has_shared;
+  int has_shared, kind;
   float slope;
   __nv_bfloat16 *act, *act_sh;
   int64_t ld_act, ld_act_sh;
@@ -325,7 +398,7 @@ struct GateUpWork {
       if (pr < 0) continue;
       const float k = s ? 1.f : R.score[pr];
       (s ? act_sh + (size_t)pr * ld_act_sh : act + (size_t)pr * ld_act)[f] =
-          __float2bfloat16(gated_clamped_fast(k * (j ? c.y : c.x), k * (j ? c.w : c.z), S.limit, slope));
+          __float2bfloat16(expert_act<true>(kind, k, j ? c.y : c.x, j ? c.w : c.z, S.limit, slope));
     }
   }
 };
@@ -397,15 +470,27 @@ struct HeadsWork {
   }
 };
 
+bool rule_ok(const RouteRule& r, int E, int top) {
+  if (!r.correction) return r.groups == 0;
+  if (r.groups < 0 || r.groups > MAX_GROUPS || top > 32) return false;
+  return r.groups == 0 || (E % r.groups == 0 && r.keep >= 1 && r.keep <= r.groups && top <= r.keep * (E / r.groups));
+}
 bool skinny_fits(int nt, int kmax) { return 8 * nt * skinny_pitch((kmax + 31) & ~31) + 64 <= SKINNY_SMEM_MAX; }
 
 }  // namespace
 
 // Choice of the `top` largest logits per token (ties: lower index first), their sigmoids, and the running position of every (token, slot) inside its
-// expert. count: int[E], zero before the launch (ft_moe_layout zeroes it again). expert, score, pos: [T * top].
-FT_EXPORT int ft_moe_topk(const float* logits, int64_t ld, int T, int E, int top, int* expert, float* score, int* pos, int* count, cudaStream_t st) {
-  if (T < 1 || E < 1 || top < 1 || top > E) return FT_ERR_ARG;
-  moe_topk_kernel<<<(T + 7) / 8, 256, 0, st>>>(logits, ld, T, E, top, expert, score, pos, count);
+// expert. count: int[E], zero before the launch (ft_moe_layout zeroes it again). expert, score, pos: [T * top]. With a correction (f32[E]) the choice goes by sigmoid +
+// correction, within the `keep` best of `groups` equal groups of neighbours (0: no groups; a group counts its two best), and the scores are the chosen sigmoids
+// divided by their sum, times scale (top up to 32, groups up to 256).
+FT_EXPORT int ft_moe_topk(const float* logits, int64_t ld, int T, int E, int top, const float* correction, int groups, int keep, float scale, int* expert, float* score,
+                          int* pos, int* count, cudaStream_t st) {
+  const RouteRule rule{correction, groups, keep, scale};
+  if (T < 1 || E < 1 || top < 1 || top > E || !rule_ok(rule, E, top)) return FT_ERR_ARG;
+  const size_t smem = correction ? (size_t)8 * (E + groups) * 4 : 0;
+  if (smem > 200 * 1024) return FT_ERR_TOO_LARGE;
+  if (smem > 48 * 1024) FT_CUDA_TRY(cudaFuncSetAttribute(moe_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
+  moe_topk_kernel<<<(T + 7) / 8, 256, smem, st>>>(logits, ld, T, E, top, rule, expert, score, pos, count);
   return (int)cudaGetLastError();
 }
 
@@ -427,40 +512,41 @@ FT_EXPORT int ft_moe_gather(const void* h, int64_t ldh_bytes, const int* expert,
   return (int)cudaGetLastError();
 }
 
-// act[r][f] = g sigmoid(slope g) (u + 1) with g = min(s gate, limit), u = clamp(s up, -limit, limit), s = row_score[r] (1 when null). gu: columns in
-// blocks of eight gate, eight up (2 * fp columns); dtype bf16 or (is_f32) f32. rows_used: device int bounding the rows, or null.
-FT_EXPORT int ft_moe_act(const void* gu, int64_t ld_gu, const float* row_score, const int* rows_used, int rows, int fp, float limit, float slope, void* act,
-                         int64_t ld_act, int is_f32, cudaStream_t st) {
-  if (rows < 1 || fp < 8 || (fp & 7) || (ld_gu & 7) || (ld_act & 7) || ld_gu < 2 * fp || ld_act < fp) return FT_ERR_ARG;
+// kind 0: act[r][f] = g sigmoid(slope g) (u + 1) with g = min(s gate, limit), u = clamp(s up, -limit, limit), s = row_score[r] (1 when null); kind 1:
+// s gate sigmoid(gate) up. gu: columns in blocks of eight gate, eight up (2 * fp columns); dtype bf16 or (is_f32) f32. rows_used: device int bounding the rows, or null.
+FT_EXPORT int ft_moe_act(const void* gu, int64_t ld_gu, const float* row_score, const int* rows_used, int rows, int fp, int kind, float limit, float slope,
+                         void* act, int64_t ld_act, int is_f32, cudaStream_t st) {
+  if (rows < 1 || kind < 0 || kind > 1 || fp < 8 || (fp & 7) || (ld_gu & 7) || (ld_act & 7) || ld_gu < 2 * fp || ld_act < fp) return FT_ERR_ARG;
   const int units = fp / 4, gx = (units + 255) / 256, threads = ((units + gx - 1) / gx + 31) / 32 * 32;
   const int gy = (148 * 8 * (256 / threads) + gx - 1) / gx;
   const dim3 grid(gx, gy < rows ? gy : rows);
-  if (is_f32) moe_act_kernel<float><<<grid, threads, 0, st>>>((const float*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (float*)act, ld_act);
-  else moe_act_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>((const __nv_bfloat16*)gu, ld_gu, row_score, rows_used, rows, fp, limit, slope, (__nv_bfloat16*)act, ld_act);
+  if (is_f32) moe_act_kernel<float><<<grid, threads, 0, st>>>((const float*)gu, ld_gu, row_score, rows_used, rows, fp, kind, limit, slope, (float*)act, ld_act);
+  else moe_act_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>((const __nv_bfloat16*)gu, ld_gu, row_score, rows_used, rows, fp, kind, limit, slope, (__nv_bfloat16*)act, ld_act);
   return (int)cudaGetLastError();
 }
 
-// Decode routing (B <= 16 tokens, bf16 operands, f32 accumulation): logits [B][E] f32 scratch, counter int zero before the first launch. Outputs:
-// n_active int[1], id int[E], cnt int[E], pair int[E][16], pair_of int[E][16], score f32 [B * top].
-FT_EXPORT int ft_moe_route_small(const void* h, int64_t ldh, const void* router, int64_t ldr, int B, int W, int E, int top, float* logits, int* counter, int* n_active,
-                                 int* id, int* cnt, int* pair, int* pair_of, float* score, cudaStream_t st) {
-  if (B < 1 || B > SMALL_TOK || E < 1 || top < 1 || top > E || top > MAX_TOP || (ldh & 7) || (ldr & 7)) return FT_ERR_ARG;
-  return (int)ft_launch_pdl(moe_route_small_kernel, dim3(E), dim3(128), 0, st, (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)router, ldr, B, W, E, top, logits,
-                            counter, SmallRoute{n_active, id, cnt, pair, pair_of, score});
+// Decode routing (B <= 16 tokens, bf16 operands, f32 accumulation): logits f32 scratch of 32 E, counter int zero before the first launch. Outputs:
+// n_active int[1], id int[E], cnt int[E], pair int[E][16], pair_of int[E][16], score f32 [B * top]. Choice and scores as in ft_moe_topk.
+FT_EXPORT int ft_moe_route_small(const void* h, int64_t ldh, const void* router, int64_t ldr, int B, int W, int E, int top, const float* correction, int groups, int keep,
+                                 float scale, float* logits, int* counter, int* n_active, int* id, int* cnt, int* pair, int* pair_of, float* score, cudaStream_t st) {
+  const RouteRule rule{correction, groups, keep, scale};
+  if (B < 1 || B > SMALL_TOK || E < 1 || top < 1 || top > E || top > MAX_TOP || (ldh & 7) || (ldr & 7) || !rule_ok(rule, E, top)) return FT_ERR_ARG;
+  return (int)ft_launch_pdl(moe_route_small_kernel, dim3(E), dim3(128), 0, st, (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)router, ldr, B, W, E, top, rule,
+                            logits, counter, SmallRoute{n_active, id, cnt, pair, pair_of, score});
 }
 
 // Gate / up projections and activation of a decode step. gu: [E][2 * fp][ld_in] interleaved rows, ld_in >= W rounded up to 32; act: bf16 [B * top][ld_act],
-// row = token * top + slot. Shared expert (shared_gu null: none): act_sh bf16 [B][ld_act_sh]. fp is the neuron count rounded up to 8.
+// row = token * top + slot; kind as in ft_moe_act. Shared expert (shared_gu null: none): act_sh bf16 [B][ld_act_sh]. fp is the neuron count rounded up to 8.
 FT_EXPORT int ft_moe_gate_up_small(const void* h, int64_t ldh, int B, int W, int E, int top, int* n_active, int* id, int* cnt, int* pair, int* pair_of, float* score,
-                                   const void* gu, int f, int64_t ld_in, float limit, const void* shared_gu, int f_sh, int64_t ld_in_sh, float limit_sh, float slope,
-                                   void* act, int64_t ld_act, void* act_sh, int64_t ld_act_sh, cudaStream_t st) {
+                                   const void* gu, int f, int64_t ld_in, float limit, const void* shared_gu, int f_sh, int64_t ld_in_sh, float limit_sh, int kind,
+                                   float slope, void* act, int64_t ld_act, void* act_sh, int64_t ld_act_sh, cudaStream_t st) {
   const int kp = (W + 31) & ~31, fp = (f + 7) & ~7, fps = (f_sh + 7) & ~7;
   if (B < 1 || B > SMALL_TOK || f < 1 || (ldh & 7) || (ld_in & 7) || ld_in < kp || ld_act < f || (shared_gu && (f_sh < 1 || (ld_in_sh & 7) || ld_in_sh < kp || ld_act_sh < f_sh)))
     return FT_ERR_ARG;
   if (!skinny_fits(1, W)) return FT_ERR_TOO_LARGE;
   GateUpWork p{(const __nv_bfloat16*)h, ldh, B, W, 0, SmallRoute{n_active, id, cnt, pair, pair_of, score},
                ExpertSet{(const __nv_bfloat16*)gu, f, fp, ld_in, 2 * fp * ld_in, limit}, ExpertSet{(const __nv_bfloat16*)shared_gu, f_sh, fps, ld_in_sh, 0, limit_sh},
-               shared_gu ? 1 : 0, slope, (__nv_bfloat16*)act, (__nv_bfloat16*)act_sh, ld_act, ld_act_sh};
+               shared_gu ? 1 : 0, kind, slope, (__nv_bfloat16*)act, (__nv_bfloat16*)act_sh, ld_act, ld_act_sh};
   const int items = (E < B * top ? E : B * top) * (fp / 8) + (shared_gu ? fps / 8 : 0);
   if (B > 8 && skinny_fits(2, W)) return skinny_launch<GateUpWork, 2>(p, W, items, st);
   for (p.tok0 = 0; p.tok0 < B; p.tok0 += 8) {

@@ -1,10 +1,12 @@
-// One f32 residual per token with the norm on the sublayer's output, and the activation of a gated feed-forward.
+// One f32 residual per token, with the norm on the sublayer's output or ahead of two sublayers that run side by side, and the activation of a gated feed-forward.
 //
 //   ft_residual_embed    x = scale * table[id];  h = x in the operand type
 //   ft_residual_update   y = sum of the sublayer's f32 planes;  x += y / rms(y) * w;  h = x, or x / rms(x) * w_last ahead of the output projection
+//   ft_parallel_embed    x = table[id];  h1 = x / rms(x) * w1, h2 = x / rms(x) * w2: the operands of two sublayers
+//   ft_parallel_update   x += mult * (what both sublayers returned: f32 planes, expert rows through an index, a bias);  h1 and h2 from the new x
 //   ft_gated_act         act(gate) * up of interleaved gate / up columns, from a 16-bit or f32 matrix or from split-K planes
 //
-// ft_residual_update takes one row per cluster of CTAs: one CTA where there are rows enough to fill the GPU, up to eight (sums of squares meet in
+// The updates take one row per cluster of CTAs: one CTA where there are rows enough to fill the GPU, up to eight (sums of squares meet in
 // distributed shared memory) for the few rows of a decode step, whose planes are then read by eight SMs instead of one. Everything a row needs stays in
 // registers between its two norms. Compiled without fast-math.
 #include <cooperative_groups.h>
@@ -140,6 +142,99 @@ __global__ void __launch_bounds__(UPD_THREADS) residual_update_kernel(float* __r
   if (ncta > 1) cluster.sync();                     // nobody leaves while a partner may still read its shared memory
 }
 
+// Two sublayers of the same x: f32 planes of either (a: the mixer, b: the feed-forward), rows of experts through row_of, and a bias
+template <typename H> struct PairOutput {
+  const float *a, *b;
+  int na, nb;
+  size_t stride_a, stride_b;
+  int64_t lda, ldb;
+  const H* rows;
+  const int* row_of;
+  int top;
+  int64_t ldr;
+  const float* bias;
+};
+FT_DEVICE void add_planes(float4& v, const float* p, int planes, size_t stride) {
+  int k = 0;
+  for (; k + 4 <= planes; k += 4) {
+    float4 t[4];
+#pragma unroll
+    for (int j = 0; j < 4; j++) t[j] = __ldcg(reinterpret_cast<const float4*>(p + (k + j) * stride));
+    v.x += (t[0].x + t[1].x) + (t[2].x + t[3].x);
+    v.y += (t[0].y + t[1].y) + (t[2].y + t[3].y);
+    v.z += (t[0].z + t[1].z) + (t[2].z + t[3].z);
+    v.w += (t[0].w + t[1].w) + (t[2].w + t[3].w);
+  }
+  for (; k < planes; k++) {
+    const float4 t = __ldcg(reinterpret_cast<const float4*>(p + k * stride));
+    v.x += t.x; v.y += t.y; v.z += t.z; v.w += t.w;
+  }
+}
+// EMBED: x starts as the embedding row of ids[row]. w2 null: one operand
+template <int NV, bool EMBED, typename H>
+__global__ void __launch_bounds__(UPD_THREADS) parallel_update_kernel(float* __restrict__ x, int64_t ldx, const int64_t* __restrict__ ids, const H* __restrict__ table,
+                                                                      int64_t ld_table, int64_t vocab, PairOutput<H> Y, float mult, const float* __restrict__ w1,
+                                                                      const float* __restrict__ w2, float eps, H* __restrict__ h1, H* __restrict__ h2, int64_t ldh, int ncta,
+                                                                      int W, int cols, int store_x) {
+  namespace cg = cooperative_groups;
+  __shared__ float red[32];
+  __shared__ float cta_ss;
+  cg::cluster_group cluster = cg::this_cluster();
+  const int row = blockIdx.x / ncta, c0 = blockIdx.x % ncta * cols, cend = min(W, c0 + cols);
+  pdl_wait();
+  pdl_launch_dependents();
+  float* xr = x + (size_t)row * ldx;
+  int64_t id = -1;
+  if constexpr (EMBED) id = ids[row];
+  float4 xv[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < cend) {
+      if constexpr (EMBED) {
+        if (id >= 0 && id < vocab) xv[i] = get4(table + (size_t)id * ld_table + c);
+      } else {
+        const float4 old = *reinterpret_cast<const float4*>(xr + c);
+        float4 v = Y.bias ? *reinterpret_cast<const float4*>(Y.bias + c) : make_float4(0.f, 0.f, 0.f, 0.f);
+        if (Y.na) add_planes(v, Y.a + (size_t)row * Y.lda + c, Y.na, Y.stride_a);
+        if (Y.nb) add_planes(v, Y.b + (size_t)row * Y.ldb + c, Y.nb, Y.stride_b);
+#pragma unroll 4
+        for (int k = 0; k < Y.top; k++) {
+          const float4 t = get4(Y.rows + (size_t)Y.row_of[(size_t)row * Y.top + k] * Y.ldr + c);
+          v.x += t.x; v.y += t.y; v.z += t.z; v.w += t.w;
+        }
+        xv[i] = make_float4(old.x + mult * v.x, old.y + mult * v.y, old.z + mult * v.z, old.w + mult * v.w);
+      }
+      xv[i] = keep4(xv[i], c, W);
+      if (store_x) *reinterpret_cast<float4*>(xr + c) = xv[i];
+      ss += sq4(xv[i]);
+    }
+  }
+  ss = block_sum(ss, red);
+  if (ncta > 1) {
+    if (threadIdx.x == 0) cta_ss = ss;
+    cluster.sync();
+    ss = 0.f;
+    for (int r = 0; r < ncta; r++) ss += *cluster.map_shared_rank(&cta_ss, r);
+  }
+  const float rstd = 1.f / sqrtf(ss / (float)W + eps);
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    if (c < cend) {
+      const float4 n = make_float4(xv[i].x * rstd, xv[i].y * rstd, xv[i].z * rstd, xv[i].w * rstd), a = *reinterpret_cast<const float4*>(w1 + c);
+      put4(h1 + (size_t)row * ldh + c, make_float4(n.x * a.x, n.y * a.y, n.z * a.z, n.w * a.w));
+      if (w2 != nullptr) {
+        const float4 b = *reinterpret_cast<const float4*>(w2 + c);
+        put4(h2 + (size_t)row * ldh + c, make_float4(n.x * b.x, n.y * b.y, n.z * b.z, n.w * b.w));
+      }
+    }
+  }
+  if (ncta > 1) cluster.sync();                     // nobody leaves while a partner may still read its shared memory
+}
+
 // ------------------------------------------------------------------------------------------------------------
 // gated activation
 // ------------------------------------------------------------------------------------------------------------
@@ -163,11 +258,18 @@ FT_DEVICE float4 unpack4(uint2 r) {
   return make_float4(a.x, a.y, b.x, b.y);
 }
 
-// columns come in blocks of eight gates and the eight ups of the same neurons; a thread takes one block (bf16: two 16-byte loads, one 16-byte store)
+FT_DEVICE float4 add4(float4 a, float4 b) { return make_float4(a.x + b.x, a.y + b.y, a.z + b.z, a.w + b.w); }
+
+// columns come in blocks of eight gates and the eight ups of the same neurons; a thread takes one block (bf16: two 16-byte loads, one 16-byte store). bias: f32 in the
+// order of the columns, or null
 template <typename T>
-__global__ void __launch_bounds__(256) gated_act_kernel(const T* __restrict__ gu, int64_t ld, int rows, int blocks, int kind, T* __restrict__ out, int64_t ldo) {
+__global__ void __launch_bounds__(256) gated_act_kernel(const T* __restrict__ gu, int64_t ld, const float* __restrict__ bias, int rows, int blocks, int kind,
+                                                        T* __restrict__ out, int64_t ldo) {
   const int b = blockIdx.x * blockDim.x + threadIdx.x;
   if (b >= blocks) return;
+  float4 bv[4];
+#pragma unroll
+  for (int i = 0; i < 4; i++) bv[i] = bias ? *reinterpret_cast<const float4*>(bias + b * 16 + i * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
   constexpr int RU = sizeof(T) == 2 ? 4 : 1;
   for (int r0 = blockIdx.y * RU; r0 < rows; r0 += gridDim.y * RU) {
     if constexpr (sizeof(T) == 2) {
@@ -180,8 +282,8 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const T* __restrict__ gu
       }
 #pragma unroll
       for (int i = 0; i < RU; i++) {
-        const float4 a = gated4<false>(unpack4(make_uint2(g[i].x, g[i].y)), unpack4(make_uint2(u[i].x, u[i].y)), kind);
-        const float4 c = gated4<false>(unpack4(make_uint2(g[i].z, g[i].w)), unpack4(make_uint2(u[i].z, u[i].w)), kind);
+        const float4 a = gated4<false>(add4(unpack4(make_uint2(g[i].x, g[i].y)), bv[0]), add4(unpack4(make_uint2(u[i].x, u[i].y)), bv[2]), kind);
+        const float4 c = gated4<false>(add4(unpack4(make_uint2(g[i].z, g[i].w)), bv[1]), add4(unpack4(make_uint2(u[i].z, u[i].w)), bv[3]), kind);
         const float e[8] = {a.x, a.y, a.z, a.w, c.x, c.y, c.z, c.w};
         if (r0 + i < rows) *reinterpret_cast<bf16x8*>(out + (size_t)(r0 + i) * ldo + b * 8) = float_to_bf16x8(e);
       }
@@ -189,13 +291,14 @@ __global__ void __launch_bounds__(256) gated_act_kernel(const T* __restrict__ gu
       const float* s = gu + (size_t)r0 * ld + b * 16;
 #pragma unroll
       for (int i = 0; i < 8; i += 4)
-        *reinterpret_cast<float4*>(out + (size_t)r0 * ldo + b * 8 + i) = gated4<true>(*reinterpret_cast<const float4*>(s + i), *reinterpret_cast<const float4*>(s + 8 + i), kind);
+        *reinterpret_cast<float4*>(out + (size_t)r0 * ldo + b * 8 + i) =
+            gated4<true>(add4(*reinterpret_cast<const float4*>(s + i), bv[i / 4]), add4(*reinterpret_cast<const float4*>(s + 8 + i), bv[2 + i / 4]), kind);
     }
   }
 }
 
-__global__ void __launch_bounds__(128) gated_act_planes_kernel(const float* __restrict__ p, int splits, int64_t ldp, size_t pstride, int rows, int quads, int kind,
-                                                               __nv_bfloat16* __restrict__ out, int64_t ldo) {
+__global__ void __launch_bounds__(128) gated_act_planes_kernel(const float* __restrict__ p, int splits, int64_t ldp, size_t pstride, const float* __restrict__ bias, int rows,
+                                                               int quads, int kind, __nv_bfloat16* __restrict__ out, int64_t ldo) {
   pdl_wait();
   pdl_launch_dependents();
   const int i = blockIdx.x * 128 + threadIdx.x;
@@ -203,6 +306,10 @@ __global__ void __launch_bounds__(128) gated_act_planes_kernel(const float* __re
   const int r = i / quads, q = i % quads;                       // four neurons
   const float* s = p + (size_t)r * ldp + (q >> 1) * 16 + (q & 1) * 4;
   float4 g = make_float4(0.f, 0.f, 0.f, 0.f), u = g;
+  if (bias) {
+    g = *reinterpret_cast<const float4*>(bias + (q >> 1) * 16 + (q & 1) * 4);
+    u = *reinterpret_cast<const float4*>(bias + (q >> 1) * 16 + (q & 1) * 4 + 8);
+  }
 #pragma unroll 4
   for (int k = 0; k < splits; k++) {
     const float4 a = __ldcg(reinterpret_cast<const float4*>(s + k * pstride)), b = __ldcg(reinterpret_cast<const float4*>(s + k * pstride + 8));
@@ -230,15 +337,46 @@ int launch_update(int ncta, int rows, cudaStream_t st, float* x, int64_t ldx, co
   return (int)cudaLaunchKernelEx(&cfg, residual_update_kernel<NV, H>, x, ldx, y, planes, (size_t)pstride, ldy, w, w_last, eps, h, ldh, ncta, W, cols, store);
 }
 
-template <typename H>
-int dispatch_update(float* x, int64_t ldx, const float* y, int planes, int64_t pstride, int64_t ldy, const float* w, const float* w_last, float eps, void* h, int64_t ldh,
-                    int rows, int W, int store, cudaStream_t st) {
+// how a row of W columns is spread: CTAs of its cluster, columns of a CTA, float4 columns of a thread
+struct RowSpread { int ncta, cols, nv; };
+RowSpread row_spread(int rows, int W) {
   // rows alone fill the GPU, or a row is spread over up to eight SMs (at least 256 columns each)
   int ncta = 1;
   while (ncta < 8 && (rows * ncta < 148 && W > 256 * ncta * 2)) ncta *= 2;
   while (ncta < 8 && (W + ncta - 1) / ncta > UPD_THREADS * 4 * 8) ncta *= 2;
   const int cols = ((W + ncta - 1) / ncta + 3) & ~3;
-  const int nv = (cols + UPD_THREADS * 4 - 1) / (UPD_THREADS * 4);
+  return RowSpread{ncta, cols, (cols + UPD_THREADS * 4 - 1) / (UPD_THREADS * 4)};
+}
+
+template <bool EMBED, typename H>
+int dispatch_parallel(float* x, int64_t ldx, const int64_t* ids, const void* table, int64_t ld_table, int64_t vocab, const PairOutput<H>& Y, float mult, const float* w1,
+                      const float* w2, float eps, void* h1, void* h2, int64_t ldh, int rows, int W, int store, cudaStream_t st) {
+  const RowSpread sp = row_spread(rows, W);
+  if (sp.nv > 8) return FT_ERR_TOO_LARGE;
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(sp.ncta * rows);
+  cfg.blockDim = dim3(UPD_THREADS);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = sp.ncta;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = ft_pdl_enabled() ? 2 : 1;
+#define FT_PU(N) return (int)cudaLaunchKernelEx(&cfg, parallel_update_kernel<N, EMBED, H>, x, ldx, ids, (const H*)table, ld_table, vocab, Y, mult, w1, w2, eps, (H*)h1, (H*)h2, ldh,                                                 sp.ncta, W, sp.cols, store)
+  if (sp.nv <= 1) FT_PU(1);
+  if (sp.nv <= 2) FT_PU(2);
+  if (sp.nv <= 4) FT_PU(4);
+  FT_PU(8);
+#undef FT_PU
+}
+
+template <typename H>
+int dispatch_update(float* x, int64_t ldx, const float* y, int planes, int64_t pstride, int64_t ldy, const float* w, const float* w_last, float eps, void* h, int64_t ldh,
+                    int rows, int W, int store, cudaStream_t st) {
+  const auto [ncta, cols, nv] = row_spread(rows, W);
   if (nv > 8) return FT_ERR_TOO_LARGE;
 #define FT_RU(N) return launch_update<N, H>(ncta, rows, st, x, ldx, y, planes, pstride, ldy, w, w_last, eps, (H*)h, ldh, W, cols, store)
   if (nv <= 1) FT_RU(1);
@@ -270,21 +408,47 @@ FT_EXPORT int ft_residual_update(float* x, int64_t ldx, const float* y, int plan
   return dispatch_update<__nv_bfloat16>(x, ldx, y, planes, plane_stride, ldy, w, w_last, eps, h, ldh, rows, W, store_x, st);
 }
 
-// out[r][f] = act(gate) * up for f < fp (a multiple of 8) from columns in blocks of eight gates and eight ups; kind 0: gelu (tanh form), 1: silu.
-FT_EXPORT int ft_gated_act(const void* gu, int64_t ld, int rows, int fp, int kind, void* out, int64_t ldo, int is_f32, cudaStream_t st) {
+// Start of a pass whose layers norm ahead of two sublayers: x [rows][ldx] f32 = table[ids[r]] (zeros for ids outside [0, vocab)), h1 = x / sqrt(mean(x^2) + eps) * w1 and, unless
+// w2 is null, h2 the same with w2; both [rows][ldh] in the table's type. Widths up to 65536.
+FT_EXPORT int ft_parallel_embed(const int64_t* ids, const void* table, int64_t ld_table, int64_t vocab, const float* w1, const float* w2, float eps, float* x, int64_t ldx,
+                                void* h1, void* h2, int64_t ldh, int is_f32, int rows, int W, cudaStream_t st) {
+  if (rows < 1 || W < 1 || !w1 || (w2 && !h2) || (ld_table & 3) || (ldx & 3) || (ldh & 3)) return FT_ERR_ARG;
+  if (is_f32) return dispatch_parallel<true, float>(x, ldx, ids, table, ld_table, vocab, PairOutput<float>{}, 0.f, w1, w2, eps, h1, h2, ldh, rows, W, 1, st);
+  return dispatch_parallel<true, __nv_bfloat16>(x, ldx, ids, table, ld_table, vocab, PairOutput<__nv_bfloat16>{}, 0.f, w1, w2, eps, h1, h2, ldh, rows, W, 1, st);
+}
+
+// x += mult * (planes of a [na][row][lda] + planes of b [nb][row][ldb] + expert rows row_of[row][0..top) (type of h) + bias); h1, h2 as in ft_parallel_embed. a, b: f32, either
+// may be absent (0 planes); bias f32 or null; all vectors readable up to W rounded up to a multiple of four. x is left alone when store_x is 0.
+FT_EXPORT int ft_parallel_update(float* x, int64_t ldx, float mult, const float* a, int na, int64_t stride_a, int64_t lda, const float* b, int nb, int64_t stride_b, int64_t ldb,
+                                 const void* expert_rows, const int* row_of, int top, int64_t ldr, const float* bias, const float* w1, const float* w2, float eps, void* h1,
+                                 void* h2, int64_t ldh, int is_f32, int rows, int W, int store_x, cudaStream_t st) {
+  if (rows < 1 || W < 1 || na < 0 || nb < 0 || top < 0 || !w1 || (w2 && !h2) || (ldx & 3) || (lda & 3) || (ldb & 3) || (ldr & 3) || (ldh & 3) || (stride_a & 3) || (stride_b & 3) ||
+      (top && (!expert_rows || !row_of)))
+    return FT_ERR_ARG;
+  if (is_f32) {
+    const PairOutput<float> Y{a, b, na, nb, (size_t)stride_a, (size_t)stride_b, lda, ldb, (const float*)expert_rows, row_of, top, ldr, bias};
+    return dispatch_parallel<false, float>(x, ldx, nullptr, nullptr, 0, 0, Y, mult, w1, w2, eps, h1, h2, ldh, rows, W, store_x, st);
+  }
+  const PairOutput<__nv_bfloat16> Y{a, b, na, nb, (size_t)stride_a, (size_t)stride_b, lda, ldb, (const __nv_bfloat16*)expert_rows, row_of, top, ldr, bias};
+  return dispatch_parallel<false, __nv_bfloat16>(x, ldx, nullptr, nullptr, 0, 0, Y, mult, w1, w2, eps, h1, h2, ldh, rows, W, store_x, st);
+}
+
+// out[r][f] = act(gate + bias) * (up + bias) for f < fp (a multiple of 8) from columns in blocks of eight gates and eight ups; kind 0: gelu (tanh form), 1: silu; bias: f32 in
+// the order of the columns, or null.
+FT_EXPORT int ft_gated_act(const void* gu, int64_t ld, const float* bias, int rows, int fp, int kind, void* out, int64_t ldo, int is_f32, cudaStream_t st) {
   if (rows < 1 || fp < 8 || (fp & 7) || (ld & 7) || (ldo & 7) || kind < 0 || kind > 1) return FT_ERR_ARG;
   const int blocks = fp / 8, threads = blocks >= 256 ? 256 : (blocks + 31) & ~31, ru = is_f32 ? 1 : 4;
   const int gx = (blocks + threads - 1) / threads, want = (rows + ru - 1) / ru, cap = 148 * 16 / gx + 1;
   const dim3 grid(gx, want < cap ? want : cap);
-  if (is_f32) gated_act_kernel<float><<<grid, threads, 0, st>>>((const float*)gu, ld, rows, blocks, kind, (float*)out, ldo);
-  else gated_act_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>((const __nv_bfloat16*)gu, ld, rows, blocks, kind, (__nv_bfloat16*)out, ldo);
+  if (is_f32) gated_act_kernel<float><<<grid, threads, 0, st>>>((const float*)gu, ld, bias, rows, blocks, kind, (float*)out, ldo);
+  else gated_act_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>((const __nv_bfloat16*)gu, ld, bias, rows, blocks, kind, (__nv_bfloat16*)out, ldo);
   return (int)cudaGetLastError();
 }
 
 // The same from split-K planes [split][row][ldp] (f32) to bf16 rows.
-FT_EXPORT int ft_gated_act_planes(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int rows, int fp, int kind, void* out, int64_t ldo, cudaStream_t st) {
+FT_EXPORT int ft_gated_act_planes(const float* planes, int splits, int64_t ldp, int64_t plane_stride, const float* bias, int rows, int fp, int kind, void* out, int64_t ldo, cudaStream_t st) {
   if (rows < 1 || splits < 1 || fp < 8 || (fp & 7) || (ldp & 3) || (plane_stride & 3) || (ldo & 3) || kind < 0 || kind > 1) return FT_ERR_ARG;
   const int quads = fp / 4;
-  return (int)ft_launch_pdl(gated_act_planes_kernel, dim3((rows * quads + 127) / 128), dim3(128), 0, st, planes, splits, ldp, (size_t)plane_stride, rows, quads, kind,
-                            (__nv_bfloat16*)out, ldo);
+  return (int)ft_launch_pdl(gated_act_planes_kernel, dim3((rows * quads + 127) / 128), dim3(128), 0, st, planes, splits, ldp, (size_t)plane_stride, bias, rows, quads,
+                            kind, (__nv_bfloat16*)out, ldo);
 }

@@ -69,20 +69,30 @@ class ExpertConfig:
 
 @dataclass
 class MoeConfig:
+    """``groups`` (0: none), of which ``keep`` stay, and ``scale`` belong to routers that choose within the best groups of experts and norm their weights."""
     experts: int
     top: int
     expert: ExpertConfig
     shared: Optional[ExpertConfig] = None
+    groups: int = 0
+    keep: int = 0
+    scale: float = 1.0
 
     @staticmethod
     def from_dict(d: dict) -> "MoeConfig":
         if d.get("kind", "moe") != "moe":
-            raise InvalidArgument(f"Ginisun: unknown feed-forward kind {d['kind']!r}")
-        return MoeConfig(int(d["router"]["experts"]), int(d["router"]["top"]), ExpertConfig.from_dict(d["expert"]),
-                         ExpertConfig.from_dict(d["shared"]) if d.get("shared") else None)
+            raise InvalidArgument(f"unknown feed-forward kind {d['kind']!r}")
+        r = d["router"]
+        g = r.get("groups") or {}
+        return MoeConfig(int(r["experts"]), int(r["top"]), ExpertConfig.from_dict(d["expert"]), ExpertConfig.from_dict(d["shared"]) if d.get("shared") else None,
+                         int(g.get("count", 0)), int(g.get("keep", 0)), float(r.get("scale", 1.0)))
 
     def to_dict(self) -> dict:
         out = dict(kind="moe", router=dict(experts=self.experts, top=self.top), expert=self.expert.to_dict())
+        if self.scale != 1.0:
+            out["router"]["scale"] = self.scale
+        if self.groups:
+            out["router"]["groups"] = dict(count=self.groups, keep=self.keep)
         if self.shared:
             out["shared"] = self.shared.to_dict()
         return out
@@ -140,6 +150,8 @@ class GinisunConfig:
                 raise InvalidArgument(f"Ginisun: layer {i}: scale must be positive")
             if l.mlp and not 1 <= l.mlp.top <= l.mlp.experts:
                 raise InvalidArgument(f"Ginisun: layer {i}: top must be between 1 and the number of experts")
+            if l.mlp and (l.mlp.groups or l.mlp.scale != 1.0):
+                raise InvalidArgument(f"Ginisun: layer {i}: the router has no groups and no scale")
 
     @staticmethod
     def uniform(layers: int, vocab: int, width: int, heads: int, dim: int, rot_dim: int, vdim: int, kv_rank: int, experts: int, top: int, ff: int, shared_ff: int = 0,

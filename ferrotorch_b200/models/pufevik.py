@@ -37,7 +37,8 @@ ACTIVATION = "gelu_tanh"             # fixed by the design
 
 @dataclass
 class AttentionConfig:
-    """Grouped-query attention; ``window`` 0 means every earlier position."""
+    """Grouped-query attention; ``window`` 0 means every earlier position, ``keep_first`` tokens stay visible beside a window; ``scaling``: YaRN scaling of the rotation (``factor``,
+    ``original``, ``fast``, ``slow``)."""
     heads: int
     kv_heads: int
     dim: int
@@ -47,17 +48,25 @@ class AttentionConfig:
     rope_base: float = 10000.0
     window: int = 0
     v_mix: bool = False
+    keep_first: int = 0
+    scaling: Optional[Dict[str, float]] = None
 
     @staticmethod
     def from_dict(d: dict) -> "AttentionConfig":
         rot, mask = d.get("rot") or {}, d.get("mask") or {}
+        s = rot.get("scaling")
         return AttentionConfig(int(d["heads"]), int(d["kv_heads"]), int(d["dim"]), int(d["vdim"]), float(d["scale"]), int(rot.get("dims", 0)), float(rot.get("base", 10000.0)),
-                               int(mask.get("size", 0)), bool(d.get("v_mix", False)))
+                               int(mask.get("size", 0)), bool(d.get("v_mix", False)), int(mask.get("keep_first", 0)),
+                               {k: float(s[k]) for k in ("factor", "original", "fast", "slow")} if s else None)
 
     def to_dict(self) -> dict:
         d = dict(heads=self.heads, kv_heads=self.kv_heads, dim=self.dim, vdim=self.vdim, scale=self.scale, rot=dict(base=self.rope_base, dims=self.rot_dims))
+        if self.scaling:
+            d["rot"]["scaling"] = dict(self.scaling)
         if self.window:
             d["mask"] = dict(size=self.window)
+            if self.keep_first:
+                d["mask"]["keep_first"] = self.keep_first
         if self.v_mix:
             d["v_mix"] = True
         return d
@@ -67,8 +76,17 @@ class AttentionConfig:
             raise InvalidArgument(f"{where}: sizes must be positive and heads a multiple of kv_heads")
         if self.rot_dims < 0 or self.rot_dims % 2 or self.rot_dims > self.dim or not self.rope_base > 0:
             raise InvalidArgument(f"{where}: rot.dims must be even and at most dim, rot.base positive")
-        if not self.scale > 0 or self.window < 0:
-            raise InvalidArgument(f"{where}: scale must be positive and the window not negative")
+        if not self.scale > 0 or self.window < 0 or self.keep_first < 0:
+            raise InvalidArgument(f"{where}: scale must be positive, the window and the number of kept tokens not negative")
+        if self.scaling and not (min(self.scaling.values()) > 0 and self.rope_base != 1.0):
+            raise InvalidArgument(f"{where}: the constants of rot.scaling must be positive")
+
+    @property
+    def rope_scaling(self) -> Optional[dict]:
+        """The scaling in the form of :func:`~ferrotorch_b200.ops.llama.rope_inv_freq`."""
+        s = self.scaling
+        return s and dict(type="yarn", factor=s["factor"], original_max_position=s["original"], beta_fast=s["fast"], beta_slow=s["slow"],
+                          attention_factor=0.1 * math.log(s["factor"]) + 1.0)
 
 
 @dataclass
@@ -167,8 +185,11 @@ class PufevikConfig:
             raise InvalidArgument("Pufevik: vocab, width and the number of layers must be positive")
         for i, l in enumerate(self.layers):
             l.mixer.validate(f"Pufevik: layer {i}")
-            if isinstance(l.mixer, AttentionConfig) and l.mixer.window:
+            a = l.mixer if isinstance(l.mixer, AttentionConfig) else l.mixer.left
+            if a is l.mixer and a.window:
                 raise InvalidArgument(f"Pufevik: layer {i}: a window stands in the left half of 'parallel' layers only")
+            if a.keep_first or a.scaling:
+                raise InvalidArgument(f"Pufevik: layer {i}: no kept first tokens, no scaled rotation")
         mix = [self.layers[i].mixer for i in self.mixing_layers]
         if any((m.kv_heads, m.vdim) != (mix[0].kv_heads, mix[0].vdim) for m in mix):
             raise InvalidArgument("Pufevik: layers that mix values must have the same kv_heads and vdim")

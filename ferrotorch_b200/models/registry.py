@@ -108,6 +108,17 @@ def _pufevik_engine(cfg, weights, device, dtype, max_tokens):
     return ServingEngine(PufevikModel(cfg, weights, device, dtype), max_tokens=max_tokens)
 
 
+def _mepupel_config(d: dict):
+    from .mepupel import MepupelConfig
+    return MepupelConfig.from_dict(d)
+
+
+def _mepupel_engine(cfg, weights, device, dtype, max_tokens):
+    from .mepupel import MepupelModel
+    from .serving import ServingEngine
+    return ServingEngine(MepupelModel(cfg, weights, device, dtype), max_tokens=max_tokens)
+
+
 def _llama_config(d: dict):
     from .llama import LlamaConfig
     return LlamaConfig.from_hf(d)
@@ -124,4 +135,5 @@ def _llama_engine(cfg, weights, device, dtype, max_tokens):
 PRODUCTS = ("gemm_tcgen05", "gemm_2sm", "gemm_simt", "fsdp_gather", "decode")      # matrix products and their split-K forms
 register_architecture(Architecture("Ginisun", _ginisun_config, _ginisun_engine, kernels=(*PRODUCTS, "stream_ops", "moe", "latent_attn")))
 register_architecture(Architecture("Pufevik", _pufevik_config, _pufevik_engine, kernels=(*PRODUCTS, "gqa_attn", "matrix_memory", "residual_ops")))
+register_architecture(Architecture("Mepupel", _mepupel_config, _mepupel_engine, kernels=(*PRODUCTS, "gqa_attn", "latent_attn", "moe", "state_space", "residual_ops")))
 register_architecture(Architecture("LlamaForCausalLM", _llama_config, _llama_engine, ("llama",)))

@@ -45,10 +45,11 @@ class StepEntry:
 class MemoryPlan:
     """How recurrent layers go over the new tokens of a batch. ``segments`` ``[n, 8]``: first row, rows, state slot, sequence, flags (1 the only segment, 2 the last, 4 the
     sequence starts), scratch state; ``inner``: those that are not last (``None`` if there are none); ``chains`` ``[sequences, 4]``: first scratch state, segments, slot,
-    whether the sequence starts; ``scratch``: number of scratch states."""
+    whether the sequence starts; ``spans`` ``[sequences, 4]``: first row, rows, slot, whether the sequence starts; ``scratch``: number of scratch states."""
     segments: torch.Tensor
     inner: Optional[torch.Tensor]
     chains: torch.Tensor
+    spans: torch.Tensor
     sequences: int
     scratch: int
 
@@ -114,7 +115,7 @@ class RowBatch:
         """Segments of the new tokens for recurrent layers whose walk takes ``ctas`` CTAs per segment: as many as fill the GPU, none shorter than ``SEGMENT_MIN`` tokens.
         ``ctas`` 0: one segment per sequence."""
         if ctas not in self._plans:
-            segs, inner, chains = [], [], []
+            segs, inner, chains, spans = [], [], [], []
             # an equal share of all new tokens per segment, as many segments as the GPU takes at once
             share = max(SEGMENT_MIN, -(-self.rows // max(1, SEGMENT_CTAS // ctas) // MEMORY_CHUNK) * MEMORY_CHUNK) if ctas else 0
             scratch = 0
@@ -129,10 +130,11 @@ class RowBatch:
                     if j + 1 < count:
                         inner.append(row)
                 chains.append((base, count, slot, fresh))
+                spans.append((r0, n, slot, fresh))
                 scratch += count if count > 1 else 0
-            packed = torch.tensor([x for r in segs + inner for x in r] + [x for r in chains for x in r], dtype=torch.int32).to(self.device)
-            a, b, c = torch.split(packed, [8 * len(segs), 8 * len(inner), 4 * len(chains)])
-            self._plans[ctas] = MemoryPlan(a.view(-1, 8), b.view(-1, 8) if inner else None, c.view(-1, 4), len(chains), scratch)
+            packed = torch.tensor([x for t in (segs, inner, chains, spans) for r in t for x in r], dtype=torch.int32).to(self.device)
+            a, b, c, d = torch.split(packed, [8 * len(segs), 8 * len(inner), 4 * len(chains), 4 * len(spans)])
+            self._plans[ctas] = MemoryPlan(a.view(-1, 8), b.view(-1, 8) if inner else None, c.view(-1, 4), d.view(-1, 4), len(chains), scratch)
         return self._plans[ctas]
 
 

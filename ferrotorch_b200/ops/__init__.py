@@ -8,12 +8,14 @@ from .loss import cross_entropy, cross_entropy_fwd_bwd
 from .optim import adamw_flat_, sgd_flat_, grad_norm_, scale_
 from .attention import attention_packed, flash_fwd, flash_bwd
 from .streams import DynamicTanhWeights, HyperWeights, SublayerOutput, dynamic_tanh, hyper_embed, hyper_update
-from .moe import ExpertStack, MoeWeights, MoeSmallBuffers, MoeRouting, moe_rows, moe_small, gated_act, grouped_linear, interleave_gate_up
-from .latent_attention import (LatentDims, LatentWeights, LatentDecodeBuffers, latent_attention_rows, latent_attention_decode, absorb_queries, expand_values,
+from .moe import ExpertStack, MoeWeights, MoeSmallBuffers, MoeRouting, RouteRule, moe_rows, moe_small, gated_act, grouped_linear, interleave_gate_up
+from .latent_attention import (LatentDims, LatentWeights, LatentDecodeBuffers, latent_context, latent_attention_rows, latent_attention_decode, absorb_queries, expand_values,
                                rotary_pair_tables)
-from .residual import DenseGatedWeights, dense_gated_rows, gated_act_planes, gated_act_rows, residual_embed, residual_update
+from .residual import (DenseGatedWeights, dense_gated_rows, gated_act_planes, gated_act_rows, parallel_embed, parallel_update, residual_embed,
+                       residual_update)
 from .gqa_attention import GqaDims, GqaWeights, GqaDecodeBuffers, gqa_attention_rows, gqa_attention_decode, pack_head_rows, pack_head_columns, pack_head_vector
 from .matrix_memory import MemoryDims, MemoryWeights, matrix_memory_rows, matrix_memory_decode
+from .state_space import SsmDims, SsmWeights, SsmDecodeBuffers, state_space_rows, state_space_decode
 from . import attention
 
 __all__ = [n for n in dir() if not n.startswith("_")]

@@ -1,6 +1,6 @@
-"""Grouped-query attention over a paged row cache on the kernels of ``csrc/kernels/gqa_attn.cu``: own key and value sizes, RMS norms on queries and keys (per head or
-over the whole projection), rotary positions on the first dimensions, an optional sliding window, an optional sink per head, values optionally mixed with an
-earlier layer's, an output gate (per element or per head) and a scale.
+"""Grouped-query attention over a paged row cache on the kernels of ``csrc/kernels/gqa_attn.cu``: own key and value sizes, optional RMS norms on queries and keys (per
+head or over the whole projection), rotary positions on the first dimensions (neighbouring pairs or halves), an optional sliding window beside which the first tokens
+may stay visible, an optional sink per head, values optionally mixed with an earlier layer's, an output gate (per element or per head) and a scale.
 
 Prompts of any ragged batch run a tcgen05 flash kernel that reads keys and values from the pages; a decode step streams the visible rows once for all heads of a
 group. f32 data takes a plain kernel.
@@ -16,6 +16,7 @@ from .. import _lib
 from .streams import padded_vector, round_up
 
 GATE_NONE, GATE_ELEMENT, GATE_HEAD = 0, 1, 2
+NORM_HEAD, NORM_WHOLE, NORM_NONE = 0, 1, 2
 SMALL_TOKENS = 16
 GROUP_ROWS = 128                     # query rows (tokens x heads of a group) of a flash sub-tile
 MAX_SPLITS = 64
@@ -23,7 +24,8 @@ MAX_SPLITS = 64
 
 @dataclass(frozen=True)
 class GqaDims:
-    """Sizes and constants of one attention layer. ``window`` 0: every earlier position is visible. Head sizes are padded to multiples of 16: projection rows
+    """Sizes and constants of one attention layer. ``window`` 0: every earlier position is visible; otherwise the last ``window`` and the first ``keep`` of them are.
+    ``halves``: dimension i turns with i + rot_dims / 2 instead of 2 i with 2 i + 1. ``norm``: whether queries and keys are normed. Head sizes are padded to multiples of 16: projection rows
     ``heads x d16 | kv_heads x d16 | kv_heads x v16``, cache rows ``kv_heads x d16 | kv_heads x v16``."""
     heads: int
     kv_heads: int
@@ -36,7 +38,12 @@ class GqaDims:
     whole_norm: bool = False
     gate: int = GATE_NONE
     out_scale: float = 1.0
+    keep: int = 0
+    halves: bool = False
+    norm: bool = True
 
+    @property
+    def norm_kind(self): return (NORM_WHOLE if self.whole_norm else NORM_HEAD) if self.norm else NORM_NONE
     @property
     def d16(self): return round_up(self.dim, 16)
     @property
@@ -83,15 +90,16 @@ def pack_head_vector(v: torch.Tensor, heads: int, size: int, device) -> torch.Te
 class GqaWeights:
     """Vectors of an attention layer (f32 on the device): query and key norm weights, ``sink`` ``[heads]``, ``mix`` (the weight of an earlier layer's values)."""
     dims: GqaDims
-    q_norm: torch.Tensor
-    k_norm: torch.Tensor
+    q_norm: Optional[torch.Tensor]
+    k_norm: Optional[torch.Tensor]
     sink: Optional[torch.Tensor] = None
     mix: Optional[torch.Tensor] = None
 
     @staticmethod
     def pack(dims: GqaDims, q_norm, k_norm, device, sink=None, mix=None) -> "GqaWeights":
         hq, hk = (dims.heads, dims.kv_heads) if dims.whole_norm else (1, 1)
-        return GqaWeights(dims, pack_head_vector(q_norm, hq, dims.dim, device), pack_head_vector(k_norm, hk, dims.dim, device),
+        qw, kw = (pack_head_vector(t, n, dims.dim, device) if dims.norm else None for t, n in ((q_norm, hq), (k_norm, hk)))
+        return GqaWeights(dims, qw, kw,
                           None if sink is None else padded_vector(sink, device), None if mix is None else mix.reshape(1).to(device, torch.float32))
 
 
@@ -102,10 +110,10 @@ def gqa_attention_rows(qkv: torch.Tensor, w: GqaWeights, batch, cache: torch.Ten
     ``w.mix``. ``batch`` holds the tables of :class:`~ferrotorch_b200.models.serving.RowBatch`, ``cache`` is this layer's page storage."""
     D, T, S = w.dims, qkv.shape[0], _lib.S()
     f32 = qkv.dtype == torch.float32
-    _lib.call("ft_gqa_prep", qkv, qkv.stride(0), T, D.heads, D.kv_heads, D.dim, D.vdim, D.rot_dims, int(D.whole_norm), w.q_norm, w.k_norm, D.eps, batch.positions, cos, sin,
-              batch.slots, cache, first_values, 0 if first_values is None else first_values.stride(0), None if first_values is None else w.mix, int(f32), S)
+    _lib.call("ft_gqa_prep", qkv, qkv.stride(0), T, D.heads, D.kv_heads, D.dim, D.vdim, D.rot_dims, D.norm_kind, int(D.halves), w.q_norm, w.k_norm, D.eps, batch.positions,
+              cos, sin, batch.slots, cache, first_values, 0 if first_values is None else first_values.stride(0), None if first_values is None else w.mix, int(f32), S)
     bt = batch.block_table
-    tail = (D.heads, D.kv_heads, D.dim, D.vdim, D.scale, D.window, w.sink, gate, 0 if gate is None else gate.stride(0), D.gate, D.out_scale, out, out.stride(0))
+    tail = (D.heads, D.kv_heads, D.dim, D.vdim, D.scale, D.window, D.keep, w.sink, gate, 0 if gate is None else gate.stride(0), D.gate, D.out_scale, out, out.stride(0))
     tile = 0 if f32 else D.flash_tile()
     if tile:
         tiles = batch.query_tiles(tile)
@@ -121,7 +129,7 @@ class GqaDecodeBuffers:
     def __init__(self, dims: GqaDims, max_batch: int, max_tokens: int, device, splits: Optional[int] = None):
         D = dims
         groups = D.kv_heads * -(-(D.heads // D.kv_heads) // 16)
-        span = min(max_tokens, D.window or max_tokens)
+        span = min(max_tokens, D.window + D.keep if D.window else max_tokens)
         # by batch size: two CTAs per SM, at least one 64-row chunk per split at the longest visible range
         self.splits = [splits or max(1, min(MAX_SPLITS, 296 // (b * groups), -(-span // 64))) for b in range(1, max_batch + 1)]
         self.q = torch.zeros(SMALL_TOKENS, D.heads, D.d16, device=device, dtype=torch.bfloat16)
@@ -136,7 +144,7 @@ def gqa_attention_decode(planes: torch.Tensor, splits: int, w: GqaWeights, b: Gq
     ``[16, out_cols]``. ``keep_values`` (f32 ``[16, kv_heads * v16]``) receives the values, ``first_values`` such values are mixed in."""
     D, S = w.dims, _lib.S()
     bt, mb = state.block_table, state.block_table.shape[1]
-    _lib.call("ft_gqa_decode_prep", planes, splits, planes.stride(1), planes.stride(0), B, D.heads, D.kv_heads, D.dim, D.vdim, D.rot_dims, int(D.whole_norm), w.q_norm, w.k_norm,
-              D.eps, state.positions, cos, sin, bt, mb, gate_col, D.gate, b.gate, keep_values, first_values, None if first_values is None else w.mix, b.q, cache, S)
-    _lib.call("ft_gqa_decode", b.q, cache, bt, mb, state.seq_lens, B, D.heads, D.kv_heads, D.dim, D.vdim, D.scale, D.window, w.sink, b.gate, D.gate, D.out_scale, b.splits[B - 1],
-              b.ws, b.counters, out, out.stride(0), S)
+    _lib.call("ft_gqa_decode_prep", planes, splits, planes.stride(1), planes.stride(0), B, D.heads, D.kv_heads, D.dim, D.vdim, D.rot_dims, D.norm_kind, int(D.halves),
+              w.q_norm, w.k_norm, D.eps, state.positions, cos, sin, bt, mb, gate_col, D.gate, b.gate, keep_values, first_values, None if first_values is None else w.mix, b.q, cache, S)
+    _lib.call("ft_gqa_decode", b.q, cache, bt, mb, state.seq_lens, B, D.heads, D.kv_heads, D.dim, D.vdim, D.scale, D.window, D.keep, w.sink, b.gate, D.gate, D.out_scale,
+              b.splits[B - 1], b.ws, b.counters, out, out.stride(0), S)

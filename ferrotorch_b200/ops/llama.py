@@ -64,7 +64,8 @@ def rope_inv_freq(head_dim: int, theta: float, scaling: dict | None = None, seq_
         def corr(n):
             return head_dim * math.log(orig / (n * 2 * math.pi)) / (2 * math.log(base))
         lo, hi = max(math.floor(corr(beta_fast)), 0), min(math.ceil(corr(beta_slow)), head_dim - 1)
-        ramp = ((torch.arange(half, dtype=torch.float64) - lo) / (hi - lo if hi != lo else 1e-3)).clamp(0, 1)
+        span = (hi - lo if hi != lo else 1e-3) if hf else max(hi - lo, 1e-3)
+        ramp = ((torch.arange(half, dtype=torch.float64) - lo) / span).clamp(0, 1)
         if hf or "attention_factor" in scaling:
             att = float(scaling.get("attention_factor") or (0.1 * math.log(factor) + 1.0 if factor > 1 else 1.0))
         return inv / factor * ramp + inv * (1 - ramp), att

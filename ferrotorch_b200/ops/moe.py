@@ -1,6 +1,6 @@
 """Mixture of experts on the kernels of ``csrc/kernels/moe.cu``: sigmoid router, the ``top`` best experts per token, experts of the clamped gated form
-``W_down (g sigmoid(slope g) (u + 1))`` with ``g = min(W_gate x, limit)`` and ``u = clamp(W_up x, -limit, limit)`` applied to ``score * x``, and an
-optional expert that every token passes through.
+``W_down (g sigmoid(slope g) (u + 1))`` with ``g = min(W_gate x, limit)`` and ``u = clamp(W_up x, -limit, limit)`` applied to ``score * x``, or of the form
+``score * W_down (silu(W_gate x) * (W_up x))``, and an optional expert that every token passes through. The choice goes by logit or by a :class:`RouteRule`.
 
 Prompts sort their (token, expert) pairs into 128-row segments and run grouped tcgen05 GEMMs; a decode step (up to 16 tokens in bf16) streams the
 weights of the experts in use through ``mma.sync`` with all tokens in shared memory.
@@ -84,6 +84,19 @@ class ExpertStack:
 
 
 @dataclass
+class RouteRule:
+    """Experts are chosen by ``sigmoid(logit) + correction``, within the ``keep`` best of ``groups`` equal groups of neighbours (0: no groups; a group's score is the sum of
+    its two best), and weighted with the chosen sigmoids divided by their sum, times ``scale``. ``correction``: f32 ``[experts]`` on the device."""
+    correction: torch.Tensor
+    groups: int = 0
+    keep: int = 0
+    scale: float = 1.0
+
+
+EXPERT_FORMS = {"clamped": 0, "silu": 1}
+
+
+@dataclass
 class MoeWeights:
     router: torch.Tensor                     # [experts, width] view with a pitch that is a multiple of 8
     experts: ExpertStack
@@ -91,6 +104,17 @@ class MoeWeights:
     width: int
     top: int
     slope: float = 1.702
+    form: str = "clamped"
+    rule: Optional[RouteRule] = None
+
+    @property
+    def kind(self) -> int:
+        return EXPERT_FORMS[self.form]
+
+    @property
+    def rule_args(self) -> tuple:
+        r = self.rule
+        return (r.correction, r.groups, r.keep, r.scale) if r else (None, 0, 0, 1.0)
 
     @property
     def num_experts(self) -> int:
@@ -125,7 +149,7 @@ class MoeSmallBuffers:
 
         def ints(*s):
             return torch.zeros(*s, device=device, dtype=torch.int32)
-        return MoeSmallBuffers(torch.zeros(SMALL_TOKENS * E, device=device), ints(1), ints(1), ints(E), ints(E), ints(E * SMALL_TOKENS), ints(E * SMALL_TOKENS),
+        return MoeSmallBuffers(torch.zeros(2 * SMALL_TOKENS * E, device=device), ints(1), ints(1), ints(E), ints(E), ints(E * SMALL_TOKENS), ints(E * SMALL_TOKENS),
                                torch.zeros(SMALL_TOKENS * top, device=device), torch.zeros(SMALL_TOKENS * top, round_up(f, 8), device=device, dtype=torch.bfloat16),
                                torch.zeros(SMALL_TOKENS, round_up(fs, 8), device=device, dtype=torch.bfloat16),
                                torch.zeros(top + 1, SMALL_TOKENS, round_up(width, 8), device=device))
@@ -135,18 +159,20 @@ def moe_small(h: torch.Tensor, w: MoeWeights, b: MoeSmallBuffers, tokens: int) -
     """Decode step: ``tokens`` (<= 16) bf16 rows of ``h``. The result's planes live in ``b`` until the next call."""
     E, x, s, S = w.num_experts, w.experts, w.shared, _lib.S()
     route = (b.n_active, b.ids, b.cnt, b.pair, b.pair_of, b.score)
-    _lib.call("ft_moe_route_small", h, h.stride(0), w.router, w.router.stride(0), tokens, w.width, E, w.top, b.logits, b.counter, *route, S)
+    _lib.call("ft_moe_route_small", h, h.stride(0), w.router, w.router.stride(0), tokens, w.width, E, w.top, *w.rule_args, b.logits, b.counter,
+              *route, S)
     _lib.call("ft_moe_gate_up_small", h, h.stride(0), tokens, w.width, E, w.top, *route, x.gu, x.ff, x.gu.stride(1), x.limit, s.gu if s else None, s.ff if s else 0,
-              s.gu.stride(1) if s else 0, s.limit if s else 0.0, w.slope, b.act, b.act.stride(0), b.act_sh, b.act_sh.stride(0), S)
+              s.gu.stride(1) if s else 0, s.limit if s else 0.0, w.kind, w.slope, b.act, b.act.stride(0), b.act_sh, b.act_sh.stride(0), S)
     _lib.call("ft_moe_down_small", b.act, b.act.stride(0), b.act_sh, b.act_sh.stride(0), tokens, w.width, E, w.top, *route, x.down, x.ff, x.down.stride(1),
               s.down if s else None, s.ff if s else 0, s.down.stride(1) if s else 0, x.down.shape[1], b.planes, b.planes.stride(0), b.planes.stride(1), S)
     return SublayerOutput(planes=b.planes, count=w.top + (1 if s else 0))
 
 
-def gated_act(gu: torch.Tensor, fp: int, limit: float, slope: float, row_score: Optional[torch.Tensor] = None, rows_used: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """Activation of interleaved gate / up columns ``[rows, 2 * fp]`` -> ``[rows, fp]``, both scaled by ``row_score`` first."""
+def gated_act(gu: torch.Tensor, fp: int, limit: float, slope: float, row_score: Optional[torch.Tensor] = None, rows_used: Optional[torch.Tensor] = None,
+              form: str = "clamped") -> torch.Tensor:
+    """Activation of interleaved gate / up columns ``[rows, 2 * fp]`` -> ``[rows, fp]``; clamped: both scaled by ``row_score`` first, silu: the result is."""
     act = torch.empty(gu.shape[0], fp, device=gu.device, dtype=gu.dtype)
-    _lib.call("ft_moe_act", gu, gu.stride(0), row_score, rows_used, gu.shape[0], fp, limit, slope, act, act.stride(0), int(gu.dtype == torch.float32), _lib.S())
+    _lib.call("ft_moe_act", gu, gu.stride(0), row_score, rows_used, gu.shape[0], fp, EXPERT_FORMS[form], limit, slope, act, act.stride(0), int(gu.dtype == torch.float32), _lib.S())
     return act
 
 
@@ -169,7 +195,7 @@ class MoeRouting:
         expert, pos, start, group, used = torch.split(ints, [T * w.top, T * w.top, E, tiles, 1])
         score = torch.empty(T * w.top, device=dev, dtype=torch.float32)
         count = torch.zeros(E, device=dev, dtype=torch.int32)
-        _lib.call("ft_moe_topk", logits, logits.stride(0), T, E, w.top, expert, score, pos, count, _lib.S())
+        _lib.call("ft_moe_topk", logits, logits.stride(0), T, E, w.top, *w.rule_args, expert, score, pos, count, _lib.S())
         _lib.call("ft_moe_layout", count, E, tiles, start, group, used, _lib.S())
         return MoeRouting(expert, score, pos, start, group, used)
 
@@ -186,12 +212,12 @@ def moe_rows(h: torch.Tensor, w: MoeWeights) -> SublayerOutput:
     _lib.call("ft_moe_gather", h, ld * es, r.expert, r.score, r.pos, r.start, T, w.top, round_up(w.width, 8) * es, xs, ld * es, row_of, row_score, _lib.S())
     gu = torch.empty(rows, 2 * x.fp, device=h.device, dtype=h.dtype)
     grouped_linear(xs, x.gu, r.tile_group, 2 * x.fp, w.width, gu)
-    act = gated_act(gu, x.fp, x.limit, w.slope, row_score, r.rows_used)
+    act = gated_act(gu, x.fp, x.limit, w.slope, row_score, r.rows_used, w.form)
     out = torch.empty(rows, round_up(w.width, 8), device=h.device, dtype=h.dtype)
     grouped_linear(act, x.down, r.tile_group, w.width, x.ff, out)
     planes = None
     if s is not None:
         sgu = linear_rows(h, s.gu[0][:, : w.width])
-        planes = linear_rows(gated_act(sgu, s.fp, s.limit, w.slope)[:, : s.ff], s.down[0][: w.width, : s.ff], out_f32=True)
+        planes = linear_rows(gated_act(sgu, s.fp, s.limit, w.slope, form=w.form)[:, : s.ff], s.down[0][: w.width, : s.ff], out_f32=True)
         planes = planes.as_strided((1, T, w.width), (0, planes.stride(0), 1))
     return SublayerOutput(planes=planes, rows=out, row_of=row_of, top=w.top)

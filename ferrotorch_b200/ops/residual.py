@@ -1,5 +1,5 @@
-"""One f32 residual per token with the RMS norm on every sublayer's output (``x <- x + norm(f(x))``), and the activation of a dense gated feed-forward, on the
-fused kernels of ``csrc/kernels/residual_ops.cu``.
+"""One f32 residual per token, with the RMS norm on every sublayer's output (``x <- x + norm(f(x))``) or ahead of two sublayers side by side
+(``x <- x + m (f(norm1(x)) + g(norm2(x)))``), and the activation of a dense gated feed-forward, on the fused kernels of ``csrc/kernels/residual_ops.cu``.
 
 Between two projections there is one kernel: it sums the sublayer's partial results, norms them, adds them to the residual and leaves the next projection's
 operand (the residual itself, or its norm ahead of the output projection).
@@ -13,7 +13,7 @@ import torch
 
 from .. import _lib
 from .moe import interleave_gate_up, linear_rows
-from .streams import SublayerOutput, round_up
+from .streams import SublayerOutput, padded_vector, round_up
 
 GATED_ACTS = {"gelu_tanh": 0, "silu": 1}
 
@@ -32,41 +32,67 @@ def residual_update(x: torch.Tensor, y: SublayerOutput, w: torch.Tensor, eps: fl
     _lib.call("ft_residual_update", x, x.stride(0), p, n, p.stride(0), p.stride(1), w, last, eps, h, h.stride(0), int(h.dtype == torch.float32), rows, width, int(store), _lib.S())
 
 
+def parallel_embed(ids: torch.Tensor, table: torch.Tensor, w1: torch.Tensor, w2: Optional[torch.Tensor], eps: float, x: torch.Tensor, h1: torch.Tensor,
+                   h2: Optional[torch.Tensor], rows: int) -> None:
+    """``x = table[ids]`` (f32) and the operands of the first layer's two sublayers: ``h1 = norm(x) * w1``, ``h2 = norm(x) * w2`` (``w2`` ``None``: the first alone)."""
+    _lib.call("ft_parallel_embed", ids, table, table.stride(0), table.shape[0], w1, w2, eps, x, x.stride(0), h1, h2, h1.stride(0), int(h1.dtype == torch.float32), rows,
+              table.shape[1], _lib.S())
+
+
+def parallel_update(x: torch.Tensor, mult: float, a: Optional[SublayerOutput], b: Optional[SublayerOutput], w1: torch.Tensor, w2: Optional[torch.Tensor], eps: float,
+                    h1: torch.Tensor, h2: Optional[torch.Tensor], rows: int, width: int, store: bool = True) -> None:
+    """``x += mult * (a + b)`` for what two sublayers of the same ``x`` returned, then the next operands as in :func:`parallel_embed`. ``a`` has planes alone; ``b`` planes,
+    expert rows and a bias."""
+    def planes(y):
+        p = None if y is None else y.planes
+        return (None, 0, 0, 0) if p is None else (p, y.count if y.count is not None else p.shape[0], p.stride(0), p.stride(1))
+    r = None if b is None else b.rows
+    _lib.call("ft_parallel_update", x, x.stride(0), mult, *planes(a), *planes(b), r, None if r is None else b.row_of, 0 if r is None else b.top, 0 if r is None else r.stride(0),
+              None if b is None else b.bias, w1, w2, eps, h1, h2, h1.stride(0), int(h1.dtype == torch.float32), rows, width, int(store), _lib.S())
+
+
 @dataclass
 class DenseGatedWeights:
-    """``down(act(gate x) * up x)``: ``gu`` ``[2 * fp, width]`` (gate and up rows interleaved in eights), ``down`` ``[width, ff]``, both with padded pitches."""
+    """``down(act(gate x) * up x)``: ``gu`` ``[2 * fp, width]`` (gate and up rows interleaved in eights), ``down`` ``[width, ff]``, both with padded pitches; biases (f32),
+    if any: ``gu_bias`` in the order of the rows of ``gu``, ``down_bias`` (added by the residual update)."""
     gu: torch.Tensor
     down: torch.Tensor
     act: str = "gelu_tanh"
+    gu_bias: Optional[torch.Tensor] = None
+    down_bias: Optional[torch.Tensor] = None
 
     @property
     def fp(self) -> int:
         return self.gu.shape[0] // 2
 
     @staticmethod
-    def pack(gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor, device, dtype, act: str = "gelu_tanh") -> "DenseGatedWeights":
+    def pack(gate: torch.Tensor, up: torch.Tensor, down: torch.Tensor, device, dtype, act: str = "gelu_tanh", gate_bias=None, up_bias=None, down_bias=None) -> "DenseGatedWeights":
         f, width = gate.shape
         gu = interleave_gate_up(gate.to(device, dtype), up.to(device, dtype), round_up(width, 32))
         d = torch.zeros(width, round_up(f, 32), device=device, dtype=dtype)
         d[:, :f] = down.to(device, dtype)
-        return DenseGatedWeights(gu[:, :width], d[:, :f], act)
+        gb = db = None
+        if gate_bias is not None:
+            gb = interleave_gate_up(*(t.reshape(-1, 1).to(device, torch.float32) for t in (gate_bias, up_bias)), 1).flatten().contiguous()
+            db = padded_vector(down_bias, device)
+        return DenseGatedWeights(gu[:, :width], d[:, :f], act, gb, db)
 
 
-def gated_act_rows(gu: torch.Tensor, fp: int, act: str) -> torch.Tensor:
-    """Activation of interleaved gate / up columns ``[rows, 2 * fp]`` -> ``[rows, fp]``."""
+def gated_act_rows(gu: torch.Tensor, fp: int, act: str, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Activation of interleaved gate / up columns ``[rows, 2 * fp]`` -> ``[rows, fp]``; ``bias`` in the order of the columns."""
     out = torch.empty(gu.shape[0], fp, device=gu.device, dtype=gu.dtype)
-    _lib.call("ft_gated_act", gu, gu.stride(0), gu.shape[0], fp, GATED_ACTS[act], out, out.stride(0), int(gu.dtype == torch.float32), _lib.S())
+    _lib.call("ft_gated_act", gu, gu.stride(0), bias, gu.shape[0], fp, GATED_ACTS[act], out, out.stride(0), int(gu.dtype == torch.float32), _lib.S())
     return out
 
 
-def gated_act_planes(planes: torch.Tensor, splits: int, rows: int, fp: int, act: str, out: torch.Tensor) -> torch.Tensor:
+def gated_act_planes(planes: torch.Tensor, splits: int, rows: int, fp: int, act: str, out: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """The same from split-K planes of the projection of a few tokens, to bf16 rows."""
-    _lib.call("ft_gated_act_planes", planes, splits, planes.stride(1), planes.stride(0), rows, fp, GATED_ACTS[act], out, out.stride(0), _lib.S())
+    _lib.call("ft_gated_act_planes", planes, splits, planes.stride(1), planes.stride(0), bias, rows, fp, GATED_ACTS[act], out, out.stride(0), _lib.S())
     return out
 
 
 def dense_gated_rows(h: torch.Tensor, w: DenseGatedWeights) -> SublayerOutput:
     """Any number of token rows (bf16 or f32)."""
-    a = gated_act_rows(linear_rows(h, w.gu), w.fp, w.act)
+    a = gated_act_rows(linear_rows(h, w.gu), w.fp, w.act, w.gu_bias)
     y = linear_rows(a[:, : w.down.shape[1]], w.down, out_f32=True)
-    return SublayerOutput(planes=y.as_strided((1, y.shape[0], y.shape[1]), (0, y.stride(0), 1)))
+    return SublayerOutput(planes=y.as_strided((1, y.shape[0], y.shape[1]), (0, y.stride(0), 1)), bias=w.down_bias)

@@ -57,12 +57,13 @@ class HyperWeights:
 @dataclass
 class SublayerOutput:
     """What a sublayer hands to the stream update: f32 ``planes`` ``[count, rows, ld]`` to be summed, and / or ``rows`` of expert output with the
-    index ``row_of`` ``[tokens, top]`` of the rows that belong to each token."""
+    index ``row_of`` ``[tokens, top]`` of the rows that belong to each token, and / or a ``bias``."""
     planes: Optional[torch.Tensor] = None
     rows: Optional[torch.Tensor] = None
     row_of: Optional[torch.Tensor] = None
     top: int = 0
     count: Optional[int] = None          # planes in use when fewer than allocated
+    bias: Optional[torch.Tensor] = None  # f32 vector added to every row
 
 
 def dynamic_tanh(x: torch.Tensor, weights: DynamicTanhWeights, out: Optional[torch.Tensor] = None) -> torch.Tensor:
