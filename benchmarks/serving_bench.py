@@ -1,5 +1,6 @@
-"""Prefill and decode throughput of the serving models on layers of realistic size with random weights: the Ginisun and Pufevik decoders beside a Llama decoder
-of the same width and the same number of feed-forward neurons per token (Pufevik also has its attention sizes; its layers alternate between the two kinds). Run through ``bench.py --serving``.
+"""Prefill and decode throughput of the serving models on layers of realistic size with random weights: the Ginisun, Pufevik and Mepupel decoders beside a Llama decoder
+of the same width and the same number of feed-forward neurons per token (Pufevik also has its attention sizes; its layers alternate between the two kinds; Mepupel has Ginisun's experts,
+and one layer of each kind in turn). Run through ``bench.py --serving``.
 
 Every kernel class is also timed (CUDA events around its launches, L2 flushed by the step's own traffic) against its roofline, the slower of algorithmic
 bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate. Times of single launches below ~5 us are dominated by launch overhead.
@@ -15,6 +16,8 @@ import torch
 from ferrotorch_b200 import _lib
 from ferrotorch_b200.models import GenerationConfig, LlamaConfig
 from ferrotorch_b200.models.ginisun import GinisunConfig, GinisunModel, RandomGinisunWeights
+from ferrotorch_b200.models.ginisun import ExpertConfig, MoeConfig
+from ferrotorch_b200.models.mepupel import MepupelConfig, MepupelModel, RandomMepupelWeights
 from ferrotorch_b200.models.pufevik import PufevikConfig, PufevikModel, RandomPufevikWeights
 from ferrotorch_b200.models.llama_infer import LlamaTPEngine, TPContext
 from ferrotorch_b200.models.serving import ServingEngine, StepEntry
@@ -28,6 +31,11 @@ PUFEVIK = {                          # matrix memory beside the attention, windo
     "1k": dict(memory_heads=4, memory_dim=128, memory_vdim=256, window=1024),
     "2k": dict(memory_heads=4, memory_dim=256, memory_vdim=512, window=1024),
     "4k": dict(memory_heads=8, memory_dim=256, memory_vdim=512, window=1024),
+}
+MEPUPEL = {                          # state space, groups of experts, latents
+    "1k": dict(ssm=dict(heads=32, vdim=64, state=128, groups=1, norm_groups=1, conv=4), groups=4, keep=2, q_rank=512, kv_rank=256),
+    "2k": dict(ssm=dict(heads=64, vdim=64, state=128, groups=8, norm_groups=8, conv=4), groups=8, keep=4, q_rank=1024, kv_rank=512),
+    "4k": dict(ssm=dict(heads=128, vdim=64, state=128, groups=8, norm_groups=8, conv=4), groups=4, keep=2, q_rank=1536, kv_rank=512),
 }
 VOCAB = 32768
 
@@ -248,6 +256,97 @@ def run_pufevik(size, layers, batch, prompt, ctx, steps, kernels=True):
             "decode_tokens_per_s": round(batch / dec_ms * 1e3), "prefill_kernels": table, "decode_kernels": dtable}
 
 
+def run_mepupel(size, layers, batch, prompt, ctx, steps, kernels=True):
+    """Layers in turn: state space, windowed attention, latent attention, latent attention on the latent before it; experts in every layer."""
+    from ferrotorch_b200.models.serving import RowBatch
+    bw, fl, _ = peaks()
+    s, e = SIZES[size], MEPUPEL[size]
+    W, T, F, SF, E, top = s["width"], prompt, s["ff"], s["shared_ff"], s["experts"], s["top"]
+    H = W // 128
+    G = max(1, H // 4)
+    att = dict(heads=H, kv_heads=G, dim=128, vdim=128, scale=128 ** -0.5, rot=dict(base=1e4, dims=64, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0)),
+               mask=dict(size=1024, keep_first=64))
+    lat = dict(heads=H, dim=128, vdim=128, q_rank=e["q_rank"], kv_rank=e["kv_rank"], scale=128 ** -0.5)
+    cfg = MepupelConfig.pattern(("mals" * layers)[:layers], VOCAB, W, e["ssm"], att, lat,
+                                MoeConfig(E, top, ExpertConfig(F), ExpertConfig(SF), e["groups"], e["keep"], 2.0), residual_mult=0.5)
+    eng = ServingEngine(MepupelModel(cfg, RandomMepupelWeights(cfg)), max_tokens=max(batch * (ctx + steps * 4 + 64), prompt + 64), max_sequences=batch + 1)
+    g = torch.Generator().manual_seed(1)
+    ids = torch.randint(0, VOCAB, (prompt,), generator=g).tolist()
+    entry = [StepEntry("p", ids, [prompt - 1])]
+    eng._admit(entry)
+    rb = RowBatch(entry, eng.cache, eng.device, eng.max_blocks)
+    device_prefill = lambda: eng.model.forward_rows(rb, eng.cache)          # the device part: tables of the batch are built once
+    pre_ms = timed(device_prefill)
+    by = {k: next((l for l in eng.model.layers if getattr(l, k)), None) for k in ("ssm", "attn", "latent")}
+    S, A, L = (by[k].mixer.dims if by[k] else None for k in ("ssm", "attn", "latent"))
+    table = dtable = None
+    def g_(n, k, out=2, m=T): return (2 * (m * k + n * k) + out * m * n, 2 * m * n * k)
+    pairs, nkv = T * top, H * (L.dim8 + L.v8)
+    common = {(S.main, W): "projection gemm (state space)", (by["attn"].proj.shape[0], W): "projection gemm (attention)", (L.proj_cols, W): "projection gemm (latent)",
+              (L.q_cols, W): "projection gemm (latent, shared)", (H * L.dim8, L.q_rank): "query expansion gemm", (W, S.out_cols): "output gemm (state space)",
+              (2 * SF, W): "shared gate/up gemm", ("grouped", 2 * F, W): "experts gate/up gemm", ("grouped", W, F): "experts down gemm"}
+    if kernels:
+        names = dict(common)
+        names.update({(S.h8, W): "step size gemm", (nkv, L.rank): "key/value expansion gemm", (E, W): "router gemm"})
+        for shape, label in (((W, A.out_cols), "output gemm (attention)"), ((W, SF), "shared down gemm")):
+            names[shape] = "output gemms and shared down gemm" if SF in (A.out_cols, S.out_cols) and shape[1] == SF else label      # one shape: one label
+        classify = _by_shape(names)
+        win, keep = A.window, A.keep
+        seen = win * T - win * (win - 1) // 2 + keep * max(0, T - win) if win < T else T * (T + 1) // 2
+        N = S.n16
+        roofs = {names[k]: g_(k[0], k[1], 4 if "output" in names[k] or "down" in names[k] or "step" in names[k] or "router" in names[k] else 2) for k in names if k[0] != "grouped"}
+        roofs.update({
+            "experts gate/up gemm": (2 * (pairs * W + E * 2 * F * W + pairs * 2 * F), 4 * pairs * F * W), "experts down gemm": (2 * (pairs * W + E * F * W + pairs * F), 2 * pairs * F * W),
+            "ft_gqa_flash": (2 * T * (A.qkv_cols + A.out_cols), 4 * H * seen * 128), "ft_gqa_prep": (4 * T * (H * A.rot_dims + A.qkv_cols - A.k_col), 0),
+            "ft_latent_flash": (2 * T * (H * L.dim8 + nkv + H * L.v8), H * T * T * (L.dim + L.vdim)), "ft_latent_prep": (2 * T * (2 * L.q_rank + L.rank + 2 * L.row), 0),
+            "ft_moe_gather": (4 * pairs * W, 0), "ft_moe_act": ((pairs * F * 6 + T * SF * 6) / 2, 0), "ft_moe_topk": (T * E * 4, 0),
+            "ft_parallel_update": (T * W * (8 + 4 + 4 + 2 * top + 4), 0), "ft_ssm_conv": (4 * T * S.channels, 0), "ft_ssm_finish": (6 * T * S.out_cols, 0),
+            "state walk (outputs)": (2 * T * (S.channels + S.out_cols), 2 * T * S.heads * (2 * N * S.v16 + 32 * (N + S.v16))),
+            "state walk (states)": (2 * T * (S.channels - S.groups * N), 2 * T * S.heads * N * S.v16)})
+        def label(fn, raw):
+            if fn == "ft_ssm_walk":
+                return "state walk (outputs)" if raw[17] else "state walk (states)"
+            return classify(fn, raw)
+        table = kernel_table(device_prefill, label, roofs, bw, fl)
+    eng.release("p")
+    seqs = [f"s{i}" for i in range(batch)]
+    for q in seqs:
+        eng.step([StepEntry(q, torch.randint(0, VOCAB, (ctx,), generator=g).tolist(), [])])
+    eng.decode_greedy(seqs, [1] * batch, 4)
+    best = []
+    for _ in range(3):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        eng.decode_greedy(seqs, [1] * batch, steps)
+        e1.record()
+        torch.cuda.synchronize()
+        best.append(e0.elapsed_time(e1) / steps)
+    dec_ms = statistics.median(best)
+    active = None
+    if kernels:
+        for q in seqs:
+            eng.cache.reserve(q, eng.cache.lengths[q] + 1)
+        eng._load_state(seqs, [1 + i for i in range(batch)])
+        positions, lens, tokens = eng.state.positions.clone(), eng.state.seq_lens.clone(), eng.state.tokens.clone()
+        def one():
+            eng.state.positions.copy_(positions); eng.state.seq_lens.copy_(lens); eng.state.tokens.copy_(tokens)
+            eng.model.decode(eng.state, batch, eng.cache)
+        one()
+        active = int(eng.model._moe_buffers.n_active)               # experts in use (of the last layer; the layers are alike)
+        n = eng.cache.lengths[seqs[0]] + 1
+        names = dict(common)
+        names.update({(S.main + S.h8, W): "projection gemm (state space)", (W, A.out_cols): "output gemm (attention)", (VOCAB, W): "head gemm"})
+        roofs = {names[k]: (2 * k[0] * k[1], 0) for k in names if k[0] != "grouped"}
+        roofs.update({"ft_gqa_decode": (2 * batch * min(n, A.window + A.keep) * A.row, 0), "ft_latent_decode": (2 * batch * n * L.row, 2 * batch * H * n * (L.row + L.r16)),
+                      "ft_latent_decode_prep": (2 * H * L.dim8 * L.rank, 0), "ft_skinny_heads": (2 * H * L.v8 * L.rank, 0), "ft_ssm_decode": (8 * batch * S.state_size, 0),
+                      "ft_moe_gate_up_small": (4 * W * (active * F + SF), 0), "ft_moe_down_small": (2 * W * (active * F + SF), 0), "ft_parallel_update": (batch * W * (12 + 4 * (top + 1) + 16), 0)})
+        dtable = kernel_table(one, _by_shape(names), roofs, bw, fl)
+    eng.check()
+    return {"prefill_ms": round(pre_ms, 3), "prefill_tokens_per_s": round(prompt / pre_ms * 1e3), "decode_ms_per_step": round(dec_ms, 4), "decode_tokens_per_s": round(batch / dec_ms * 1e3),
+            "active_experts": active, "prefill_kernels": table, "decode_kernels": dtable}
+
+
 def run_llama(size, layers, batch, prompt, ctx, steps, kernels=True):
     bw, fl, _ = peaks()
     s = SIZES[size]
@@ -306,7 +405,7 @@ def main(sizes="1k,2k,4k", layers=4, batch=8, prompt=4096, ctx=2048, steps=64, k
     res = {}
     for size in sizes.split(","):
         res[size] = {}
-        for name, run in (("ginisun", run_ginisun), ("pufevik", run_pufevik), ("llama", run_llama)):
+        for name, run in (("ginisun", run_ginisun), ("pufevik", run_pufevik), ("mepupel", run_mepupel), ("llama", run_llama)):
             if models and name not in models.split(","):
                 continue
             res[size][name] = run(size, layers, batch, prompt, ctx, steps, kernels)

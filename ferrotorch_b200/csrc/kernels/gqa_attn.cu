@@ -158,6 +158,32 @@ __global__ void __launch_bounds__(PREP_T) gqa_prep_kernel(T* __restrict__ qkv, i
         finish(i / hv, i % hv, i < nq, x, i < nq ? rq : rk);
       }
     }
+  } else if (!normed && A.halves && (half & 7) == 0) {
+    const int hw = half / 8, tail = hv - 2 * hw;     // nothing to reduce: pairs of vectors of all heads in a row, then the keys' columns behind the rotated ones
+    for (int i = threadIdx.x; i < (D.H + D.G) * hw; i += PREP_T) {
+      const int head = i / hw, vi = i % hw;
+      const T* src = row + head * D.d16 + vi * 8;
+      T* to = head < D.H ? row + head * D.d16 + vi * 8 : dst + (head - D.H) * D.d16 + vi * 8;
+      float a[8], b[8], c[8], s[8];
+      load8(src, a);
+      load8(src + half, b);
+      load8(ct + vi * 8, c);
+      load8(st + vi * 8, s);
+#pragma unroll
+      for (int e = 0; e < 8; e++) {
+        const float u = a[e];
+        a[e] = u * c[e] - b[e] * s[e];
+        b[e] = b[e] * c[e] + u * s[e];
+      }
+      store8(to, a);
+      store8(to + half, b);
+    }
+    for (int i = threadIdx.x; i < D.G * tail; i += PREP_T) {
+      const int at = i / tail * D.d16 + (2 * hw + i % tail) * 8;
+      float a[8];
+      load8(row + D.H * D.d16 + at, a);
+      store8(dst + at, a);
+    }
   } else {
     int lanes = 1;                                   // lanes of a head: a power of two that covers its columns, at most a warp
     while (lanes < hv && lanes < 32) lanes *= 2;

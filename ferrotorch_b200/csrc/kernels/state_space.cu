@@ -60,7 +60,7 @@ template <> FT_DEVICE void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (
 // convolution: grid (channel blocks, row blocks), 128 threads, eight channels a thread. spans int4[sequence] {first row, rows, slot, 1 if the sequence starts}. TAPS: number
 // of taps with the window of earlier inputs in registers, or 0 to read it again for every row.
 // ------------------------------------------------------------------------------------------------------------
-constexpr int CONV_ROWS = 16;
+constexpr int CONV_ROWS = 8;
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(128) ssm_conv_kernel(const T* __restrict__ x, int64_t ld, int rows, const int* __restrict__ seq_of, const int4* __restrict__ spans,
                                                        const float* __restrict__ w, const float* __restrict__ bias, const float* __restrict__ slots, size_t slot_stride, SsmDims D,
@@ -86,6 +86,37 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const T* __restrict__ x, 
     float wt[TAPS][8], win[TAPS][8];
 #pragma unroll
     for (int k = 0; k < TAPS; k++) load8(w + (size_t)k * cc + c, wt[k]);
+    auto tap = [&](T* dst) {
+      float a[8];
+#pragma unroll
+      for (int e = 0; e < 8; e++) {
+        float t = b[e];
+#pragma unroll
+        for (int k = 0; k < TAPS; k++) t += wt[k][e] * win[k][e];
+        a[e] = silu_for<T>(t);
+      }
+      store8(dst, a);
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; k++)
+#pragma unroll
+        for (int e = 0; e < 8; e++) win[k][e] = win[k + 1][e];
+    };
+    const int first = seq_of[r0];
+    if (r1 - r0 == CONV_ROWS && seq_of[r1 - 1] == first) {      // rows of one sequence: all of them on their way at once
+      const int4 sp = spans[first];
+      uint4 raw[CONV_ROWS];
+      static_assert(sizeof(T) == 2, "eight channels in 16 bytes");
+#pragma unroll
+      for (int j = 0; j < CONV_ROWS; j++) raw[j] = *reinterpret_cast<const uint4*>(x + (size_t)(r0 + j) * ld + c);
+#pragma unroll
+      for (int k = 0; k < TAPS - 1; k++) input(sp, r0, TAPS - 1 - k, win[k]);
+#pragma unroll
+      for (int j = 0; j < CONV_ROWS; j++) {
+        bf16x8_to_float(*reinterpret_cast<const bf16x8*>(&raw[j]), win[TAPS - 1]);
+        tap(out + (size_t)(r0 + j) * cc + c);
+      }
+      return;
+    }
     int cur = -1;
     for (int r = r0; r < r1; r++) {
       const int s = seq_of[r];
@@ -96,19 +127,7 @@ __global__ void __launch_bounds__(128) ssm_conv_kernel(const T* __restrict__ x, 
         cur = s;
       }
       load8(x + (size_t)r * ld + c, win[TAPS - 1]);
-      float a[8];
-#pragma unroll
-      for (int e = 0; e < 8; e++) {
-        float t = b[e];
-#pragma unroll
-        for (int k = 0; k < TAPS; k++) t += wt[k][e] * win[k][e];
-        a[e] = silu_for<T>(t);
-      }
-      store8(out + (size_t)r * cc + c, a);
-#pragma unroll
-      for (int k = 0; k < TAPS - 1; k++)
-#pragma unroll
-        for (int e = 0; e < 8; e++) win[k][e] = win[k + 1][e];
+      tap(out + (size_t)r * cc + c);
     }
   } else {
     for (int r = r0; r < r1; r++) {

@@ -187,16 +187,17 @@ class MepupelConfig:
                     raise InvalidArgument(f"{where}: experts have no limit")
 
     @staticmethod
-    def pattern(kinds: str, vocab: int, width: int, ssm: dict, attention: dict, latent: dict, mlp: Union[DenseConfig, MoeConfig, None], residual_mult: float = 1.0,
-                eps: float = 1e-5) -> "MepupelConfig":
+    def pattern(kinds: str, vocab: int, width: int, ssm: dict, attention: dict, latent: dict, mlp: Union[DenseConfig, MoeConfig, None], first_ff: int = 0,
+                residual_mult: float = 1.0, eps: float = 1e-5) -> "MepupelConfig":
         """Layers by letter: ``m`` (state space), ``a`` (attention), ``l`` (latent attention), ``s`` (latent attention on the latent of the ``l`` before it), each kind with the
-        sizes of its dictionary (as in ``config.json``) and all with the same feed-forward."""
+        sizes of its dictionary (as in ``config.json``) and all with the same feed-forward, but for a dense one of ``first_ff`` neurons in the first layer."""
         layers = []
         for i, k in enumerate(kinds):
+            f = DenseConfig(first_ff) if first_ff and i == 0 else mlp
             if k in "ls":
-                layers.append(MepupelLayer(LatentConfig(**latent, kv_from=kinds.rindex("l", 0, i) if k == "s" else None), mlp))
+                layers.append(MepupelLayer(LatentConfig(**latent, kv_from=kinds.rindex("l", 0, i) if k == "s" else None), f))
             else:
-                layers.append(MepupelLayer(Mamba2Config(**ssm) if k == "m" else AttentionConfig.from_dict(attention), mlp))
+                layers.append(MepupelLayer(Mamba2Config(**ssm) if k == "m" else AttentionConfig.from_dict(attention), f))
         c = MepupelConfig(vocab, width, eps, residual_mult, layers)
         c.validate()
         return c
