@@ -103,7 +103,17 @@ FT_EXPORT int ft_status_read_clear(uint32_t* out) {
 FT_EXPORT int ft_abi_version() { return 1; }
 
 static bool g_pdl = false;
-bool ft_pdl_enabled() { return g_pdl; }
+static bool g_pdl_break = false;
+bool ft_pdl_enabled() {
+  const bool on = g_pdl && !g_pdl_break;
+  g_pdl_break = false;
+  return on;
+}
+// The next launch that asks is an ordinary one: for the first kernel behind an event of another stream, which has to wait for all it depends on.
+FT_EXPORT int ft_pdl_break() {
+  g_pdl_break = true;
+  return 0;
+}
 // Switch programmatic dependent launch on or off for the kernels that support it (the decode path). Returns the previous setting.
 FT_EXPORT int ft_set_pdl(int enabled) {
   const int prev = g_pdl ? 1 : 0;

@@ -435,6 +435,7 @@ class MepupelModel:
                 l.g_expand = _SplitKGemm(l.latent.uq, dev, planes.setdefault("expand", {}))
             if l.dense:
                 l.g_gu, l.g_down = _SplitKGemm(l.dense.gu, dev, planes.setdefault("gate", {})), _SplitKGemm(l.dense.down, dev, planes.setdefault("feed-forward", {}))
+        self._side = torch.cuda.Stream(dev)
         self._g_head = _SplitKGemm(self.head, dev)
         moes = [l.moe for l in self.layers if l.moe]
         self._moe_buffers = MoeSmallBuffers.allocate(moes, dev) if moes else None
@@ -472,9 +473,19 @@ class MepupelModel:
         """One token for the first ``B`` sequences of ``state``; returns the logits buffer ``[16, vocab]`` (rows below ``B`` are valid)."""
         cfg, W, x, h1, h2 = self.cfg, self.cfg.width, self._x, self._h1, self._h2
         parallel_embed(state.tokens, self.embed, *self._next_norms(0), cfg.eps, x, h1, h2, B)
+        main, side, lib = torch.cuda.current_stream(self.device), self._side, _lib.kernels()
         for i, l in enumerate(self.layers):
+            # the two sublayers of a layer do not depend on one another: the feed-forward streams its weights beside the mixer's chain of small kernels
+            b = None
+            if l.norm2 is not None:
+                side.wait_stream(main)
+                with torch.cuda.stream(side):
+                    lib.ft_pdl_break()
+                    b = self._feed_decode(l, B)
             a = self._mix_decode(l, i, state, B, cache)
-            b = self._feed_decode(l, B)
+            if b is not None:
+                main.wait_stream(side)
+                lib.ft_pdl_break()
             parallel_update(x, cfg.residual_mult, a, b, *self._next_norms(i + 1), cfg.eps, h1, h2, B, W, store=i + 1 < len(self.layers))
         self._g_head(h1)
         g = self._g_head
