@@ -162,7 +162,11 @@ FT_DEVICE bool mw_wait(uint64_t* bar, uint32_t parity) {
     if ((i & 0xff) == 0 && globaltimer_ns() - t0 > 2000000000ull) return false;
   }
 }
-FT_DEVICE void bar_named(int id, int threads) { asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory"); }
+// bar.sync counts whole warps: lanes that a wait has let go one by one come together first
+FT_DEVICE void bar_named(int id, int threads) {
+  __syncwarp();
+  asm volatile("bar.sync %0, %1;" ::"r"(id), "r"(threads) : "memory");
+}
 template <int N> FT_DEVICE void reg_inc() { asm volatile("setmaxnreg.inc.sync.aligned.u32 %0;" ::"n"(N)); }
 template <int N> FT_DEVICE void reg_dec() { asm volatile("setmaxnreg.dec.sync.aligned.u32 %0;" ::"n"(N)); }
 // two neighbouring f32 values as bf16 high parts and bf16 remainders (16 mantissa bits together)
