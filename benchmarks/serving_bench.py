@@ -334,6 +334,7 @@ def run_mepupel(size, layers, batch, prompt, ctx, steps, kernels=True):
             eng.model.decode(eng.state, batch, eng.cache)
         one()
         active = int(eng.model._moe_buffers.n_active)               # experts in use (of the last layer; the layers are alike)
+        eng.model.side_by_side = False                              # kernels one by one
         n = eng.cache.lengths[seqs[0]] + 1
         names = dict(common)
         names.update({(S.main + S.h8, W): "projection gemm (state space)", (W, A.out_cols): "output gemm (attention)", (VOCAB, W): "head gemm"})

@@ -295,6 +295,7 @@ class MepupelModel:
         if dtype not in (torch.bfloat16, torch.float32):
             raise InvalidArgument("Mepupel runs in bfloat16 or float32")
         self.cfg, self.device, self.dtype, self.vocab = cfg, torch.device(device), dtype, cfg.vocab
+        self.side_by_side = True             # decode: the two sublayers of a layer on two streams
         if self.device.type != "cuda":
             raise InvalidArgument("Mepupel runs on a CUDA device (its operators are CUDA kernels)")
         self._load(weights)
@@ -476,16 +477,18 @@ class MepupelModel:
         main, side, lib = torch.cuda.current_stream(self.device), self._side, _lib.kernels()
         for i, l in enumerate(self.layers):
             # the two sublayers of a layer do not depend on one another: the feed-forward streams its weights beside the mixer's chain of small kernels
-            b = None
-            if l.norm2 is not None:
+            two = self.side_by_side and l.norm2 is not None
+            if two:
                 side.wait_stream(main)
                 with torch.cuda.stream(side):
                     lib.ft_pdl_break()
                     b = self._feed_decode(l, B)
             a = self._mix_decode(l, i, state, B, cache)
-            if b is not None:
+            if two:
                 main.wait_stream(side)
                 lib.ft_pdl_break()
+            else:
+                b = self._feed_decode(l, B)
             parallel_update(x, cfg.residual_mult, a, b, *self._next_norms(i + 1), cfg.eps, h1, h2, B, W, store=i + 1 < len(self.layers))
         self._g_head(h1)
         g = self._g_head
