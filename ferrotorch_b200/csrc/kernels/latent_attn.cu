@@ -1,7 +1,7 @@
 // Latent attention: keys and values are linear images of one small vector per token (the latent c, RMS-normalised) plus one rotated key part shared by
 // all heads, so a token's cache row is [c | k_rot] whatever the number of heads. Rows are padded: c to a multiple of 16 elements (`r16`), k_rot to a
 // multiple of 16 (`row` = r16 + padded rot), zeros in the padding. Pages hold 16 rows. The rotated part may be absent (rot = 0), queries may come through a
-// normalised latent of their own, and a layer may read the latent that an earlier layer cached.
+// normalised latent of their own, a layer may read the latent that an earlier layer cached, and the heads' outputs may be gated (per element or per head).
 //
 //   score(q, j) = scale (q_plain . W_uk c_j + q_rot . k_rot_j) = scale (W_uk^T q_plain | q_rot) . (c_j | k_rot_j)
 //   out         = W_uv sum_j p_j c_j
@@ -14,6 +14,7 @@
 //   ft_latent_decode        one query token per sequence over the cached rows, all heads of a tile share every loaded row (mma.sync), split over the
 //                           sequence; ft_latent_combine merges the splits
 //   ft_latent_rows          plain f32-arithmetic kernel for f32 or bf16 data and any sizes (the 32-bit path)
+//   ft_latent_gate          the output gate as a pass of its own, behind ft_latent_rows
 // Compiled without fast-math.
 #include "common.cuh"
 #include "host_common.h"
@@ -33,6 +34,17 @@ FT_DEVICE float ex2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
   return y;
 }
+
+FT_DEVICE float sigmoid_exact(float x) { return 1.f / (1.f + expf(-x)); }
+FT_DEVICE float sigmoid_fast(float x) { return 1.f / (1.f + __expf(-x)); }
+
+// Output gate: pre-activations [rows][ldg] in the data type, a column per element (heads padded to 8) or per head
+enum { GATE_NONE = 0, GATE_ELEMENT = 1, GATE_HEAD = 2 };
+struct OutputGate {
+  const void* p;
+  int64_t ldg;
+  int kind;
+};
 
 // Column layout of a projection row: heads of [plain padded to d8 | rot padded to dr8] (or, with q_rank, the query latent padded to a multiple of 8), then the latent
 // (rank padded to rank8), then the shared rot part.
@@ -182,8 +194,21 @@ __global__ void __launch_bounds__(128) latent_rows_kernel(const T* __restrict__ 
     if (threadIdx.x + 128 * i < D.r16) dst[threadIdx.x + 128 * i] = from_f<T>(o[i] / l);
 }
 
+// a [rows][lda], heads of v8 columns, gated in place; four columns a thread
+template <typename T>
+__global__ void __launch_bounds__(256) latent_gate_kernel(T* __restrict__ a, int64_t lda, OutputGate gate, int quads, int v8) {
+  const int i = blockIdx.x * 256 + threadIdx.x;
+  if (i >= quads) return;
+  T* x = a + (size_t)blockIdx.y * lda + i * 4;
+  const T* g = reinterpret_cast<const T*>(gate.p) + (size_t)blockIdx.y * gate.ldg;
+  const int hd = i * 4 / v8;
+#pragma unroll
+  for (int e = 0; e < 4; e++) x[e] = from_f<T>(to_f(x[e]) * sigmoid_exact(to_f(g[gate.kind == GATE_HEAD ? hd : i * 4 + e])));
+}
+
 // ------------------------------------------------------------------------------------------------------------
-// decode preparation on split-K planes: CTAs [0, H * slices) absorb 64 latent columns of one head for every token, the rest handle one token's cache row
+// decode preparation on split-K planes: CTAs [0, H * slices) absorb 64 latent columns of one head for every token, then one CTA per token handles its cache row, and with a
+// gate the rest take 256 of its columns each
 // ------------------------------------------------------------------------------------------------------------
 constexpr int DEC_TOK = 16, ABS_COLS = 64, PREP_THREADS = 256;
 FT_DEVICE float plane_sum(const float* __restrict__ p, int splits, size_t stride, size_t idx) {
@@ -202,7 +227,8 @@ __global__ void __launch_bounds__(PREP_THREADS) latent_decode_prep_kernel(const 
                                                                           const __nv_bfloat16* __restrict__ wuk, int64_t ldw, const float* __restrict__ w, float eps,
                                                                           const int* __restrict__ positions, const float* __restrict__ cos_t,
                                                                           const float* __restrict__ sin_t, const int* __restrict__ block_table, int max_blocks,
-                                                                          __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache) {
+                                                                          __nv_bfloat16* __restrict__ q, __nv_bfloat16* __restrict__ cache, int gate_cols,
+                                                                          float* __restrict__ gate) {
   extern __shared__ __align__(16) uint8_t prep_smem[];
   __shared__ float red[32];
   const int slices = (D.r16 + ABS_COLS - 1) / ABS_COLS, half = D.dr / 2;
@@ -261,7 +287,14 @@ __global__ void __launch_bounds__(PREP_THREADS) latent_decode_prep_kernel(const 
     }
     return;
   }
-  const int b = blockIdx.x - D.H * slices, pos = positions[b];
+  const int extra = blockIdx.x - D.H * slices, rows = cache ? B : 0;
+  if (extra >= rows) {                                // sigmoid of the gate's columns, behind the shared rotated part
+    const int per = (gate_cols + PREP_THREADS - 1) / PREP_THREADS, tk = (extra - rows) / per, c = (extra - rows) % per * PREP_THREADS + threadIdx.x;
+    if (c < gate_cols)
+      gate[(size_t)tk * gate_cols + c] = sigmoid_exact(plane_sum(planes, splits, pstride, (size_t)tk * ldp + (size_t)D.H * (D.d8 + D.dr8) + (cache ? D.rank8 + D.dr8 : 0) + c));
+    return;
+  }
+  const int b = extra, pos = positions[b];
   const size_t base = (size_t)b * ldp + (size_t)D.H * (D.d8 + D.dr8);
   float* lat = reinterpret_cast<float*>(prep_smem);     // rank floats (the launcher sizes the buffer for both uses)
   float ss = 0.f;
@@ -620,7 +653,7 @@ template <int NT, int NQ, int NV>
 __global__ void __launch_bounds__(64 + 128 * NT, (NT == 1 && NV == 1) ? 2 : 1)
 latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmQr, const __grid_constant__ CUtensorMap tmK,
                     const __grid_constant__ CUtensorMap tmKr, const __grid_constant__ CUtensorMap tmV, const int4* __restrict__ tiles, FlashDims F, float scale_log2,
-                    __nv_bfloat16* __restrict__ out, int64_t ldo, uint32_t* status) {
+                    OutputGate gate, __nv_bfloat16* __restrict__ out, int64_t ldo, uint32_t* status) {
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int nq = NQ > 0 ? NQ : F.nn + F.nr, nv = NV > 0 ? NV : F.nv;
@@ -821,9 +854,14 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
     }
     if (ok && nb > 0) {
       tc_fence_after();
-      const float inv_l = 1.f / l;
+      float inv_l = 1.f / l;
       const bool live = t * LF_BM + r < tl.y;
-      __nv_bfloat16* dst = out + (size_t)(tl.x + t * LF_BM + r) * ldo + (size_t)hd * F.dv8;
+      const size_t row = (size_t)(tl.x + t * LF_BM + r);
+      const __nv_bfloat16* gp = reinterpret_cast<const __nv_bfloat16*>(gate.p) + row * gate.ldg;
+      if (gate.kind == GATE_HEAD && live) inv_l *= sigmoid_fast(__bfloat162float(gp[hd]));
+      const bool gated = gate.kind == GATE_ELEMENT;
+      gp += (size_t)hd * F.dv8;
+      __nv_bfloat16* dst = out + row * ldo + (size_t)hd * F.dv8;
       // rows past the end of the sequence only skip the stores: the warp-wide TMEM loads stay in code that all lanes run together
 #pragma unroll 1
       for (int c = 0; c < nv * 2; c++) {
@@ -832,6 +870,17 @@ latent_flash_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_consta
         tmem_ld_32x32b_x32(tO + lane_off + t * nv * 64 + c * 32, ov);
         tmem_ld_wait();
         uint4 w[4];
+        if (gated) {
+#pragma unroll
+          for (int c8 = 0; c8 < 4; c8++) {
+            if (live && c * 32 + c8 * 8 + 8 <= F.dv8) {
+              float gv[8];
+              bf16x8_to_float(*reinterpret_cast<const bf16x8*>(gp + c * 32 + c8 * 8), gv);
+#pragma unroll
+              for (int i = 0; i < 8; i++) ov[8 * c8 + i] = __float_as_uint(__uint_as_float(ov[8 * c8 + i]) * sigmoid_fast(gv[i]));
+            }
+          }
+        }
 #pragma unroll
         for (int c8 = 0; c8 < 4; c8++) {
           uint32_t e[4];
@@ -874,14 +923,15 @@ int flash_smem(int NT, int nq, int nv) { return NT * nq * LF_QB + 2 * (nq + nv) 
 constexpr int SMEM_MAX = 232448;
 
 template <int NT, int NQ, int NV>
-int launch_flash(const CUtensorMap (&m)[5], const int* tiles, int ntiles, int H, const FlashDims& F, float scale, void* out, int64_t ldo, int smem, cudaStream_t st) {
+int launch_flash(const CUtensorMap (&m)[5], const int* tiles, int ntiles, int H, const FlashDims& F, float scale, const OutputGate& gate, void* out, int64_t ldo, int smem,
+                 cudaStream_t st) {
   static bool configured = false;
   if (!configured) {
     FT_CUDA_TRY(cudaFuncSetAttribute(latent_flash_kernel<NT, NQ, NV>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_MAX));
     configured = true;
   }
   latent_flash_kernel<NT, NQ, NV><<<dim3(ntiles, H), 64 + 128 * NT, smem, st>>>(m[0], m[1], m[2], m[3], m[4], reinterpret_cast<const int4*>(tiles), F,
-                                                                       scale * 1.4426950408889634f, (__nv_bfloat16*)out, ldo, ft_status_ptr());
+                                                                       scale * 1.4426950408889634f, gate, (__nv_bfloat16*)out, ldo, ft_status_ptr());
   return (int)cudaGetLastError();
 }
 
@@ -936,6 +986,21 @@ FT_EXPORT int ft_latent_rows(const void* q, const void* cache, const int* block_
   return (int)cudaGetLastError();
 }
 
+// a [rows][lda] (heads of v8 columns, v8 a multiple of 8) times the sigmoid of gate [rows][ldg], kinds as in ft_latent_flash; both f32 (is_f32) or bf16.
+FT_EXPORT int ft_latent_gate(void* a, int64_t lda, const void* gate, int64_t ldg, int gate_kind, int rows, int H, int v8, int is_f32, cudaStream_t st) {
+  if (rows < 1 || H < 1 || v8 < 8 || (v8 & 7) || (gate_kind != GATE_ELEMENT && gate_kind != GATE_HEAD) || !gate) return FT_ERR_ARG;
+  const int quads = H * v8 / 4, es = is_f32 ? 4 : 2;
+  for (int r0 = 0; r0 < rows; r0 += 65535) {
+    const int n = rows - r0 < 65535 ? rows - r0 : 65535;
+    char* x = (char*)a + (size_t)r0 * lda * es;
+    const OutputGate G{(const char*)gate + (size_t)r0 * ldg * es, ldg, gate_kind};
+    const dim3 grid((quads + 255) / 256, n);
+    if (is_f32) latent_gate_kernel<float><<<grid, 256, 0, st>>>((float*)x, lda, G, quads, v8);
+    else latent_gate_kernel<__nv_bfloat16><<<grid, 256, 0, st>>>((__nv_bfloat16*)x, lda, G, quads, v8);
+  }
+  return (int)cudaGetLastError();
+}
+
 // Decode step of B <= 16 sequences whose queries come through a latent, from split-K planes [query latent padded to 8 | latent padded to 8]: the normalised query
 // latent (bf16 [B][ldq]) and, unless cache is null, the cache row of every sequence's current position. Latents of up to 12288.
 FT_EXPORT int ft_latent_decode_norms(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int B, int q_rank, int rank, const float* wq, const float* w, float eps,
@@ -949,18 +1014,20 @@ FT_EXPORT int ft_latent_decode_norms(const float* planes, int splits, int64_t ld
 
 // Decode step of B <= 16 sequences, from the split-K planes of the fused query / latent projection (column layout as in ft_latent_prep): absorbed and
 // rotated queries q [B][H][row] bf16, cache row of every sequence's current position (cache null: the planes hold queries alone). wuk: bf16 [H * d8][ldw], ldw >= rank padded to 16, zeros past rank.
+// gate_cols > 0: gate (f32 [B][gate_cols]) gets the sigmoid of the columns behind those.
 FT_EXPORT int ft_latent_decode_prep(const float* planes, int splits, int64_t ldp, int64_t plane_stride, int B, int H, int d, int dr, int rank, const void* wuk,
                                     int64_t ldw, const float* w, float eps, const int* positions, const float* cos_t, const float* sin_t, const int* block_table,
-                                    int max_blocks, void* q, void* cache, cudaStream_t st) {
-  if (B < 1 || B > DEC_TOK || splits < 1 || !dims_ok(H, d, dr, rank)) return FT_ERR_ARG;
+                                    int max_blocks, void* q, void* cache, int gate_cols, float* gate, cudaStream_t st) {
+  if (B < 1 || B > DEC_TOK || splits < 1 || !dims_ok(H, d, dr, rank) || gate_cols < 0 || (gate_cols && !gate)) return FT_ERR_ARG;
   const LatentDims D = make_dims(H, d, dr, rank);
   if ((ldw & 7) || ldw < D.r16) return FT_ERR_ARG;
   const int slices = (D.r16 + ABS_COLS - 1) / ABS_COLS;
   const size_t absorb = (size_t)d * (ABS_COLS * 2 + DEC_TOK * 4), norm = sizeof(float) * (size_t)rank;
   const size_t smem = absorb > norm ? absorb : norm;
   if (smem > 48 * 1024) return FT_ERR_TOO_LARGE;
-  return (int)ft_launch_pdl(latent_decode_prep_kernel, dim3(H * slices + (cache ? B : 0)), dim3(PREP_THREADS), smem, st, planes, splits, ldp, (size_t)plane_stride, D, B,
-                            (const __nv_bfloat16*)wuk, ldw, w, eps, positions, cos_t, sin_t, block_table, max_blocks, (__nv_bfloat16*)q, (__nv_bfloat16*)cache);
+  return (int)ft_launch_pdl(latent_decode_prep_kernel, dim3(H * slices + (cache ? B : 0) + B * ((gate_cols + PREP_THREADS - 1) / PREP_THREADS)), dim3(PREP_THREADS), smem, st, planes, splits, ldp, (size_t)plane_stride, D, B,
+                            (const __nv_bfloat16*)wuk, ldw, w, eps, positions, cos_t, sin_t, block_table, max_blocks, (__nv_bfloat16*)q, (__nv_bfloat16*)cache, gate_cols,
+                            gate);
 }
 
 // Attention of one token per sequence over its cached rows (seq_lens[b] rows, the newest included); q as written by ft_latent_decode_prep. Partial
@@ -1006,9 +1073,12 @@ FT_EXPORT int ft_latent_flash_tile(int d, int dr, int dv) {
 // Causal attention over ragged sequences. q: [q_rows][ldq] with heads of [d padded to 8 | dr padded to 8]; kv: [ctx_rows][ldkv] with H heads of keys (d
 // padded to 8), then H heads of values (dv padded to 8); kr: rotated key part, [ctx_rows][ldkr]; out: [q_rows][ldo], heads of dv padded to 8. tiles: int4
 // per tile {first query row, rows (<= the tile size), position of the first row, first context row of its sequence}: the row at position p sees context
-// rows 0..p of its sequence. dr may be 0 (kr is not read then). All bf16, leading dimensions multiples of 8.
+// rows 0..p of its sequence. dr may be 0 (kr is not read then). gate_kind 1: gate rows (pitch ldg) of H * (dv padded to 8) pre-activations, 2: of H; 0: none. All bf16, leading
+// dimensions multiples of 8.
 FT_EXPORT int ft_latent_flash(const void* q, int64_t ldq, int q_rows, const void* kv, int64_t ldkv, const void* kr, int64_t ldkr, int ctx_rows, const int* tiles, int ntiles,
-                              int H, int d, int dr, int dv, float scale, void* out, int64_t ldo, cudaStream_t st) {
+                              int H, int d, int dr, int dv, float scale, const void* gate, int64_t ldg, int gate_kind, void* out, int64_t ldo, cudaStream_t st) {
+  const OutputGate G{gate, ldg, gate_kind};
+  if (gate_kind < 0 || gate_kind > 2 || (gate_kind && !gate) || (gate_kind == GATE_ELEMENT && ((ldg & 7) || (reinterpret_cast<uintptr_t>(gate) & 15)))) return FT_ERR_ARG;
   if (q_rows < 1 || ctx_rows < 1 || ntiles < 1 || H < 1 || H > 65535 || d < 1 || dr < 0 || dv < 1 || (ldq & 7) || (ldkv & 7) || (ldkr & 7) || (ldo & 7)) return FT_ERR_ARG;
   const int tile = ft_latent_flash_tile(d, dr, dv);
   if (tile == 0) return FT_ERR_TOO_LARGE;
@@ -1029,7 +1099,7 @@ FT_EXPORT int ft_latent_flash(const void* q, int64_t ldq, int q_rows, const void
   const FlashDims F{d, dr, dv, (d + 63) / 64, (dr + 63) / 64, (dv + 63) / 64, dv8};
   const int nq = F.nn + F.nr;
   const int smem = flash_smem(tile / 128, nq, F.nv);
-#define FT_LF(T, Q, V) return launch_flash<T, Q, V>(m, tiles, ntiles, H, F, scale, out, ldo, smem, st)
+#define FT_LF(T, Q, V) return launch_flash<T, Q, V>(m, tiles, ntiles, H, F, scale, G, out, ldo, smem, st)
   if (tile == 256) {
     if (nq == 2 && F.nv == 2) FT_LF(2, 2, 2);
     if (nq == 3 && F.nv == 1) FT_LF(2, 3, 1);

@@ -2,8 +2,8 @@
 //   clamped   g = min(W_gate x, limit),  u = clamp(W_up x, -limit, limit),  expert(x) = W_down (g sigmoid(slope g) (u + 1)), applied to score * x: the
 //             projections are linear, so W (score x) = score (W x), and the score multiplies the f32 accumulators: no scaled copy of the tokens is made (or rounded)
 //   silu      expert(x) = score W_down (g sigmoid(g) u): the score multiplies the activation, in f32, ahead of the down projection
-// The router takes the largest logits, or (RouteRule) the largest sums of sigmoid and a per-expert correction, among the experts of the best groups, with weights that
-// are normed to a given sum.
+// The router takes the largest logits, weighted with their sigmoids, or (RouteRule) the largest sums of sigmoid and a per-expert correction, or of logit and bias, among the
+// experts of the best groups, with weights that are normed to a given sum.
 //
 // Weights: gate and up rows are interleaved in blocks of eight (eight gate rows, then the eight up rows of the same neurons), so that a warp's 16
 // weight rows -- and a thread's accumulators -- hold a neuron's gate and up together, and the tiles of the grouped GEMM hold both as well.
@@ -59,10 +59,13 @@ FT_DEVICE void next_best(const float* z, int E, float pv, int pi, float& bv, int
   }
 }
 
-// How a router with a correction chooses: experts by sigmoid(logit) + correction, within the `keep` groups (of neighbours) whose two best experts have the largest sum
-// (groups 0: all experts); the weights are the chosen sigmoids divided by their sum, times scale. correction null: by logit, weights are the sigmoids.
+// How a router chooses: by logit, weights are the sigmoids (ROUTE_SIGMOID); or by a choice score within the `keep` groups (of neighbours) whose two best experts have the
+// largest sum (groups 0: all experts), weights normed to the sum `scale`: sigmoid(logit) + vector, weights proportional to the chosen sigmoids (ROUTE_CORRECTED); logit +
+// vector, weights proportional to the exponentials of the chosen scores (ROUTE_SOFTMAX).
+enum { ROUTE_SIGMOID = 0, ROUTE_CORRECTED = 1, ROUTE_SOFTMAX = 2 };
 struct RouteRule {
-  const float* correction;
+  int kind;
+  const float* vector;
   int groups, keep;
   float scale;
 };
@@ -72,7 +75,7 @@ constexpr int MAX_GROUPS = 256;
 // whole warp: ch[e] = choice score of expert e, minus infinity outside the best groups. gs: [groups] scratch
 FT_DEVICE void choice_scores(const float* z, float* ch, int E, const RouteRule& rule, float* gs) {
   const int lane = threadIdx.x & 31;
-  for (int e = lane; e < E; e += 32) ch[e] = sigmoid_f(__ldcg(z + e)) + rule.correction[e];
+  for (int e = lane; e < E; e += 32) ch[e] = (rule.kind == ROUTE_SOFTMAX ? __ldcg(z + e) : sigmoid_f(__ldcg(z + e))) + rule.vector[e];
   __syncwarp();
   if (rule.groups == 0) return;
   const int size = E / rule.groups;
@@ -101,19 +104,21 @@ FT_DEVICE void choice_scores(const float* z, float* ch, int E, const RouteRule& 
   }
   __syncwarp();
 }
-// whole warp: the `top` best of ch in order, take(slot, expert, sigmoid of its logit) on every lane; a ruled router's normed weights follow, lane j with take(-1 - j, 0, weight)
+// whole warp: the `top` best of ch in order, take(slot, expert, its weight before norming) on every lane; a ruled router's normed weights follow, lane j with
+// take(-1 - j, 0, weight)
 template <typename Take>
 FT_DEVICE void choose(const float* z, const float* ch, int E, int top, const RouteRule& rule, Take take) {
-  float pv = INFINITY, sum = 0.f;
+  float pv = INFINITY, sum = 0.f, best = 0.f;
   int pi = -1;
-  const bool ruled = rule.correction != nullptr;
+  const bool ruled = rule.kind != ROUTE_SIGMOID;
   float mine = 0.f;                                  // lane j keeps the weight of slot j (of a ruled router: top <= 32)
   for (int j = 0; j < top; j++) {
     float v;
     int e;
     next_best(ch, E, pv, pi, v, e);
     if (e >= E) e = j;                               // only with NaN logits
-    const float s = sigmoid_f(ruled ? __ldcg(z + e) : v);
+    if (j == 0) best = v;
+    const float s = rule.kind == ROUTE_SOFTMAX ? expf(v - best) : sigmoid_f(ruled ? __ldcg(z + e) : v);
     sum += s;
     if ((threadIdx.x & 31) == j) mine = s;
     take(j, e, s);
@@ -134,14 +139,15 @@ __global__ void __launch_bounds__(256) moe_topk_kernel(const float* __restrict__
   if (tok >= T) return;
   const float* z = logits + (size_t)tok * ld;
   float* ch = choice_sh + (size_t)warp * (E + rule.groups);
-  if (rule.correction) choice_scores(z, ch, E, rule, ch + E);
+  const bool ruled = rule.kind != ROUTE_SIGMOID;
+  if (ruled) choice_scores(z, ch, E, rule, ch + E);
   const size_t at = (size_t)tok * top;
-  choose(z, rule.correction ? ch : z, E, top, rule, [&](int j, int e, float s) {
+  choose(z, ruled ? ch : z, E, top, rule, [&](int j, int e, float s) {
     if (j < 0) {                                     // final weights, a lane each
       score[at - 1 - j] = s;
     } else if (lane == 0) {
       expert[at + j] = e;
-      if (!rule.correction) score[at + j] = s;
+      if (!ruled) score[at + j] = s;
       pos[at + j] = atomicAdd(&count[e], 1);
     }
   });
@@ -306,21 +312,21 @@ __global__ void __launch_bounds__(128) moe_route_small_kernel(const __nv_bfloat1
   __syncthreads();
   if (!is_last) return;
   __threadfence();
-  const bool staged = B * E <= ROUTE_LOGITS;
-  if (staged && !rule.correction) {
+  const bool staged = B * E <= ROUTE_LOGITS, ruled = rule.kind != ROUTE_SIGMOID;
+  if (staged && !ruled) {
     for (int i = threadIdx.x; i < B * E; i += 128) zs[i] = __ldcg(logits + i);
     __syncthreads();
   }
   for (int b = warp; b < B; b += 4) {
     const float* z = logits + (size_t)b * E;
     float* ch = staged ? zs + (size_t)b * E : logits + (size_t)SMALL_TOK * E + (size_t)b * E;
-    if (rule.correction) choice_scores(z, ch, E, rule, gs[warp]);
-    choose(z, rule.correction || staged ? ch : z, E, top, rule, [&](int j, int c, float s) {
+    if (ruled) choice_scores(z, ch, E, rule, gs[warp]);
+    choose(z, ruled || staged ? ch : z, E, top, rule, [&](int j, int c, float s) {
       if (j < 0) {
         R.score[b * top - 1 - j] = s;
       } else if (lane == 0) {
         chosen[b * top + j] = c;
-        if (!rule.correction) R.score[b * top + j] = s;
+        if (!ruled) R.score[b * top + j] = s;
       }
     });
   }
@@ -451,6 +457,9 @@ struct HeadsWork {
   int B, heads, N, Kin;
   __nv_bfloat16* out;
   int64_t ldo, head_o;
+  const float* gate;                 // factors [token][ldg] or null: head_g columns between heads, elem_g (0 or 1) between a head's outputs
+  int64_t ldg;
+  int head_g, elem_g;
 
   FT_DEVICE SkinnyShape shape() const { return SkinnyShape{{heads, 0}, {(N + 15) / 16, 1}, {1, 1}}; }
   FT_DEVICE int K(int) const { return Kin; }
@@ -464,14 +473,16 @@ struct HeadsWork {
     for (int j = 0; j < 2; j++) {
       if (tk + j >= B) break;
       __nv_bfloat16* o = out + (size_t)(tk + j) * ldo + (size_t)g * head_o;
-      if (r < N) o[r] = __float2bfloat16(j ? c.y : c.x);
-      if (r + 8 < N) o[r + 8] = __float2bfloat16(j ? c.w : c.z);
+      const float* f = gate ? gate + (size_t)(tk + j) * ldg + (size_t)g * head_g : nullptr;
+      if (r < N) o[r] = __float2bfloat16((j ? c.y : c.x) * (f ? f[r * elem_g] : 1.f));
+      if (r + 8 < N) o[r + 8] = __float2bfloat16((j ? c.w : c.z) * (f ? f[(r + 8) * elem_g] : 1.f));
     }
   }
 };
 
 bool rule_ok(const RouteRule& r, int E, int top) {
-  if (!r.correction) return r.groups == 0;
+  if (r.kind < ROUTE_SIGMOID || r.kind > ROUTE_SOFTMAX || (r.kind != ROUTE_SIGMOID) != (r.vector != nullptr)) return false;
+  if (r.kind == ROUTE_SIGMOID) return r.groups == 0;
   if (r.groups < 0 || r.groups > MAX_GROUPS || top > 32) return false;
   return r.groups == 0 || (E % r.groups == 0 && r.keep >= 1 && r.keep <= r.groups && top <= r.keep * (E / r.groups));
 }
@@ -480,14 +491,14 @@ bool skinny_fits(int nt, int kmax) { return 8 * nt * skinny_pitch((kmax + 31) & 
 }  // namespace
 
 // Choice of the `top` largest logits per token (ties: lower index first), their sigmoids, and the running position of every (token, slot) inside its
-// expert. count: int[E], zero before the launch (ft_moe_layout zeroes it again). expert, score, pos: [T * top]. With a correction (f32[E]) the choice goes by sigmoid +
-// correction, within the `keep` best of `groups` equal groups of neighbours (0: no groups; a group counts its two best), and the scores are the chosen sigmoids
-// divided by their sum, times scale (top up to 32, groups up to 256).
-FT_EXPORT int ft_moe_topk(const float* logits, int64_t ld, int T, int E, int top, const float* correction, int groups, int keep, float scale, int* expert, float* score,
+// expert. count: int[E], zero before the launch (ft_moe_layout zeroes it again). expert, score, pos: [T * top]. rule 1 with a vector (f32[E]): the choice goes by sigmoid +
+// vector, within the `keep` best of `groups` equal groups of neighbours (0: no groups; a group counts its two best), and the scores are the chosen sigmoids
+// divided by their sum, times scale (top up to 32, groups up to 256); rule 2: by logit + vector, and the scores are the softmax over the chosen, times scale.
+FT_EXPORT int ft_moe_topk(const float* logits, int64_t ld, int T, int E, int top, int rule_kind, const float* vector, int groups, int keep, float scale, int* expert, float* score,
                           int* pos, int* count, cudaStream_t st) {
-  const RouteRule rule{correction, groups, keep, scale};
+  const RouteRule rule{rule_kind, vector, groups, keep, scale};
   if (T < 1 || E < 1 || top < 1 || top > E || !rule_ok(rule, E, top)) return FT_ERR_ARG;
-  const size_t smem = correction ? (size_t)8 * (E + groups) * 4 : 0;
+  const size_t smem = rule_kind ? (size_t)8 * (E + groups) * 4 : 0;
   if (smem > 200 * 1024) return FT_ERR_TOO_LARGE;
   if (smem > 48 * 1024) FT_CUDA_TRY(cudaFuncSetAttribute(moe_topk_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024));
   moe_topk_kernel<<<(T + 7) / 8, 256, smem, st>>>(logits, ld, T, E, top, rule, expert, score, pos, count);
@@ -527,9 +538,9 @@ FT_EXPORT int ft_moe_act(const void* gu, int64_t ld_gu, const float* row_score, 
 
 // Decode routing (B <= 16 tokens, bf16 operands, f32 accumulation): logits f32 scratch of 32 E, counter int zero before the first launch. Outputs:
 // n_active int[1], id int[E], cnt int[E], pair int[E][16], pair_of int[E][16], score f32 [B * top]. Choice and scores as in ft_moe_topk.
-FT_EXPORT int ft_moe_route_small(const void* h, int64_t ldh, const void* router, int64_t ldr, int B, int W, int E, int top, const float* correction, int groups, int keep,
+FT_EXPORT int ft_moe_route_small(const void* h, int64_t ldh, const void* router, int64_t ldr, int B, int W, int E, int top, int rule_kind, const float* vector, int groups, int keep,
                                  float scale, float* logits, int* counter, int* n_active, int* id, int* cnt, int* pair, int* pair_of, float* score, cudaStream_t st) {
-  const RouteRule rule{correction, groups, keep, scale};
+  const RouteRule rule{rule_kind, vector, groups, keep, scale};
   if (B < 1 || B > SMALL_TOK || E < 1 || top < 1 || top > E || top > MAX_TOP || (ldh & 7) || (ldr & 7) || !rule_ok(rule, E, top)) return FT_ERR_ARG;
   return (int)ft_launch_pdl(moe_route_small_kernel, dim3(E), dim3(128), 0, st, (const __nv_bfloat16*)h, ldh, (const __nv_bfloat16*)router, ldr, B, W, E, top, rule,
                             logits, counter, SmallRoute{n_active, id, cnt, pair, pair_of, score});
@@ -580,11 +591,12 @@ FT_EXPORT int ft_moe_down_small(const void* act, int64_t ld_act, const void* act
 
 // out[b][head][n] = sum_k w[head][n][k] x[b][head][k] for B <= 16 tokens: x bf16 (ldx between tokens, head_x between heads, 16-byte aligned), w bf16 rows of
 // ldw >= K rounded up to 32 elements with head_w elements between heads (16-row blocks are read whole: the buffer extends past the last head's rows
-// to the next multiple of 16), out bf16.
+// to the next multiple of 16), out bf16, times gate[b][head * head_g + n * elem_g] (f32 rows of ldg) unless gate is null.
 FT_EXPORT int ft_skinny_heads(const void* x, int64_t ldx, int64_t head_x, const void* w, int64_t ldw, int64_t head_w, int B, int heads, int N, int K, void* out,
-                              int64_t ldo, int64_t head_o, cudaStream_t st) {
+                              int64_t ldo, int64_t head_o, const float* gate, int64_t ldg, int head_g, int elem_g, cudaStream_t st) {
   if (B < 1 || B > SMALL_TOK || heads < 1 || N < 1 || K < 1 || (ldx & 7) || (head_x & 7) || (ldw & 7) || ldw < ((K + 31) & ~31) || (head_w & 7)) return FT_ERR_ARG;
-  const HeadsWork p{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, ldx, head_x, ldw, head_w, B, heads, N, K, (__nv_bfloat16*)out, ldo, head_o};
+  const HeadsWork p{(const __nv_bfloat16*)x, (const __nv_bfloat16*)w, ldx, head_x, ldw, head_w, B, heads, N, K, (__nv_bfloat16*)out, ldo, head_o, gate,
+                    ldg, head_g, elem_g};
   const int items = heads * ((N + 15) / 16);
   if (!skinny_fits(B > 8 ? 2 : 1, K)) return FT_ERR_TOO_LARGE;
   return B > 8 ? skinny_launch<HeadsWork, 2>(p, K, items, st) : skinny_launch<HeadsWork, 1>(p, K, items, st);

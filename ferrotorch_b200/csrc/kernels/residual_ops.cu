@@ -1,15 +1,21 @@
-// One f32 residual per token, with the norm on the sublayer's output or ahead of two sublayers that run side by side, and the activation of a gated feed-forward.
+// One f32 residual per token, with the norm on the sublayer's output or ahead of two sublayers that run side by side, averages over the layers' results, the token shift ahead of a
+// mixer, and the activations of feed-forwards.
 //
 //   ft_residual_embed    x = scale * table[id];  h = x in the operand type
 //   ft_residual_update   y = sum of the sublayer's f32 planes;  x += y / rms(y) * w;  h = x, or x / rms(x) * w_last ahead of the output projection
 //   ft_parallel_embed    x = table[id];  h1 = x / rms(x) * w1, h2 = x / rms(x) * w2: the operands of two sublayers
 //   ft_parallel_update   x += mult * (what both sublayers returned: f32 planes, expert rows through an index, a bias);  h1 and h2 from the new x
+//   ft_depth_update      X = x + y / rms(y) * w, kept beside the results of the earlier layers;  x = a weighted sum of all of them;  its norm, shifted by one token or not
+//   ft_token_shift       h = n + (n of the token before - n) * s with n = x / rms(x) * w:  the shifted operand of a prompt's rows
 //   ft_gated_act         act(gate) * up of interleaved gate / up columns, from a 16-bit or f32 matrix or from split-K planes
+//   ft_poly_norm         a N(z) + b N(z^2) + c N(z^3) + e with N dividing a row by its root mean square, from a 16-bit or f32 matrix or from split-K planes
 //
 // The updates take one row per cluster of CTAs: one CTA where there are rows enough to fill the GPU, up to eight (sums of squares meet in
 // distributed shared memory) for the few rows of a decode step, whose planes are then read by eight SMs instead of one. Everything a row needs stays in
 // registers between its two norms. Compiled without fast-math.
 #include <cooperative_groups.h>
+
+#include <utility>
 
 #include "common.cuh"
 #include "host_common.h"
@@ -236,6 +242,239 @@ __global__ void __launch_bounds__(UPD_THREADS) parallel_update_kernel(float* __r
 }
 
 // ------------------------------------------------------------------------------------------------------------
+// averages over depth, token shift
+// ------------------------------------------------------------------------------------------------------------
+// results[j]: what layer j - 1 returned (0: the embedding output). The update stores results[count] and hands on x = sum over j <= count of avg[j] results[j]. What becomes of
+// the norm of x: `rstd` set: only its factor is stored, per row (ft_token_shift does the rest); `shift` set (a decode step): h = n + (n of the token before - n) shift, with
+// the state of this row's slot; else h = n.
+template <typename H> struct DepthArgs {
+  const float* y;                    // f32 planes of the sublayer, or
+  int planes;
+  size_t pstride;
+  int64_t ldy;
+  const H* rows;                     // rows of experts through row_of
+  const int* row_of;
+  int top;
+  int64_t ldr;
+  const float* w_out;
+  float* x;
+  float* results;
+  size_t rstride;
+  int64_t ldx;
+  int count;
+  const float* avg;
+  const float* w_next;
+  float eps;
+  H* h;
+  int64_t ldh;
+  float* rstd;
+  const float* shift;
+  float* state;
+  int64_t ld_state;
+  const int *slots, *positions;
+  int store;                         // 0: neither x nor the result is needed any more
+};
+FT_DEVICE void fma4(float4& a, float k, float4 v) { a.x += k * v.x; a.y += k * v.y; a.z += k * v.z; a.w += k * v.w; }
+FT_DEVICE float4 mul4(float4 a, float k, float4 w) { return make_float4(a.x * k * w.x, a.y * k * w.y, a.z * k * w.z, a.w * k * w.w); }
+// shifted operand from this token's and the previous token's normed values
+FT_DEVICE float4 shift4(float4 n, float4 before, float4 s) {
+  return make_float4(n.x + (before.x - n.x) * s.x, n.y + (before.y - n.y) * s.y, n.z + (before.z - n.z) * s.z, n.w + (before.w - n.w) * s.w);
+}
+
+template <int NV, bool EMBED, typename H>
+__global__ void __launch_bounds__(UPD_THREADS) depth_update_kernel(DepthArgs<H> A, const int64_t* __restrict__ ids, const H* __restrict__ table, int64_t ld_table, int64_t vocab,
+                                                                   int ncta, int W, int cols) {
+  namespace cg = cooperative_groups;
+  __shared__ float red[32];
+  __shared__ float cta_ss[2];
+  cg::cluster_group cluster = cg::this_cluster();
+  const int row = blockIdx.x / ncta, c0 = blockIdx.x % ncta * cols, cend = min(W, c0 + cols);
+  pdl_wait();
+  pdl_launch_dependents();
+  auto row_sum = [&](float ss, int slot) -> float {
+    ss = block_sum(ss, red);
+    if (ncta == 1) return ss;
+    if (threadIdx.x == 0) cta_ss[slot] = ss;
+    cluster.sync();
+    float t = 0.f;
+    for (int r = 0; r < ncta; r++) t += *cluster.map_shared_rank(&cta_ss[slot], r);
+    return t;
+  };
+  float* xr = A.x + (size_t)row * A.ldx;
+  float* res = A.results + (size_t)row * A.ldx;
+  float4 xv[NV];
+  float s2 = 0.f;
+  if constexpr (EMBED) {
+    const int64_t id = ids[row];
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < cend) {
+        if (id >= 0 && id < vocab) xv[i] = keep4(get4(table + (size_t)id * ld_table + c), c, W);
+        *reinterpret_cast<float4*>(xr + c) = xv[i];
+        *reinterpret_cast<float4*>(res + c) = xv[i];
+        s2 += sq4(xv[i]);
+      }
+    }
+  } else {
+    float4 v[NV];
+    float ss = 0.f;
+    const float last = A.avg[A.count];
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      v[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (c < cend) {
+        if (A.planes) add_planes(v[i], A.y + (size_t)row * A.ldy + c, A.planes, A.pstride);
+#pragma unroll 4
+        for (int k = 0; k < A.top; k++) {
+          const float4 t = get4(A.rows + (size_t)A.row_of[(size_t)row * A.top + k] * A.ldr + c);
+          v[i].x += t.x; v[i].y += t.y; v[i].z += t.z; v[i].w += t.w;
+        }
+        v[i] = keep4(v[i], c, W);
+        ss += sq4(v[i]);
+#pragma unroll 4
+        for (int j = 0; j < A.count; j++) fma4(xv[i], A.avg[j], *reinterpret_cast<const float4*>(res + j * A.rstride + c));
+      }
+    }
+    const float rstd = 1.f / sqrtf(row_sum(ss, 0) / (float)W + A.eps);
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      if (c < cend) {
+        float4 r = *reinterpret_cast<const float4*>(xr + c);
+        const float4 w = *reinterpret_cast<const float4*>(A.w_out + c);
+        r = keep4(make_float4(r.x + v[i].x * rstd * w.x, r.y + v[i].y * rstd * w.y, r.z + v[i].z * rstd * w.z, r.w + v[i].w * rstd * w.w), c, W);
+        fma4(xv[i], last, r);
+        if (A.store) {
+          *reinterpret_cast<float4*>(res + A.count * A.rstride + c) = r;
+          *reinterpret_cast<float4*>(xr + c) = xv[i];
+        }
+        s2 += sq4(xv[i]);
+      }
+    }
+  }
+  const float r2 = 1.f / sqrtf(row_sum(s2, 1) / (float)W + A.eps);
+  if (A.rstd != nullptr) {
+    if (blockIdx.x % ncta == 0 && threadIdx.x == 0) A.rstd[row] = r2;
+  } else {
+    float* state = A.shift ? A.state + (size_t)A.slots[row] * A.ld_state : nullptr;
+    const bool first = A.shift && A.positions[row] == 0;
+#pragma unroll
+    for (int i = 0; i < NV; i++) {
+      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      if (c < cend) {
+        float4 n = mul4(xv[i], r2, *reinterpret_cast<const float4*>(A.w_next + c));
+        if (A.shift) {
+          const float4 before = first ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(state + c);
+          *reinterpret_cast<float4*>(state + c) = n;
+          n = shift4(n, before, *reinterpret_cast<const float4*>(A.shift + c));
+        }
+        put4(A.h + (size_t)row * A.ldh + c, n);
+      }
+    }
+  }
+  if (ncta > 1) cluster.sync();                     // nobody leaves while a partner may still read its shared memory
+}
+
+// A thread takes four columns of SHIFT_ROWS neighbouring rows, and the row ahead of them where that belongs to the same sequence. The thread that meets a sequence's first
+// row of this batch replaces its state, after it has read it: spans[sequence] = {first row, rows, state slot, whether the sequence starts here}.
+constexpr int SHIFT_ROWS = 8;
+template <typename H>
+__global__ void __launch_bounds__(256) token_shift_kernel(const float* __restrict__ x, int64_t ldx, const float* __restrict__ rstd, const float* __restrict__ w,
+                                                          const float* __restrict__ shift, const int4* __restrict__ spans, const int* __restrict__ seq_of,
+                                                          float* __restrict__ state, int64_t ld_state, H* __restrict__ h, int64_t ldh, int rows, int W) {
+  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+  if (c >= W) return;
+  const float4 wv = *reinterpret_cast<const float4*>(w + c), sv = *reinterpret_cast<const float4*>(shift + c);
+  const int r0 = blockIdx.y * SHIFT_ROWS;
+  float4 v[SHIFT_ROWS + 1];
+#pragma unroll
+  for (int i = 0; i <= SHIFT_ROWS; i++) {
+    const int r = min(max(r0 + i - 1, 0), rows - 1);
+    v[i] = mul4(*reinterpret_cast<const float4*>(x + (size_t)r * ldx + c), rstd[r], wv);
+  }
+#pragma unroll
+  for (int i = 0; i < SHIFT_ROWS; i++) {
+    const int r = r0 + i;
+    if (r >= rows) break;
+    float4 before = v[i];
+    const int4 sp = spans[seq_of[r]];
+    if (r == sp.x) {
+      float* st = state + (size_t)sp.z * ld_state + c;
+      before = sp.w ? make_float4(0.f, 0.f, 0.f, 0.f) : *reinterpret_cast<const float4*>(st);
+      const int e = sp.x + sp.y - 1;
+      *reinterpret_cast<float4*>(st) = mul4(*reinterpret_cast<const float4*>(x + (size_t)e * ldx + c), rstd[e], wv);
+    }
+    put4(h + (size_t)r * ldh + c, shift4(v[i + 1], before, sv));
+  }
+}
+
+// ------------------------------------------------------------------------------------------------------------
+// polynomial of normed powers: one row per cluster as in the updates above
+// ------------------------------------------------------------------------------------------------------------
+template <int NV, typename I, typename O>
+__global__ void __launch_bounds__(UPD_THREADS) poly_norm_kernel(const I* __restrict__ z, int planes, size_t pstride, int64_t ldz, const float* __restrict__ coef, float eps,
+                                                                O* __restrict__ out, int64_t ldo, int ncta, int W, int cols) {
+  namespace cg = cooperative_groups;
+  __shared__ float red[3][32];
+  __shared__ float cta_ss[3];
+  cg::cluster_group cluster = cg::this_cluster();
+  const int row = blockIdx.x / ncta, c0 = blockIdx.x % ncta * cols, cend = min(W, c0 + cols), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  pdl_wait();
+  pdl_launch_dependents();
+  float4 v[NV];
+  float s[3] = {0.f, 0.f, 0.f};                      // sums of z^2, z^4 and z^6
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < cend) {
+      if constexpr (sizeof(I) == 4) add_planes(v[i], z + (size_t)row * ldz + c, planes, pstride);
+      else v[i] = get4(z + (size_t)row * ldz + c);
+      v[i] = keep4(v[i], c, W);
+      const float e[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
+#pragma unroll
+      for (int k = 0; k < 4; k++) {
+        const float q = e[k] * e[k];
+        s[0] += q; s[1] += q * q; s[2] += q * q * q;
+      }
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < 3; k++) {
+    s[k] = warp_sum(s[k]);
+    if (lane == 0) red[k][warp] = s[k];
+  }
+  __syncthreads();
+#pragma unroll
+  for (int k = 0; k < 3; k++) {
+    s[k] = 0.f;
+#pragma unroll
+    for (int i = 0; i < UPD_THREADS / 32; i++) s[k] += red[k][i];
+  }
+  if (ncta > 1) {
+    if (threadIdx.x < 3) cta_ss[threadIdx.x] = threadIdx.x == 0 ? s[0] : threadIdx.x == 1 ? s[1] : s[2];
+    cluster.sync();
+#pragma unroll
+    for (int k = 0; k < 3; k++) {
+      s[k] = 0.f;
+      for (int r = 0; r < ncta; r++) s[k] += *cluster.map_shared_rank(&cta_ss[k], r);
+    }
+  }
+  const float inv = 1.f / (float)W;
+  const float a = coef[0] / sqrtf(s[0] * inv + eps), b = coef[1] / sqrtf(s[1] * inv + eps), d = coef[2] / sqrtf(s[2] * inv + eps), e0 = coef[3];
+  auto f = [&](float t) { return ((d * t + b) * t + a) * t + e0; };
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    if (c < cend) put4(out + (size_t)row * ldo + c, keep4(make_float4(f(v[i].x), f(v[i].y), f(v[i].z), f(v[i].w)), c, W));
+  }
+  if (ncta > 1) cluster.sync();                     // nobody leaves while a partner may still read its shared memory
+}
+
+// ------------------------------------------------------------------------------------------------------------
 // gated activation
 // ------------------------------------------------------------------------------------------------------------
 enum { ACT_GELU_TANH = 0, ACT_SILU = 1 };
@@ -348,6 +587,48 @@ RowSpread row_spread(int rows, int W) {
   return RowSpread{ncta, cols, (cols + UPD_THREADS * 4 - 1) / (UPD_THREADS * 4)};
 }
 
+// one row per cluster of sp.ncta CTAs
+template <typename... K, typename... A>
+int launch_rows(const RowSpread& sp, int rows, cudaStream_t st, void (*kernel)(K...), A&&... args) {
+  cudaLaunchConfig_t cfg = {};
+  cfg.gridDim = dim3(sp.ncta * rows);
+  cfg.blockDim = dim3(UPD_THREADS);
+  cfg.stream = st;
+  cudaLaunchAttribute attr[2];
+  attr[0].id = cudaLaunchAttributeClusterDimension;
+  attr[0].val.clusterDim.x = sp.ncta;
+  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
+  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+  attr[1].val.programmaticStreamSerializationAllowed = 1;
+  cfg.attrs = attr;
+  cfg.numAttrs = ft_pdl_enabled() ? 2 : 1;
+  return (int)cudaLaunchKernelEx(&cfg, kernel, std::forward<A>(args)...);
+}
+
+template <bool EMBED, typename H>
+int dispatch_depth(const DepthArgs<H>& A, const int64_t* ids, const void* table, int64_t ld_table, int64_t vocab, int rows, int W, cudaStream_t st) {
+  const RowSpread sp = row_spread(rows, W);
+  if (sp.nv > 8) return FT_ERR_TOO_LARGE;
+#define FT_DU(N) return launch_rows(sp, rows, st, depth_update_kernel<N, EMBED, H>, A, ids, (const H*)table, ld_table, vocab, sp.ncta, W, sp.cols)
+  if (sp.nv <= 1) FT_DU(1);
+  if (sp.nv <= 2) FT_DU(2);
+  if (sp.nv <= 4) FT_DU(4);
+  FT_DU(8);
+#undef FT_DU
+}
+
+template <typename I, typename O>
+int dispatch_poly(const void* z, int planes, int64_t pstride, int64_t ldz, const float* coef, float eps, void* out, int64_t ldo, int rows, int W, cudaStream_t st) {
+  const RowSpread sp = row_spread(rows, W);
+  if (sp.nv > 8) return FT_ERR_TOO_LARGE;
+#define FT_PN(N) return launch_rows(sp, rows, st, poly_norm_kernel<N, I, O>, (const I*)z, planes, (size_t)pstride, ldz, coef, eps, (O*)out, ldo, sp.ncta, W, sp.cols)
+  if (sp.nv <= 1) FT_PN(1);
+  if (sp.nv <= 2) FT_PN(2);
+  if (sp.nv <= 4) FT_PN(4);
+  FT_PN(8);
+#undef FT_PN
+}
+
 template <bool EMBED, typename H>
 int dispatch_parallel(float* x, int64_t ldx, const int64_t* ids, const void* table, int64_t ld_table, int64_t vocab, const PairOutput<H>& Y, float mult, const float* w1,
                       const float* w2, float eps, void* h1, void* h2, int64_t ldh, int rows, int W, int store, cudaStream_t st) {
@@ -431,6 +712,74 @@ FT_EXPORT int ft_parallel_update(float* x, int64_t ldx, float mult, const float*
   }
   const PairOutput<__nv_bfloat16> Y{a, b, na, nb, (size_t)stride_a, (size_t)stride_b, lda, ldb, (const __nv_bfloat16*)expert_rows, row_of, top, ldr, bias};
   return dispatch_parallel<false, __nv_bfloat16>(x, ldx, nullptr, nullptr, 0, 0, Y, mult, w1, w2, eps, h1, h2, ldh, rows, W, store_x, st);
+}
+
+// Start of a pass with averages over depth: x and results, both [rows][ldx] f32, = table[ids[r]] (zeros for ids outside [0, vocab)). What becomes of the norm n = x / sqrt(mean(x^2)
+// + eps) * w_next: rstd (f32 [rows]) not null: only 1 / sqrt(mean(x^2) + eps) is stored; else h [rows][ldh] in the table's type, shifted with the state of row slots[r] (f32 rows of
+// ld_state; not read at position 0, replaced by n) unless shift is null. Widths up to 65536.
+FT_EXPORT int ft_depth_embed(const int64_t* ids, const void* table, int64_t ld_table, int64_t vocab, float* x, float* results, int64_t ldx, const float* w_next, float eps,
+                             void* h, int64_t ldh, float* rstd, const float* shift, float* state, int64_t ld_state, const int* slots, const int* positions, int is_f32, int rows,
+                             int W, cudaStream_t st) {
+  if (rows < 1 || W < 1 || (!rstd && (!w_next || !h)) || (shift && (!state || !slots || !positions)) || (ld_table & 3) || (ldx & 3) || (ldh & 3) || (ld_state & 3)) return FT_ERR_ARG;
+#define FT_DE(T)                                                                                                                                                       \
+  {                                                                                                                                                                    \
+    DepthArgs<T> A{};                                                                                                                                                  \
+    A.x = x; A.results = results; A.ldx = ldx; A.w_next = w_next; A.eps = eps; A.h = (T*)h; A.ldh = ldh; A.rstd = rstd; A.shift = shift; A.state = state;               \
+    A.ld_state = ld_state; A.slots = slots; A.positions = positions; A.store = 1;                                                                                      \
+    return dispatch_depth<true, T>(A, ids, table, ld_table, vocab, rows, W, st);                                                                                       \
+  }
+  if (is_f32) FT_DE(float);
+  FT_DE(__nv_bfloat16);
+#undef FT_DE
+}
+
+// X = x + y / sqrt(mean(y^2) + eps) * w_out with y = sum of f32 planes [planes][row][ldy] + expert rows row_of[row][0..top) (type of h); results[count] = X; x = sum over j <= count
+// of avg[j] results[j] (f32, results_stride elements apart, rows of ldx); then as in ft_depth_embed. x and results[count] are left alone when store is 0. All vectors readable up to W
+// rounded up to a multiple of four.
+FT_EXPORT int ft_depth_update(float* x, float* results, int64_t results_stride, int64_t ldx, int count, const float* avg, const float* y, int planes, int64_t plane_stride,
+                              int64_t ldy, const void* expert_rows, const int* row_of, int top, int64_t ldr, const float* w_out, const float* w_next, float eps, void* h,
+                              int64_t ldh, float* rstd, const float* shift, float* state, int64_t ld_state, const int* slots, const int* positions, int is_f32, int rows, int W,
+                              int store, cudaStream_t st) {
+  if (rows < 1 || W < 1 || count < 1 || planes < 0 || top < 0 || !w_out || !avg || (!rstd && (!w_next || !h)) || (shift && (!state || !slots || !positions)) || (ldx & 3) ||
+      (ldy & 3) || (ldr & 3) || (ldh & 3) || (ld_state & 3) || (results_stride & 3) || (plane_stride & 3) || (top && (!expert_rows || !row_of)))
+    return FT_ERR_ARG;
+#define FT_DU(T)                                                                                                                                                        \
+  {                                                                                                                                                                     \
+    const DepthArgs<T> A{y, planes, (size_t)plane_stride, ldy, (const T*)expert_rows, row_of, top, ldr, w_out, x, results, (size_t)results_stride, ldx, count, avg, w_next, \
+                         eps, (T*)h, ldh, rstd, shift, state, ld_state, slots, positions, store};                                                                       \
+    return dispatch_depth<false, T>(A, nullptr, nullptr, 0, 0, rows, W, st);                                                                                            \
+  }
+  if (is_f32) FT_DU(float);
+  FT_DU(__nv_bfloat16);
+#undef FT_DU
+}
+
+// h[r] = n[r] + (n before r - n[r]) * shift with n[r] = x[r] * rstd[r] * w, for a batch of sequences whose rows lie one after another: spans int4 per sequence {first row, rows, slot,
+// whether it starts here}, seq_of[r] the sequence of a row. Before a sequence's first row comes its state (f32 row `slot` of ld_state) or, where it starts, zeros; the state
+// becomes n of its last row. h in bf16, or f32 with is_f32.
+FT_EXPORT int ft_token_shift(const float* x, int64_t ldx, const float* rstd, const float* w, const float* shift, const int* spans, const int* seq_of, float* state, int64_t ld_state,
+                             void* h, int64_t ldh, int is_f32, int rows, int W, cudaStream_t st) {
+  if (rows < 1 || W < 1 || !rstd || !w || !shift || !spans || !seq_of || !state || (ldx & 3) || (ldh & 3) || (ld_state & 3) || (reinterpret_cast<uintptr_t>(spans) & 15)) return FT_ERR_ARG;
+  const int quads = (W + 3) / 4, threads = quads >= 256 ? 256 : (quads + 31) & ~31, groups = (rows + SHIFT_ROWS - 1) / SHIFT_ROWS;
+  if (groups > 65535) return FT_ERR_TOO_LARGE;
+  const dim3 grid((quads + threads - 1) / threads, groups);
+  if (is_f32) token_shift_kernel<float><<<grid, threads, 0, st>>>(x, ldx, rstd, w, shift, (const int4*)spans, seq_of, state, ld_state, (float*)h, ldh, rows, W);
+  else token_shift_kernel<__nv_bfloat16><<<grid, threads, 0, st>>>(x, ldx, rstd, w, shift, (const int4*)spans, seq_of, state, ld_state, (__nv_bfloat16*)h, ldh, rows, W);
+  return (int)cudaGetLastError();
+}
+
+// out[r] = a N(z) + b N(z^2) + c N(z^3) + e for rows z of n columns, powers element by element, N(v) = v / sqrt(mean(v^2) + eps); coef: f32 {a, b, c, e}. z and out bf16, or f32 with is_f32.
+FT_EXPORT int ft_poly_norm(const void* z, int64_t ldz, const float* coef, float eps, int rows, int n, void* out, int64_t ldo, int is_f32, cudaStream_t st) {
+  if (rows < 1 || n < 1 || !coef || (ldz & 3) || (ldo & 3)) return FT_ERR_ARG;
+  if (is_f32) return dispatch_poly<float, float>(z, 1, 0, ldz, coef, eps, out, ldo, rows, n, st);
+  return dispatch_poly<__nv_bfloat16, __nv_bfloat16>(z, 1, 0, ldz, coef, eps, out, ldo, rows, n, st);
+}
+
+// The same from split-K planes [split][row][ldp] (f32) to bf16 rows.
+FT_EXPORT int ft_poly_norm_planes(const float* planes, int splits, int64_t ldp, int64_t plane_stride, const float* coef, float eps, int rows, int n, void* out, int64_t ldo,
+                                  cudaStream_t st) {
+  if (rows < 1 || splits < 1 || n < 1 || !coef || (ldp & 3) || (plane_stride & 3) || (ldo & 3)) return FT_ERR_ARG;
+  return dispatch_poly<float, __nv_bfloat16>(planes, splits, plane_stride, ldp, coef, eps, out, ldo, rows, n, st);
 }
 
 // out[r][f] = act(gate + bias) * (up + bias) for f < fp (a multiple of 8) from columns in blocks of eight gates and eight ups; kind 0: gelu (tanh form), 1: silu; bias: f32 in

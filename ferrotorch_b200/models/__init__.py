@@ -1,4 +1,4 @@
-"""Model zoo: Llama (training, tensor-parallel inference, generation), Ginisun (latent attention + mixture of experts, serving), Pufevik (attention beside a matrix memory, serving), Mepupel (state space, windowed and latent attention beside experts, serving), BERT, Whisper, Stable Diffusion, GCN, RL policies."""
+"""Model zoo: Llama (training, tensor-parallel inference, generation), Ginisun (latent attention + mixture of experts, serving), Pufevik (attention beside a matrix memory, serving), Mepupel (state space, windowed and latent attention beside experts, serving), Vemepel (differential attention in chunks, gated latent attention, averages over depth, serving), BERT, Whisper, Stable Diffusion, GCN, RL policies."""
 from . import llama, llama_gen, bert, whisper, diffusion, graph, rl
 from .llama import LlamaConfig, LlamaModel, LlamaForCausalLM, LlamaDecoderLayer
 from .llama_gen import (CachedLlama, KvCache, LlamaKvCache, LayerKvCache, GenerationConfig, generate, generate_with_streamer, beam_search, SpecDecodeConfig,
@@ -9,6 +9,7 @@ from .llama_gen import (CachedLlama, KvCache, LlamaKvCache, LayerKvCache, Genera
 from .ginisun import GinisunConfig, GinisunLayer, GinisunModel, LatentMixerConfig, MoeConfig, ExpertConfig, RandomGinisunWeights
 from .pufevik import PufevikConfig, PufevikLayer, PufevikModel, AttentionConfig, MemoryConfig, ParallelConfig, RandomPufevikWeights
 from .mepupel import MepupelConfig, MepupelLayer, MepupelModel, Mamba2Config, LatentConfig, DenseConfig, RandomMepupelWeights
+from .vemepel import VemepelConfig, VemepelLayer, VemepelModel, DifferentialConfig, GatedLatentConfig, RotaryGatedLatentConfig, RandomVemepelWeights
 from .serving import (ServingEngine, Scheduler, StepEntry, RowBatch, MemoryPlan, DecodeState, EngineCache, CachedEngineModel, CachedModelEngine)
 from .registry import Architecture, checked_weights, register_architecture, architectures, architecture_of, load_engine, load_model_config, load_checkpoint_weights
 from .llama_blocks import LlamaActivation, LlamaMLP, LlamaAttention, LlamaGpuLayer, LlamaGpuInferencer, ProfiledForwardResult

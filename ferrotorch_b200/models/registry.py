@@ -119,6 +119,17 @@ def _mepupel_engine(cfg, weights, device, dtype, max_tokens):
     return ServingEngine(MepupelModel(cfg, weights, device, dtype), max_tokens=max_tokens)
 
 
+def _vemepel_config(d: dict):
+    from .vemepel import VemepelConfig
+    return VemepelConfig.from_dict(d)
+
+
+def _vemepel_engine(cfg, weights, device, dtype, max_tokens):
+    from .serving import ServingEngine
+    from .vemepel import VemepelModel
+    return ServingEngine(VemepelModel(cfg, weights, device, dtype), max_tokens=max_tokens)
+
+
 def _llama_config(d: dict):
     from .llama import LlamaConfig
     return LlamaConfig.from_hf(d)
@@ -136,4 +147,5 @@ PRODUCTS = ("gemm_tcgen05", "gemm_2sm", "gemm_simt", "fsdp_gather", "decode")   
 register_architecture(Architecture("Ginisun", _ginisun_config, _ginisun_engine, kernels=(*PRODUCTS, "stream_ops", "moe", "latent_attn")))
 register_architecture(Architecture("Pufevik", _pufevik_config, _pufevik_engine, kernels=(*PRODUCTS, "gqa_attn", "matrix_memory", "residual_ops")))
 register_architecture(Architecture("Mepupel", _mepupel_config, _mepupel_engine, kernels=(*PRODUCTS, "gqa_attn", "latent_attn", "moe", "state_space", "residual_ops")))
+register_architecture(Architecture("Vemepel", _vemepel_config, _vemepel_engine, kernels=(*PRODUCTS, "gqa_attn", "latent_attn", "moe", "residual_ops")))
 register_architecture(Architecture("LlamaForCausalLM", _llama_config, _llama_engine, ("llama",)))

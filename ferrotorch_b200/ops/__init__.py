@@ -11,9 +11,9 @@ from .streams import DynamicTanhWeights, HyperWeights, SublayerOutput, dynamic_t
 from .moe import ExpertStack, MoeWeights, MoeSmallBuffers, MoeRouting, RouteRule, moe_rows, moe_small, gated_act, grouped_linear, interleave_gate_up
 from .latent_attention import (LatentDims, LatentWeights, LatentDecodeBuffers, latent_context, latent_attention_rows, latent_attention_decode, absorb_queries, expand_values,
                                rotary_pair_tables)
-from .residual import (DenseGatedWeights, dense_gated_rows, gated_act_planes, gated_act_rows, parallel_embed, parallel_update, residual_embed,
+from .residual import (DenseGatedWeights, DensePolyWeights, TokenShift, dense_poly_rows, depth_embed, depth_update, poly_norm_planes, poly_norm_rows, token_shift, dense_gated_rows, gated_act_planes, gated_act_rows, parallel_embed, parallel_update, residual_embed,
                        residual_update)
-from .gqa_attention import GqaDims, GqaWeights, GqaDecodeBuffers, gqa_attention_rows, gqa_attention_decode, pack_head_rows, pack_head_columns, pack_head_vector
+from .gqa_attention import GqaDims, GqaWeights, GqaDecodeBuffers, gqa_attention_rows, gqa_attention_decode, pack_head_rows, pack_head_columns, pack_head_vector, differential_blend
 from .matrix_memory import MemoryDims, MemoryWeights, matrix_memory_rows, matrix_memory_decode
 from .state_space import SsmDims, SsmWeights, SsmDecodeBuffers, state_space_rows, state_space_decode
 from . import attention

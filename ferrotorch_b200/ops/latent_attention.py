@@ -1,5 +1,6 @@
 """Latent attention (keys and values expanded from one small cached vector per token, optionally one rotated key part shared by all heads) on the kernels of
-``csrc/kernels/latent_attn.cu``. Queries may come through a latent of their own, and a layer may read the latent that an earlier layer cached.
+``csrc/kernels/latent_attn.cu``. Queries may come through a latent of their own, a layer may read the latent that an earlier layer cached, and the heads' outputs may be
+gated (per element or per head).
 
 Prompts expand keys and values per head with a GEMM and run a tcgen05 flash kernel over ragged sequences; a decode step folds ``W_uk`` into the query
 and ``W_uv`` into the output, so that it reads nothing but the cached rows. f32 data takes the folded form everywhere, on a plain kernel.
@@ -14,6 +15,7 @@ import torch
 from .. import _lib
 from ..errors import InvalidArgument
 from .gemm import gemm
+from .gqa_attention import GATE_ELEMENT, GATE_NONE
 from .moe import linear_rows
 from .streams import SublayerOutput, padded_vector, round_up
 
@@ -24,7 +26,7 @@ _SMEM_MAX = 232448
 @dataclass(frozen=True)
 class LatentDims:
     """Sizes of one latent-attention layer: per head ``dim`` plain and ``rot_dim`` (possibly 0) rotated query / key dimensions and ``vdim`` value dimensions; a
-    latent of ``rank``. The padded sizes give the layouts the kernels share: projection rows ``heads x [dim8 | rot8] | rank8 | rot``, cache rows ``[r16 | rot16]``."""
+    latent of ``rank``. The padded sizes give the layouts the kernels share: projection rows ``heads x [dim8 | rot8] | rank8 | rot8 | gate``, cache rows ``[r16 | rot16]``."""
     heads: int
     dim: int
     rot_dim: int
@@ -34,6 +36,7 @@ class LatentDims:
     eps: float
     q_rank: int = 0                      # queries from a normalised latent of this size (without a rotated part)
     own: bool = True                     # the layer has a latent of its own; otherwise it reads an earlier layer's
+    gate: int = GATE_NONE                # of the heads' outputs
 
     @property
     def dim8(self): return round_up(self.dim, 8)
@@ -50,7 +53,11 @@ class LatentDims:
     @property
     def q_cols(self): return round_up(self.q_rank, 8) if self.q_rank else self.heads * (self.dim8 + self.rot8)
     @property
-    def proj_cols(self): return self.q_cols + (self.rank8 + self.rot8 if self.own else 0)
+    def gate_col(self): return self.q_cols + (self.rank8 + self.rot8 if self.own else 0)
+    @property
+    def gate_cols(self): return 0 if self.gate == GATE_NONE else self.heads * self.v8 if self.gate == GATE_ELEMENT else self.heads
+    @property
+    def proj_cols(self): return self.gate_col + round_up(self.gate_cols, 8)
 
     def flash_tile(self) -> int:
         """Query rows per tile of the flash kernel, 0 when these sizes do not fit it."""
@@ -78,7 +85,7 @@ class LatentDims:
 
 @dataclass
 class LatentWeights:
-    """Packed projections: ``proj`` ``[proj_cols, width]`` (queries or query latent, latent, shared rotated key), ``ukv`` ``[heads * dim8 + heads * v8 (+ 16), rank32]``
+    """Packed projections: ``proj`` ``[proj_cols, width]`` (queries or query latent, latent, shared rotated key, gate), ``ukv`` ``[heads * dim8 + heads * v8 (+ 16), rank32]``
     (key, then value expansion of every head), ``out`` ``[width, heads * v8]``, ``norm`` f32; with a query latent its expansion ``uq`` ``[heads * dim8, q_rank]``
     and norm ``q_norm``."""
     dims: LatentDims
@@ -90,12 +97,12 @@ class LatentWeights:
     q_norm: Optional[torch.Tensor] = None
 
     @staticmethod
-    def pack(dims: LatentDims, q, dkv, norm, uk, uv, out, device, dtype, dq=None, q_norm=None) -> "LatentWeights":
+    def pack(dims: LatentDims, q, dkv, norm, uk, uv, out, device, dtype, dq=None, q_norm=None, gate=None) -> "LatentWeights":
         """With a query latent, ``dq`` projects to it, ``q_norm`` norms it and ``q`` expands it; ``dkv`` and ``norm`` are ``None`` where the latent is an earlier layer's."""
         D, W = dims, out.shape[0]
         H = D.heads
-        if (D.q_rank > 0) != (dq is not None) or (D.q_rank and D.rot_dim) or D.own != (dkv is not None):
-            raise InvalidArgument("latent attention: weights and sizes must agree on the query latent (which has no rotated part) and on the latent")
+        if (D.q_rank > 0) != (dq is not None) or (D.q_rank and (D.rot_dim or D.gate)) or D.own != (dkv is not None) or (D.gate != GATE_NONE) != (gate is not None):
+            raise InvalidArgument("latent attention: weights and sizes must agree on the query latent (which has no rotated part and no gate), on the latent and on the gate")
 
         def place(rows, cols):
             return torch.zeros(rows, round_up(cols, 32), device=device, dtype=dtype)
@@ -113,6 +120,12 @@ class LatentWeights:
         if D.own:
             proj[D.q_cols: D.q_cols + D.rank, :W] = dkv[: D.rank].to(device, dtype)
             proj[D.q_cols + D.rank8: D.q_cols + D.rank8 + D.rot_dim, :W] = dkv[D.rank:].to(device, dtype)
+        if gate is not None:
+            g = gate.to(device, dtype)
+            if D.gate == GATE_ELEMENT:
+                proj[D.gate_col: D.gate_col + H * D.v8].view(H, D.v8, -1)[:, : D.vdim, :W] = g.reshape(H, D.vdim, W)
+            else:
+                proj[D.gate_col: D.gate_col + H, :W] = g
         ukv = place(H * (D.dim8 + D.v8) + 16, D.rank)                  # 16 spare rows: the decode kernel reads whole 16-row blocks
         ukv[: H * D.dim8].view(H, D.dim8, -1)[:, : D.dim, : D.rank] = uk.to(device, dtype).reshape(H, D.dim, D.rank)
         ukv[H * D.dim8: H * (D.dim8 + D.v8)].view(H, D.v8, -1)[:, : D.vdim, : D.rank] = uv.to(device, dtype).reshape(H, D.vdim, D.rank)
@@ -184,6 +197,8 @@ def latent_attention_rows(h: torch.Tensor, w: LatentWeights, batch, cache: torch
               batch.ctx_rows if fill else None, cache if D.own else None, ctx if fill else None, int(f32), _lib.S())
     if fill and batch.past_slots is not None:
         _lib.call("ft_latent_ctx_gather", cache, ctx, D.row * 2, batch.past_slots, batch.past_rows, batch.past_slots.numel(), _lib.S())
+    gate = q[:, D.gate_col:] if D.gate else None
+    gating = (gate, 0 if gate is None else gate.stride(0), D.gate)
     if D.q_rank:
         q = linear_rows(q[:, : D.q_rank], w.uq)
     if flash:
@@ -191,7 +206,7 @@ def latent_attention_rows(h: torch.Tensor, w: LatentWeights, batch, cache: torch
         a = torch.empty(T, D.heads * D.v8, device=h.device, dtype=h.dtype)
         tiles = batch.tiles_for(D)
         _lib.call("ft_latent_flash", q, q.stride(0), T, kv, kv.stride(0), ctx[:, D.r16:] if D.rot_dim else None, D.row, batch.ctx_total, tiles, tiles.shape[0], D.heads, D.dim, D.rot_dim,
-                  D.vdim, D.scale, a, a.stride(0), _lib.S())
+                  D.vdim, D.scale, *gating, a, a.stride(0), _lib.S())
     else:
         full = absorb_queries(q, w)
         o = torch.empty(T, D.heads, D.r16, device=h.device, dtype=h.dtype)
@@ -200,6 +215,8 @@ def latent_attention_rows(h: torch.Tensor, w: LatentWeights, batch, cache: torch
             _lib.call("ft_latent_rows", full[r0:r1], cache, batch.block_table, batch.block_table.shape[1], batch.seq_of[r0:r1], batch.positions[r0:r1], r1 - r0,
                       D.heads, D.rot_dim, D.rank, D.scale, o[r0:r1], int(f32), _lib.S())
         a = expand_values(o, w)
+        if D.gate:
+            _lib.call("ft_latent_gate", a, a.stride(0), *gating, T, D.heads, D.v8, int(f32), _lib.S())
     y = linear_rows(a, w.out, out_f32=True)
     return SublayerOutput(planes=y.as_strided((1, T, y.shape[1]), (0, y.stride(0), 1)))
 
@@ -217,6 +234,7 @@ class LatentDecodeBuffers:
         self.lat = torch.zeros(SMALL_TOKENS, D.heads, D.r16, device=device, dtype=torch.bfloat16)
         self.ws = torch.zeros(max(b * n for b, n in enumerate(self.splits, 1)) * self.tiles * self.mt * 16 * (D.r16 + 4), device=device)
         self.attn = torch.zeros(SMALL_TOKENS, D.heads * D.v8, device=device, dtype=torch.bfloat16)
+        self.gate = torch.zeros(SMALL_TOKENS, max(D.gate_cols, 1), device=device)
         self.cq = torch.zeros(SMALL_TOKENS, round_up(max(D.q_rank, 1), 8), device=device, dtype=torch.bfloat16)[:, : D.q_rank]
 
 
@@ -226,16 +244,16 @@ def latent_attention_decode(planes: torch.Tensor, splits: int, w: LatentWeights,
     product of ``w.uq`` where queries come through a latent."""
     D, S = w.dims, _lib.S()
     bt, mb, nsplit = state.block_table, state.block_table.shape[1], b.splits[B - 1]
-    own = cache if D.own else None
+    own, gate = cache if D.own else None, b.gate if D.gate else None
     if D.q_rank:
         _lib.call("ft_latent_decode_norms", planes, splits, planes.stride(1), planes.stride(0), B, D.q_rank, D.rank, w.q_norm, w.norm, D.eps, state.positions, bt, mb,
                   b.cq, b.cq.stride(0), own, S)
         expand(b.cq)
         planes, splits, own = expand.planes, expand.splits, None
     _lib.call("ft_latent_decode_prep", planes, splits, planes.stride(1), planes.stride(0), B, D.heads, D.dim, D.rot_dim, D.rank, w.ukv, w.ukv.stride(0), w.norm, D.eps,
-              state.positions, cos, sin, bt, mb, b.q, own, S)
+              state.positions, cos, sin, bt, mb, b.q, own, D.gate_cols, gate, S)
     _lib.call("ft_latent_decode", b.q, cache, bt, mb, state.seq_lens, B, D.heads, D.rot_dim, D.rank, D.scale, nsplit, b.mt, b.ws, S)
     _lib.call("ft_latent_combine", b.ws, B, D.heads, D.rank, nsplit, b.mt, b.lat, S)
     _lib.call("ft_skinny_heads", b.lat, b.lat.stride(0), b.lat.stride(1), w.uv, w.uv.stride(0), D.v8 * w.uv.stride(0), B, D.heads, D.vdim, D.rank, b.attn,
-              b.attn.stride(0), D.v8, S)
+              b.attn.stride(0), D.v8, gate, D.gate_cols, D.v8 if D.gate == GATE_ELEMENT else 1, int(D.gate == GATE_ELEMENT), S)
     return b.attn

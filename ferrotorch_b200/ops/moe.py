@@ -1,4 +1,4 @@
-"""Mixture of experts on the kernels of ``csrc/kernels/moe.cu``: sigmoid router, the ``top`` best experts per token, experts of the clamped gated form
+"""Mixture of experts on the kernels of ``csrc/kernels/moe.cu``: sigmoid or softmax router, the ``top`` best experts per token, experts of the clamped gated form
 ``W_down (g sigmoid(slope g) (u + 1))`` with ``g = min(W_gate x, limit)`` and ``u = clamp(W_up x, -limit, limit)`` applied to ``score * x``, or of the form
 ``score * W_down (silu(W_gate x) * (W_up x))``, and an optional expert that every token passes through. The choice goes by logit or by a :class:`RouteRule`.
 
@@ -85,12 +85,14 @@ class ExpertStack:
 
 @dataclass
 class RouteRule:
-    """Experts are chosen by ``sigmoid(logit) + correction``, within the ``keep`` best of ``groups`` equal groups of neighbours (0: no groups; a group's score is the sum of
-    its two best), and weighted with the chosen sigmoids divided by their sum, times ``scale``. ``correction``: f32 ``[experts]`` on the device."""
+    """Experts are chosen by ``sigmoid(logit) + correction`` (``softmax``: by ``logit + correction``), within the ``keep`` best of ``groups`` equal groups of neighbours (0: no
+    groups; a group's score is the sum of its two best), and weighted with the chosen sigmoids divided by their sum (``softmax``: the softmax over the chosen sums), times
+    ``scale``. ``correction``: f32 ``[experts]`` on the device."""
     correction: torch.Tensor
     groups: int = 0
     keep: int = 0
     scale: float = 1.0
+    softmax: bool = False
 
 
 EXPERT_FORMS = {"clamped": 0, "silu": 1}
@@ -114,7 +116,7 @@ class MoeWeights:
     @property
     def rule_args(self) -> tuple:
         r = self.rule
-        return (r.correction, r.groups, r.keep, r.scale) if r else (None, 0, 0, 1.0)
+        return (2 if r.softmax else 1, r.correction, r.groups, r.keep, r.scale) if r else (0, None, 0, 0, 1.0)
 
     @property
     def num_experts(self) -> int:

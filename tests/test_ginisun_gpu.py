@@ -263,7 +263,7 @@ def test_one_far_key_in_prompts(dn, dr, dv):
         v = rounded(v, BF16)
         qd, kvd, krd = dev(q.reshape(T, -1), BF16), dev(np.concatenate([k.reshape(T, -1), v.reshape(T, -1)], 1), BF16), dev(kr, BF16)
         out = torch.full((T, H * D.v8), float("nan"), device="cuda", dtype=BF16)
-        _lib.call("ft_latent_flash", qd, qd.stride(0), T, kvd, kvd.stride(0), krd, krd.stride(0), T, tl, len(tiles), H, dn, dr, dv, D.scale, out, out.stride(0), _lib.S())
+        _lib.call("ft_latent_flash", qd, qd.stride(0), T, kvd, kvd.stride(0), krd, krd.stride(0), T, tl, len(tiles), H, dn, dr, dv, D.scale, None, 0, 0, out, out.stride(0), _lib.S())
         got = out.view(T, H, D.v8)[:, :, :dv].float().cpu().numpy()
         assert np.isfinite(got).all()
         for o, n in ((0, lens[0]), (lens[0], lens[1])):

@@ -163,9 +163,9 @@ def test_packed_weights_keep_every_row_where_the_kernels_look():
     d = DenseGatedWeights.pack(torch.ones(9, 5), torch.ones(9, 5), torch.ones(5, 9), "cpu", torch.float32, "silu", torch.arange(1.0, 10), 10 * torch.arange(1.0, 10), torch.ones(5))
     assert d.gu_bias.tolist() == [*range(1, 9), *range(10, 90, 10), 9] + [0] * 7 + [90] + [0] * 7 and d.down_bias.tolist() == [1] * 5 + [0] * 3
     m = MoeWeights(torch.zeros(4, 8), None, None, 8, 2)
-    assert m.rule_args == (None, 0, 0, 1.0) and m.kind == 0
+    assert m.rule_args == (0, None, 0, 0, 1.0) and m.kind == 0
     r = RouteRule(torch.zeros(8), 2, 1, 1.5)
-    assert MoeWeights(torch.zeros(4, 8), None, None, 8, 2, form="silu", rule=r).rule_args == (r.correction, 2, 1, 1.5)
+    assert MoeWeights(torch.zeros(4, 8), None, None, 8, 2, form="silu", rule=r).rule_args == (1, r.correction, 2, 1, 1.5)
 
 
 def test_size_limits_of_the_kernels():

@@ -94,7 +94,7 @@ def test_packed_weights_keep_every_row_where_the_kernels_look():
 def test_size_limits_of_the_kernels():
     L = _lib.kernels()
     for heads, kv, d, dv, sub in ((8, 1, 64, 64, 1), (8, 2, 128, 128, 1), (4, 4, 96, 100, 1), (4, 4, 192, 100, 2), (1, 1, 256, 256, 1), (2, 1, 1024, 64, 0), (130, 1, 64, 64, 0)):
-        assert L.ft_gqa_flash_subtiles(heads, kv, d, dv) == sub, (heads, kv, d, dv)
+        assert L.ft_gqa_flash_subtiles(heads, kv, d, dv, 1) == sub, (heads, kv, d, dv)
         assert GqaDims(heads, kv, d, dv, 0, 1.0, 1e-5).flash_tile() == sub * (128 // (heads // kv))
     assert GqaDims(130, 1, 64, 64, 0, 1.0, 1e-5).decode_supported() and not GqaDims(1, 1, 600, 64, 0, 1.0, 1e-5).decode_supported()
     assert MemoryDims(1, 256, 999, 1.0, 1e-5).walk_supported() and not MemoryDims(1, 272, 16, 1.0, 1e-5).walk_supported()
