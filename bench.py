@@ -44,7 +44,7 @@ def _parse():
                     help="after the timed runs, time every kernel class of one step with CUDA events (optimizer serialised on the compute "
                          "stream so that the classes add up to the step) and add the table to the JSON line")
     ap.add_argument("--serving", nargs="?", const="1k,2k,4k", default=None, metavar="SIZES",
-                    help="instead of the headline: prefill and decode throughput of the serving models (Ginisun, Pufevik and Mepupel beside Llama) on a few layers of "
+                    help="instead of the headline: prefill and decode throughput of the serving models (Ginisun, Pufevik, Mepupel and Vemepel beside Llama) on a few layers of "
                          "the named sizes with random weights, and every kernel class against its roofline")
     return ap.parse_args()
 

@@ -1,6 +1,6 @@
-"""Prefill and decode throughput of the serving models on layers of realistic size with random weights: the Ginisun, Pufevik and Mepupel decoders beside a Llama decoder
-of the same width and the same number of feed-forward neurons per token (Pufevik also has its attention sizes; its layers alternate between the two kinds; Mepupel has Ginisun's experts,
-and one layer of each kind in turn). Run through ``bench.py --serving``.
+"""Prefill and decode throughput of the serving models on layers of realistic size with random weights: the Ginisun, Pufevik, Mepupel and Vemepel decoders beside a Llama decoder
+of the same width and the same number of feed-forward neurons per token (Pufevik also has its attention sizes; its layers alternate between the two kinds; Mepupel and Vemepel have
+Ginisun's experts, and one layer of each kind in turn; every second layer of Vemepel is dense). Run through ``bench.py --serving``.
 
 Every kernel class is also timed (CUDA events around its launches, L2 flushed by the step's own traffic) against its roofline, the slower of algorithmic
 bytes / measured copy bandwidth and FLOPs / measured bf16 GEMM rate. Times of single launches below ~5 us are dominated by launch overhead.
@@ -19,6 +19,7 @@ from ferrotorch_b200.models.ginisun import GinisunConfig, GinisunModel, RandomGi
 from ferrotorch_b200.models.ginisun import ExpertConfig, MoeConfig
 from ferrotorch_b200.models.mepupel import MepupelConfig, MepupelModel, RandomMepupelWeights
 from ferrotorch_b200.models.pufevik import PufevikConfig, PufevikModel, RandomPufevikWeights
+from ferrotorch_b200.models.vemepel import RandomVemepelWeights, VemepelConfig, VemepelModel
 from ferrotorch_b200.models.llama_infer import LlamaTPEngine, TPContext
 from ferrotorch_b200.models.serving import ServingEngine, StepEntry
 
@@ -210,7 +211,7 @@ def run_pufevik(size, layers, batch, prompt, ctx, steps, kernels=True):
                  "ft_mm_finish": (T * M.heads * M.v16 * 8, 0)}
         def label(fn, raw):
             if fn == "ft_gqa_flash":
-                return "flash (window)" if raw[14] else "flash (full)"
+                return "flash (window)" if raw[15] else "flash (full)"
             if fn == "ft_mm_walk":
                 return "memory walk (outputs)" if raw[17] else "memory walk (states)"
             return classify(fn, raw)
@@ -248,7 +249,7 @@ def run_pufevik(size, layers, batch, prompt, ctx, steps, kernels=True):
                  "attention (window)": (2 * batch * min(L, win) * D.row, 0), "attention (full)": (2 * batch * L * D.row, 0), "ft_mm_decode": (2 * batch * M.state_size * 4, 0)}
         def label_d(fn, raw):
             if fn == "ft_gqa_decode":
-                return "attention (window)" if raw[11] else "attention (full)"
+                return "attention (window)" if raw[12] else "attention (full)"
             return classify(fn, raw)
         dtable = kernel_table(one, label_d, roofs, bw, fl)
     eng.check()
@@ -348,6 +349,101 @@ def run_mepupel(size, layers, batch, prompt, ctx, steps, kernels=True):
             "active_experts": active, "prefill_kernels": table, "decode_kernels": dtable}
 
 
+def run_vemepel(size, layers, batch, prompt, ctx, steps, kernels=True):
+    """Layers in turn: differential attention in chunks, latent attention with a rotated part, without positions, differential attention on the first one's keys and values; dense
+    and mixture-of-experts feed-forwards alternate."""
+    from ferrotorch_b200.models.serving import RowBatch
+    bw, fl, _ = peaks()
+    s = SIZES[size]
+    W, T, F, E, top, R = s["width"], prompt, s["ff"], s["experts"], s["top"], s["kv_rank"]
+    H, DF = W // 128, top * F + s["shared_ff"]
+    G = max(1, H // 4)
+    chunk = 1024
+    att = dict(heads=H, kv_heads=G, dim=64, vdim=128, scale=64 ** -0.5, diff=0.5, mask=dict(size=chunk))
+    lat = dict(heads=H, dim=128, vdim=128, kv_rank=R, scale=128 ** -0.5)
+    cfg = VemepelConfig.pattern(("arls" * layers)[:layers], VOCAB, W, att, lat, dict(lat, rot_dim=64, rot=dict(base=1e4, dims=64)), MoeConfig(E, top, ExpertConfig(F)), dense_ff=DF)
+    eng = ServingEngine(VemepelModel(cfg, RandomVemepelWeights(cfg)), max_tokens=max(batch * (ctx + steps * 4 + 64), prompt + 64), max_sequences=batch + 1)
+    g = torch.Generator().manual_seed(1)
+    ids = torch.randint(0, VOCAB, (prompt,), generator=g).tolist()
+    entry = [StepEntry("p", ids, [prompt - 1])]
+    eng._admit(entry)
+    rb = RowBatch(entry, eng.cache, eng.device, eng.max_blocks)
+    device_prefill = lambda: eng.model.forward_rows(rb, eng.cache)          # the device part: tables of the batch are built once
+    pre_ms = timed(device_prefill)
+    A = next(l.attn.dims for l in eng.model.layers if l.attn)
+    P, L = (next((l.latent.dims for l in eng.model.layers if l.latent and bool(l.latent.dims.rot_dim) == rotated), None) for rotated in (True, False))
+    n_layers, pairs, nkv = len(eng.model.layers), T * top, H * (L.dim8 + L.v8)
+    deep = sum(range(1, n_layers + 1)) / n_layers                           # results that an average reads, over the layers
+    common = {(A.qkv_cols, W): "projection gemm (attention)", (A.k_col, W): "projection gemm (attention, shared keys)", (P.proj_cols, W): "projection gemm (latent, rotated)",
+              (L.proj_cols, W): "projection gemm (latent)", (W, A.out_cols): "output gemm", (DF, W): "up gemm", (W, DF): "down gemm",
+              ("grouped", 2 * F, W): "experts gate/up gemm", ("grouped", W, F): "experts down gemm"}
+    table = dtable = active = None
+    def g_(n, k, out=2, m=T): return (2 * (m * k + n * k) + out * m * n, 2 * m * n * k)
+    if kernels:
+        names = dict(common)
+        names.update({(nkv, R): "key/value expansion gemm", (E, W): "router gemm"})
+        seen = sum(min(i % chunk, chunk) + 1 for i in range(T))             # keys that the chunks' queries see
+        roofs = {names[k]: g_(k[0], k[1], 4 if "output" in names[k] or "down" in names[k] or "router" in names[k] else 2) for k in names if k[0] != "grouped"}
+        roofs.update({
+            "experts gate/up gemm": (2 * (pairs * W + E * 2 * F * W + pairs * 2 * F), 4 * pairs * F * W), "experts down gemm": (2 * (pairs * W + E * F * W + pairs * F), 2 * pairs * F * W),
+            "ft_gqa_flash": (2 * T * (A.qkv_cols + A.out_cols), 2 * 2 * H * seen * (A.dim + A.vdim)), "ft_gqa_prep": (4 * T * (A.qkv_cols - A.k_col), 0),
+            "flash (latent, rotated)": (2 * T * (H * (P.dim8 + P.rot8) + nkv + 2 * H * P.v8), H * T * T * (P.dim + P.rot_dim + P.vdim)),
+            "flash (latent)": (2 * T * (H * L.dim8 + nkv + H * L.v8), H * T * T * (L.dim + L.vdim)),
+            "prep (latent, rotated)": (2 * T * (2 * H * P.rot8 + R + P.rot8 + 2 * P.row), 0), "prep (latent)": (2 * T * (R + 2 * L.row), 0),
+            "ft_moe_gather": (4 * pairs * W, 0), "ft_moe_act": (pairs * F * 6, 0), "ft_moe_topk": (T * E * 4, 0), "ft_poly_norm": (4 * T * DF, 0), "ft_token_shift": (6 * T * W, 0),
+            "ft_residual_update": (T * W * 14, 0), "ft_depth_update": (T * W * (4 * deep + 12 + (4 + 2 * top) / 2), 0), "ft_depth_embed": (T * W * 10, 0)})
+        classify = _by_shape(names)
+        def label(fn, raw):
+            if fn == "ft_latent_flash":
+                return "flash (latent, rotated)" if raw[12] else "flash (latent)"
+            if fn == "ft_latent_prep":
+                return "prep (latent, rotated)" if raw[5] else "prep (latent)"
+            return classify(fn, raw)
+        table = kernel_table(device_prefill, label, roofs, bw, fl)
+    eng.release("p")
+    seqs = [f"s{i}" for i in range(batch)]
+    for q in seqs:
+        eng.step([StepEntry(q, torch.randint(0, VOCAB, (ctx,), generator=g).tolist(), [])])
+    eng.decode_greedy(seqs, [1] * batch, 4)
+    best = []
+    for _ in range(3):
+        e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        torch.cuda.synchronize()
+        e0.record()
+        eng.decode_greedy(seqs, [1] * batch, steps)
+        e1.record()
+        torch.cuda.synchronize()
+        best.append(e0.elapsed_time(e1) / steps)
+    dec_ms = statistics.median(best)
+    if kernels:
+        for q in seqs:
+            eng.cache.reserve(q, eng.cache.lengths[q] + 1)
+        eng._load_state(seqs, [1 + i for i in range(batch)])
+        positions, lens, tokens = eng.state.positions.clone(), eng.state.seq_lens.clone(), eng.state.tokens.clone()
+        def one():
+            eng.state.positions.copy_(positions); eng.state.seq_lens.copy_(lens); eng.state.tokens.copy_(tokens)
+            eng.model.decode(eng.state, batch, eng.cache)
+        one()
+        active = int(eng.model._moe_buffers.n_active)               # experts in use (of the last layer; the layers are alike)
+        n = eng.cache.lengths[seqs[0]] + 1
+        names = dict(common)
+        names[(VOCAB, W)] = "head gemm"
+        roofs = {names[k]: (2 * k[0] * k[1], 0) for k in names if k[0] != "grouped"}
+        roofs.update({"ft_gqa_decode": (2 * batch * ((n - 1) % chunk + 1) * A.row, 0),
+                      "attention (latent, rotated)": (2 * batch * n * P.row, 2 * batch * H * n * (P.row + P.r16)), "attention (latent)": (2 * batch * n * L.row, 2 * batch * H * n * (L.row + L.r16)),
+                      "ft_latent_decode_prep": (2 * H * L.dim8 * R, 0), "ft_skinny_heads": (2 * H * L.v8 * R, 0), "ft_moe_gate_up_small": (4 * W * active * F, 0),
+                      "ft_moe_down_small": (2 * W * active * F, 0)})
+        classify_d = _by_shape(names)
+        def label_d(fn, raw):
+            if fn == "ft_latent_decode":
+                return "attention (latent, rotated)" if raw[7] else "attention (latent)"
+            return classify_d(fn, raw)
+        dtable = kernel_table(one, label_d, roofs, bw, fl)
+    eng.check()
+    return {"prefill_ms": round(pre_ms, 3), "prefill_tokens_per_s": round(prompt / pre_ms * 1e3), "decode_ms_per_step": round(dec_ms, 4), "decode_tokens_per_s": round(batch / dec_ms * 1e3),
+            "active_experts": active, "prefill_kernels": table, "decode_kernels": dtable}
+
+
 def run_llama(size, layers, batch, prompt, ctx, steps, kernels=True):
     bw, fl, _ = peaks()
     s = SIZES[size]
@@ -406,7 +502,7 @@ def main(sizes="1k,2k,4k", layers=4, batch=8, prompt=4096, ctx=2048, steps=64, k
     res = {}
     for size in sizes.split(","):
         res[size] = {}
-        for name, run in (("ginisun", run_ginisun), ("pufevik", run_pufevik), ("mepupel", run_mepupel), ("llama", run_llama)):
+        for name, run in (("ginisun", run_ginisun), ("pufevik", run_pufevik), ("mepupel", run_mepupel), ("vemepel", run_vemepel), ("llama", run_llama)):
             if models and name not in models.split(","):
                 continue
             res[size][name] = run(size, layers, batch, prompt, ctx, steps, kernels)

@@ -194,7 +194,7 @@ class VemepelConfig:
         for i, l in enumerate(self.layers):
             where, m, f = f"Vemepel: layer {i}", l.mixer, l.mlp
             m.validate(where)
-            if self.source(i) != i:
+            if getattr(m, "kv_from", None) is not None:
                 j = self.layers[m.kv_from].mixer if 0 <= m.kv_from < i else None
                 if not isinstance(j, DifferentialConfig) or j.kv_from is not None or (j.kv_heads, j.dim, j.vdim) != (m.kv_heads, m.dim, m.vdim):
                     raise InvalidArgument(f"{where}: kv_from must name an earlier attention layer with keys and values of its own and the same kv_heads, dim and vdim")

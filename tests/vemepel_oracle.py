@@ -109,8 +109,8 @@ def latent_mixer(h, W, m, eps):
     c, kr = latent_of(h, W, m, eps)
     k = np.concatenate([(c @ W["uk"].T).reshape(T, H, d), np.repeat(kr[:, None], H, 1)], -1)
     o = attend(q, k, (c @ W["uv"].T).reshape(T, H, dv), m["scale"], visible(T))
-    g = sigmoid(h @ W["g"].T)
-    return (o * (g[:, :, None] if g.shape[1] == H and H * dv != H else g.reshape(T, H, dv))).reshape(T, H * dv) @ W["o"].T
+    g = sigmoid(h @ W["g"].T).reshape(T, H, -1)                      # one or ``vdim`` per head
+    return (o * g).reshape(T, H * dv) @ W["o"].T
 
 
 # -- feed-forward ---------------------------------------------------------------------------------------------------------------------------
@@ -185,3 +185,55 @@ def bf16(a):
     """Values rounded to bf16."""
     u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
     return (((u.astype(np.uint64) + 0x7FFF + ((u >> 16) & 1)) >> 16) << 16).astype(np.uint32).view(np.float32).reshape(np.shape(a))
+
+
+def random_model(seed, kinds="arl", vocab=90, width=56, logit_scale=0.7, eps=1e-5, heads=4, kv_heads=2, dim=12, vdim=20, scale=None, diff=0.35, chunk=24, kv_from=None, lat_heads=3,
+                 lat_dim=16, lat_vdim=20, kv_rank=32, rot=8, base=10000.0, mlp="moe", ff=40, dense_ff=72, experts=8, top=3, overrides=None):
+    """A configuration with one layer per letter of ``kinds`` (``a``: differential attention, ``l``: latent attention without positions, ``r``: with a rotated part) and random
+    weights rounded to bf16. ``overrides[i]`` replaces keyword values for layer i; ``mlp`` is ``moe``, ``dense`` or ``None``; ``chunk=0`` leaves the chunks out."""
+    rng = np.random.default_rng(seed)
+
+    def mat(o, i, s=1.0):
+        return bf16(rng.standard_normal((o, i)) * s / math.sqrt(i))
+
+    def vec(n, mean=0.0, s=0.2):
+        return bf16(mean + s * rng.standard_normal(n))
+    W, layers = {"embed": bf16(rng.standard_normal((vocab, width)))}, []
+    given = {k: v for k, v in locals().items() if k in ("heads kv_heads dim vdim scale diff chunk kv_from lat_heads lat_dim lat_vdim kv_rank rot base mlp ff dense_ff experts top").split()}
+    for i, kind in enumerate(kinds):
+        o, p = dict(given, **(overrides or {}).get(i, {})), f"l{i}."
+        q = p + "mix."
+        W.update({p + "norm1": vec(width), p + "norm1b": vec(width, -0.2), p + "shift": bf16(rng.uniform(0.0, 1.0, width)), p + "dwa": vec(i + 2, 0.1, 0.3)})
+        W[p + "dwa"][-1] += 1.0
+        W[p + "dwa"] = bf16(W[p + "dwa"])
+        if kind == "a":
+            H, G, d, dv = o["heads"], o["kv_heads"], o["dim"], o["vdim"]
+            W.update({q + "q": mat(2 * H * d, width, 1.5), q + "o": mat(width, H * dv), **{q + n: vec(d, 0.0, 0.3) for n in ("lq1", "lk1", "lq2", "lk2")}})
+            m = dict(heads=H, kv_heads=G, dim=d, vdim=dv, scale=o["scale"] or d ** -0.5, diff=o["diff"])
+            if o["kv_from"] is None:
+                W.update({q + "k": mat(2 * G * d, width, 1.5), q + "v": mat(G * dv, width)})
+            else:
+                m["kv_from"] = o["kv_from"]
+            if o["chunk"]:
+                m["mask"] = dict(size=o["chunk"])
+        else:
+            H, d, dv, r, e = o["lat_heads"], o["lat_dim"], o["lat_vdim"], o["kv_rank"], o["rot"] if kind == "r" else 0
+            W.update({q + "q": mat(H * (d + e), width, 1.5), q + "dkv": mat(r + e, width), q + "dkv.norm": vec(r, 1.0), q + "uk": mat(H * d, r, 1.5), q + "uv": mat(H * dv, r),
+                      q + "g": mat(H * dv if e else H, width, 1.5), q + "o": mat(width, H * dv)})
+            m = dict(heads=H, dim=d, vdim=dv, kv_rank=r, scale=o["scale"] or (d + e) ** -0.5)
+            if e:
+                m.update(rot_dim=e, rot=dict(base=o["base"], dims=e))
+        f, F = p + "mlp.", None
+        if o["mlp"]:
+            W.update({p + "norm2": vec(width), p + "norm2b": vec(width, -0.2)})
+        if o["mlp"] == "dense":
+            F = dict(kind="dense", ff=o["dense_ff"])
+            W.update({f + "up": mat(o["dense_ff"], width, 1.5), f + "down": mat(width, o["dense_ff"]), f + "act": vec(4, 0.3, 0.5)})
+        elif o["mlp"] == "moe":
+            F = dict(kind="moe", router=dict(experts=o["experts"], top=o["top"]), expert=dict(ff=o["ff"]))
+            W.update({f + "router": mat(o["experts"], width, 2.0), f + "router.b": vec(o["experts"], 0.0, 0.5)})
+            for n in range(o["experts"]):
+                W.update({f"{f}e{n}.gate": mat(o["ff"], width, 1.5), f"{f}e{n}.up": mat(o["ff"], width), f"{f}e{n}.down": mat(width, o["ff"])})
+        layers.append(dict(type=dict(a="attention", l="latent_attention", r="latent_attention_2")[kind], mixer=m, mlp=F))
+    W["final.norm"], W["head"] = vec(width), mat(vocab, width, 2.0)
+    return dict(architecture="Vemepel", vocab=vocab, width=width, norm=dict(eps=eps), logit_scale=logit_scale, layers=layers), W
