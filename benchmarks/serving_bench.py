@@ -358,7 +358,7 @@ def run_vemepel(size, layers, batch, prompt, ctx, steps, kernels=True):
     W, T, F, E, top, R = s["width"], prompt, s["ff"], s["experts"], s["top"], s["kv_rank"]
     H, DF = W // 128, top * F + s["shared_ff"]
     G = max(1, H // 4)
-    chunk = 1024
+    chunk = 1280                                        # not a divisor of the context: the decoded tokens' chunk is three quarters full
     att = dict(heads=H, kv_heads=G, dim=64, vdim=128, scale=64 ** -0.5, diff=0.5, mask=dict(size=chunk))
     lat = dict(heads=H, dim=128, vdim=128, kv_rank=R, scale=128 ** -0.5)
     cfg = VemepelConfig.pattern(("arls" * layers)[:layers], VOCAB, W, att, lat, dict(lat, rot_dim=64, rot=dict(base=1e4, dims=64)), MoeConfig(E, top, ExpertConfig(F)), dense_ff=DF)

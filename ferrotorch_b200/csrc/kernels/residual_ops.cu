@@ -66,9 +66,9 @@ __global__ void __launch_bounds__(256) residual_embed_kernel(const int64_t* __re
 }
 
 constexpr int UPD_THREADS = 256;
-// NV: float4 columns per thread
-template <int NV, typename H>
-__global__ void __launch_bounds__(UPD_THREADS) residual_update_kernel(float* __restrict__ x, int64_t ldx, const float* __restrict__ y, int planes, size_t pstride, int64_t ldy,
+// NV: float4 columns per thread, of TH threads
+template <int NV, int TH, typename H>
+__global__ void __launch_bounds__(TH) residual_update_kernel(float* __restrict__ x, int64_t ldx, const float* __restrict__ y, int planes, size_t pstride, int64_t ldy,
                                                                       const float* __restrict__ w, const float* __restrict__ w_last, float eps, H* __restrict__ h,
                                                                       int64_t ldh, int ncta, int W, int cols, int store_x) {
   namespace cg = cooperative_groups;
@@ -79,7 +79,7 @@ __global__ void __launch_bounds__(UPD_THREADS) residual_update_kernel(float* __r
   float4 wv[NV];                                    // weights do not depend on the predecessor
 #pragma unroll
   for (int i = 0; i < NV; i++) {
-    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    const int c = c0 + (i * TH + threadIdx.x) * 4;
     wv[i] = c < cend ? *reinterpret_cast<const float4*>(w + c) : make_float4(0.f, 0.f, 0.f, 0.f);
   }
   pdl_wait();
@@ -99,7 +99,7 @@ __global__ void __launch_bounds__(UPD_THREADS) residual_update_kernel(float* __r
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; i++) {
-    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    const int c = c0 + (i * TH + threadIdx.x) * 4;
     v[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
     if (c < cend) {
       xv[i] = *reinterpret_cast<const float4*>(xr + c);
@@ -125,7 +125,7 @@ __global__ void __launch_bounds__(UPD_THREADS) residual_update_kernel(float* __r
   float s2 = 0.f;
 #pragma unroll
   for (int i = 0; i < NV; i++) {
-    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    const int c = c0 + (i * TH + threadIdx.x) * 4;
     xv[i] = make_float4(xv[i].x + v[i].x * rstd * wv[i].x, xv[i].y + v[i].y * rstd * wv[i].y, xv[i].z + v[i].z * rstd * wv[i].z, xv[i].w + v[i].w * rstd * wv[i].w);
     if (c < cend) {
       xv[i] = keep4(xv[i], c, W);
@@ -138,7 +138,7 @@ __global__ void __launch_bounds__(UPD_THREADS) residual_update_kernel(float* __r
     const float r2 = 1.f / sqrtf(row_sum(s2, 1) / (float)W + eps);
 #pragma unroll
     for (int i = 0; i < NV; i++) {
-      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      const int c = c0 + (i * TH + threadIdx.x) * 4;
       if (c < cend) {
         const float4 l = *reinterpret_cast<const float4*>(w_last + c);
         put4(h + (size_t)row * ldh + c, make_float4(xv[i].x * r2 * l.x, xv[i].y * r2 * l.y, xv[i].z * r2 * l.z, xv[i].w * r2 * l.w));
@@ -281,8 +281,9 @@ FT_DEVICE float4 shift4(float4 n, float4 before, float4 s) {
   return make_float4(n.x + (before.x - n.x) * s.x, n.y + (before.y - n.y) * s.y, n.z + (before.z - n.z) * s.z, n.w + (before.w - n.w) * s.w);
 }
 
-template <int NV, bool EMBED, typename H>
-__global__ void __launch_bounds__(UPD_THREADS) depth_update_kernel(DepthArgs<H> A, const int64_t* __restrict__ ids, const H* __restrict__ table, int64_t ld_table, int64_t vocab,
+// TH threads per CTA: at most two float4 columns a thread, of which it holds three sets
+template <int NV, int TH, bool EMBED, typename H>
+__global__ void __launch_bounds__(TH) depth_update_kernel(DepthArgs<H> A, const int64_t* __restrict__ ids, const H* __restrict__ table, int64_t ld_table, int64_t vocab,
                                                                    int ncta, int W, int cols) {
   namespace cg = cooperative_groups;
   __shared__ float red[32];
@@ -308,7 +309,7 @@ __global__ void __launch_bounds__(UPD_THREADS) depth_update_kernel(DepthArgs<H> 
     const int64_t id = ids[row];
 #pragma unroll
     for (int i = 0; i < NV; i++) {
-      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      const int c = c0 + (i * TH + threadIdx.x) * 4;
       xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (c < cend) {
         if (id >= 0 && id < vocab) xv[i] = keep4(get4(table + (size_t)id * ld_table + c), c, W);
@@ -318,14 +319,15 @@ __global__ void __launch_bounds__(UPD_THREADS) depth_update_kernel(DepthArgs<H> 
       }
     }
   } else {
-    float4 v[NV];
+    float4 v[NV], old[NV];
     float ss = 0.f;
     const float last = A.avg[A.count];
 #pragma unroll
     for (int i = 0; i < NV; i++) {
-      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
-      v[i] = xv[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+      const int c = c0 + (i * TH + threadIdx.x) * 4;
+      v[i] = xv[i] = old[i] = make_float4(0.f, 0.f, 0.f, 0.f);
       if (c < cend) {
+        old[i] = *reinterpret_cast<const float4*>(xr + c);
         if (A.planes) add_planes(v[i], A.y + (size_t)row * A.ldy + c, A.planes, A.pstride);
 #pragma unroll 4
         for (int k = 0; k < A.top; k++) {
@@ -341,11 +343,10 @@ __global__ void __launch_bounds__(UPD_THREADS) depth_update_kernel(DepthArgs<H> 
     const float rstd = 1.f / sqrtf(row_sum(ss, 0) / (float)W + A.eps);
 #pragma unroll
     for (int i = 0; i < NV; i++) {
-      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      const int c = c0 + (i * TH + threadIdx.x) * 4;
       if (c < cend) {
-        float4 r = *reinterpret_cast<const float4*>(xr + c);
-        const float4 w = *reinterpret_cast<const float4*>(A.w_out + c);
-        r = keep4(make_float4(r.x + v[i].x * rstd * w.x, r.y + v[i].y * rstd * w.y, r.z + v[i].z * rstd * w.z, r.w + v[i].w * rstd * w.w), c, W);
+        const float4 w = *reinterpret_cast<const float4*>(A.w_out + c), o = old[i];
+        const float4 r = keep4(make_float4(o.x + v[i].x * rstd * w.x, o.y + v[i].y * rstd * w.y, o.z + v[i].z * rstd * w.z, o.w + v[i].w * rstd * w.w), c, W);
         fma4(xv[i], last, r);
         if (A.store) {
           *reinterpret_cast<float4*>(res + A.count * A.rstride + c) = r;
@@ -363,7 +364,7 @@ __global__ void __launch_bounds__(UPD_THREADS) depth_update_kernel(DepthArgs<H> 
     const bool first = A.shift && A.positions[row] == 0;
 #pragma unroll
     for (int i = 0; i < NV; i++) {
-      const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+      const int c = c0 + (i * TH + threadIdx.x) * 4;
       if (c < cend) {
         float4 n = mul4(xv[i], r2, *reinterpret_cast<const float4*>(A.w_next + c));
         if (A.shift) {
@@ -412,36 +413,15 @@ __global__ void __launch_bounds__(256) token_shift_kernel(const float* __restric
 }
 
 // ------------------------------------------------------------------------------------------------------------
-// polynomial of normed powers: one row per cluster as in the updates above
+// polynomial of normed powers
 // ------------------------------------------------------------------------------------------------------------
-template <int NV, typename I, typename O>
-__global__ void __launch_bounds__(UPD_THREADS) poly_norm_kernel(const I* __restrict__ z, int planes, size_t pstride, int64_t ldz, const float* __restrict__ coef, float eps,
-                                                                O* __restrict__ out, int64_t ldo, int ncta, int W, int cols) {
-  namespace cg = cooperative_groups;
-  __shared__ float red[3][32];
-  __shared__ float cta_ss[3];
-  cg::cluster_group cluster = cg::this_cluster();
-  const int row = blockIdx.x / ncta, c0 = blockIdx.x % ncta * cols, cend = min(W, c0 + cols), warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  pdl_wait();
-  pdl_launch_dependents();
-  float4 v[NV];
-  float s[3] = {0.f, 0.f, 0.f};                      // sums of z^2, z^4 and z^6
-#pragma unroll
-  for (int i = 0; i < NV; i++) {
-    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
-    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
-    if (c < cend) {
-      if constexpr (sizeof(I) == 4) add_planes(v[i], z + (size_t)row * ldz + c, planes, pstride);
-      else v[i] = get4(z + (size_t)row * ldz + c);
-      v[i] = keep4(v[i], c, W);
-      const float e[4] = {v[i].x, v[i].y, v[i].z, v[i].w};
-#pragma unroll
-      for (int k = 0; k < 4; k++) {
-        const float q = e[k] * e[k];
-        s[0] += q; s[1] += q * q; s[2] += q * q * q;
-      }
-    }
-  }
+FT_DEVICE void add_powers(float (&s)[3], float z) {
+  const float q = z * z, f = q * q;
+  s[0] += q; s[1] += f; s[2] += f * q;
+}
+// sums of z^2, z^4 and z^6 over a CTA
+FT_DEVICE void block_powers(float (&s)[3], float (*red)[32]) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
 #pragma unroll
   for (int k = 0; k < 3; k++) {
     s[k] = warp_sum(s[k]);
@@ -451,9 +431,46 @@ __global__ void __launch_bounds__(UPD_THREADS) poly_norm_kernel(const I* __restr
 #pragma unroll
   for (int k = 0; k < 3; k++) {
     s[k] = 0.f;
-#pragma unroll
-    for (int i = 0; i < UPD_THREADS / 32; i++) s[k] += red[k][i];
+    for (int i = 0; i < warps; i++) s[k] += red[k][i];
   }
+}
+struct PolyNorm {
+  float a, b, d, e;
+  FT_DEVICE PolyNorm(const float (&s)[3], const float* coef, float eps, int W) {
+    const float inv = 1.f / (float)W;
+    a = coef[0] / sqrtf(s[0] * inv + eps);
+    b = coef[1] / sqrtf(s[1] * inv + eps);
+    d = coef[2] / sqrtf(s[2] * inv + eps);
+    e = coef[3];
+  }
+  FT_DEVICE float operator()(float t) const { return ((d * t + b) * t + a) * t + e; }
+};
+
+// one row per cluster as in the updates above
+template <int NV, typename I, typename O>
+__global__ void __launch_bounds__(UPD_THREADS) poly_norm_kernel(const I* __restrict__ z, int planes, size_t pstride, int64_t ldz, const float* __restrict__ coef, float eps,
+                                                                O* __restrict__ out, int64_t ldo, int ncta, int W, int cols) {
+  namespace cg = cooperative_groups;
+  __shared__ float red[3][32];
+  __shared__ float cta_ss[3];
+  cg::cluster_group cluster = cg::this_cluster();
+  const int row = blockIdx.x / ncta, c0 = blockIdx.x % ncta * cols, cend = min(W, c0 + cols);
+  pdl_wait();
+  pdl_launch_dependents();
+  float4 v[NV];
+  float s[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
+    v[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (c < cend) {
+      if constexpr (sizeof(I) == 4) add_planes(v[i], z + (size_t)row * ldz + c, planes, pstride);
+      else v[i] = get4(z + (size_t)row * ldz + c);
+      v[i] = keep4(v[i], c, W);
+      add_powers(s, v[i].x); add_powers(s, v[i].y); add_powers(s, v[i].z); add_powers(s, v[i].w);
+    }
+  }
+  block_powers(s, red);
   if (ncta > 1) {
     if (threadIdx.x < 3) cta_ss[threadIdx.x] = threadIdx.x == 0 ? s[0] : threadIdx.x == 1 ? s[1] : s[2];
     cluster.sync();
@@ -463,15 +480,52 @@ __global__ void __launch_bounds__(UPD_THREADS) poly_norm_kernel(const I* __restr
       for (int r = 0; r < ncta; r++) s[k] += *cluster.map_shared_rank(&cta_ss[k], r);
     }
   }
-  const float inv = 1.f / (float)W;
-  const float a = coef[0] / sqrtf(s[0] * inv + eps), b = coef[1] / sqrtf(s[1] * inv + eps), d = coef[2] / sqrtf(s[2] * inv + eps), e0 = coef[3];
-  auto f = [&](float t) { return ((d * t + b) * t + a) * t + e0; };
+  const PolyNorm f(s, coef, eps, W);
 #pragma unroll
   for (int i = 0; i < NV; i++) {
     const int c = c0 + (i * UPD_THREADS + threadIdx.x) * 4;
     if (c < cend) put4(out + (size_t)row * ldo + c, keep4(make_float4(f(v[i].x), f(v[i].y), f(v[i].z), f(v[i].w)), c, W));
   }
   if (ncta > 1) cluster.sync();                     // nobody leaves while a partner may still read its shared memory
+}
+
+// many bf16 rows: one CTA each, which keeps the row in registers as it was loaded (16 bytes at a time; pitches are multiples of eight)
+template <int NV>
+__global__ void __launch_bounds__(UPD_THREADS) poly_norm_rows_kernel(const __nv_bfloat16* __restrict__ z, int64_t ldz, const float* __restrict__ coef, float eps,
+                                                                     __nv_bfloat16* __restrict__ out, int64_t ldo, int W) {
+  __shared__ float red[3][32];
+  const __nv_bfloat16* zr = z + (size_t)blockIdx.x * ldz;
+  bf16x8 v[NV];
+  float s[3] = {0.f, 0.f, 0.f};
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = (i * UPD_THREADS + threadIdx.x) * 8;
+    if (c < W) v[i] = *reinterpret_cast<const bf16x8*>(zr + c);
+  }
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = (i * UPD_THREADS + threadIdx.x) * 8;
+    if (c < W) {
+      float x[8];
+      bf16x8_to_float(v[i], x);
+#pragma unroll
+      for (int e = 0; e < 8; e++)
+        if (c + e < W) add_powers(s, x[e]);
+    }
+  }
+  block_powers(s, red);
+  const PolyNorm f(s, coef, eps, W);
+#pragma unroll
+  for (int i = 0; i < NV; i++) {
+    const int c = (i * UPD_THREADS + threadIdx.x) * 8;
+    if (c < W) {
+      float x[8];
+      bf16x8_to_float(v[i], x);
+#pragma unroll
+      for (int e = 0; e < 8; e++) x[e] = c + e < W ? f(x[e]) : 0.f;
+      *reinterpret_cast<bf16x8*>(out + (size_t)blockIdx.x * ldo + c) = float_to_bf16x8(x);
+    }
+  }
 }
 
 // ------------------------------------------------------------------------------------------------------------
@@ -558,24 +612,6 @@ __global__ void __launch_bounds__(128) gated_act_planes_kernel(const float* __re
   put4(out + (size_t)r * ldo + q * 4, gated4<false>(g, u, kind));
 }
 
-template <int NV, typename H>
-int launch_update(int ncta, int rows, cudaStream_t st, float* x, int64_t ldx, const float* y, int planes, int64_t pstride, int64_t ldy, const float* w, const float* w_last,
-                  float eps, H* h, int64_t ldh, int W, int cols, int store) {
-  cudaLaunchConfig_t cfg = {};
-  cfg.gridDim = dim3(ncta * rows);
-  cfg.blockDim = dim3(UPD_THREADS);
-  cfg.stream = st;
-  cudaLaunchAttribute attr[2];
-  attr[0].id = cudaLaunchAttributeClusterDimension;
-  attr[0].val.clusterDim.x = ncta;
-  attr[0].val.clusterDim.y = attr[0].val.clusterDim.z = 1;
-  attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
-  attr[1].val.programmaticStreamSerializationAllowed = 1;
-  cfg.attrs = attr;
-  cfg.numAttrs = ft_pdl_enabled() ? 2 : 1;
-  return (int)cudaLaunchKernelEx(&cfg, residual_update_kernel<NV, H>, x, ldx, y, planes, (size_t)pstride, ldy, w, w_last, eps, h, ldh, ncta, W, cols, store);
-}
-
 // how a row of W columns is spread: CTAs of its cluster, columns of a CTA, float4 columns of a thread
 struct RowSpread { int ncta, cols, nv; };
 RowSpread row_spread(int rows, int W) {
@@ -589,10 +625,10 @@ RowSpread row_spread(int rows, int W) {
 
 // one row per cluster of sp.ncta CTAs
 template <typename... K, typename... A>
-int launch_rows(const RowSpread& sp, int rows, cudaStream_t st, void (*kernel)(K...), A&&... args) {
+int launch_rows(const RowSpread& sp, int rows, int threads, cudaStream_t st, void (*kernel)(K...), A&&... args) {
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(sp.ncta * rows);
-  cfg.blockDim = dim3(UPD_THREADS);
+  cfg.blockDim = dim3(threads);
   cfg.stream = st;
   cudaLaunchAttribute attr[2];
   attr[0].id = cudaLaunchAttributeClusterDimension;
@@ -609,11 +645,11 @@ template <bool EMBED, typename H>
 int dispatch_depth(const DepthArgs<H>& A, const int64_t* ids, const void* table, int64_t ld_table, int64_t vocab, int rows, int W, cudaStream_t st) {
   const RowSpread sp = row_spread(rows, W);
   if (sp.nv > 8) return FT_ERR_TOO_LARGE;
-#define FT_DU(N) return launch_rows(sp, rows, st, depth_update_kernel<N, EMBED, H>, A, ids, (const H*)table, ld_table, vocab, sp.ncta, W, sp.cols)
-  if (sp.nv <= 1) FT_DU(1);
-  if (sp.nv <= 2) FT_DU(2);
-  if (sp.nv <= 4) FT_DU(4);
-  FT_DU(8);
+#define FT_DU(N, TH) return launch_rows(sp, rows, TH, st, depth_update_kernel<N, TH, EMBED, H>, A, ids, (const H*)table, ld_table, vocab, sp.ncta, W, sp.cols)
+  if (sp.nv <= 1) FT_DU(1, 256);
+  if (sp.nv <= 2) FT_DU(2, 256);
+  if (sp.nv <= 4) FT_DU(2, 512);
+  FT_DU(2, 1024);
 #undef FT_DU
 }
 
@@ -621,7 +657,7 @@ template <typename I, typename O>
 int dispatch_poly(const void* z, int planes, int64_t pstride, int64_t ldz, const float* coef, float eps, void* out, int64_t ldo, int rows, int W, cudaStream_t st) {
   const RowSpread sp = row_spread(rows, W);
   if (sp.nv > 8) return FT_ERR_TOO_LARGE;
-#define FT_PN(N) return launch_rows(sp, rows, st, poly_norm_kernel<N, I, O>, (const I*)z, planes, (size_t)pstride, ldz, coef, eps, (O*)out, ldo, sp.ncta, W, sp.cols)
+#define FT_PN(N) return launch_rows(sp, rows, UPD_THREADS, st, poly_norm_kernel<N, I, O>, (const I*)z, planes, (size_t)pstride, ldz, coef, eps, (O*)out, ldo, sp.ncta, W, sp.cols)
   if (sp.nv <= 1) FT_PN(1);
   if (sp.nv <= 2) FT_PN(2);
   if (sp.nv <= 4) FT_PN(4);
@@ -657,13 +693,13 @@ int dispatch_parallel(float* x, int64_t ldx, const int64_t* ids, const void* tab
 template <typename H>
 int dispatch_update(float* x, int64_t ldx, const float* y, int planes, int64_t pstride, int64_t ldy, const float* w, const float* w_last, float eps, void* h, int64_t ldh,
                     int rows, int W, int store, cudaStream_t st) {
-  const auto [ncta, cols, nv] = row_spread(rows, W);
-  if (nv > 8) return FT_ERR_TOO_LARGE;
-#define FT_RU(N) return launch_update<N, H>(ncta, rows, st, x, ldx, y, planes, pstride, ldy, w, w_last, eps, (H*)h, ldh, W, cols, store)
-  if (nv <= 1) FT_RU(1);
-  if (nv <= 2) FT_RU(2);
-  if (nv <= 4) FT_RU(4);
-  FT_RU(8);
+  const RowSpread sp = row_spread(rows, W);
+  if (sp.nv > 8) return FT_ERR_TOO_LARGE;
+#define FT_RU(N, TH) return launch_rows(sp, rows, TH, st, residual_update_kernel<N, TH, H>, x, ldx, y, planes, (size_t)pstride, ldy, w, w_last, eps, (H*)h, ldh, sp.ncta, W, sp.cols, store)
+  if (sp.nv <= 1) FT_RU(1, 256);
+  if (sp.nv <= 2) FT_RU(2, 256);
+  if (sp.nv <= 4) FT_RU(2, 512);
+  FT_RU(2, 1024);
 #undef FT_RU
 }
 
@@ -768,10 +804,22 @@ FT_EXPORT int ft_token_shift(const float* x, int64_t ldx, const float* rstd, con
   return (int)cudaGetLastError();
 }
 
-// out[r] = a N(z) + b N(z^2) + c N(z^3) + e for rows z of n columns, powers element by element, N(v) = v / sqrt(mean(v^2) + eps); coef: f32 {a, b, c, e}. z and out bf16, or f32 with is_f32.
+// out[r] = a N(z) + b N(z^2) + c N(z^3) + e for rows z of n columns, powers element by element, N(v) = v / sqrt(mean(v^2) + eps); coef: f32 {a, b, c, e}. z and out bf16, or f32 with is_f32;
+// rows end with a whole group of four columns (of eight where a pitch is a multiple of eight). Up to 65536 columns.
 FT_EXPORT int ft_poly_norm(const void* z, int64_t ldz, const float* coef, float eps, int rows, int n, void* out, int64_t ldo, int is_f32, cudaStream_t st) {
   if (rows < 1 || n < 1 || !coef || (ldz & 3) || (ldo & 3)) return FT_ERR_ARG;
   if (is_f32) return dispatch_poly<float, float>(z, 1, 0, ldz, coef, eps, out, ldo, rows, n, st);
+  const int nv = (n + UPD_THREADS * 8 - 1) / (UPD_THREADS * 8);
+  if (rows >= 148 && nv <= 8 && !(ldz & 7) && !(ldo & 7) && !((reinterpret_cast<uintptr_t>(z) | reinterpret_cast<uintptr_t>(out)) & 15)) {
+#define FT_PR(N) poly_norm_rows_kernel<N><<<rows, UPD_THREADS, 0, st>>>((const __nv_bfloat16*)z, ldz, coef, eps, (__nv_bfloat16*)out, ldo, n)
+    if (nv <= 1) FT_PR(1);
+    else if (nv <= 2) FT_PR(2);
+    else if (nv <= 4) FT_PR(4);
+    else if (nv <= 6) FT_PR(6);
+    else FT_PR(8);
+#undef FT_PR
+    return (int)cudaGetLastError();
+  }
   return dispatch_poly<__nv_bfloat16, __nv_bfloat16>(z, 1, 0, ldz, coef, eps, out, ldo, rows, n, st);
 }
 

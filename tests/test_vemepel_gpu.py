@@ -200,7 +200,7 @@ def test_residual_with_norms_behind_sublayers_and_averages_over_depth(dtype, row
 
 # -- dense feed-forward ----------------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", [F32, BF16])
-@pytest.mark.parametrize("width,ff", [(24, 8), (40, 33), (64, 700), (16, 2050), (8, 9001)])
+@pytest.mark.parametrize("width,ff", [(24, 8), (40, 33), (64, 700), (16, 2050), (8, 9001), (8, 16390)])
 def test_dense_feed_forward_of_normed_powers(dtype, width, ff):
     rng = np.random.default_rng(ff)
     act = rounded([0.7, -0.4, 1.3, 0.25], F32)
@@ -208,7 +208,7 @@ def test_dense_feed_forward_of_normed_powers(dtype, width, ff):
     W["act"] = act
     eps = 1e-2
     w = DensePolyWeights.pack(torch.tensor(W["up"]), torch.tensor(W["down"]), torch.tensor(act), eps, "cuda", dtype)
-    for rows in (1, 5, 130):
+    for rows in (1, 5, 130, 150):
         h = rounded(2.0 * rng.standard_normal((rows, width)), dtype)
         assert rel(dense_poly_rows(padded(h, dtype), w).planes[0], O.dense(h, W, eps)) < (1e-5 if dtype == F32 else 3e-2)
         z = rounded(np.exp(rng.standard_normal((rows, 1))) * rng.standard_normal((rows, ff)), dtype)
