@@ -3,7 +3,7 @@
 
     python examples/llama_generate.py --prompt-len 16 --new 32 [--weights /path/to/model.safetensors --config /path/to/config.json]
 
-With `--model DIR` any registered architecture is loaded from its checkpoint directory (`config.json` + safetensors; Llama, Ginisun, Pufevik, Mepupel) and run by the
+With `--model DIR` any registered architecture is loaded from its checkpoint directory (`config.json` + safetensors; Llama, Ginisun, Pufevik, Mepupel, Vemepel) and run by the
 serving engine: `python examples/llama_generate.py --model DIR --prompt 5,17,3 --prompt 8 --new 32 [--temperature 0.8 --top-k 50 --top-p 0.95]`.
 
 On a B200 the same model runs through the tensor-parallel engine (`LlamaTPEngine`: paged KV cache, CUDA-graph decode) with `--engine tp`

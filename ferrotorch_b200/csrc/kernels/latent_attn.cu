@@ -131,6 +131,43 @@ __global__ void __launch_bounds__(128) latent_prep_kernel(T* __restrict__ qkv, i
   }
 }
 
+// Rows that have nothing but a latent to norm (no rotated part, no query latent): a warp each, eight columns a lane
+template <typename T> FT_DEVICE void load8(const T* p, float (&v)[8]);
+template <> FT_DEVICE void load8<float>(const float* p, float (&v)[8]) {
+  const float4 a = reinterpret_cast<const float4*>(p)[0], b = reinterpret_cast<const float4*>(p)[1];
+  v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; v[4] = b.x; v[5] = b.y; v[6] = b.z; v[7] = b.w;
+}
+template <> FT_DEVICE void load8<__nv_bfloat16>(const __nv_bfloat16* p, float (&v)[8]) { bf16x8_to_float(*reinterpret_cast<const bf16x8*>(p), v); }
+template <typename T> FT_DEVICE void store8(T* p, const float (&v)[8]);
+template <> FT_DEVICE void store8<float>(float* p, const float (&v)[8]) {
+  reinterpret_cast<float4*>(p)[0] = make_float4(v[0], v[1], v[2], v[3]);
+  reinterpret_cast<float4*>(p)[1] = make_float4(v[4], v[5], v[6], v[7]);
+}
+template <> FT_DEVICE void store8<__nv_bfloat16>(__nv_bfloat16* p, const float (&v)[8]) { *reinterpret_cast<bf16x8*>(p) = float_to_bf16x8(v); }
+template <typename T>
+__global__ void __launch_bounds__(128) latent_norm_kernel(const T* __restrict__ lat, int64_t ld, int rows, LatentDims D, const float* __restrict__ w, float eps,
+                                                          const int* __restrict__ slots, const int* __restrict__ ctx_rows, T* __restrict__ cache, T* __restrict__ ctx) {
+  const int r = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+  if (r >= rows) return;
+  const T* src = lat + (size_t)r * ld;
+  float ss = 0.f, v[8];
+  for (int i = lane * 8; i < D.rank8; i += 256) {
+    load8(src + i, v);
+#pragma unroll
+    for (int e = 0; e < 8; e++) ss += i + e < D.rank ? v[e] * v[e] : 0.f;
+  }
+  const float rstd = 1.f / sqrtf(warp_sum(ss) / (float)D.rank + eps);
+  T* dst = cache + (size_t)slots[r] * D.row;
+  T* dense = ctx ? ctx + (size_t)ctx_rows[r] * D.row : nullptr;
+  for (int i = lane * 8; i < D.r16; i += 256) {
+    if (i < D.rank8) load8(src + i, v);
+#pragma unroll
+    for (int e = 0; e < 8; e++) v[e] = i + e < D.rank ? v[e] * rstd * w[i + e] : 0.f;
+    store8(dst + i, v);
+    if (dense) store8(dense + i, v);
+  }
+}
+
 __global__ void __launch_bounds__(128) latent_ctx_gather_kernel(const uint4* __restrict__ cache, uint4* __restrict__ ctx, int vecs, const int* __restrict__ slots,
                                                                 const int* __restrict__ rows) {
   const uint4* src = cache + (size_t)slots[blockIdx.x] * vecs;
@@ -959,6 +996,12 @@ FT_EXPORT int ft_latent_prep(void* qkv, int64_t ld, int rows, int H, int d, int 
   if (rows < 1 || !dims_ok(H, d, dr, rank) || q_rank < 0 || (ctx && !ctx_rows) || (q_rank ? dr != 0 || !wq : !cache)) return FT_ERR_ARG;
   const LatentDims D = make_dims(H, d, dr, rank, q_rank);
   if (ld < (int64_t)D.q_cols + (cache ? D.rank8 + dr : 0) || (ld & 7)) return FT_ERR_ARG;
+  if (dr == 0 && q_rank == 0) {
+    const int ctas = (rows + 3) / 4;
+    if (is_f32) latent_norm_kernel<float><<<ctas, 128, 0, st>>>((const float*)qkv + D.q_cols, ld, rows, D, w, eps, slots, ctx_rows, (float*)cache, (float*)ctx);
+    else latent_norm_kernel<__nv_bfloat16><<<ctas, 128, 0, st>>>((const __nv_bfloat16*)qkv + D.q_cols, ld, rows, D, w, eps, slots, ctx_rows, (__nv_bfloat16*)cache, (__nv_bfloat16*)ctx);
+    return (int)cudaGetLastError();
+  }
   if (is_f32) latent_prep_kernel<float><<<rows, 128, 0, st>>>((float*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (float*)cache, (float*)ctx, wq);
   else latent_prep_kernel<__nv_bfloat16><<<rows, 128, 0, st>>>((__nv_bfloat16*)qkv, ld, D, w, eps, positions, cos_t, sin_t, slots, ctx_rows, (__nv_bfloat16*)cache,
                                                                (__nv_bfloat16*)ctx, wq);

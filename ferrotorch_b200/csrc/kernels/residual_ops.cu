@@ -698,8 +698,8 @@ int dispatch_update(float* x, int64_t ldx, const float* y, int planes, int64_t p
 #define FT_RU(N, TH) return launch_rows(sp, rows, TH, st, residual_update_kernel<N, TH, H>, x, ldx, y, planes, (size_t)pstride, ldy, w, w_last, eps, (H*)h, ldh, sp.ncta, W, sp.cols, store)
   if (sp.nv <= 1) FT_RU(1, 256);
   if (sp.nv <= 2) FT_RU(2, 256);
-  if (sp.nv <= 4) FT_RU(2, 512);
-  FT_RU(2, 1024);
+  if (sp.nv <= 4) FT_RU(4, 256);
+  FT_RU(8, 256);
 #undef FT_RU
 }
 
